@@ -7,6 +7,10 @@ torch headers; everything is linked into one shared object that
 ``torch.ops.load_library`` loads.  Objects are cached under ``build/`` keyed
 by a hash of the source, its local headers and the flags, so a rebuild only
 recompiles what changed.  nvcc cross-compiles, so this runs without a GPU.
+
+``build(subset)`` compiles only the sources one model family needs and links
+them into a library of its own (``_C_<subset>.so``): what a fresh checkout does
+when a single model is to be run and the whole library has not been built.
 """
 from __future__ import annotations
 
@@ -22,6 +26,18 @@ CSRC = PKG / "csrc"
 ROOT = PKG.parent
 BUILD = ROOT / "build" / "obj"
 LIB = PKG / "_C.so"
+
+# model family -> sources (relative to csrc) of its stand-alone library
+SUBSETS = {
+    "layered": ("common/tensor_map.cpp", "core_bindings.cpp", "layered_bindings.cpp", "gemm/gemm_bf16.cu", "gemm/gemm_f32.cu",
+                "pointwise/rows32.cu", "attention/qkv_append.cu", "attention/head_mix_token.cu",
+                "attention/head_mix_prefill.cu", "mlstm/mlstm_recurrent.cu", "mlstm/mlstm_chunked.cu",
+                "sampling/sampling.cu", "runtime/page_pool.cpp"),
+}
+
+
+def library_path(subset: str = "") -> Path:
+    return PKG / f"_C_{subset}.so" if subset else LIB
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
@@ -43,7 +59,10 @@ def _headers_digest() -> str:
     return h.hexdigest()
 
 
-def _sources():
+def _sources(subset: str = ""):
+    if subset:
+        files = [CSRC / name for name in SUBSETS[subset]]
+        return [p for p in files if p.suffix == ".cu"], [p for p in files if p.suffix == ".cpp"]
     cu = sorted(CSRC.rglob("*.cu"))
     cpp = sorted(p for p in CSRC.rglob("*.cpp"))
     return cu, cpp
@@ -60,7 +79,8 @@ def _compile(src: Path, cmd_prefix: list[str], tag: str, hdr: str, verbose: bool
         return obj, False
     for stale in BUILD.glob(f"{rel}.*.o"):
         stale.unlink()
-    cmd = cmd_prefix + ["-c", str(src), "-o", str(obj)]
+    part = obj.with_suffix(f".{os.getpid()}.part")   # renamed when complete: an interrupted compile leaves no object behind
+    cmd = cmd_prefix + ["-c", str(src), "-o", str(part)]
     if verbose:
         print(f"[build] {tag} {src.relative_to(ROOT)}", flush=True)
     r = subprocess.run(cmd, capture_output=True, text=True)
@@ -68,11 +88,12 @@ def _compile(src: Path, cmd_prefix: list[str], tag: str, hdr: str, verbose: bool
         raise RuntimeError(f"compile failed: {' '.join(cmd)}\n{r.stdout}\n{r.stderr}")
     if verbose and r.stderr.strip():
         print(r.stderr, flush=True)
+    os.replace(part, obj)
     return obj, True
 
 
-def build(verbose: bool = True, ptxas_info: bool = False) -> Path:
-    """Compile (if needed) and link ``_C.so``; returns its path."""
+def build(verbose: bool = True, ptxas_info: bool = False, subset: str = "") -> Path:
+    """Compile (if needed) and link ``_C.so`` (or the library of one model family); returns its path."""
     import torch
     from torch.utils import cpp_extension as ce
 
@@ -83,13 +104,14 @@ def build(verbose: bool = True, ptxas_info: bool = False) -> Path:
     inc = [f"-I{CSRC}", f"-I{cuda}/include"]
     torch_inc = [f"-I{p}" for p in ce.include_paths()]
     abi = f"-D_GLIBCXX_USE_CXX11_ABI={int(torch._C._GLIBCXX_USE_CXX11_ABI)}"
-    cu, cpp = _sources()
+    lib = library_path(subset)
+    cu, cpp = _sources(subset)
     jobs = []
     nv = [nvcc] + NVCC_FLAGS + (["-Xptxas", "-v"] if ptxas_info else []) + inc
     for s in cu:
         jobs.append((s, nv, "nvcc"))
     for s in cpp:
-        uses_torch = "torch/" in s.read_text() or "ATen/" in s.read_text()
+        uses_torch = any(k in s.read_text() for k in ("torch/", "ATen/", "binding_util.h"))
         cx = ["g++"] + CXX_FLAGS + inc + ([abi] + torch_inc if uses_torch else [])
         jobs.append((s, cx, "g++ "))
     workers = max(1, min(len(jobs), os.cpu_count() or 4))
@@ -98,23 +120,23 @@ def build(verbose: bool = True, ptxas_info: bool = False) -> Path:
     objs = [r[0] for r in res]
     changed = any(r[1] for r in res)
     # (objects may also have been compiled by an earlier, link-less pass: compare against the library's age)
-    stale = LIB.exists() and any(o.stat().st_mtime > LIB.stat().st_mtime for o in objs)
-    if changed or stale or not LIB.exists():
+    stale = lib.exists() and any(o.stat().st_mtime > lib.stat().st_mtime for o in objs)
+    if changed or stale or not lib.exists():
         tl = ce.library_paths()
         # link beside the final name and rename: a reader (a process that loads the library, a copy of the tree) never
         # sees a half-written file
-        tmp = LIB.with_suffix(".so.tmp")
+        tmp = lib.with_suffix(".so.tmp")
         link = ["g++", "-shared", "-o", str(tmp)] + [str(o) for o in objs]
         for p in tl:
             link += [f"-L{p}", f"-Wl,-rpath,{p}"]
         link += [f"-L{cuda}/lib64", "-lc10", "-ltorch_cpu", "-ltorch", "-lc10_cuda", "-ltorch_cuda", "-lcudart"]
         if verbose:
-            print(f"[build] link {LIB.relative_to(ROOT)}", flush=True)
+            print(f"[build] link {lib.relative_to(ROOT)}", flush=True)
         r = subprocess.run(link, capture_output=True, text=True)
         if r.returncode != 0:
             raise RuntimeError(f"link failed: {' '.join(link)}\n{r.stdout}\n{r.stderr}")
-        os.replace(tmp, LIB)
-    return LIB
+        os.replace(tmp, lib)
+    return lib
 
 
 if __name__ == "__main__":

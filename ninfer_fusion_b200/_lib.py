@@ -9,33 +9,44 @@ from __future__ import annotations
 
 import os
 from pathlib import Path
+from typing import Optional
 
 import torch
 
 _LIB = Path(__file__).resolve().parent / "_C.so"
-_loaded = False
+_loaded: Optional[Path] = None
 
 
 def native_available() -> bool:
     return _LIB.exists()
 
 
-def load_native(build_if_missing: bool = False):
-    """Load ``_C.so`` once and return ``torch.ops.nfb200``."""
-    global _loaded
-    if not _loaded:
-        if not _LIB.exists():
-            if build_if_missing or os.environ.get("NFB200_BUILD_ON_IMPORT") == "1":
-                from ._build import build
+def native_path() -> Path:
+    """The library this process loaded, or the full one."""
+    return _loaded or _LIB
 
-                build(verbose=False)
+
+def load_native(build_if_missing: bool = False, subset: str = ""):
+    """Load ``_C.so`` once and return ``torch.ops.nfb200``.
+
+    `subset`: a process that runs one model family only may use that family's own library (see ``_build.SUBSETS``)
+    when the full one is not there; it is compiled if need be."""
+    global _loaded
+    if _loaded is None:
+        path = _LIB
+        if not _LIB.exists():
+            from . import _build
+            if subset:
+                path = _build.build(verbose=False, subset=subset)
+            elif build_if_missing or os.environ.get("NFB200_BUILD_ON_IMPORT") == "1":
+                _build.build(verbose=False)
             else:
                 raise RuntimeError(
                     f"{_LIB} is missing: run `python -m ninfer_fusion_b200._build` "
                     "(or __graft_entry__.build()) first; the CUDA kernels have no fallback"
                 )
-        torch.ops.load_library(str(_LIB))
-        _loaded = True
+        torch.ops.load_library(str(path))
+        _loaded = path
     return torch.ops.nfb200
 
 

@@ -40,7 +40,9 @@ def add_model_args(ap: argparse.ArgumentParser) -> None:
     ap.add_argument("--artifact", help=".ninfer artifact (weights + embedded tokenizer / chat template)")
     ap.add_argument("--model", default="tiny-dense", help="registered geometry for --random-init (see models/config.py); an "
                     "attention-only package (spark-x2.5-4b, muse-glimmer-30b, gemma4-31b, optionally NAME@LAYERS) runs on "
-                    "the CPU oracle at a reduced debug geometry unless --full-geometry is given")
+                    "the CPU oracle at a reduced debug geometry unless --full-geometry is given; a folder with config.json and "
+                    "safetensors, or a geometry of models/architectures.py (kuzanex-tiny, kuzanex-1b, ...), runs as a layer-list model")
+    ap.add_argument("--float32", action="store_true", help="layer-list models: activations, cache and matrix products in true 32-bit")
     ap.add_argument("--full-geometry", action="store_true", help="attention-only packages: the full widths and vocabulary")
     ap.add_argument("--random-init", action="store_true", help="random weights of --model instead of an artifact")
     ap.add_argument("--layers", type=int, default=0, help="shrink the geometry to this many layers (debug)")
@@ -160,6 +162,11 @@ def _oracle_package(args):
                             vocab=0 if full else 2048, hidden_div=1 if full else 8)
 
 
+def _layered_model(args) -> bool:
+    from .models.architectures import LAYERED_REGISTRY, is_model_folder
+    return args.model in LAYERED_REGISTRY or is_model_folder(args.model)
+
+
 def load_model(args) -> Tuple[ModelConfig, Dict[str, object], Tokenizer, str]:
     tok: Optional[Tokenizer] = None
     template: Optional[str] = None
@@ -202,6 +209,27 @@ def load_model(args) -> Tuple[ModelConfig, Dict[str, object], Tokenizer, str]:
         cfg = package_model_config(pkg, args.max_context)
         weights = random_package_weights(pkg, seed=args.seed)
         name = f"{pkg.model_id}:random-init"
+    elif _layered_model(args):
+        # a model folder (config.json + safetensors) or a registered geometry of a layer-list design
+        from .models import architectures as AR
+        if not str(args.device).startswith("cuda"):
+            raise SystemExit(f"{args.model}: layer-list models run on the GPU kernels only")
+        if args.weights not in ("bf16", "stored"):
+            raise SystemExit(f"{args.model}: layer-list models take bf16 weights, not --weights {args.weights}")
+        folder = AR.is_model_folder(args.model)
+        dtype = torch.float32 if getattr(args, "float32", False) else torch.bfloat16
+        try:
+            if folder and not args.random_init:
+                cfg, weights = AR.load_folder(args.model, args.device, dtype)
+            else:
+                cfg = AR.read_config(args.model) if folder else AR.LAYERED_REGISTRY[args.model]
+                cfg = cfg.shrink(args.layers) if args.layers else cfg
+                weights = AR.random_layered_weights(cfg, args.device, args.seed, dtype)
+        except (ValueError, OSError) as e:
+            raise SystemExit(str(e)) from None
+        name = cfg.name if folder and not args.random_init else f"{cfg.name}:random-init"
+        if folder and not args.tokenizer and os.path.exists(os.path.join(args.model, "tokenizer.json")):
+            tok = Tokenizer.from_file(os.path.join(args.model, "tokenizer.json"))
     else:
         cfg = get_config(args.model)
         if args.layers:
@@ -310,6 +338,9 @@ def build_engine(args, cfg: ModelConfig, weights, ranks=None) -> Optional[Engine
     kv = args.kv_dtype
     check_device_routes(args, weights)
     _kv_spec_from_ceilings(args, cfg)
+    if _layered_model(args) and not args.artifact:
+        if ranks is not None or getattr(args, "spec", "none") not in ("none", "off") or getattr(args, "vision", False) or args.weight_budget_gib > 0:
+            raise SystemExit(f"{cfg.name}: layer-list models run on one GPU, without --tp / --ep / --dp, --spec, --vision or --weight-budget-gib")
     if ranks is not None and max(int(getattr(args, "ep", 1)), int(getattr(args, "dp", 1))) > 1:
         # every request lives on one rank (parallel/partitioned.py); expert parallelism adds the MoE exchange between
         # the ranks inside every forward pass, hence lock step

@@ -1,0 +1,78 @@
+// Attention whose scores are shaped per head and then mixed across heads before the softmax (plain C++ ABI).
+//
+//   c_g(i, j)  = cap * tanh(scale * q_g(i) . k_{g / (H/G)}(j) / cap)          (cap = 0: no cap)
+//   s_h(i, j)  = sum_g mix[h, g] * c_g(i, j)  -  slope[h] * (i - j)            (mix = null: the identity)
+//   visible    : 0 <= i - j < window (window = 0: all of the past)
+//   a_h(i, j)  = exp(s_h) / (sink_one + sum_j exp(s_h))
+//   out_h(i)   = sigmoid(gate[i, h]) * sum_j a_h(i, j) v(j)                    (gate = null: no gate)
+//
+// `slope` is the bias AFTER mixing: a per-head bias b_g taken off before the mix is slope[h] = sum_g mix[h, g] b_g.
+// Scores, weights and sums are fp32.  K and V live in paged planes [page, kv_head, token in page, width]; widths are
+// multiples of 16, zero-padded by the producer.  q, k, v and out are bf16 or (f32) fp32.
+#pragma once
+#include <cuda_runtime.h>
+#include <stdint.h>
+
+namespace nfb {
+
+struct HeadMixArgs {
+  const void* q = nullptr;          // [T, n_heads * dim], leading dimension ldq
+  int64_t ldq = 0;
+  const void* k_pages = nullptr;    // [pages, n_kv, page_size, dim]
+  const void* v_pages = nullptr;    // [pages, n_kv, page_size, vdim]
+  const int* block_table = nullptr; // [rows, table_ld]
+  int table_ld = 0;
+  const int* table_row = nullptr;   // [T]
+  const int* kv_len = nullptr;      // [T] position + 1
+  int T = 0;
+  int n_heads = 0, n_kv = 0, dim = 0, vdim = 0, page_size = 0, window = 0;
+  float scale = 1.f, softcap = 0.f, sink = 0.f;   // sink: what is added to the softmax denominator (0 or 1)
+  const float* mix = nullptr;       // [H, H] row-major, or null
+  const float* slope = nullptr;     // [H], or null
+  const float* gate = nullptr;      // [T, *] raw gate values of head h at gate[t * ld_gate + h], or null
+  int64_t ld_gate = 0;
+  void* out = nullptr;              // [T, n_heads * vdim], leading dimension ldo
+  int64_t ldo = 0;
+  bool f32 = false;
+  cudaStream_t stream = nullptr;
+  bool pdl = false;
+};
+
+// One CTA per (token, split of its visible keys); a second kernel merges the splits.  part_o: fp32
+// [T, n_splits, H, vdim], part_ml: fp32 [T, n_splits, H, 2]; both unused with one split.
+const char* head_mix_token_attention(const HeadMixArgs& a, int split_keys, int n_splits, float* part_o, float* part_ml);
+
+// bf16 prefill: query blocks of up to 64 consecutive tokens of one sequence (blk_start / blk_count, n_blocks).
+// `max_keys` bounds the visible key range of a block (host).  Mixed scores pass through `scratch` (scratch_bytes) in
+// register-fragment order, as many blocks at a time as fit.
+const char* head_mix_prefill(const HeadMixArgs& a, const int* blk_start, const int* blk_count, int n_blocks, int max_keys,
+                             void* scratch, int64_t scratch_bytes);
+// Scratch for `blocks` query blocks at a time.
+int64_t head_mix_prefill_scratch(int n_heads, int max_keys, int window, int blocks);
+constexpr int kHeadMixBlock = 64;
+
+struct QkvAppendArgs {
+  const void* proj = nullptr;       // [T, ldp]: q heads at q_off, k heads at k_off, v heads at v_off
+  int64_t ldp = 0;
+  int q_off = 0, k_off = 0, v_off = 0;
+  int T = 0, n_heads = 0, n_kv = 0;
+  int dim = 0, dim_true = 0, vdim = 0;     // padded q / k width, width the norm's mean runs over, padded v width
+  const float* q_norm = nullptr;    // [dim] fp32 weights, or null = no norm
+  const float* k_norm = nullptr;
+  float eps = 0.f;
+  const int* table_row = nullptr;
+  const int* cache_pos = nullptr;
+  const int* block_table = nullptr;
+  int table_ld = 0, page_size = 0;
+  void* q_out = nullptr;            // [T, n_heads * dim], leading dimension ldq
+  int64_t ldq = 0;
+  void* k_pages = nullptr;
+  void* v_pages = nullptr;
+  bool f32 = false;
+  cudaStream_t stream = nullptr;
+  bool pdl = false;
+};
+// Per-head RMS norm of q and k, k and v rows appended to their pages.
+const char* qkv_append(const QkvAppendArgs& a);
+
+}  // namespace nfb

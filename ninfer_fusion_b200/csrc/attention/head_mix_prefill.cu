@@ -1,0 +1,376 @@
+// Head-mixing attention for prompt portions (bf16 operands, tensor cores).  A mixed score needs every head's score of
+// the same (query, key), while the weighted sum over values is per head, so the work is cut in two kernels that meet in
+// an L2-sized scratch of fp32 scores:
+//
+//   scores   one warp = 16 queries x 8 NT keys x ALL heads.  The scores of one head come out of mma.sync in registers,
+//            are soft-capped there and added into the mixed scores of every head, acc[h] += mix[h, g] * c_g (outer
+//            product form: no score ever crosses a thread).  Distance bias and mask are applied to the finished sums,
+//            which are stored in accumulator-fragment order.  Query and key fragments are read straight from global /
+//            L1: the k index of an MMA may be permuted freely as long as both operands agree, so each lane takes four
+//            consecutive values per 16-wide step.
+//   values   one CTA = (64 queries, head): flash-style running softmax over score fragments read back in the same
+//            order (they are exactly the A operand of the value MMA), V tiles staged with cp.async.
+//
+// Query blocks are processed as many at a time as the scratch holds.
+#include "head_mix.h"
+
+#include <math_constants.h>
+
+#include "../common/elem.cuh"
+#include "../common/launch.h"
+#include "../common/mma_sync.cuh"
+
+namespace nfb {
+
+namespace {
+
+using bf16 = __nv_bfloat16;
+
+struct PrefillParams {
+  HeadMixArgs a;
+  const int* blk_start;
+  const int* blk_count;
+  int blk0;            // first query block of this launch
+  int n_tiles;         // 8-key tiles reserved per query block
+  float4* scratch;     // [block][tile][q tile 0..3][head][lane]
+};
+
+// Key range of a query block and of one of its 16-query tiles, in 8-key tiles counted from the block's first key.
+struct BlockRange {
+  int t0, cnt, row, pos0, last, lo, k0;
+  __device__ __forceinline__ BlockRange(const PrefillParams& p, int blk) {
+    t0 = p.blk_start[blk];
+    cnt = p.blk_count[blk];
+    row = p.a.table_row[t0];
+    pos0 = p.a.kv_len[t0] - 1;
+    last = pos0 + cnt - 1;
+    lo = p.a.window > 0 ? max(0, pos0 - p.a.window + 1) : 0;
+    k0 = lo & ~7;
+  }
+  __device__ __forceinline__ int first_query(int qt) const { return pos0 + qt * 16; }
+  __device__ __forceinline__ int last_query(int qt) const { return min(pos0 + qt * 16 + 15, last); }
+  __device__ __forceinline__ int first_tile(int qt, int window) const {
+    const int f = window > 0 ? max(0, first_query(qt) - window + 1) : 0;
+    return (f - k0) >> 3;
+  }
+  __device__ __forceinline__ int last_tile(int qt) const { return (last_query(qt) - k0) >> 3; }
+};
+
+// HMAX: heads rounded up (mixed scores of all of them are live in registers); NT: 8-key tiles per warp.
+// blockDim 256: 8 warps = 4 query tiles x 2 key groups.  grid: (query block, key group pair, group of HMAX output heads)
+template <int HMAX, int NT>
+__global__ void __launch_bounds__(256) head_mix_scores_kernel(const PrefillParams p) {
+  extern __shared__ __align__(16) float mix_s[];   // [H][HMAX]: mix_s[g][h] = mix[h0 + h, g]
+  const HeadMixArgs& a = p.a;
+  const int H = a.n_heads, G = a.n_kv, R = H / G, D = a.dim, P = a.page_size, W = a.window;
+  const int h0 = blockIdx.z * HMAX;
+  for (int i = threadIdx.x; i < H * HMAX; i += blockDim.x) {
+    const int g = i / HMAX, h = h0 + i % HMAX;
+    mix_s[i] = h < H ? (a.mix != nullptr ? a.mix[h * H + g] : (h == g ? 1.f : 0.f)) : 0.f;
+  }
+  pdl_launch_next();
+  pdl_wait_prior();
+  __syncthreads();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int qt = warp & 3;
+  const BlockRange br(p, p.blk0 + blockIdx.x);
+  if (qt * 16 >= br.cnt) return;
+  const int tile0 = (blockIdx.y * 2 + (warp >> 2)) * NT;
+  if (tile0 > br.last_tile(qt) || tile0 + NT <= br.first_tile(qt, W)) return;
+  const int r4 = lane >> 2, c4 = lane & 3;
+
+  // query rows (A fragment rows r4, r4 + 8), clamped to the block
+  const bf16* qrow0;
+  const bf16* qrow1;
+  {
+    const int i0 = min(qt * 16 + r4, br.cnt - 1), i1 = min(qt * 16 + r4 + 8, br.cnt - 1);
+    qrow0 = static_cast<const bf16*>(a.q) + (br.t0 + i0) * a.ldq + c4 * 4;
+    qrow1 = static_cast<const bf16*>(a.q) + (br.t0 + i1) * a.ldq + c4 * 4;
+  }
+  // key rows (B fragment column r4 of each tile), clamped to mapped positions; the mask below removes the others
+  const bf16* krow[NT];
+#pragma unroll
+  for (int n = 0; n < NT; ++n) {
+    const int key = min(max(br.k0 + (tile0 + n) * 8 + r4, br.lo), br.last);
+    const int page = max(a.block_table[static_cast<long long>(br.row) * a.table_ld + key / P], 0);
+    krow[n] = static_cast<const bf16*>(a.k_pages) + (static_cast<long long>(page) * G * P + key % P) * D + c4 * 4;
+  }
+  float acc[HMAX][NT * 4];
+#pragma unroll
+  for (int h = 0; h < HMAX; ++h)
+#pragma unroll
+    for (int j = 0; j < NT * 4; ++j) acc[h][j] = 0.f;
+  const float inv_cap = a.softcap > 0.f ? a.scale / a.softcap : 0.f;
+  for (int g = 0; g < H; ++g) {
+    float c[NT * 4];
+#pragma unroll
+    for (int j = 0; j < NT * 4; ++j) c[j] = 0.f;
+    const long long kofs = static_cast<long long>(g / R) * P * D;
+    const bf16* q0 = qrow0 + g * D;
+    const bf16* q1 = qrow1 + g * D;
+#pragma unroll 4
+    for (int d = 0; d < D; d += 16) {
+      const uint2 x0 = *reinterpret_cast<const uint2*>(q0 + d);
+      const uint2 x1 = *reinterpret_cast<const uint2*>(q1 + d);
+      const uint32_t af[4] = {x0.x, x1.x, x0.y, x1.y};
+#pragma unroll
+      for (int n = 0; n < NT; ++n) {
+        const uint2 y = *reinterpret_cast<const uint2*>(krow[n] + kofs + d);
+        mma_bf16_16816(c + 4 * n, af, y.x, y.y);
+      }
+    }
+    if (a.softcap > 0.f) {
+#pragma unroll
+      for (int j = 0; j < NT * 4; ++j) c[j] = a.softcap * tanh_of<bf16>(c[j] * inv_cap);
+    } else {
+#pragma unroll
+      for (int j = 0; j < NT * 4; ++j) c[j] *= a.scale;
+    }
+    const float4* mg = reinterpret_cast<const float4*>(mix_s + g * HMAX);
+#pragma unroll
+    for (int h = 0; h < HMAX; h += 4) {
+      const float4 m = mg[h / 4];
+#pragma unroll
+      for (int j = 0; j < NT * 4; ++j) {
+        acc[h][j] = fmaf(m.x, c[j], acc[h][j]);
+        acc[h + 1][j] = fmaf(m.y, c[j], acc[h + 1][j]);
+        acc[h + 2][j] = fmaf(m.z, c[j], acc[h + 2][j]);
+        acc[h + 3][j] = fmaf(m.w, c[j], acc[h + 3][j]);
+      }
+    }
+  }
+#pragma unroll
+  for (int n = 0; n < NT; ++n) {
+    const int tile = tile0 + n;
+    if (tile >= p.n_tiles) break;
+    const int j0 = br.k0 + tile * 8 + c4 * 2;             // key of accumulator columns 0, 1
+    const int i0 = br.first_query(qt) + r4;               // query of rows 0, 1 (i0, i0 + 8)
+    float dist[4];
+    bool vis[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int d = (i0 + (e >> 1) * 8) - (j0 + (e & 1));
+      dist[e] = static_cast<float>(d);
+      vis[e] = d >= 0 && (W <= 0 || d < W);
+    }
+    float4* dst = p.scratch + ((static_cast<long long>(blockIdx.x) * p.n_tiles + tile) * 4 + qt) * H * 32 + lane;
+#pragma unroll
+    for (int h = 0; h < HMAX; ++h) {
+      if (h0 + h < H) {
+        const float sl = a.slope != nullptr ? a.slope[h0 + h] : 0.f;
+        float4 o;
+        o.x = vis[0] ? acc[h][4 * n] - sl * dist[0] : -CUDART_INF_F;
+        o.y = vis[1] ? acc[h][4 * n + 1] - sl * dist[1] : -CUDART_INF_F;
+        o.z = vis[2] ? acc[h][4 * n + 2] - sl * dist[2] : -CUDART_INF_F;
+        o.w = vis[3] ? acc[h][4 * n + 3] - sl * dist[3] : -CUDART_INF_F;
+        dst[(h0 + h) * 32] = o;
+      }
+    }
+  }
+}
+
+constexpr int kVTile = 64;   // keys per V tile
+
+// VT: 16-wide value column tiles per CTA.  blockDim 128: warp = query tile.  grid: (query block, head, value chunk)
+template <int VT>
+__global__ void __launch_bounds__(128) head_mix_values_kernel(const PrefillParams p) {
+  constexpr int kLd = VT * 16 + 8;
+  extern __shared__ __align__(16) bf16 v_s[];   // [2][kVTile][kLd]
+  const HeadMixArgs& a = p.a;
+  const int H = a.n_heads, G = a.n_kv, V = a.vdim, P = a.page_size, W = a.window;
+  const int h = blockIdx.y, g = h / (H / G), v0 = blockIdx.z * VT * 16;
+  pdl_launch_next();
+  pdl_wait_prior();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int qt = warp;
+  const BlockRange br(p, p.blk0 + blockIdx.x);
+  const bool live = qt * 16 < br.cnt;
+  const int first = live ? br.first_tile(qt, W) : 1, last = live ? br.last_tile(qt) : 0;
+  const int r4 = lane >> 2, c4 = lane & 3;
+  const int n_vt = (br.last - br.k0) / kVTile + 1;
+  const int* table = a.block_table + static_cast<long long>(br.row) * a.table_ld;
+  const bf16* vp = static_cast<const bf16*>(a.v_pages) + static_cast<long long>(g) * P * V;
+  const uint32_t vs_base = smem_u32(v_s);
+  auto stage = [&](int vt) {
+    const uint32_t dst = vs_base + (vt & 1) * (kVTile * kLd * 2);
+    for (int i = threadIdx.x; i < kVTile * VT * 2; i += 128) {
+      const int r = i / (VT * 2), c = (i % (VT * 2)) * 8;
+      const int key = br.k0 + vt * kVTile + r;
+      bool ok = key >= br.lo && key <= br.last && v0 + c < V;
+      const int page = ok ? table[key / P] : -1;
+      ok = ok && page >= 0;
+      const bf16* src = ok ? vp + (static_cast<long long>(page) * G * P + key % P) * V + v0 + c : vp;
+      cp_async16(dst + (r * kLd + c) * 2, src, ok);
+    }
+    cp_async_commit();
+  };
+  float o[VT * 2][4];
+#pragma unroll
+  for (int n = 0; n < VT * 2; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) o[n][e] = 0.f;
+  float m[2] = {-CUDART_INF_F, -CUDART_INF_F}, l[2] = {0.f, 0.f};
+  const float4* sc = p.scratch + ((static_cast<long long>(blockIdx.x) * p.n_tiles) * 4 + qt) * H * 32 + h * 32 + lane;
+  const long long sc_tile = static_cast<long long>(4) * H * 32;
+  stage(0);
+  for (int vt = 0; vt < n_vt; ++vt) {
+    const bool mine = vt * 8 <= last && vt * 8 + 7 >= first;
+    float4 s[8];
+    if (mine) {
+#pragma unroll
+      for (int n = 0; n < 8; ++n) {
+        const int tile = vt * 8 + n;
+        s[n] = (tile >= first && tile <= last) ? sc[tile * sc_tile]
+                                               : make_float4(-CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F);
+      }
+    }
+    if (vt + 1 < n_vt) { stage(vt + 1); cp_async_wait<1>(); } else { cp_async_wait<0>(); }
+    __syncthreads();
+    if (mine) {
+      float mx0 = m[0], mx1 = m[1];
+#pragma unroll
+      for (int n = 0; n < 8; ++n) {
+        mx0 = fmaxf(mx0, fmaxf(s[n].x, s[n].y));
+        mx1 = fmaxf(mx1, fmaxf(s[n].z, s[n].w));
+      }
+#pragma unroll
+      for (int d = 1; d < 4; d <<= 1) {
+        mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, d));
+        mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, d));
+      }
+      // a row without a visible key so far keeps maximum -inf; its weights are exp(-inf - 0) = 0
+      const float b0 = mx0 == -CUDART_INF_F ? 0.f : mx0, b1 = mx1 == -CUDART_INF_F ? 0.f : mx1;
+      const float cr0 = __expf(m[0] - b0), cr1 = __expf(m[1] - b1);
+      m[0] = mx0;
+      m[1] = mx1;
+      l[0] *= cr0;
+      l[1] *= cr1;
+#pragma unroll
+      for (int n = 0; n < VT * 2; ++n) {
+        o[n][0] *= cr0; o[n][1] *= cr0; o[n][2] *= cr1; o[n][3] *= cr1;
+      }
+      const uint32_t tile_base = vs_base + (vt & 1) * (kVTile * kLd * 2);
+#pragma unroll
+      for (int kk = 0; kk < 4; ++kk) {
+        float w[8];
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          const float4 x = s[2 * kk + u];
+          w[4 * u] = __expf(x.x - b0); w[4 * u + 1] = __expf(x.y - b0);
+          w[4 * u + 2] = __expf(x.z - b1); w[4 * u + 3] = __expf(x.w - b1);
+          l[0] += w[4 * u] + w[4 * u + 1];
+          l[1] += w[4 * u + 2] + w[4 * u + 3];
+        }
+        const uint32_t af[4] = {pack_bf16x2(w[0], w[1]), pack_bf16x2(w[2], w[3]), pack_bf16x2(w[4], w[5]), pack_bf16x2(w[6], w[7])};
+#pragma unroll
+        for (int n = 0; n < VT; ++n) {
+          uint32_t b[4];
+          ldsm_x4_trans(tile_base + ((kk * 16 + (lane & 15)) * kLd + n * 16 + (lane >> 4) * 8) * 2, b);
+          mma_bf16_16816(o[2 * n], af, b[0], b[1]);
+          mma_bf16_16816(o[2 * n + 1], af, b[2], b[3]);
+        }
+      }
+    }
+    __syncthreads();
+  }
+  if (!live) return;
+#pragma unroll
+  for (int d = 1; d < 4; d <<= 1) {
+    l[0] += __shfl_xor_sync(0xffffffffu, l[0], d);
+    l[1] += __shfl_xor_sync(0xffffffffu, l[1], d);
+  }
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    const int i = qt * 16 + r4 + r * 8;
+    if (i >= br.cnt) continue;
+    const long long t = br.t0 + i;
+    float f;
+    if (a.sink > 0.f) {
+      const float mx = fmaxf(m[r], 0.f);
+      const float e = expf(m[r] - mx);
+      f = e / (a.sink * expf(-mx) + l[r] * e);
+    } else {
+      f = 1.f / l[r];
+    }
+    if (a.gate != nullptr) f *= sigmoid_of<bf16>(a.gate[t * a.ld_gate + h]);
+    bf16* dst = static_cast<bf16*>(a.out) + t * a.ldo + static_cast<long long>(h) * V + v0 + c4 * 2;
+#pragma unroll
+    for (int n = 0; n < VT * 2; ++n)
+      if (v0 + n * 8 < V) *reinterpret_cast<uint32_t*>(dst + n * 8) = pack_bf16x2(o[n][2 * r] * f, o[n][2 * r + 1] * f);
+  }
+}
+
+int tiles_for(int max_keys, int window) {
+  // 8-key tiles of the widest query block: its first query reaches window - 1 keys back, the start is rounded down
+  int keys = max_keys;
+  if (window > 0 && window + kHeadMixBlock - 1 < keys) keys = window + kHeadMixBlock - 1;
+  return (keys + 7 + 7) / 8;
+}
+
+template <int HMAX, int NT>
+cudaError_t launch_scores(const PrefillParams& p, int n_blocks) {
+  auto kern = head_mix_scores_kernel<HMAX, NT>;
+  const size_t smem = sizeof(float) * static_cast<size_t>(p.a.n_heads) * HMAX;
+  const int groups = (p.n_tiles + 2 * NT - 1) / (2 * NT);
+  const dim3 grid(n_blocks, groups, (p.a.n_heads + HMAX - 1) / HMAX);
+  if (smem > 48 * 1024) {
+    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    if (e != cudaSuccess) return e;
+  }
+  return launch_kernel(kern, grid, dim3(256), smem, p.a.stream, p.a.pdl, 1, p);
+}
+
+template <int VT>
+cudaError_t launch_values(const PrefillParams& p, int n_blocks) {
+  auto kern = head_mix_values_kernel<VT>;
+  constexpr int smem = 2 * kVTile * (VT * 16 + 8) * 2;
+  static bool attr_set = false;
+  if (smem > 48 * 1024 && !attr_set) {
+    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return e;
+    attr_set = true;
+  }
+  const dim3 grid(n_blocks, p.a.n_heads, (p.a.vdim + VT * 16 - 1) / (VT * 16));
+  return launch_kernel(kern, grid, dim3(128), smem, p.a.stream, p.a.pdl, 1, p);
+}
+
+}  // namespace
+
+int64_t head_mix_prefill_scratch(int n_heads, int max_keys, int window, int blocks) {
+  return static_cast<int64_t>(blocks) * tiles_for(max_keys, window) * 4 * n_heads * 32 * 16;
+}
+
+const char* head_mix_prefill(const HeadMixArgs& a, const int* blk_start, const int* blk_count, int n_blocks, int max_keys,
+                             void* scratch, int64_t scratch_bytes) {
+  if (a.T <= 0 || n_blocks <= 0) return nullptr;
+  if (a.f32) return "head_mix_prefill: bf16 only";
+  if (a.dim % 16 || a.vdim % 16 || a.n_kv <= 0 || a.n_heads % a.n_kv) return "head_mix_prefill: bad head geometry";
+  if (a.n_heads > 512) return "head_mix_prefill: too many heads";
+  if (a.ldq % 4 || a.ldo % 2) return "head_mix_prefill: misaligned rows";
+  PrefillParams p;
+  p.a = a;
+  p.blk_start = blk_start;
+  p.blk_count = blk_count;
+  p.scratch = static_cast<float4*>(scratch);
+  p.n_tiles = tiles_for(max_keys, a.window);
+  const int64_t per_block = head_mix_prefill_scratch(a.n_heads, max_keys, a.window, 1);
+  const int at_once = static_cast<int>(scratch_bytes / per_block < n_blocks ? scratch_bytes / per_block : n_blocks);
+  if (at_once < 1) return "head_mix_prefill: the scratch does not hold one query block";
+  for (p.blk0 = 0; p.blk0 < n_blocks; p.blk0 += at_once) {
+    const int n = n_blocks - p.blk0 < at_once ? n_blocks - p.blk0 : at_once;
+    cudaError_t e;
+    if (a.n_heads <= 4) e = launch_scores<4, 4>(p, n);
+    else if (a.n_heads <= 8) e = launch_scores<8, 2>(p, n);
+    else if (a.n_heads <= 16) e = launch_scores<16, 2>(p, n);
+    else e = launch_scores<32, 1>(p, n);
+    if (e != cudaSuccess) return cudaGetErrorString(e);
+    if (a.vdim <= 32) e = launch_values<2>(p, n);
+    else if (a.vdim <= 64) e = launch_values<4>(p, n);
+    else if (a.vdim <= 128) e = launch_values<8>(p, n);
+    else e = launch_values<16>(p, n);
+    if (e != cudaSuccess) return cudaGetErrorString(e);
+  }
+  return nullptr;
+}
+
+}  // namespace nfb

@@ -51,7 +51,8 @@ struct GemmGather {
   float eps = 0.f;
 };
 
-enum GemmActivation : int { kActNone = 0, kActGeluTanh = 1, kActGeluErf = 2 };
+// kActXielu: z > 0: a z^2 + z / 2;  z <= 0: b (exp(z) - 1 - z) + z / 2, with (a, b) = act_params[0..1] (both positive).
+enum GemmActivation : int { kActNone = 0, kActGeluTanh = 1, kActGeluErf = 2, kActXielu = 3 };
 
 constexpr int kMaxRanks = 8;
 
@@ -78,6 +79,12 @@ struct GemmArgs {
   int64_t ldr = 0;
   const float* bias = nullptr;   // [N] fp32, added by kEpiStore and kEpiResidual
   int act = kActNone;            // kEpiStore: out = act(acc + bias)
+  const float* act_params = nullptr;  // kActXielu: two floats on the device
+  // kEpiStore: columns n >= out32_from are stored as fp32 in out32[t, n - out32_from] instead of bf16 in `out` (gate
+  // rows whose consumers work in 32-bit, or a whole 32-bit result with out32_from = 0; `out` may then be null)
+  float* out32 = nullptr;
+  int64_t ldo32 = 0;
+  int out32_from = 0;
   float* partial = nullptr;
   int splits = 1;
   int epi = kEpiStore;

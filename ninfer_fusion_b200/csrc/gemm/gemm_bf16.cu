@@ -77,7 +77,11 @@ struct KernelParams {
   const __nv_bfloat16* resid;
   long long ldr;
   const float* bias;
-  int act;  // kActNone / kActGeluTanh / kActGeluErf, applied after the bias (kEpiStore only)
+  int act;  // GemmActivation, applied after the bias (kEpiStore only)
+  const float* act_params;
+  float* out32;        // kEpiStore: columns >= out32_from as fp32 (nullptr: none)
+  long long ldo32;
+  int out32_from;
   float* partial;      // [splits, T, N] fp32
   int* status;
   // kEpiPushPartial: tensor-parallel reduce-scatter by peer stores
@@ -122,6 +126,12 @@ __device__ __forceinline__ float gelu(float x, int mode) {
     return 0.5f * x * (1.f + tanhf(u));
   }
   return 0.5f * x * (1.f + erff(x * 0.7071067811865476f));
+}
+
+__device__ __forceinline__ float activate(float z, int mode, float a, float b) {
+  if (mode == kActXielu)
+    return z > 0.f ? (a * z + 0.5f) * z : b * (__expf(z) - 1.f - z) + 0.5f * z;
+  return gelu(z, mode);
 }
 
 template <int TN, int EPI, bool DEEP>
@@ -602,6 +612,8 @@ __global__ void __launch_bounds__(128) gemm_ws_kernel(const __grid_constant__ CU
     } else {
       const int n = n0 + warp * 32 + lane;
       const float bias = ((EPI == kEpiStore || EPI == kEpiResidual) && p.bias != nullptr && n < p.N) ? p.bias[n] : 0.f;
+      const float act_a = EPI == kEpiStore && p.act_params != nullptr ? p.act_params[0] : 0.f;
+      const float act_b = EPI == kEpiStore && p.act_params != nullptr ? p.act_params[1] : 0.f;
       // tiles of conv channels (kEpiStore at decode): taps + SiLU + history roll here, activation to conv_out
       const bool conv_tile = EPI == kEpiStore && p.conv_state != nullptr && n0 < p.conv_C;
       float cw[4] = {0.f, 0.f, 0.f, 0.f};
@@ -690,8 +702,8 @@ __global__ void __launch_bounds__(128) gemm_ws_kernel(const __grid_constant__ CU
             float a1 = v[2 * m + 1] + bias;
             if constexpr (EPI == kEpiStore) {
               if (p.act != kActNone) {
-                a0 = gelu(a0, p.act);
-                a1 = gelu(a1, p.act);
+                a0 = activate(a0, p.act, act_a, act_b);
+                a1 = activate(a1, p.act, act_a, act_b);
               }
             }
             const float send = (lane & 1) ? a0 : a1;
@@ -705,7 +717,10 @@ __global__ void __launch_bounds__(128) gemm_ws_kernel(const __grid_constant__ CU
                 lo += __bfloat162float(r2[m].x);
                 hi += __bfloat162float(r2[m].y);
               }
-              *reinterpret_cast<uint32_t*>(outp + static_cast<long long>(t) * ldo + ne) = pack_bf16x2(lo, hi);
+              if (EPI == kEpiStore && p.out32 != nullptr && ne >= p.out32_from)
+                *reinterpret_cast<float2*>(p.out32 + static_cast<long long>(t) * p.ldo32 + ne - p.out32_from) = make_float2(lo, hi);
+              else
+                *reinterpret_cast<uint32_t*>(outp + static_cast<long long>(t) * ldo + ne) = pack_bf16x2(lo, hi);
             }
           }
         }
@@ -942,6 +957,8 @@ __global__ void __launch_bounds__(kPersistThreads, 1) gemm_persist_kernel(const 
       } else {
         const int n = n0 + lg * 32 + lane;
         const float bias = (p.bias != nullptr && n < p.N) ? p.bias[n] : 0.f;
+        const float act_a = EPI == kEpiStore && p.act_params != nullptr ? p.act_params[0] : 0.f;
+        const float act_b = EPI == kEpiStore && p.act_params != nullptr ? p.act_params[1] : 0.f;
         for (int c = 0; c < TN; c += kChunk) {
           if (t0 + c >= p.T) break;
           uint32_t v[kChunk];
@@ -964,8 +981,8 @@ __global__ void __launch_bounds__(kPersistThreads, 1) gemm_persist_kernel(const 
             float a1 = __uint_as_float(v[2 * m + 1]) + bias;
             if constexpr (EPI == kEpiStore) {
               if (p.act != kActNone) {
-                a0 = gelu(a0, p.act);
-                a1 = gelu(a1, p.act);
+                a0 = activate(a0, p.act, act_a, act_b);
+                a1 = activate(a1, p.act, act_a, act_b);
               }
             }
             const float send = (lane & 1) ? a0 : a1;
@@ -979,7 +996,10 @@ __global__ void __launch_bounds__(kPersistThreads, 1) gemm_persist_kernel(const 
                 lo += __bfloat162float(r2[m].x);
                 hi += __bfloat162float(r2[m].y);
               }
-              *reinterpret_cast<uint32_t*>(p.out + static_cast<long long>(t) * p.ldo + ne) = pack_bf16x2(lo, hi);
+              if (EPI == kEpiStore && p.out32 != nullptr && ne >= p.out32_from)
+                *reinterpret_cast<float2*>(p.out32 + static_cast<long long>(t) * p.ldo32 + ne - p.out32_from) = make_float2(lo, hi);
+              else
+                *reinterpret_cast<uint32_t*>(p.out + static_cast<long long>(t) * p.ldo + ne) = pack_bf16x2(lo, hi);
             }
           }
         }
@@ -1273,6 +1293,13 @@ const char* gemm_bf16(const GemmArgs& a) {
   if ((reinterpret_cast<uintptr_t>(a.w) | reinterpret_cast<uintptr_t>(a.x)) & 15)
     return "gemm_bf16: operands must be 16-byte aligned";
   if ((a.N & 1) || (a.ldo & 1)) return "gemm_bf16: N and ldo must be even";
+  if (a.act == kActXielu && a.act_params == nullptr) return "gemm_bf16: xIELU needs its two parameters";
+  if (a.out32 != nullptr) {
+    if (a.epi != kEpiStore || a.conv.state != nullptr) return "gemm_bf16: fp32 columns need the plain store epilogue";
+    if ((a.ldo32 & 1) || (a.out32_from & 1) || a.out32_from < 0 || a.out32_from >= a.N ||
+        a.ldo32 < a.N - a.out32_from || (reinterpret_cast<uintptr_t>(a.out32) & 7))
+      return "gemm_bf16: fp32 columns must start at an even column and have an even leading dimension";
+  }
   const int tn = gemm_tile_tokens(static_cast<int>(a.T));
   const bool global_split = a.epi == kEpiPartial || a.epi == kEpiPushPartial;
   KernelParams kp = {};
@@ -1374,7 +1401,9 @@ const char* gemm_bf16(const GemmArgs& a) {
   kp.bias = a.bias; kp.act = a.epi == kEpiStore ? a.act : kActNone; kp.partial = a.partial; kp.status = a.status;
   if (a.epi == kEpiResidual && a.resid == nullptr) return "gemm_bf16: residual epilogue without residual";
   if (a.epi == kEpiPartial && a.partial == nullptr) return "gemm_bf16: split-K without workspace";
-  const bool needs_out = a.epi == kEpiStore || a.epi == kEpiResidual || a.epi == kEpiSwiglu;
+  kp.act_params = a.act_params; kp.out32 = a.out32; kp.ldo32 = a.ldo32; kp.out32_from = a.out32_from;
+  const bool all32 = a.out32 != nullptr && a.out32_from == 0;
+  const bool needs_out = !all32 && (a.epi == kEpiStore || a.epi == kEpiResidual || a.epi == kEpiSwiglu);
   if (needs_out && a.out == nullptr) return "gemm_bf16: no output";
 
   CUtensorMap tw, tx;

@@ -10,6 +10,7 @@
 
 #include <math_constants.h>
 
+#include "../common/elem.cuh"
 #include "../common/ptx.cuh"
 
 namespace nfb {
@@ -46,25 +47,25 @@ __device__ __forceinline__ Best block_best(Best x, Best* red) {
   return y;  // identical in every warp
 }
 
-__global__ void __launch_bounds__(kThreads) argmax_kernel(const __nv_bfloat16* __restrict__ logits, long long ld,
-                                                          int V, int* __restrict__ out) {
+template <typename A>
+__global__ void __launch_bounds__(kThreads) argmax_kernel(const A* __restrict__ logits, long long ld, int V, int* __restrict__ out) {
   __shared__ Best red[32];
   pdl_launch_next();
   pdl_wait_prior();
-  const __nv_bfloat16* row = logits + blockIdx.x * ld;
+  const A* row = logits + blockIdx.x * ld;
   Best b{-CUDART_INF_F, 0x7fffffff};
   const int nvec = V / 8;
   for (int c = threadIdx.x; c < nvec; c += kThreads) {
-    const uint4 r = *reinterpret_cast<const uint4*>(row + c * 8);
-    const __nv_bfloat16* e = reinterpret_cast<const __nv_bfloat16*>(&r);
+    float e[8];
+    load8(row + c * 8, e);
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
-      const float f = __bfloat162float(e[j]);
+      const float f = e[j];
       if (f > b.v) { b.v = f; b.i = c * 8 + j; }  // ascending index: strict > keeps the lowest id
     }
   }
   for (int i = nvec * 8 + threadIdx.x; i < V; i += kThreads) {
-    const float f = __bfloat162float(row[i]);
+    const float f = elem_to_f(row[i]);
     if (f > b.v || (f == b.v && i < b.i)) { b.v = f; b.i = i; }
   }
   b = block_best(b, red);
@@ -84,6 +85,7 @@ __device__ __forceinline__ uint4 philox(uint4 ctr, uint2 key) {
   return ctr;
 }
 
+template <typename A>
 __global__ void __launch_bounds__(kThreads) sample_kernel(const SampleParams p) {
   __shared__ Best red[32];
   __shared__ float top_v[kMaxTopK];
@@ -91,7 +93,7 @@ __global__ void __launch_bounds__(kThreads) sample_kernel(const SampleParams p) 
   pdl_launch_next();
   pdl_wait_prior();
   const int row_id = blockIdx.x;
-  const __nv_bfloat16* row = p.logits + row_id * p.ld;
+  const A* row = static_cast<const A*>(p.logits) + row_id * p.ld;
   const float temp = p.temperature ? p.temperature[row_id] : 1.f;
   const int top_k_req = p.top_k ? p.top_k[row_id] : kMaxTopK;
   const float top_p = p.top_p ? p.top_p[row_id] : 1.f;
@@ -107,7 +109,7 @@ __global__ void __launch_bounds__(kThreads) sample_kernel(const SampleParams p) 
   for (int k = 0; k < K; ++k) {
     Best b{-CUDART_INF_F, 0x7fffffff};
     for (int i = threadIdx.x; i < p.V; i += kThreads) {
-      float f = __bfloat162float(row[i]);
+      float f = elem_to_f(row[i]);
       if (counts != nullptr) {
         const int c = counts[i];
         if (c > 0) f -= pres + freq * static_cast<float>(c);
@@ -286,7 +288,7 @@ __global__ void accept_greedy_tree_kernel(const int* __restrict__ target_ids, co
 
 }  // namespace
 
-const char* argmax_rows(const void* logits, long long ld, int T, int V, int* out, cudaStream_t stream, bool pdl) {
+const char* argmax_rows(const void* logits, long long ld, int T, int V, int* out, bool f32, cudaStream_t stream, bool pdl) {
   if (T <= 0) return nullptr;
   if (ld % 8) return "argmax_rows: leading dimension must be a multiple of 8";
   cudaLaunchConfig_t cfg = {};
@@ -295,13 +297,15 @@ const char* argmax_rows(const void* logits, long long ld, int T, int V, int* out
   attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
   attr[0].val.programmaticStreamSerializationAllowed = 1;
   cfg.attrs = attr; cfg.numAttrs = pdl ? 1 : 0;
-  cudaError_t e = cudaLaunchKernelEx(&cfg, argmax_kernel, static_cast<const __nv_bfloat16*>(logits), ld, V, out);
+  cudaError_t e = f32 ? cudaLaunchKernelEx(&cfg, argmax_kernel<float>, static_cast<const float*>(logits), ld, V, out)
+                      : cudaLaunchKernelEx(&cfg, argmax_kernel<__nv_bfloat16>, static_cast<const __nv_bfloat16*>(logits), ld, V, out);
   return e == cudaSuccess ? nullptr : cudaGetErrorString(e);
 }
 
 const char* sample_rows(const SampleParams& p, cudaStream_t stream) {
   if (p.T <= 0) return nullptr;
-  sample_kernel<<<p.T, kThreads, 0, stream>>>(p);
+  if (p.logits_f32) sample_kernel<float><<<p.T, kThreads, 0, stream>>>(p);
+  else sample_kernel<__nv_bfloat16><<<p.T, kThreads, 0, stream>>>(p);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? nullptr : cudaGetErrorString(e);
 }

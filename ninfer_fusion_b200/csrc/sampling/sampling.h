@@ -8,10 +8,12 @@ namespace nfb {
 
 constexpr int kMaxTopK = 32;
 
-const char* argmax_rows(const void* logits, long long ld, int T, int V, int* out, cudaStream_t stream, bool pdl);
+// logits bf16, or fp32 with `f32`
+const char* argmax_rows(const void* logits, long long ld, int T, int V, int* out, bool f32, cudaStream_t stream, bool pdl);
 
 struct SampleParams {
-  const __nv_bfloat16* logits;  // [T, ld]
+  const void* logits;           // [T, ld] bf16, or fp32 with logits_f32
+  bool logits_f32;
   long long ld;
   int T, V;
   const float* temperature;     // per row; <= 0 means greedy.  Null = 1

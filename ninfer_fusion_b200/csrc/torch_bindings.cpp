@@ -1,9 +1,6 @@
 // torch.ops.nfb200.* : thin, checked adapters from torch tensors to the plain
 // C++ launchers.  No kernel code lives here.
-#include <ATen/cuda/CUDAContext.h>
-#include <c10/cuda/CUDAGuard.h>
-#include <torch/library.h>
-#include <ATen/ATen.h>
+#include "binding_util.h"
 
 #include "attention/attention.h"
 #include "comm/comm.h"
@@ -14,103 +11,7 @@
 
 namespace {
 
-using at::Tensor;
-using OptT = const std::optional<Tensor>&;
-
-inline cudaStream_t cur_stream() { return at::cuda::getCurrentCUDAStream().stream(); }
-
-inline void chk(const char* err) { TORCH_CHECK(err == nullptr, err ? err : ""); }
-
-inline void need_cuda(const Tensor& t, const char* name) {
-  TORCH_CHECK(t.is_cuda(), name, " must be a CUDA tensor");
-}
-inline void need(const Tensor& t, at::ScalarType dt, const char* name) {
-  need_cuda(t, name);
-  TORCH_CHECK(t.scalar_type() == dt, name, " has the wrong dtype");
-}
-inline void need_rows(const Tensor& t, const char* name) {
-  TORCH_CHECK(t.dim() == 2 && t.stride(1) == 1, name, " must be 2-D with unit inner stride");
-}
-template <typename T>
-inline T* ptr_or_null(OptT t) {
-  return t.has_value() && t->defined() ? static_cast<T*>(t->data_ptr()) : nullptr;
-}
-
-int64_t sm_count() {
-  static int n = 0;
-  if (n == 0) n = at::cuda::getCurrentDeviceProperties()->multiProcessorCount;
-  return n;
-}
-
-// Optional L2 prefetch hint: a (contiguous) tensor the next kernel will stream; at most the first 32 MB are asked for.
-void fill_prefetch(nfb::GemmArgs& a, OptT next) {
-  if (!(next.has_value() && next->defined() && next->is_cuda() && next->is_contiguous())) return;
-  a.prefetch = next->data_ptr();
-  const int64_t bytes = next->numel() * next->element_size();
-  a.prefetch_bytes = bytes < (32 << 20) ? bytes : (32 << 20);
-}
-
-// Optional decode conv epilogue (nfb::GemmConv): all four tensors or none.
-void fill_conv(nfb::GemmArgs& a, OptT conv_w, OptT conv_state, OptT conv_slot, OptT conv_out) {
-  if (!(conv_state.has_value() && conv_state->defined())) return;
-  TORCH_CHECK(conv_w.has_value() && conv_slot.has_value() && conv_out.has_value(), "conv epilogue: all four tensors");
-  need(*conv_w, at::kBFloat16, "conv_w"); need(*conv_state, at::kBFloat16, "conv_state");
-  need(*conv_slot, at::kInt, "conv_slot"); need(*conv_out, at::kBFloat16, "conv_out");
-  TORCH_CHECK(conv_w->dim() == 2 && conv_w->size(1) == 4 && conv_w->is_contiguous(), "conv_w must be [C, 4]");
-  const int64_t C = conv_w->size(0);
-  TORCH_CHECK(conv_state->dim() == 3 && conv_state->size(1) == 3 && conv_state->size(2) == C && conv_state->is_contiguous(),
-              "conv_state must be [slots, 3, C]");
-  TORCH_CHECK(conv_out->dim() == 2 && conv_out->size(0) == a.T && conv_out->size(1) == C && conv_out->is_contiguous(),
-              "conv_out must be [T, C]");
-  TORCH_CHECK(conv_slot->numel() >= a.T && conv_slot->is_contiguous(), "conv_slot must hold one slot per token");
-  a.conv.w = conv_w->data_ptr(); a.conv.state = conv_state->data_ptr();
-  a.conv.slot = static_cast<const int*>(conv_slot->data_ptr()); a.conv.out = conv_out->data_ptr();
-  a.conv.C = static_cast<int>(C);
-}
-
-// out = epilogue(x @ w^T).  epi: 0 store(+bias), 1 residual add, 2 swiglu, 3 split-K partials.
-void gemm_bf16(const Tensor& x, const Tensor& w, OptT out, int64_t epi, OptT resid, OptT bias, OptT partial,
-               int64_t splits, OptT status, bool pdl, int64_t act, OptT conv_w, OptT conv_state, OptT conv_slot,
-               OptT conv_out, OptT prefetch) {
-  need(x, at::kBFloat16, "x"); need(w, at::kBFloat16, "w");
-  need_rows(x, "x"); need_rows(w, "w");
-  TORCH_CHECK(x.size(1) == w.size(1), "gemm_bf16: K mismatch");
-  TORCH_CHECK(act >= 0 && act <= 2 && (act == 0 || epi == nfb::kEpiStore), "gemm_bf16: activation needs the store epilogue");
-  c10::cuda::CUDAGuard guard(x.device());
-  nfb::GemmArgs a;
-  a.w = w.data_ptr(); a.N = w.size(0); a.K = w.size(1); a.ldw = w.stride(0);
-  a.x = x.data_ptr(); a.T = x.size(0); a.ldx = x.stride(0);
-  const int64_t out_cols = epi == nfb::kEpiSwiglu ? a.N / 2 : a.N;
-  if (epi != nfb::kEpiPartial) {
-    TORCH_CHECK(out.has_value(), "gemm_bf16: out required");
-    need(*out, at::kBFloat16, "out"); need_rows(*out, "out");
-    TORCH_CHECK(out->size(0) == a.T && out->size(1) == out_cols, "gemm_bf16: out shape");
-    a.out = out->data_ptr(); a.ldo = out->stride(0);
-  }
-  if (epi == nfb::kEpiResidual) {
-    TORCH_CHECK(resid.has_value(), "gemm_bf16: resid required");
-    need(*resid, at::kBFloat16, "resid"); need_rows(*resid, "resid");
-    TORCH_CHECK(resid->size(0) == a.T && resid->size(1) == a.N, "gemm_bf16: resid shape");
-    a.resid = resid->data_ptr(); a.ldr = resid->stride(0);
-  }
-  if (bias.has_value() && bias->defined()) {
-    need(*bias, at::kFloat, "bias");
-    TORCH_CHECK(bias->numel() == a.N && bias->is_contiguous(), "gemm_bf16: bias shape");
-    a.bias = static_cast<const float*>(bias->data_ptr());
-  }
-  if (epi == nfb::kEpiPartial) {
-    TORCH_CHECK(partial.has_value(), "gemm_bf16: partial workspace required");
-    need(*partial, at::kFloat, "partial");
-    TORCH_CHECK(partial->is_contiguous() && partial->numel() >= splits * a.T * a.N, "gemm_bf16: workspace too small");
-    a.partial = static_cast<float*>(partial->data_ptr());
-  }
-  a.splits = static_cast<int>(splits); a.epi = static_cast<int>(epi); a.act = static_cast<int>(act);
-  a.status = ptr_or_null<int>(status);
-  a.stream = cur_stream(); a.pdl = pdl;
-  fill_conv(a, conv_w, conv_state, conv_slot, conv_out);
-  fill_prefetch(a, prefetch);
-  chk(nfb::gemm_bf16(a));
-}
+using namespace nfb_bind;
 
 Tensor gemm_trace(bool enable, int64_t n_ctas) {
   nfb::gemm_trace_enable(enable);
@@ -130,11 +31,6 @@ std::tuple<int64_t, Tensor> gemm_timeline(int64_t mode) {
   const int used = nfb::gemm_timeline_end(reinterpret_cast<unsigned long long*>(out.data_ptr()), &slots, &ctas);
   TORCH_CHECK(slots == 64 && ctas == 256, "timeline geometry changed");
   return {used, out};
-}
-
-int64_t gemm_pick_splits(int64_t T, int64_t N, int64_t K, int64_t epi) {
-  return nfb::gemm_pick_splits(static_cast<int>(T), static_cast<int>(N), static_cast<int>(K), static_cast<int>(epi),
-                               static_cast<int>(sm_count()));
 }
 
 void add_rmsnorm(OptT partial, int64_t splits, OptT delta, OptT resid_in, OptT resid_out, OptT norm_w, OptT normed,
@@ -550,62 +446,6 @@ int64_t gdn_chunked_workspace_bytes(int64_t T, int64_t n_seq, int64_t n_v_heads)
       nfb::gdn_chunked_max_chunks(static_cast<int>(T), static_cast<int>(n_seq)), static_cast<int>(n_v_heads)));
 }
 
-void argmax_rows(const Tensor& logits, const Tensor& out, bool pdl) {
-  need(logits, at::kBFloat16, "logits"); need_rows(logits, "logits"); need(out, at::kInt, "out");
-  TORCH_CHECK(out.numel() == logits.size(0));
-  c10::cuda::CUDAGuard guard(logits.device());
-  chk(nfb::argmax_rows(logits.data_ptr(), logits.stride(0), static_cast<int>(logits.size(0)),
-                       static_cast<int>(logits.size(1)), static_cast<int*>(out.data_ptr()), cur_stream(), pdl));
-}
-
-void sample_rows(const Tensor& logits, OptT temperature, OptT top_k, OptT top_p, OptT min_p, OptT presence,
-                 OptT frequency, OptT token_counts, OptT seeds, OptT positions, int64_t purpose, const Tensor& out,
-                 OptT out_prob, OptT draft_ids, OptT accepted, OptT draft_dist_ids, OptT draft_dist_probs,
-                 OptT out_dist_ids, OptT out_dist_probs) {
-  need(logits, at::kBFloat16, "logits"); need_rows(logits, "logits"); need(out, at::kInt, "out");
-  c10::cuda::CUDAGuard guard(logits.device());
-  nfb::SampleParams p = {};
-  p.logits = static_cast<const __nv_bfloat16*>(logits.data_ptr()); p.ld = logits.stride(0);
-  p.T = static_cast<int>(logits.size(0)); p.V = static_cast<int>(logits.size(1));
-  p.temperature = ptr_or_null<const float>(temperature); p.top_k = ptr_or_null<const int>(top_k);
-  p.top_p = ptr_or_null<const float>(top_p); p.min_p = ptr_or_null<const float>(min_p);
-  p.presence = ptr_or_null<const float>(presence); p.frequency = ptr_or_null<const float>(frequency);
-  p.token_counts = ptr_or_null<const int>(token_counts);
-  p.seeds = ptr_or_null<const unsigned long long>(seeds); p.positions = ptr_or_null<const int>(positions);
-  p.purpose = static_cast<unsigned int>(purpose);
-  p.out = static_cast<int*>(out.data_ptr()); p.out_prob = ptr_or_null<float>(out_prob);
-  if (draft_ids.has_value() && draft_ids->defined()) {
-    need(*draft_ids, at::kInt, "draft_ids");
-    TORCH_CHECK(draft_ids->numel() >= p.T, "draft_ids: one entry per row");
-    p.draft_ids = static_cast<const int*>(draft_ids->data_ptr());
-  }
-  if (accepted.has_value() && accepted->defined()) {
-    need(*accepted, at::kInt, "accepted");
-    TORCH_CHECK(accepted->numel() >= p.T, "accepted: one entry per row");
-    p.accepted = static_cast<int*>(accepted->data_ptr());
-  }
-  if (draft_dist_ids.has_value() && draft_dist_ids->defined()) {
-    TORCH_CHECK(draft_dist_probs.has_value() && draft_dist_probs->defined() && p.draft_ids != nullptr,
-                "draft distribution needs ids, probabilities and draft_ids");
-    need(*draft_dist_ids, at::kInt, "draft_dist_ids"); need(*draft_dist_probs, at::kFloat, "draft_dist_probs");
-    TORCH_CHECK(draft_dist_ids->is_contiguous() && draft_dist_probs->is_contiguous() && draft_dist_ids->dim() == 2 &&
-                draft_dist_ids->size(0) >= p.T && draft_dist_probs->sizes() == draft_dist_ids->sizes(), "draft distribution shapes");
-    p.draft_dist_ids = static_cast<const int*>(draft_dist_ids->data_ptr());
-    p.draft_dist_probs = static_cast<const float*>(draft_dist_probs->data_ptr());
-    p.dist_k = static_cast<int>(draft_dist_ids->size(1));
-  }
-  if (out_dist_ids.has_value() && out_dist_ids->defined()) {
-    TORCH_CHECK(out_dist_probs.has_value() && out_dist_probs->defined(), "out_dist needs ids and probabilities");
-    need(*out_dist_ids, at::kInt, "out_dist_ids"); need(*out_dist_probs, at::kFloat, "out_dist_probs");
-    TORCH_CHECK(out_dist_ids->is_contiguous() && out_dist_probs->is_contiguous() && out_dist_ids->dim() == 2 &&
-                out_dist_ids->size(0) >= p.T && out_dist_probs->sizes() == out_dist_ids->sizes(), "out distribution shapes");
-    p.out_dist_ids = static_cast<int*>(out_dist_ids->data_ptr());
-    p.out_dist_probs = static_cast<float*>(out_dist_probs->data_ptr());
-    p.dist_out_k = static_cast<int>(out_dist_ids->size(1));
-  }
-  chk(nfb::sample_rows(p, cur_stream()));
-}
-
 void accept_greedy_chain(const Tensor& target_ids, const Tensor& draft_ids, const Tensor& n_accepted,
                          const Tensor& out_tokens) {
   need(target_ids, at::kInt, "target_ids"); need(draft_ids, at::kInt, "draft_ids");
@@ -902,11 +742,9 @@ TORCH_LIBRARY(nfb200, m) {
   m.def("tp_gather_norm(Tensor x, Tensor norm_w, Tensor normed, int my_base, int xflag_off, float eps, bool unit_offset, Tensor state, Tensor? status, bool pdl) -> ()", &tp_gather_norm);
   m.def("gemm_bf16_push_all(Tensor x, Tensor w, int splits, int world, int rank, int[] peer_bases, int recv_off, int flag_off, int T_cap, Tensor state, Tensor? status, bool pdl) -> ()", &gemm_bf16_push_all);
   m.def("tp_sum_norm(int world, int T_cap, int arrivals, int my_base, int recv_off, int flag_off, Tensor x, Tensor? norm_w, Tensor? normed, float eps, bool unit_offset, Tensor state, Tensor? status, bool pdl) -> ()", &tp_sum_norm);
-  m.def("gemm_bf16(Tensor x, Tensor w, Tensor? out, int epi, Tensor? resid, Tensor? bias, Tensor? partial, int splits, Tensor? status, bool pdl, int act=0, Tensor? conv_w=None, Tensor? conv_state=None, Tensor? conv_slot=None, Tensor? conv_out=None, Tensor? prefetch=None) -> ()", &gemm_bf16);
   m.def("gemm_trace(bool enable, int n_ctas) -> Tensor", &gemm_trace);
   m.def("gemm_timeline(int mode) -> (int, Tensor)", &gemm_timeline);
   m.def("attn_tc_trace(bool enable) -> Tensor", &attn_tc_trace);
-  m.def("gemm_pick_splits(int T, int N, int K, int epi) -> int", &gemm_pick_splits);
   m.def("add_rmsnorm(Tensor? partial, int splits, Tensor? delta, Tensor? resid_in, Tensor? resid_out, Tensor? norm_w, Tensor? normed, int T, int N, float eps, bool unit_offset, bool pdl, Tensor? q_codes=None, Tensor? q_sf=None) -> ()", &add_rmsnorm);
   m.def("embed_gather(Tensor ids, Tensor table, Tensor out, bool pdl) -> ()", &embed_gather);
   m.def("attn_prep(Tensor proj, int q_off, int k_off, int v_off, int n_q_heads, int n_kv_heads, int head_dim, Tensor? q_norm_w, Tensor? k_norm_w, float eps, bool unit_offset, int rot_dim, Tensor inv_freq, float attn_factor, Tensor rope_pos, Tensor token_seq, Tensor cache_pos, Tensor block_table, Tensor q_out, Tensor k_codes, Tensor v_codes, Tensor? k_scales, Tensor? v_scales, int page_size, int format, int group, bool pdl, bool k_hadamard=False, Tensor? k_row_scale=None, Tensor? tiers=None) -> ()", &attn_prep);
@@ -919,8 +757,6 @@ TORCH_LIBRARY(nfb200, m) {
   m.def("gdn_chunked_workspace_bytes(int T, int n_seq, int n_v_heads) -> int", &gdn_chunked_workspace_bytes);
   m.def("gdn_prefill_trace(bool enable) -> Tensor", &gdn_prefill_trace);
   m.def("kv_move_rows(Tensor block_table, Tensor table_row, Tensor src_pos, Tensor dst_pos, Tensor k_codes, Tensor v_codes, Tensor? k_scales, Tensor? v_scales, int page_size, int n_kv_heads, int head_dim, int format, int group) -> ()", &kv_move_rows);
-  m.def("argmax_rows(Tensor logits, Tensor out, bool pdl) -> ()", &argmax_rows);
-  m.def("sample_rows(Tensor logits, Tensor? temperature, Tensor? top_k, Tensor? top_p, Tensor? min_p, Tensor? presence, Tensor? frequency, Tensor? token_counts, Tensor? seeds, Tensor? positions, int purpose, Tensor out, Tensor? out_prob, Tensor? draft_ids=None, Tensor? accepted=None, Tensor? draft_dist_ids=None, Tensor? draft_dist_probs=None, Tensor? out_dist_ids=None, Tensor? out_dist_probs=None) -> ()", &sample_rows);
   m.def("accept_greedy_chain(Tensor target_ids, Tensor draft_ids, Tensor n_accepted, Tensor out_tokens) -> ()", &accept_greedy_chain);
   m.def("accept_greedy_tree(Tensor target_ids, Tensor node_tok, Tensor parent, int max_depth, Tensor n_accepted, Tensor out_tokens, Tensor out_nodes) -> ()", &accept_greedy_tree);
 }

@@ -153,4 +153,4 @@ def get_config(name: str) -> ModelConfig:
     try:
         return REGISTRY[name]
     except KeyError:
-        raise KeyError(f"unknown model '{name}'; registered: {sorted(REGISTRY)}") from None
+        raise KeyError(f"unknown model '{name}'; registered: {sorted(REGISTRY)} (layer-list designs: models/architectures.py)") from None

@@ -44,6 +44,7 @@ class StepBatch:
     n_tokens: int
     n_seqs: int
     one_token_per_seq: bool = False
+    max_seq_tokens: int = 1    # longest portion of the step (host copy, picks prefill or token-by-token kernels)
     qblk_start: Optional[torch.Tensor] = None   # [NB] first token of each attention query block
     qblk_count: Optional[torch.Tensor] = None   # [NB] tokens per query block
     # draft-tree verification (all optional): per token, the parent's token index (-1 = root of its window), whether
@@ -165,7 +166,7 @@ def pick_attention_split(max_kv_len: int, n_work: int, sm_count: int = 148, max_
 class LaunchCounter:
     """Proxy over torch.ops.nfb200 that counts the CUDA kernels each call launches."""
 
-    KERNELS = {"paged_attention": 2}
+    KERNELS = {"paged_attention": 2, "head_mix_prefill": 2}
 
     def __init__(self, ops):
         self._ops = ops
@@ -177,11 +178,16 @@ class LaunchCounter:
         fn = self._cache.get(name)
         if fn is None:
             raw = getattr(self._ops, name)
-            if name in ("gemm_pick_splits", "prefill_attn_block_tokens", "packed_attention_tile"):
+            if name in ("gemm_pick_splits", "prefill_attn_block_tokens", "packed_attention_tile", "head_mix_prefill_scratch",
+                        "head_mix_block_tokens"):
                 fn = raw
             elif name == "causal_conv1d_silu":
                 def fn(*a, _raw=raw):
                     self.count += 2 if (a[9] and not a[10]) else 1  # + history roll unless the decode fast path
+                    return _raw(*a)
+            elif name == "head_mix_attention":
+                def fn(*a, _raw=raw):
+                    self.count += 2 if a[15] > 1 else 1  # + merge of the key splits
                     return _raw(*a)
             else:
                 k = self.KERNELS.get(name, 1)
@@ -684,6 +690,12 @@ class HybridModel:
         self._materialize_normed(ws)
         return ws.normed[:T] if end_layer == cfg.n_layers else x
 
+    def head(self, ws: Workspace, head_in: torch.Tensor) -> torch.Tensor:
+        """Logits of final-normed hidden states (at most the workspace's logit rows)."""
+        out = ws.logits[: head_in.shape[0]]
+        self._gemm(head_in, self.w[f"{self.prefix}/lm_head"], out)
+        return out
+
     def logits(self, ws: Workspace, b: StepBatch, hidden: torch.Tensor) -> torch.Tensor:
         R = b.logit_rows.numel()
         head_in = ws.head_in[:R]
@@ -691,9 +703,7 @@ class HybridModel:
             head_in = hidden  # decode: every row is a logit row, in order
         else:
             torch.index_select(hidden, 0, b.logit_rows.long(), out=head_in)
-        out = ws.logits[:R]
-        self._gemm(head_in, self.w[f"{self.prefix}/lm_head"], out)
-        return out
+        return self.head(ws, head_in)
 
     def forward_greedy(self, ws: Workspace, b: StepBatch, kv: PagedKvCache, st: GdnStatePool) -> torch.Tensor:
         """One step ending in arg-max token ids for `b.logit_rows` (int32 [R], ws.next_ids)."""

@@ -12,11 +12,13 @@ src/targets/declared_capabilities.h, src/targets/{spark_x2_5_4b,muse_glimmer_30b
 from __future__ import annotations
 
 from dataclasses import dataclass, field
-from typing import Dict, FrozenSet, Optional, Tuple
+from typing import Dict, FrozenSet, Optional, Tuple, Union
 
+from .architectures import LAYERED_REGISTRY
 from .config import REGISTRY, ModelConfig
+from .layered_config import LayeredConfig
 
-FULL, SLIDING, GDN = "full", "sliding", "gdn"
+FULL, SLIDING, GDN, MLSTM = "full", "sliding", "gdn", "mlstm"
 
 # what the engine's forward pass, kernels and cache can do today
 ENGINE_CAPABILITIES: FrozenSet[str] = frozenset({
@@ -28,12 +30,14 @@ ENGINE_CAPABILITIES: FrozenSet[str] = frozenset({
     "head-dim-256", "head-dim-128",
     "kv:bf16", "kv:fp8", "kv:int8", "kv:nvfp4",
     "vision-tower",
+    # layer-list decoders (models/layered.py)
+    "layer-list-schedule", "head-mixing-attention", "attention-sink", "matrix-memory", "post-sum-norm", "xielu-mlp",
 })
 
 
 @dataclass(frozen=True)
 class LayerKind:
-    kind: str                     # FULL | SLIDING | GDN
+    kind: str                     # FULL | SLIDING | GDN | MLSTM
     rotary_dim: int = 0           # 0 = no positional rotation on this layer (NoPE)
     rope_theta: float = 0.0
     window: int = 0               # sliding layers
@@ -54,7 +58,7 @@ class Package:
     activation: str = "swiglu"
     final_logit_softcap: float = 0.0
     tie_word_embeddings: bool = False
-    config: Optional[ModelConfig] = None      # set for packages the hybrid runtime serves
+    config: Optional[Union[ModelConfig, LayeredConfig]] = None      # set for packages a runtime serves on the GPU
     notes: str = ""
     qk_scale: float = 1.0                     # learned-constant factor on q . k (on top of 1 / sqrt(head_dim))
     output_multiplier: float = 1.0            # factor on the logits before soft-capping
@@ -79,6 +83,24 @@ def _hybrid(cfg: ModelConfig) -> Package:
         needs.add("mtp-draft")
     inter = cfg.ffn_inter if cfg.moe is None else cfg.moe.expert_inter
     return Package(cfg.name, cfg.hidden, cfg.n_layers, inter, cfg.vocab, kinds, frozenset(needs), config=cfg)
+
+
+def _layered(cfg: LayeredConfig) -> Package:
+    kinds, needs = [], {"layer-list-schedule", "post-sum-norm"}
+    for l in cfg.layers:
+        m = l.mixer
+        if m.kind == "attention":
+            kinds.append(LayerKind(SLIDING if m.window else FULL, 0, 0.0, m.window, m.heads, m.kv_heads, m.dim))
+            needs |= {c for c, on in (("sliding-window-attention", m.window), ("head-mixing-attention", m.head_mixing),
+                                      ("attention-sink", m.sink), ("qk-norm", m.qk_norm)) if on}
+        else:
+            kinds.append(LayerKind(MLSTM, q_heads=m.heads, kv_heads=m.heads, head_dim=m.dim))
+            needs.add("matrix-memory")
+        if l.mlp is not None:
+            needs.add(f"{l.mlp.activation}-mlp")
+    inter = max((l.mlp.ff for l in cfg.layers if l.mlp is not None), default=0)
+    return Package(cfg.name, cfg.hidden, cfg.n_layers, inter, cfg.vocab, tuple(kinds), frozenset(needs), activation="xielu",
+                   config=cfg, notes=f"layer-list decoder ({cfg.architecture})")
 
 
 def _spark() -> Package:
@@ -119,6 +141,7 @@ def _gemma() -> Package:
 
 def _table() -> Dict[str, Package]:
     out = {name: _hybrid(cfg) for name, cfg in REGISTRY.items()}
+    out.update({name: _layered(cfg) for name, cfg in LAYERED_REGISTRY.items()})
     for p in (_spark(), _muse(), _gemma()):
         out[p.model_id] = p
     return out
@@ -141,7 +164,7 @@ def construct(model_id: str, have: FrozenSet[str] = ENGINE_CAPABILITIES) -> Mode
         raise PackageRefused(f"{model_id}: the engine lacks {', '.join(miss)}")
     if p.config is None:
         raise PackageRefused(f"{model_id}: registered as a geometry description only")
-    if sum(p.count(k) for k in (FULL, SLIDING, GDN)) != p.n_layers:
+    if sum(p.count(k) for k in (FULL, SLIDING, GDN, MLSTM)) != p.n_layers:
         raise PackageRefused(f"{model_id}: the layer table does not cover all {p.n_layers} layers")
     return p.config
 
@@ -151,7 +174,7 @@ def construct_oracle(model_id: str, layers: int = 0, vocab: int = 0, hidden_div:
     the GPU gate says about them.  `model_id@N` or `layers` takes the first N layers of the schedule."""
     base, _, n = model_id.partition("@")
     p = lookup(base)
-    if p.count(GDN):
+    if p.count(GDN) or p.count(MLSTM):
         raise PackageRefused(f"{base}: a GDN hybrid is served by the hybrid runtime, not by the attention-only oracle")
     n_layers = int(n) if n else int(layers)
     if n_layers or vocab or hidden_div > 1:
@@ -163,7 +186,7 @@ def construct_oracle(model_id: str, layers: int = 0, vocab: int = 0, hidden_div:
 def describe(model_id: str) -> dict:
     p = lookup(model_id)
     return {"model_id": p.model_id, "hidden": p.hidden, "layers": p.n_layers, "full": p.count(FULL),
-            "sliding": p.count(SLIDING), "gdn": p.count(GDN), "intermediate": p.intermediate, "vocab": p.vocab,
+            "sliding": p.count(SLIDING), "gdn": p.count(GDN), "mlstm": p.count(MLSTM), "intermediate": p.intermediate, "vocab": p.vocab,
             "activation": p.activation, "final_logit_softcap": p.final_logit_softcap,
             "needs": sorted(p.needs), "missing": list(p.missing()), "servable": not p.missing() and p.config is not None,
-            "oracle_runtime": p.count(GDN) == 0 or p.config is not None, "notes": p.notes}
+            "oracle_runtime": (p.count(GDN) == 0 and p.count(MLSTM) == 0) or isinstance(p.config, ModelConfig), "notes": p.notes}

@@ -16,7 +16,8 @@ import torch
 E2M1_GRID = torch.tensor([0.0, 0.5, 1.0, 1.5, 2.0, 3.0, 4.0, 6.0])
 
 KV_BF16, KV_FP8_ROW, KV_INT8_GROUP, KV_NVFP4 = 0, 1, 2, 3
-KV_FORMAT_NAMES = {"bf16": KV_BF16, "fp8": KV_FP8_ROW, "int8": KV_INT8_GROUP, "nvfp4": KV_NVFP4}
+KV_FP32 = 5   # (4 = mixed tiers, runtime/kv_cache.py) rows of models that run in 32-bit
+KV_FORMAT_NAMES = {"bf16": KV_BF16, "fp8": KV_FP8_ROW, "int8": KV_INT8_GROUP, "nvfp4": KV_NVFP4, "fp32": KV_FP32}
 
 
 def bf16_round(x: torch.Tensor) -> torch.Tensor:

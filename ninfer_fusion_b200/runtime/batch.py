@@ -9,7 +9,7 @@ pinned "ingress" struct (src/targets/qwen3_6/impl/runtime/program_impl.h:18436-1
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import List, Sequence
+from typing import List, Optional, Sequence
 
 import numpy as np
 import torch
@@ -26,6 +26,7 @@ class SeqChunk:
     tokens: Sequence[int]
     want_logits: bool = True   # logits for the chunk's last token
     all_logits: bool = False   # logits for every token of the chunk (speculative verify)
+    want: Optional[Sequence[int]] = None   # logits for these places of the chunk (overrides the two flags above)
     positions: object = None   # optional int [n, 3] rope positions (multimodal prefill); default = cache positions
 
 
@@ -73,7 +74,8 @@ class StepBuffers:
         cpos, kvl = self._hview("cache_pos", T), self._hview("kv_len", T)
         rpos = self._hview("rope_pos", T * self.pos_axes)
         cu, slot = self._hview("cu_seqlens", B + 1), self._hview("state_slot", B)
-        lrows = self._hview("logit_rows", sum(len(c.tokens) if c.all_logits else 1 for c in chunks))
+        lrows = self._hview("logit_rows", sum(len(c.want) if c.want is not None else len(c.tokens) if c.all_logits else 1
+                                              for c in chunks))
         t = 0
         n_logit = 0
         qt = self.attn_block_tokens
@@ -104,7 +106,10 @@ class StepBuffers:
                 blk_c.append(min(qt, n - o))
             t += n
             cu[b + 1] = t
-            if c.all_logits:
+            if c.want is not None:
+                lrows[n_logit:n_logit + len(c.want)] = [t - n + j for j in c.want]
+                n_logit += len(c.want)
+            elif c.all_logits:
                 lrows[n_logit:n_logit + n] = range(t - n, t)
                 n_logit += n
             elif c.want_logits:
@@ -125,4 +130,5 @@ class StepBuffers:
                          state_slot=self._dview("state_slot", B), logit_rows=self._dview("logit_rows", n_logit),
                          max_kv_len=max_kv, n_tokens=T, n_seqs=B,
                          one_token_per_seq=all(len(c.tokens) == 1 for c in chunks),
+                         max_seq_tokens=max((len(c.tokens) for c in chunks), default=1),
                          qblk_start=self._dview("qblk_start", nb), qblk_count=self._dview("qblk_count", nb))

@@ -53,6 +53,9 @@ def kv_page_bytes(cfg: ModelConfig, formats: Union[str, Sequence[str]], page_siz
     """Bytes one physical page takes over all attention layers (K and V codes + their scales), from the same row
     geometry the cache allocates with."""
     from .kv_cache import KV_FORMAT_NAMES, kv_row_bytes, kv_scale_bytes
+    if hasattr(cfg, "kv_geometry"):      # one geometry per layer, uncoded rows
+        elem = 4 if formats == "fp32" else 2
+        return sum(h * page_size * (kw + vw) * elem for h, kw, vw in cfg.kv_geometry)
     names = [formats] * len(cfg.attn_layers) if isinstance(formats, str) else list(formats)
     if len(names) != len(cfg.attn_layers):
         raise CapacityError(f"{len(names)} KV formats for {len(cfg.attn_layers)} attention layers")
@@ -71,9 +74,12 @@ def build_curve(cfg: ModelConfig, formats, page_size: int, max_context: int, max
     m_min, m_max = page_range(max_context, max_concurrency, page_size)
     step = kv_page_bytes(cfg, formats, page_size, n_kv_heads)
     slots = max_concurrency + (max_concurrency if checkpoint_slots is None else checkpoint_slots)
-    hv = cfg.gdn_v_heads if gdn_v_heads is None else gdn_v_heads
-    d = cfg.gdn_head_dim
-    state = len(cfg.gdn_layers) * slots * (hv * d * d * 4 + 3 * cfg.gdn_conv_dim * 2)      # fp32 state + bf16 conv taps
+    if hasattr(cfg, "state_bytes_per_slot"):
+        state = slots * cfg.state_bytes_per_slot()
+    else:
+        hv = cfg.gdn_v_heads if gdn_v_heads is None else gdn_v_heads
+        d = cfg.gdn_head_dim
+        state = len(cfg.gdn_layers) * slots * (hv * d * d * 4 + 3 * cfg.gdn_conv_dim * 2)  # fp32 state + bf16 conv taps
     L = -(-max_context // page_size)
     tables = max_concurrency * L * 4
     fixed = state + tables + workspace_bytes + graph_allowance_bytes

@@ -15,9 +15,8 @@ import numpy as np
 import torch
 
 from ..models.config import ModelConfig
-from ..models.hybrid import HybridModel, ShardGeometry, StepBatch, Workspace, pick_attention_split
+from ..models.hybrid import ShardGeometry, StepBatch
 from .batch import SeqChunk, StepBuffers
-from .kv_cache import GdnStatePool, PagedKvCache
 
 
 def context_bucket(n: int) -> int:
@@ -46,17 +45,15 @@ class Generator:
         self.page_size = page_size
         self.prefill_chunk = prefill_chunk
         self.use_graph = use_graph and self.device.type == "cuda"
-        self.model = HybridModel(cfg, weights, device, pdl=pdl, shard=shard)
-        self.model.comm = comm
-        g = self.model.g
+        from .family import build_runtime
         pages_per_row = (max_context + page_size - 1) // page_size
-        self.kv = PagedKvCache(cfg, max_batch * pages_per_row, page_size, max_batch, pages_per_row, device,
-                               formats=kv_format, int8_group=int8_group, n_kv_heads=g.n_kv_heads)
-        self.states = GdnStatePool(cfg, max_batch, device, n_qk_heads=g.gdn_qk_heads, n_v_heads=g.gdn_v_heads)
         cap = max(prefill_chunk, max_batch)
-        self.ws = Workspace(cfg, cap, max(max_batch, max_logit_rows), device, shard=shard,
-                            x_buffer=None if comm is None else comm.x)
-        qt = int(self.model.ops.prefill_attn_block_tokens(g.n_q_heads, g.n_kv_heads)) if self.device.type == "cuda" else 16
+        rt = build_runtime(cfg, weights, device, rows=max_batch, pages_per_row=pages_per_row,
+                           n_pages=max_batch * pages_per_row, page_size=page_size, state_slots=max_batch, step_tokens=cap,
+                           logit_rows=max(max_batch, max_logit_rows), kv_format=kv_format, pdl=pdl, int8_group=int8_group,
+                           shard=shard, comm=comm)
+        self.model, self.kv, self.states, self.ws = rt.model, rt.kv, rt.states, rt.ws
+        qt = rt.block_tokens
         self.bufs_prefill = StepBuffers(cap, max_batch, device, attn_block_tokens=qt)
         self.bufs_decode = StepBuffers(max_batch, max_batch, device, attn_block_tokens=qt)
         pin = self.device.type == "cuda"
@@ -211,13 +208,11 @@ class Generator:
 
     def _snapshot_states(self) -> None:
         """Warm-up / capture runs must not advance the recurrent state."""
-        self._saved = [(c.clone(), s.clone()) for c, s in zip(self.states.conv, self.states.ssm)]
+        self._saved = self.states.save()
 
     def _rollback_states(self) -> None:
         torch.cuda.synchronize(self.device)
-        for (c0, s0), c, s in zip(self._saved, self.states.conv, self.states.ssm):
-            c.copy_(c0)
-            s.copy_(s0)
+        self.states.load(self._saved)
         self._saved = None
 
     def decode_step(self) -> List[int]:

@@ -15,10 +15,10 @@ import torch
 from ..utils import trace
 
 from ..models.config import ModelConfig
-from ..models.hybrid import HybridModel, ShardGeometry, StepBatch, Workspace
+from ..models.hybrid import ShardGeometry, StepBatch
 from .batch import SeqChunk, StepBuffers
+from .family import build_runtime
 from .generator import context_bucket
-from .kv_cache import GdnStatePool, PagedKvCache
 from .program import Lane, ProgramBase, SamplingParams
 
 
@@ -44,24 +44,20 @@ class GpuProgram(ProgramBase):
         self.device = torch.device(device)
         self.prefill_chunk = prefill_chunk
         self.use_graph = use_graph
-        self.model = HybridModel(cfg, weights, device, pdl=pdl, shard=shard)
-        self.model.comm = comm
-        g = self.model.g
         pages_per_row = (max_context + page_size - 1) // page_size
         n_pages = kv_pages if kv_pages is not None else max_lanes * pages_per_row
-        self.kv = PagedKvCache(cfg, n_pages, page_size, max_lanes, pages_per_row, device, formats=kv_format,
-                               int8_group=int8_group, n_kv_heads=g.n_kv_heads, mixed_capacity=mixed_capacity,
-                               mixed_hot_tier=mixed_hot_tier)
+        cap = max(prefill_chunk, max_lanes)
+        rt = build_runtime(cfg, weights, device, rows=max_lanes, pages_per_row=pages_per_row, n_pages=n_pages,
+                           page_size=page_size, state_slots=max_lanes + self.checkpoint_slots, step_tokens=cap,
+                           logit_rows=max_lanes, kv_format=kv_format, pdl=pdl, int8_group=int8_group, shard=shard, comm=comm,
+                           mixed_capacity=mixed_capacity, mixed_hot_tier=mixed_hot_tier)
+        self.model, self.kv, self.states, self.ws = rt.model, rt.kv, rt.states, rt.ws
+        self._lookahead = rt.page_lookahead
         self.descent = descent
         self.descent_stats = {"passes": 0, "cells_moved": 0}
-        self.states = GdnStatePool(cfg, max_lanes + self.checkpoint_slots, device, n_qk_heads=g.gdn_qk_heads,
-                                   n_v_heads=g.gdn_v_heads)
         self._ckpt_slots_free = self.checkpoint_slots
-        cap = max(prefill_chunk, max_lanes)
-        self.ws = Workspace(cfg, cap, max_lanes, device, shard=shard, x_buffer=None if comm is None else comm.x)
-        qt = int(self.model.ops.prefill_attn_block_tokens(g.n_q_heads, g.n_kv_heads))
-        self.bufs_prefill = StepBuffers(cap, max_lanes, device, attn_block_tokens=qt)
-        self.bufs_decode = StepBuffers(max_lanes, max_lanes, device, attn_block_tokens=qt)
+        self.bufs_prefill = StepBuffers(cap, max_lanes, device, attn_block_tokens=rt.block_tokens, max_logit_rows=cap)
+        self.bufs_decode = StepBuffers(max_lanes, max_lanes, device, attn_block_tokens=rt.block_tokens)
         self.out_host = torch.zeros(max_lanes, dtype=torch.int32, pin_memory=True)
         # per-row sampling parameters (pinned host + device twins), filled every sampled round
         B = max_lanes
@@ -73,7 +69,7 @@ class GpuProgram(ProgramBase):
                         "positions": torch.zeros(B, dtype=torch.int32, pin_memory=True)}
         self.sp_dev = {k: v.to(self.device) for k, v in self.sp_host.items()}
         self.penalties = penalties
-        self.token_counts = (torch.zeros((B, g.vocab_rows), dtype=torch.int32, device=self.device)
+        self.token_counts = (torch.zeros((B, rt.vocab_rows), dtype=torch.int32, device=self.device)
                              if penalties and comm is None else None)
         self._graphs: Dict[tuple, torch.cuda.CUDAGraph] = {}
         self.vision = None
@@ -115,7 +111,11 @@ class GpuProgram(ProgramBase):
     def _demote(self, handle):
         """Device frontier -> pinned host copy (KV pages of every layer + the state image)."""
         pages, slot = handle
-        return {"n_pages": len(pages), "tensors": [self.kv.export_pages(pages), self.states.export_slot(slot)]}
+        live = [p for p in pages if p >= 0]
+        cold = {"n_pages": len(live), "tensors": [self.kv.export_pages(live), self.states.export_slot(slot)]}
+        if len(live) != len(pages):          # a windowed cache: pages it had already given back stay holes
+            cold["holes"] = [i for i, p in enumerate(pages) if p < 0]
+        return cold
 
     def _promote(self, cold):
         if self._ckpt_slots_free <= 0:
@@ -123,6 +123,8 @@ class GpuProgram(ProgramBase):
         pages = self.kv.import_pages(cold["tensors"][0], cold["n_pages"])
         if pages is None:
             return None
+        for i in cold.get("holes", ()):      # ascending positions
+            pages.insert(i, -1)
         self._ckpt_slots_free -= 1
         slot = self.states.alloc()
         self.states.import_slot(cold["tensors"][1], slot)
@@ -140,13 +142,13 @@ class GpuProgram(ProgramBase):
         self.device_wait_s += time.perf_counter() - t0
 
     def _pages_for(self, n_tokens: int) -> int:
-        return (max(0, n_tokens) + self.kv.page_size - 1) // self.kv.page_size
+        return self.kv.pages_for(n_tokens, self.prefill_chunk)
 
     def _pages_free(self) -> int:
         return int(self.kv.pool.free_pages)
 
     def _pages_held(self, lane: Lane) -> int:
-        return len(self.kv.row_pages.get(lane.row, ()))
+        return self.kv.live_pages(lane.row)
 
     def _kv_room(self, n_tokens: int) -> bool:
         need = self._pages_for(n_tokens)
@@ -248,11 +250,33 @@ class GpuProgram(ProgramBase):
         self._select(lg, rows, greedy, out)
         return out
 
+    def step(self, entries: Sequence[tuple]) -> torch.Tensor:
+        """One ragged step with the tokens given by the caller: `entries` = (lane, tokens, places whose logits are wanted),
+        portions of prompts beside single tokens, all in one batch.  Nothing is sampled; returns the wanted logits
+        [rows, vocab] fp32 on the host, in the order of the entries and of their places.  Lanes come from `open_empty`."""
+        chunks = []
+        for lane, tokens, want in entries:
+            self.kv.advance(lane.row, lane.n_cached, lane.n_cached + len(tokens))
+            chunks.append(SeqChunk(lane.row, lane.slot, lane.n_cached, tokens, want=list(want)))
+        self.kv.publish()
+        batch = self.bufs_prefill.build(chunks)
+        hidden = self.model.forward_hidden(self.ws, batch, self.kv, self.states)
+        rows, out = batch.logit_rows.long(), []
+        for r0 in range(0, rows.numel(), self.max_lanes):
+            lg = self.model.head(self.ws, hidden.index_select(0, rows[r0:r0 + self.max_lanes]))
+            out.append(lg.float().cpu())
+        self._wait_device()
+        self.model.status.check("after step")
+        for lane, tokens, _ in entries:
+            lane.tokens.extend(tokens)
+            lane.n_cached += len(tokens)
+        return torch.cat(out) if out else torch.zeros((0, self.cfg.vocab))
+
     # ------------------------------------------------------------------ prefill
     def prefill_step(self, lane: Lane, budget: int) -> Optional[int]:
         n = min(budget, self.prefill_chunk, len(lane.tokens) - lane.n_cached)
         done = lane.n_cached + n == len(lane.tokens)
-        self.kv.ensure(lane.row, lane.n_cached + n + 1)
+        self.kv.advance(lane.row, lane.n_cached, lane.n_cached + n + self._lookahead)
         self.kv.publish()
         chunk = SeqChunk(lane.row, lane.slot, lane.n_cached, lane.tokens[lane.n_cached:lane.n_cached + n], done)
         if lane.media is not None:
@@ -314,7 +338,7 @@ class GpuProgram(ProgramBase):
         batch = self.bufs_decode.build(self._chunks(lanes), upload=True, rope_delta=[l.rope_delta for l in lanes])
         batch.max_kv_len = bucket
         rows = batch.table_row
-        saved = [(c.clone(), s.clone()) for c, s in zip(self.states.conv, self.states.ssm)]
+        saved = self.states.save()
         stream = torch.cuda.Stream(device=self.device)
         stream.wait_stream(torch.cuda.current_stream())
         with torch.cuda.stream(stream):
@@ -326,9 +350,7 @@ class GpuProgram(ProgramBase):
         with torch.cuda.graph(g):
             self._forward_select(batch, greedy, rows)
         torch.cuda.synchronize(self.device)
-        for (c0, s0), c, s in zip(saved, self.states.conv, self.states.ssm):
-            c.copy_(c0)
-            s.copy_(s0)
+        self.states.load(saved)
         self._graphs[key] = g
         return g
 
@@ -338,7 +360,7 @@ class GpuProgram(ProgramBase):
             return []
         for l in lanes:
             l.tokens.append(l.last_token)
-            self.kv.ensure(l.row, l.n_cached + 2)
+            self.kv.advance(l.row, l.n_cached, l.n_cached + 1 + self._lookahead)
         self.kv.publish()
         greedy = self._fill_sampling(lanes)
         if self.use_graph:

@@ -20,10 +20,12 @@ from typing import Dict, List, Optional, Sequence
 import torch
 
 from ..models.config import ModelConfig
-from ..ops.reference import KV_BF16, KV_FORMAT_NAMES, KV_FP8_ROW, KV_INT8_GROUP, KV_NVFP4
+from ..ops.reference import KV_BF16, KV_FORMAT_NAMES, KV_FP32, KV_FP8_ROW, KV_INT8_GROUP, KV_NVFP4
 
 
 def kv_row_bytes(fmt: int, head_dim: int) -> int:
+    if fmt == KV_FP32:
+        return 4 * head_dim
     return 2 * head_dim if fmt == KV_BF16 else (head_dim // 2 if fmt == KV_NVFP4 else head_dim)
 
 
@@ -49,6 +51,12 @@ class KvLayerPlanes:
     # set when this layer's pages are addressed through ANOTHER cache's block table (a model whose sliding-window
     # layers live in a CyclicKvCache while its other layers live in a full cache); None = the owning cache's table
     block_table: Optional[torch.Tensor] = None
+
+    def typed(self, dtype: torch.dtype):
+        """K and V planes of an uncoded layer (bf16 / fp32 rows) as [pages, kv heads, page size, width] of `dtype`."""
+        if self.fmt != (KV_FP32 if dtype == torch.float32 else KV_BF16):
+            raise ValueError("the cache format does not match the activation type")
+        return self.k_codes.view(dtype), self.v_codes.view(dtype)
 
     def bytes(self) -> int:
         n = self.k_codes.numel() + self.v_codes.numel()
@@ -150,12 +158,12 @@ class MixedKvPlanes(KvLayerPlanes):
 
 def _load_pool_lib():
     import ctypes
-    import os
-    path = os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "_C.so")
-    if not os.path.exists(path):
+    from .._lib import native_path
+    path = native_path()
+    if not path.exists():
         return None
     try:
-        lib = ctypes.CDLL(path)
+        lib = ctypes.CDLL(str(path))
         lib.nfb200_pool_create.restype = ctypes.c_void_p
         lib.nfb200_pool_create.argtypes = [ctypes.c_int32]
         lib.nfb200_pool_destroy.argtypes = [ctypes.c_void_p]
@@ -235,8 +243,12 @@ class PagedKvCache:
     def __init__(self, cfg: ModelConfig, n_pages: int, page_size: int, max_rows: int, max_pages_per_row: int,
                  device, formats: Sequence[str] | str = "bf16", int8_group: int = 64,
                  n_kv_heads: Optional[int] = None, n_layers: Optional[int] = None,
-                 mixed_capacity: Optional[Sequence[int]] = None, mixed_hot_tier: int = 0):
-        """`formats` entry "mixed": that layer keeps its cells in three tiers (MixedKvPlanes); `mixed_capacity` =
+                 mixed_capacity: Optional[Sequence[int]] = None, mixed_hot_tier: int = 0,
+                 geometry: Optional[Sequence[tuple]] = None, look_back: int = 0):
+        """`geometry`: (kv heads, key width, value width) per attention layer, for models whose layers differ (uncoded
+        formats only); default: one geometry from `cfg`.  `look_back`: no layer looks at more than this many newest keys, so
+        `advance` returns earlier pages to the pool (0 = all keys stay).
+        `formats` entry "mixed": that layer keeps its cells in three tiers (MixedKvPlanes); `mixed_capacity` =
         cells per tier (default: every tier can hold every page), `mixed_hot_tier` = where new pages start."""
         self.cfg = cfg
         self.page_size = page_size
@@ -244,13 +256,26 @@ class PagedKvCache:
         self.device = torch.device(device)
         self.n_kv_heads = n_kv_heads if n_kv_heads is not None else cfg.n_kv_heads
         n_attn = n_layers if n_layers is not None else len(cfg.attn_layers)
+        self.geometry = list(geometry) if geometry is not None else None
+        self.look_back = look_back
         if isinstance(formats, str):
             formats = [formats] * n_attn
         if len(formats) != n_attn:
             raise ValueError(f"need one KV format per full-attention layer ({n_attn}), got {len(formats)}")
         D = cfg.head_dim
         self.layers: List[KvLayerPlanes] = []
-        for name in formats:
+        for i, name in enumerate(formats):
+            if self.geometry is not None:
+                if name not in ("bf16", "fp32"):
+                    raise ValueError(f"layers with their own KV geometry are stored as bf16 or fp32 rows, not '{name}'")
+                heads, kw, vw = self.geometry[i]
+                fmt = KV_FORMAT_NAMES[name]
+                k, v = (torch.zeros((n_pages, heads, page_size, kv_row_bytes(fmt, width)), dtype=torch.uint8, device=self.device)
+                        for width in (kw, vw))
+                self.layers.append(KvLayerPlanes(fmt, kw, k, v, None, None))
+                continue
+            if name == "fp32":
+                raise ValueError("this model's kernels have no fp32 KV rows")
             if name == "mixed":
                 cap = list(mixed_capacity) if mixed_capacity is not None else [n_pages, n_pages, n_pages]
                 self.layers.append(MixedKvPlanes(n_pages, self.n_kv_heads, page_size, D, self.device, cap, mixed_hot_tier))
@@ -366,6 +391,23 @@ class PagedKvCache:
             pages.append(p)
             self._dirty_rows.add(row)
 
+    def advance(self, row: int, start: int, end: int) -> None:
+        """Before a step that writes positions [start, end) of `row`: pages that no query of the step can see any more go
+        back to the pool (windowed caches), and the new positions get theirs."""
+        if self.look_back > 0:
+            self.release_before(row, start, self.look_back, 0)
+        self.ensure(row, end)
+
+    def pages_for(self, n_tokens: int, step_tokens: int) -> int:
+        """Most pages a sequence of `n_tokens` holds at any time when steps bring at most `step_tokens` of it."""
+        need = (max(0, n_tokens) + self.page_size - 1) // self.page_size
+        if self.look_back > 0:
+            need = min(need, (self.look_back + step_tokens + self.page_size - 1) // self.page_size + 1)
+        return need
+
+    def live_pages(self, row: int) -> int:
+        return sum(1 for p in self.row_pages.get(row, ()) if p >= 0)
+
     def trim(self, row: int, n_tokens: int) -> None:
         """Drop pages that lie wholly beyond n_tokens (speculative rollback)."""
         pages = self.row_pages.get(row, [])
@@ -434,11 +476,12 @@ class PagedKvCache:
         if tail and self.pool.free_pages < 1:
             return None
         src = self.row_pages[src_row]
-        if any(p < 0 for p in src[: full + (1 if tail else 0)]):
+        if self.look_back <= 0 and any(p < 0 for p in src[: full + (1 if tail else 0)]):
             return None   # early pages were released (sliding window): this history cannot become a frontier
         pages = []
         for i in range(full):
-            self.pool.retain(src[i])
+            if src[i] >= 0:   # (a windowed cache: released pages stay holes, nothing will look at them again)
+                self.pool.retain(src[i])
             pages.append(src[i])
         if tail:
             p_new = self._page_alloc()
@@ -452,7 +495,8 @@ class PagedKvCache:
         full = n_tokens // self.page_size
         mine = self.row_pages.setdefault(dst_row, [])
         for i in range(full):
-            self.pool.retain(pages[i])
+            if pages[i] >= 0:
+                self.pool.retain(pages[i])
             mine.append(pages[i])
             self.table_host[dst_row, i] = pages[i]
         if n_tokens % self.page_size:
@@ -527,7 +571,8 @@ class PagedKvCache:
 
     def drop_pages(self, pages: List[int]) -> None:
         for p in pages:
-            self._page_release(p)
+            if p >= 0:
+                self._page_release(p)
 
     def _copy_page(self, p_src: int, p_dst: int) -> None:
         for l in self.layers:
@@ -592,30 +637,24 @@ class CyclicKvCache(PagedKvCache):
             pages.append(p)
             self._dirty_rows.add(row)
 
-    def live_pages(self, row: int) -> int:
-        return sum(1 for p in self.row_pages.get(row, []) if p >= 0)
 
+class RecurrentStatePool:
+    """Per-sequence recurrent state in `n_slots` slots: for every recurrent layer a tuple of arrays [n_slots, ...].
+    `shapes`: per layer, the (shape without the slot, type) of each array."""
 
-class GdnStatePool:
-    """Conv history + fp32 recurrent state for every GDN layer, `n_slots` sequence slots."""
-
-    def __init__(self, cfg: ModelConfig, n_slots: int, device, n_qk_heads: Optional[int] = None,
-                 n_v_heads: Optional[int] = None, n_layers: Optional[int] = None):
-        self.cfg = cfg
+    def __init__(self, shapes: Sequence[Sequence[tuple]], n_slots: int, device):
         self.n_slots = n_slots
-        hk = n_qk_heads if n_qk_heads is not None else cfg.gdn_qk_heads
-        hv = n_v_heads if n_v_heads is not None else cfg.gdn_v_heads
-        n_gdn = n_layers if n_layers is not None else len(cfg.gdn_layers)
-        d = cfg.gdn_head_dim
-        self.conv_dim = (2 * hk + hv) * d
-        self.conv = [torch.zeros((n_slots, 3, self.conv_dim), dtype=torch.bfloat16, device=device)
-                     for _ in range(n_gdn)]
-        self.ssm = [torch.zeros((n_slots, hv, d, d), dtype=torch.float32, device=device) for _ in range(n_gdn)]
+        self.device = torch.device(device)
+        self.layers = [tuple(torch.zeros((n_slots,) + tuple(shape), dtype=dt, device=device) for shape, dt in layer)
+                       for layer in shapes]
         self._free = list(range(n_slots - 1, -1, -1))
+
+    def tensors(self) -> List[torch.Tensor]:
+        return [t for layer in self.layers for t in layer]
 
     def alloc(self) -> int:
         if not self._free:
-            raise MemoryError("GDN state slots exhausted")
+            raise MemoryError("recurrent state slots exhausted")
         s = self._free.pop()
         self.reset(s)
         return s
@@ -624,34 +663,53 @@ class GdnStatePool:
         self._free.append(slot)
 
     def reset(self, slot: int) -> None:
-        for c, s in zip(self.conv, self.ssm):
-            c[slot].zero_()
-            s[slot].zero_()
+        for t in self.tensors():
+            t[slot].zero_()
 
     def copy_slot(self, src: int, dst: int) -> None:
         """Checkpoint / fork a sequence's recurrent state."""
-        for c, s in zip(self.conv, self.ssm):
-            c[dst].copy_(c[src])
-            s[dst].copy_(s[src])
+        for t in self.tensors():
+            t[dst].copy_(t[src])
+
+    def save(self) -> List[torch.Tensor]:
+        """Copies of every slot: warm-up and capture runs must not advance the state (see `load`)."""
+        return [t.clone() for t in self.tensors()]
+
+    def load(self, saved: List[torch.Tensor]) -> None:
+        for t, c in zip(self.tensors(), saved):
+            t.copy_(c)
 
     def export_slot(self, slot: int) -> List[torch.Tensor]:
-        """State image of one slot (conv history + recurrent state of every layer) as pinned host tensors."""
-        pin = self.conv[0].device.type == "cuda"
+        """State image of one slot (every array of every layer) as pinned host tensors."""
+        pin = self.device.type == "cuda"
         out = []
-        for c, s in zip(self.conv, self.ssm):
-            for t in (c[slot], s[slot]):
-                host = torch.empty(t.shape, dtype=t.dtype, pin_memory=pin)
-                host.copy_(t, non_blocking=True)
-                out.append(host)
+        for t in self.tensors():
+            host = torch.empty(t[slot].shape, dtype=t.dtype, pin_memory=pin)
+            host.copy_(t[slot], non_blocking=True)
+            out.append(host)
         if pin:
-            torch.cuda.current_stream(self.conv[0].device).synchronize()
+            torch.cuda.current_stream(self.device).synchronize()
         return out
 
     def import_slot(self, image: List[torch.Tensor], slot: int) -> None:
-        it = iter(image)
-        for c, s in zip(self.conv, self.ssm):
-            c[slot].copy_(next(it), non_blocking=True)
-            s[slot].copy_(next(it), non_blocking=True)
+        for t, host in zip(self.tensors(), image):
+            t[slot].copy_(host, non_blocking=True)
 
     def total_bytes(self) -> int:
-        return sum(c.numel() * 2 + s.numel() * 4 for c, s in zip(self.conv, self.ssm))
+        return sum(t.numel() * t.element_size() for t in self.tensors())
+
+
+class GdnStatePool(RecurrentStatePool):
+    """Conv history + fp32 recurrent state for every GDN layer, `n_slots` sequence slots."""
+
+    def __init__(self, cfg: ModelConfig, n_slots: int, device, n_qk_heads: Optional[int] = None,
+                 n_v_heads: Optional[int] = None, n_layers: Optional[int] = None):
+        self.cfg = cfg
+        hk = n_qk_heads if n_qk_heads is not None else cfg.gdn_qk_heads
+        hv = n_v_heads if n_v_heads is not None else cfg.gdn_v_heads
+        n_gdn = n_layers if n_layers is not None else len(cfg.gdn_layers)
+        d = cfg.gdn_head_dim
+        self.conv_dim = (2 * hk + hv) * d
+        super().__init__([[((3, self.conv_dim), torch.bfloat16), ((hv, d, d), torch.float32)]] * n_gdn, n_slots, device)
+        self.conv = [layer[0] for layer in self.layers]
+        self.ssm = [layer[1] for layer in self.layers]

@@ -549,6 +549,16 @@ class ProgramBase:
             ck.hits += 1
         return lane
 
+    def open_empty(self) -> Lane:
+        """A lane without a prompt, for callers that bring the tokens of every step themselves (`GpuProgram.step`)."""
+        if not self._free_rows:
+            raise MemoryError("no free lane")
+        slot = self._alloc_slot()
+        lane = Lane(self._next_id, self._free_rows.pop(), slot)
+        self._next_id += 1
+        self.lanes[lane.lane_id] = lane
+        return lane
+
     def force_next_token(self, lane: Lane, token: int) -> None:
         """The token that is fed next on `lane` instead of the one the last step sampled (that one has not been run
         through the model yet, so replacing it rewrites nothing)."""
