@@ -214,6 +214,8 @@ def load_model(args) -> Tuple[ModelConfig, Dict[str, object], Tokenizer, str]:
         from .models import architectures as AR
         if not str(args.device).startswith("cuda"):
             raise SystemExit(f"{args.model}: layer-list models run on the GPU kernels only")
+        if getattr(args, "kv_rowscale", None):
+            raise SystemExit(f"{args.model}: layer-list models have no K row scales")
         if args.weights not in ("bf16", "stored"):
             raise SystemExit(f"{args.model}: layer-list models take bf16 weights, not --weights {args.weights}")
         folder = AR.is_model_folder(args.model)
@@ -244,10 +246,12 @@ def load_model(args) -> Tuple[ModelConfig, Dict[str, object], Tokenizer, str]:
         weights = quantize_weights(weights, args.weights)
     if args.tokenizer:
         tok = Tokenizer.from_file(args.tokenizer)
-    if tok is None:
+    toy_tokenizer = tok is None
+    if toy_tokenizer:
         tok = Tokenizer.train_toy(DEFAULT_CORPUS, n_merges=min(200, max(0, cfg.vocab - 256 - len(SPECIAL_TOKENS))),
                                   added_tokens=SPECIAL_TOKENS)
-    if tok.vocab_size > cfg.vocab:
+    # (a prompt of token ids is not encoded: a small vocabulary without a tokenizer of its own still runs)
+    if tok.vocab_size > cfg.vocab and not (toy_tokenizer and getattr(args, "prompt_ids", None)):
         raise SystemExit(f"tokenizer has {tok.vocab_size} ids but the model's vocabulary is {cfg.vocab}")
     if getattr(args, "vision", False) and not any(k.startswith("vision/") for k in weights):
         if not args.random_init:

@@ -116,4 +116,4 @@ def write_safetensors(path: str, tensors: Dict[str, torch.Tensor], metadata: Dic
         f.write(struct.pack("<Q", len(blob)))
         f.write(blob)
         for _, t in items:
-            f.write(t.view(torch.uint8).numpy().tobytes() if t.numel() else b"")
+            f.write(t.reshape(-1).view(torch.uint8).numpy().tobytes() if t.numel() else b"")

@@ -1,0 +1,56 @@
+"""Small Kuzanex configurations of the tests and weights that make faults visible."""
+import numpy as np
+import torch
+
+from ninfer_fusion_b200.models import kuzanex
+
+
+def att(H, G, D, V, W, scale=0.25, cap=15.0, ff=72):
+    return {"type": "attention", "mixer": {"heads": H, "kv_heads": G, "dim": D, "vdim": V, "scale": scale, "softcap": cap,
+                                           "mask": {"size": W}}, "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def mem(H, D, V, cap=9.0, ff=72):
+    return {"type": "mlstm", "mixer": {"heads": H, "dim": D, "vdim": V, "gate_cap": cap}, "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def conf(width, vocab, layers, alpha=1.5, eps=1e-4):
+    return {"architecture": "Kuzanex", "width": width, "vocab": vocab, "norm": {"eps": eps}, "postln_alpha": alpha, "layers": layers}
+
+
+CASES = {
+    "mixed": conf(96, 211, [mem(2, 32, 48), att(6, 2, 32, 16, 19), att(4, 4, 16, 32, 70, cap=8.0, ff=40), mem(3, 16, 16, cap=5.0)]),
+    # widths that are no multiple of anything, layers without feed-forward, unit alpha, a window of one key
+    "odd": conf(90, 77, [att(3, 1, 20, 36, 1, ff=0), mem(1, 24, 40, ff=0), att(5, 5, 12, 12, 7, ff=30), mem(5, 12, 20, ff=0)],
+                alpha=1.0, eps=1e-2),
+    "attention_only": conf(64, 128, [att(2, 1, 48, 64, 33), att(2, 1, 48, 64, 5)]),
+    "memory_only": conf(64, 130, [mem(2, 48, 32), mem(4, 16, 64)]),
+    "many_heads": conf(128, 96, [att(20, 4, 16, 16, 40), mem(9, 16, 16)]),
+}
+
+
+def build(name, seed=0):
+    """(config dict, LayeredConfig, checkpoint tensors bf16, the same as float64 arrays)."""
+    c = CASES[name]
+    cfg = kuzanex.parse_config(c, name)
+    t = kuzanex.random_tensors(cfg, seed)
+    for n in list(t):
+        if n.endswith((".q.norm", ".k.norm")):
+            t[n] = (t[n].float() * 2.5).to(torch.bfloat16)        # scores that use the cap and single keys out
+        if n.endswith(".act"):
+            t[n] = torch.tensor([0.4, -0.7]).to(torch.bfloat16)
+        if n.endswith("mix.i.b"):
+            t[n] = torch.linspace(-2.0, 4.0, t[n].numel()).to(torch.bfloat16)
+    return c, cfg, t, {n: v.double().numpy() for n, v in t.items()}
+
+
+def prompt(n, vocab, seed):
+    return np.random.default_rng(seed).integers(0, vocab, n).tolist()
+
+
+def err(got, want):
+    """Largest position error: rms over the vocabulary (mean taken off) relative to the rms of all expected logits."""
+    d = np.asarray(got, dtype=np.float64) - want
+    assert np.isfinite(d).all()
+    d -= d.mean(axis=1, keepdims=True)
+    return float(np.sqrt((d * d).mean(axis=1)).max() / np.sqrt(((want - want.mean(1, keepdims=True)) ** 2).mean()))
