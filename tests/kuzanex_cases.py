@@ -48,9 +48,23 @@ def prompt(n, vocab, seed):
     return np.random.default_rng(seed).integers(0, vocab, n).tolist()
 
 
-def err(got, want):
-    """Largest position error: rms over the vocabulary (mean taken off) relative to the rms of all expected logits."""
+def position_errors(got, want):
+    """Per position: rms over the vocabulary (mean taken off) relative to the rms of all expected logits."""
     d = np.asarray(got, dtype=np.float64) - want
     assert np.isfinite(d).all()
     d -= d.mean(axis=1, keepdims=True)
-    return float(np.sqrt((d * d).mean(axis=1)).max() / np.sqrt(((want - want.mean(1, keepdims=True)) ** 2).mean()))
+    return np.sqrt((d * d).mean(axis=1)) / np.sqrt(((want - want.mean(1, keepdims=True)) ** 2).mean())
+
+
+def err(got, want):
+    return float(position_errors(got, want).max())
+
+
+def check(got, want, dt, what=""):
+    """fp32: every position within 3e-5.  bf16: within 0.05, but for one in twenty (or one) up to 0.25: where the head
+    norm divides by an almost cancelled sum (q . k near 0 at the start of a sequence) rounding alone is that large."""
+    e = position_errors(got, want)
+    if dt == torch.float32:
+        assert e.max() < 3e-5, (what, e.max())
+    else:
+        assert e.max() < 0.25 and (e > 0.05).sum() <= max(1, len(e) // 20), (what, np.sort(e)[-5:])

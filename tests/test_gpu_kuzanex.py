@@ -13,7 +13,6 @@ import kuzanex_oracle as K
 
 pytestmark = pytest.mark.gpu
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
-TOL = {torch.float32: 3e-5, torch.bfloat16: 0.05}
 DTYPES = [torch.float32, torch.bfloat16]
 
 
@@ -60,8 +59,8 @@ def test_every_cut_of_a_prompt_gives_the_oracles_logits(name, dt):
     """Whole prompt, token by token, portions down to two tokens, decoding past windows, pages and chunks."""
     ids, want = oracle(name, 141, 1)
     prog = program(name, dt, tokens=160)
-    for cut in CUTS.values():
-        assert C.err(run(prog, ids, cut), want) < TOL[dt]
+    for what, cut in CUTS.items():
+        C.check(run(prog, ids, cut), want, dt, what)
     assert prog.kv.pool.free_pages == prog.kv.n_pages          # every page and slot came back
     assert len(prog._free_rows) == 4 and len(prog.states._free) == 4
 
@@ -96,7 +95,7 @@ def test_mixed_batches_equal_each_request_alone(name, dt):
                 prog.close(live.pop(i)[0])
     for i, n in enumerate(lens):
         ids, want = oracle(name, n, 10 + i)
-        assert C.err(np.concatenate(got[i]), want) < TOL[dt], i
+        C.check(np.concatenate(got[i]), want, dt, i)
     assert prog.kv.pool.free_pages == prog.kv.n_pages
 
 
@@ -106,7 +105,8 @@ def test_prefill_kernels_and_token_kernels_agree():
     a = run(prog, ids, [141])
     prog.model.prefill_kernels = False
     b = run(prog, ids, [141])
-    assert C.err(a, want) < 0.05 and C.err(b, want) < 0.05 and C.err(a, b) < 0.05
+    for got, ref in ((a, want), (b, want), (a, b)):
+        C.check(got, ref, torch.bfloat16)
 
 
 @pytest.mark.parametrize("dt", DTYPES)
@@ -116,14 +116,14 @@ def test_padding_stays_zero_and_only_wanted_places_come_back(dt):
     lane = prog.open_empty()
     assert prog.step([(lane, ids[:20], [])]).shape == (0, want.shape[1])
     lg = prog.step([(lane, ids[20:], [39, 0, 7])]).numpy()
-    assert C.err(lg, want[[59, 20, 27]]) < TOL[dt]
+    C.check(lg, want[[59, 20, 27]], dt)
     assert not prog.ws.x[:40, prog.cfg.hidden:].any()
 
 
 def test_long_decoding_in_32_bit():
     ids, want = oracle("mixed", 420, 4)
     prog = program("mixed", torch.float32, tokens=432, page=8)
-    assert C.err(run(prog, ids, [30] + [1] * 390), want) < 3e-5
+    C.check(run(prog, ids, [30] + [1] * 390), want, torch.float32)
 
 
 # ---------------------------------------------------------------------------- engine
