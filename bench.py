@@ -300,9 +300,20 @@ def main() -> int:
     ap.add_argument("--tree-ranks", type=int, default=1, help="candidates per depth of the draft tree (1 = chain)")
     ap.add_argument("--parallel", default="", choices=["", "tp", "ep"],
                     help="multi-GPU plan: tp = tensor parallel (dense default), ep = data parallel + expert parallel (MoE default)")
+    ap.add_argument("--compare", default="",
+                    help="not the headline benchmark: a layer-list geometry (kuzanex-1b, kuzanex-7b) beside the hybrid decoder of "
+                         "equal size, throughput and per-kernel roofline fractions, one JSON line (one GPU; --layers shrinks both)")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm(args)
+    if args.compare:
+        from ninfer_fusion_b200.utils.layerbench import compare
+        sampler = ClockSampler(0)
+        sampler.start()
+        res = compare(args.compare, args.layers)
+        res["clocks"] = sampler.stop()
+        print(json.dumps(res), flush=True)
+        return 0
     if args.warmup < 3:
         args.warmup = 3
 

@@ -30,7 +30,7 @@ LIB = PKG / "_C.so"
 # model family -> sources (relative to csrc) of its stand-alone library
 SUBSETS = {
     "layered": ("common/tensor_map.cpp", "core_bindings.cpp", "layered_bindings.cpp", "gemm/gemm_bf16.cu", "gemm/gemm_f32.cu",
-                "pointwise/rows32.cu", "attention/qkv_append.cu", "attention/head_mix_token.cu",
+                "pointwise/rows32.cu", "attention/qkv_append.cu", "attention/head_mix_token.cu", "attention/head_mix_decode.cu",
                 "attention/head_mix_prefill.cu", "mlstm/mlstm_recurrent.cu", "mlstm/mlstm_chunked.cu",
                 "sampling/sampling.cu", "runtime/page_pool.cpp"),
 }

@@ -42,6 +42,21 @@ struct HeadMixArgs {
 // [T, n_splits, H, vdim], part_ml: fp32 [T, n_splits, H, 2]; both unused with one split.
 const char* head_mix_token_attention(const HeadMixArgs& a, int split_keys, int n_splits, float* part_o, float* part_ml);
 
+// The tensor-core form of the same (bf16; head_mix_token_attention picks it by itself); leaves the splits unmerged.
+bool head_mix_decode_supported(const HeadMixArgs& a);
+const char* head_mix_decode(const HeadMixArgs& a, int split_keys, int n_splits, float* part_o, float* part_ml);
+
+#ifdef __CUDACC__
+// What the sum of exp(s - m) v, with m the maximum and l the sum of exp(s - m), is multiplied with.
+__device__ __forceinline__ float head_mix_finish(float m, float l, float sink) {
+  if (!(m > -3.0e38f)) return 0.f;   // no visible key
+  if (sink <= 0.f) return 1.f / l;
+  const float mx = fmaxf(m, 0.f);
+  const float e = expf(m - mx);
+  return e / (sink * expf(-mx) + l * e);
+}
+#endif
+
 // bf16 prefill: query blocks of up to 64 consecutive tokens of one sequence (blk_start / blk_count, n_blocks).
 // `max_keys` bounds the visible key range of a block (host).  Mixed scores pass through `scratch` (scratch_bytes) in
 // register-fragment order, as many blocks at a time as fit.

@@ -2,7 +2,8 @@
 // the same (query, key), while the weighted sum over values is per head, so the work is cut in two kernels that meet in
 // an L2-sized scratch of fp32 scores:
 //
-//   scores   one warp = 16 queries x 8 NT keys x ALL heads.  The scores of one head come out of mma.sync in registers,
+//   scores   one warp = 16 queries x 8 NT keys x ALL heads (two kernels: query heads resident in shared memory, or, for
+//            head counts and widths that do not fit there, every operand from global memory).  The scores of one head come out of mma.sync in registers,
 //            are soft-capped there and added into the mixed scores of every head, acc[h] += mix[h, g] * c_g (outer
 //            product form: no score ever crosses a thread).  Distance bias and mask are applied to the finished sums,
 //            which are stored in accumulator-fragment order.  Query and key fragments are read straight from global /
@@ -169,6 +170,181 @@ __global__ void __launch_bounds__(256) head_mix_scores_kernel(const PrefillParam
   }
 }
 
+// The same tile of work with the query heads of its 16 queries resident in shared memory: one CTA = 16 queries, eight
+// warps side by side along the keys, each walking `iters` groups of 8 NT keys.  Key fragments are private to a warp, so
+// they go straight from global memory to registers, one kv head ahead of their use; query fragments come through
+// ldmatrix.  The mixing multiply-adds run as packed pairs.
+__device__ __forceinline__ void fma2(unsigned long long& acc, unsigned long long a, unsigned long long b) {
+  asm("fma.rn.f32x2 %0, %1, %2, %0;" : "+l"(acc) : "l"(a), "l"(b));
+}
+__device__ __forceinline__ unsigned long long pack2(float x, float y) {
+  unsigned long long r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(x), "f"(y));
+  return r;
+}
+__device__ __forceinline__ void unpack2(unsigned long long v, float& x, float& y) {
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(v));
+}
+
+template <int HMAX, int NT, int KS>   // KS: upper bound of dim / 16
+__global__ void __launch_bounds__(256) head_mix_scores_resident_kernel(const PrefillParams p, int iters) {
+  extern __shared__ __align__(16) uint8_t smem_raw[];
+  const HeadMixArgs& a = p.a;
+  const int H = a.n_heads, G = a.n_kv, R = H / G, D = a.dim, P = a.page_size, W = a.window;
+  const int ldq = D + 8, steps = D / 16;
+  float2* mix_s = reinterpret_cast<float2*>(smem_raw);                             // [H][HMAX]: (mix[h, g], mix[h, g])
+  bf16* q_s = reinterpret_cast<bf16*>(smem_raw + sizeof(float2) * H * HMAX);       // [H][16][ldq], k order of the fragments
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r4 = lane >> 2, c4 = lane & 3;
+  for (int i = tid; i < H * HMAX; i += 256) {
+    const int g = i / HMAX, h = i % HMAX;
+    const float m = h < H ? (a.mix != nullptr ? a.mix[h * H + g] : (h == g ? 1.f : 0.f)) : 0.f;
+    mix_s[i] = make_float2(m, m);
+  }
+  pdl_launch_next();
+  pdl_wait_prior();
+  const int qt = blockIdx.x & 3;
+  const BlockRange br(p, p.blk0 + (blockIdx.x >> 2));
+  if (qt * 16 >= br.cnt) return;
+  const int first = br.first_tile(qt, W), last = br.last_tile(qt);
+  const int span = 8 * NT;                                   // tiles per iteration of the CTA
+  const int cta0 = blockIdx.y * iters * span;
+  if (cta0 > last || cta0 + iters * span <= first) return;
+  {
+    const int vecs = D / 8;
+    for (int i = tid; i < H * 16 * vecs; i += 256) {
+      const int v = i % vecs, row = (i / vecs) & 15, h = i / (vecs * 16);
+      const int qi = min(qt * 16 + row, br.cnt - 1);
+      const uint4 x = *reinterpret_cast<const uint4*>(static_cast<const bf16*>(a.q) + (br.t0 + qi) * a.ldq + h * D + v * 8);
+      uint32_t* dst = reinterpret_cast<uint32_t*>(q_s + (h * 16 + row) * ldq);
+      const int d = v * 8, b32 = d & ~31;
+      if (b32 + 32 <= D) {            // a lane's fragment words of two 16-wide steps are eight consecutive values
+        const int c = (d & 31) >> 3;
+        dst[(b32 + 2 * c) / 2] = x.x;
+        dst[(b32 + 8 + 2 * c) / 2] = x.y;
+        dst[(b32 + 16 + 2 * c) / 2] = x.z;
+        dst[(b32 + 24 + 2 * c) / 2] = x.w;
+      } else {                        // last single step: four consecutive values per lane
+        const int c = (d & 15) >> 2;
+        dst[(b32 + 2 * c) / 2] = x.x;
+        dst[(b32 + 8 + 2 * c) / 2] = x.y;
+        dst[(b32 + 2 * c + 2) / 2] = x.z;
+        dst[(b32 + 8 + 2 * c + 2) / 2] = x.w;
+      }
+    }
+  }
+  __syncthreads();
+  const uint32_t q_a = smem_u32(q_s) + ((lane & 15) * ldq + (lane >> 4) * 8) * 2;
+  const float inv_cap = a.softcap > 0.f ? a.scale / a.softcap : 0.f;
+  const long long k_head = static_cast<long long>(P) * D;
+  for (int it = 0; it < iters; ++it) {
+    const int tile0 = cta0 + it * span + warp * NT;
+    if (tile0 > last || tile0 + NT <= first) continue;
+    const bf16* krow[NT];
+#pragma unroll
+    for (int n = 0; n < NT; ++n) {
+      const int key = min(max(br.k0 + (tile0 + n) * 8 + r4, br.lo), br.last);
+      const int page = max(a.block_table[static_cast<long long>(br.row) * a.table_ld + key / P], 0);
+      krow[n] = static_cast<const bf16*>(a.k_pages) + (static_cast<long long>(page) * G * P + key % P) * D;
+    }
+    auto load_k = [&](int g, uint32_t (*k)[KS][2]) {
+#pragma unroll
+      for (int n = 0; n < NT; ++n) {
+        const bf16* kr = krow[n] + g * k_head;
+#pragma unroll
+        for (int s = 0; s < KS; s += 2) {
+          if (s + 1 < steps) {
+            const uint4 x = *reinterpret_cast<const uint4*>(kr + s * 16 + c4 * 8);
+            k[n][s][0] = x.x; k[n][s][1] = x.y;
+            if (s + 1 < KS) { k[n][s + 1][0] = x.z; k[n][s + 1][1] = x.w; }
+          } else if (s < steps) {
+            const uint2 x = *reinterpret_cast<const uint2*>(kr + s * 16 + c4 * 4);
+            k[n][s][0] = x.x; k[n][s][1] = x.y;
+          }
+        }
+      }
+    };
+    unsigned long long acc[HMAX][NT * 2];
+#pragma unroll
+    for (int h = 0; h < HMAX; ++h)
+#pragma unroll
+      for (int j = 0; j < NT * 2; ++j) acc[h][j] = 0ull;
+    uint32_t kf[NT][KS][2], kn[NT][KS][2];
+    load_k(0, kf);
+    for (int g = 0; g < G; ++g) {
+      if (g + 1 < G) load_k(g + 1, kn);
+      for (int r = 0; r < R; ++r) {
+        const int hq = g * R + r;
+        const uint32_t qa = q_a + hq * 16 * ldq * 2;
+        float c[NT][4];
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) c[n][e] = 0.f;
+#pragma unroll
+        for (int s = 0; s < KS; ++s) {
+          if (s < steps) {
+            uint32_t af[4];
+            ldsm_x4(qa + s * 32, af);
+#pragma unroll
+            for (int n = 0; n < NT; ++n) mma_bf16_16816(c[n], af, kf[n][s][0], kf[n][s][1]);
+          }
+        }
+        unsigned long long cp[NT * 2];
+#pragma unroll
+        for (int n = 0; n < NT; ++n) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) c[n][e] = a.softcap > 0.f ? a.softcap * tanh_of<bf16>(c[n][e] * inv_cap) : c[n][e] * a.scale;
+          cp[2 * n] = pack2(c[n][0], c[n][1]);
+          cp[2 * n + 1] = pack2(c[n][2], c[n][3]);
+        }
+        const ulonglong2* mg = reinterpret_cast<const ulonglong2*>(mix_s + hq * HMAX);
+#pragma unroll
+        for (int h = 0; h < HMAX; h += 2) {
+          const ulonglong2 m = mg[h / 2];
+#pragma unroll
+          for (int j = 0; j < NT * 2; ++j) {
+            fma2(acc[h][j], m.x, cp[j]);
+            fma2(acc[h + 1][j], m.y, cp[j]);
+          }
+        }
+      }
+#pragma unroll
+      for (int n = 0; n < NT; ++n)
+#pragma unroll
+        for (int s = 0; s < KS; ++s) { kf[n][s][0] = kn[n][s][0]; kf[n][s][1] = kn[n][s][1]; }
+    }
+#pragma unroll
+    for (int n = 0; n < NT; ++n) {
+      const int tile = tile0 + n;
+      if (tile >= p.n_tiles) break;
+      const int j0 = br.k0 + tile * 8 + c4 * 2, i0 = br.first_query(qt) + r4;
+      float dist[4];
+      bool vis[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int d = (i0 + (e >> 1) * 8) - (j0 + (e & 1));
+        dist[e] = static_cast<float>(d);
+        vis[e] = d >= 0 && (W <= 0 || d < W);
+      }
+      float4* dst = p.scratch + ((static_cast<long long>(blockIdx.x >> 2) * p.n_tiles + tile) * 4 + qt) * H * 32 + lane;
+#pragma unroll
+      for (int h = 0; h < HMAX; ++h) {
+        if (h < H) {
+          const float sl = a.slope != nullptr ? a.slope[h] : 0.f;
+          float4 o;
+          unpack2(acc[h][2 * n], o.x, o.y);
+          unpack2(acc[h][2 * n + 1], o.z, o.w);
+          o.x = vis[0] ? o.x - sl * dist[0] : -CUDART_INF_F;
+          o.y = vis[1] ? o.y - sl * dist[1] : -CUDART_INF_F;
+          o.z = vis[2] ? o.z - sl * dist[2] : -CUDART_INF_F;
+          o.w = vis[3] ? o.w - sl * dist[3] : -CUDART_INF_F;
+          dst[h * 32] = o;
+        }
+      }
+    }
+  }
+}
+
 constexpr int kVTile = 64;   // keys per V tile
 
 // VT: 16-wide value column tiles per CTA.  blockDim 128: warp = query tile.  grid: (query block, head, value chunk)
@@ -284,14 +460,7 @@ __global__ void __launch_bounds__(128) head_mix_values_kernel(const PrefillParam
     const int i = qt * 16 + r4 + r * 8;
     if (i >= br.cnt) continue;
     const long long t = br.t0 + i;
-    float f;
-    if (a.sink > 0.f) {
-      const float mx = fmaxf(m[r], 0.f);
-      const float e = expf(m[r] - mx);
-      f = e / (a.sink * expf(-mx) + l[r] * e);
-    } else {
-      f = 1.f / l[r];
-    }
+    float f = head_mix_finish(m[r], l[r], a.sink);
     if (a.gate != nullptr) f *= sigmoid_of<bf16>(a.gate[t * a.ld_gate + h]);
     bf16* dst = static_cast<bf16*>(a.out) + t * a.ldo + static_cast<long long>(h) * V + v0 + c4 * 2;
 #pragma unroll
@@ -318,6 +487,34 @@ cudaError_t launch_scores(const PrefillParams& p, int n_blocks) {
     if (e != cudaSuccess) return e;
   }
   return launch_kernel(kern, grid, dim3(256), smem, p.a.stream, p.a.pdl, 1, p);
+}
+
+constexpr size_t kResidentSmem = 200 * 1024;
+size_t resident_smem(int H, int hmax, int D) {
+  return sizeof(float2) * static_cast<size_t>(H) * hmax + sizeof(bf16) * static_cast<size_t>(H) * 16 * (D + 8);
+}
+
+template <int HMAX, int NT, int KS>
+cudaError_t launch_resident(const PrefillParams& p, int n_blocks) {
+  auto kern = head_mix_scores_resident_kernel<HMAX, NT, KS>;
+  const size_t smem = resident_smem(p.a.n_heads, HMAX, p.a.dim);
+  if (smem > 48 * 1024) {
+    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    if (e != cudaSuccess) return e;
+  }
+  constexpr int span = 8 * NT;
+  const int groups = (p.n_tiles + span - 1) / span;
+  // several key groups per CTA amortise the staging of the queries, as long as the grid still fills the GPU
+  int iters = 4;
+  while (iters > 1 && static_cast<long long>(n_blocks) * 4 * ((groups + iters - 1) / iters) < 4 * 148) iters >>= 1;
+  const dim3 grid(n_blocks * 4, (groups + iters - 1) / iters);
+  return launch_kernel(kern, grid, dim3(256), smem, p.a.stream, p.a.pdl, 1, p, iters);
+}
+
+template <int HMAX, int NT>
+cudaError_t launch_resident_dim(const PrefillParams& p, int n_blocks) {
+  if (p.a.dim <= 64) return launch_resident<HMAX, NT, 4>(p, n_blocks);
+  return launch_resident<HMAX, NT, 8>(p, n_blocks);
 }
 
 template <int VT>
@@ -359,7 +556,11 @@ const char* head_mix_prefill(const HeadMixArgs& a, const int* blk_start, const i
   for (p.blk0 = 0; p.blk0 < n_blocks; p.blk0 += at_once) {
     const int n = n_blocks - p.blk0 < at_once ? n_blocks - p.blk0 : at_once;
     cudaError_t e;
-    if (a.n_heads <= 4) e = launch_scores<4, 4>(p, n);
+    const bool resident = a.n_heads <= 32 && a.dim <= 128 && a.ldq % 8 == 0 && resident_smem(a.n_heads, 32, a.dim) <= kResidentSmem;
+    if (resident && a.n_heads <= 8) e = launch_resident_dim<8, 2>(p, n);
+    else if (resident && a.n_heads <= 16) e = launch_resident_dim<16, 2>(p, n);
+    else if (resident) e = launch_resident_dim<32, 1>(p, n);
+    else if (a.n_heads <= 4) e = launch_scores<4, 4>(p, n);
     else if (a.n_heads <= 8) e = launch_scores<8, 2>(p, n);
     else if (a.n_heads <= 16) e = launch_scores<16, 2>(p, n);
     else e = launch_scores<32, 1>(p, n);

@@ -1,5 +1,5 @@
-// Head-mixing attention, one query token per CTA (decode, and every size in 32-bit): the CTA holds ALL heads of its
-// token, because a mixed score needs every head's score of the same key.  Keys are walked in blocks of 32:
+// Head-mixing attention, one query token per CTA, on the FP32 pipes (every size, bf16 or 32-bit; bf16 head geometries
+// that suit the tensor cores take head_mix_decode.cu instead): the CTA holds ALL heads of its token, because a mixed score needs every head's score of the same key.  Keys are walked in blocks of 32:
 //   scores   eight lanes per (key, kv head): 16-byte loads along the key row, reduced by shuffles, soft-capped
 //   mix      one thread per (head, key): the row of the mixing matrix times the column of scores, bias, mask
 //   softmax  one warp per head, lane = key: running maximum and sum
@@ -19,15 +19,6 @@ namespace {
 constexpr int kThreads = 256;
 constexpr int kKeys = 32;
 constexpr int kMaxItems = 8;   // (head, 8 value columns) items per thread and pass
-
-__device__ __forceinline__ float finish_scale(float m, float l, float sink) {
-  // 1 / (sink + sum exp(s)) relative to exp(-m): o (sum of exp(s - m) v) times this is the output
-  if (m == -CUDART_INF_F) return 0.f;
-  if (sink <= 0.f) return 1.f / l;
-  const float mx = fmaxf(m, 0.f);
-  const float e = expf(m - mx);
-  return e / (sink * expf(-mx) + l * e);
-}
 
 template <typename A, int NI>
 __global__ void __launch_bounds__(kThreads) head_mix_token_kernel(const HeadMixArgs p, int split_keys, int n_splits,
@@ -184,7 +175,7 @@ __global__ void __launch_bounds__(kThreads) head_mix_token_kernel(const HeadMixA
     const int it = tid + i * kThreads;
     if (it < items) {
       const int h = it / vecs;
-      float f = finish_scale(ms[h], ls[h], p.sink);
+      float f = head_mix_finish(ms[h], ls[h], p.sink);
       if (p.gate != nullptr) f *= sigmoid_of<A>(p.gate[t * p.ld_gate + h]);
 #pragma unroll
       for (int j = 0; j < 8; ++j) acc[i][j] *= f;
@@ -218,11 +209,20 @@ __global__ void __launch_bounds__(128) head_mix_merge_kernel(const HeadMixArgs p
 #pragma unroll
     for (int j = 0; j < 8; ++j) o[j] = fmaf(e, v[j], o[j]);
   }
-  float f = finish_scale(m, l, p.sink);
+  float f = head_mix_finish(m, l, p.sink);
   if (p.gate != nullptr) f *= sigmoid_of<A>(p.gate[t * p.ld_gate + h]);
 #pragma unroll
   for (int j = 0; j < 8; ++j) o[j] *= f;
   store8(static_cast<A*>(p.out) + t * p.ldo + it * 8, o);
+}
+
+template <typename A>
+const char* merge_splits(const HeadMixArgs& a, int n_splits, const float* part_o, const float* part_ml) {
+  if (n_splits <= 1) return nullptr;
+  const int items = a.n_heads * a.vdim / 8;
+  const cudaError_t e = launch_kernel(head_mix_merge_kernel<A>, dim3((items + 127) / 128, a.T), dim3(128), 0, a.stream, a.pdl, 1, a,
+                                      n_splits, part_o, part_ml);
+  return e == cudaSuccess ? nullptr : cudaGetErrorString(e);
 }
 
 template <typename A, int NI>
@@ -249,14 +249,9 @@ const char* launch_token(const HeadMixArgs& a, int split_keys, int n_splits, flo
     if (a.gate != nullptr) b.gate = a.gate + t0 * a.ld_gate;
     float* po = part_o == nullptr ? nullptr : part_o + static_cast<int64_t>(t0) * n_splits * H * a.vdim;
     float* pm = part_ml == nullptr ? nullptr : part_ml + static_cast<int64_t>(t0) * n_splits * H * 2;
-    cudaError_t e = launch_kernel(kern, dim3(n_splits, b.T), dim3(kThreads), smem, a.stream, a.pdl, 1, b, split_keys, n_splits, po, pm);
+    const cudaError_t e = launch_kernel(kern, dim3(n_splits, b.T), dim3(kThreads), smem, a.stream, a.pdl, 1, b, split_keys, n_splits, po, pm);
     if (e != cudaSuccess) return cudaGetErrorString(e);
-    if (n_splits > 1) {
-      const int items = H * a.vdim / 8;
-      e = launch_kernel(head_mix_merge_kernel<A>, dim3((items + 127) / 128, b.T), dim3(128), 0, a.stream, a.pdl, 1, b, n_splits,
-                        static_cast<const float*>(po), static_cast<const float*>(pm));
-      if (e != cudaSuccess) return cudaGetErrorString(e);
-    }
+    if (const char* err = merge_splits<A>(b, n_splits, po, pm)) return err;
   }
   return nullptr;
 }
@@ -280,6 +275,10 @@ const char* head_mix_token_attention(const HeadMixArgs& a, int split_keys, int n
   if (a.ldq % align || a.ldo % align) return "head_mix attention: misaligned rows";
   if (split_keys <= 0 || n_splits <= 0 || (n_splits > 1 && (part_o == nullptr || part_ml == nullptr)))
     return "head_mix attention: bad split";
+  if (head_mix_decode_supported(a)) {
+    if (const char* err = head_mix_decode(a, split_keys, n_splits, part_o, part_ml)) return err;
+    return merge_splits<__nv_bfloat16>(a, n_splits, part_o, part_ml);
+  }
   return a.f32 ? launch_items<float>(a, split_keys, n_splits, part_o, part_ml)
                : launch_items<__nv_bfloat16>(a, split_keys, n_splits, part_o, part_ml);
 }

@@ -197,7 +197,7 @@ int64_t head_mix_block_tokens() { return nfb::kHeadMixBlock; }
 void mlstm(const Tensor& proj, int64_t q_off, int64_t k_off, int64_t v_off, int64_t g_off, const Tensor& gates, int64_t i_off,
            int64_t f_off, int64_t vdim_true, double q_scale, double gate_cap, double eps, const Tensor& norm,
            const Tensor& cu_seqlens, const Tensor& state_slot, const Tensor& S, const Tensor& n, const Tensor& m,
-           const Tensor& out, bool write_state, OptT chunk_ws, bool pdl) {
+           const Tensor& out, bool write_state, OptT chunk_ws, bool pdl, bool one_token) {
   nfb::MlstmArgs a;
   a.f32 = act_f32(proj, "proj");
   need_rows(proj, "proj"); need_rows(out, "out"); need(out, proj.scalar_type(), "out");
@@ -224,6 +224,8 @@ void mlstm(const Tensor& proj, int64_t q_off, int64_t k_off, int64_t v_off, int6
   a.T = static_cast<int>(T); a.n_seq = static_cast<int>(B);
   a.S = static_cast<float*>(S.data_ptr()); a.n = static_cast<float*>(n.data_ptr()); a.m = static_cast<float*>(m.data_ptr());
   a.out = out.data_ptr(); a.ldo = out.stride(0); a.write_state = write_state;
+  TORCH_CHECK(!one_token || T == B, "mlstm: one token per sequence expected");
+  a.one_token = one_token;
   c10::cuda::CUDAGuard guard(proj.device());
   a.stream = cur_stream(); a.pdl = pdl;
   if (chunk_ws.has_value() && chunk_ws->defined()) {
@@ -253,7 +255,7 @@ TORCH_LIBRARY_FRAGMENT(nfb200, m) {
   m.def("head_mix_prefill(Tensor q, Tensor k_pages, Tensor v_pages, Tensor block_table, Tensor table_row, Tensor kv_len, int window, float scale, float softcap, float sink, Tensor? mix, Tensor? slope, Tensor? gate, Tensor out, Tensor blk_start, Tensor blk_count, int max_keys, Tensor scratch, bool pdl) -> ()", &head_mix_prefill);
   m.def("head_mix_prefill_scratch(int n_heads, int max_keys, int window, int blocks) -> int", &head_mix_prefill_scratch);
   m.def("head_mix_block_tokens() -> int", &head_mix_block_tokens);
-  m.def("mlstm(Tensor proj, int q_off, int k_off, int v_off, int g_off, Tensor gates, int i_off, int f_off, int vdim_true, float q_scale, float gate_cap, float eps, Tensor norm, Tensor cu_seqlens, Tensor state_slot, Tensor S, Tensor n, Tensor m, Tensor out, bool write_state, Tensor? chunk_ws, bool pdl) -> ()", &mlstm);
+  m.def("mlstm(Tensor proj, int q_off, int k_off, int v_off, int g_off, Tensor gates, int i_off, int f_off, int vdim_true, float q_scale, float gate_cap, float eps, Tensor norm, Tensor cu_seqlens, Tensor state_slot, Tensor S, Tensor n, Tensor m, Tensor out, bool write_state, Tensor? chunk_ws, bool pdl, bool one_token=False) -> ()", &mlstm);
   m.def("mlstm_chunked_workspace_bytes(int T, int n_seq, int n_heads, int dim, int vdim) -> int", &mlstm_chunked_workspace_bytes);
   m.def("mlstm_chunked_supported(int dim, int vdim) -> bool", &mlstm_chunked_supported);
 }

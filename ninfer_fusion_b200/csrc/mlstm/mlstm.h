@@ -31,6 +31,7 @@ struct MlstmArgs {
   void* out = nullptr;            // [T, H * vdim], leading dimension ldo
   int64_t ldo = 0;
   bool write_state = true;
+  bool one_token = false;         // every sequence brings exactly one token
   bool f32 = false;
   cudaStream_t stream = nullptr;
   bool pdl = false;

@@ -2,7 +2,7 @@
 // and keeps its slice of the matrix memory in registers over all tokens of the step: a thread holds four columns of
 // every (256 / (VC / 4))-th row.  Per token: state update and both contractions (S^T q and n . q) in one pass over the
 // registers, one shuffle + shared-memory reduction, then the head norm (sum of squares exchanged inside the cluster),
-// the output gate and the store.  Decode is this kernel with one token: bound by reading and writing the state once.
+// the output gate and the store.  Steps with one token per sequence take a variant that streams the state.
 #include "mlstm.h"
 
 #include <cooperative_groups.h>
@@ -175,6 +175,149 @@ __global__ void __launch_bounds__(kThreads) mlstm_recurrent_kernel(const MlstmAr
   if (tid == 0 && blockIdx.x == 0) *mg = m;
 }
 
+// One token per sequence: the state slice is streamed instead of kept (read, updated, written and contracted row by row),
+// so few registers and many CTAs keep HBM busy.
+template <typename A, int VC>
+__global__ void __launch_bounds__(kThreads, 3) mlstm_decode_kernel(const MlstmArgs p) {
+  constexpr int kCg = VC / 4, kRg = kThreads / kCg, kAhead = 8;
+  constexpr int kPartials = kThreads / 32;
+  extern __shared__ __align__(16) float smem[];
+  const int D = p.dim, V = p.vdim, H = p.n_heads;
+  float* qs = smem;            // [D]
+  float* ks = qs + D;          // [D]
+  float* ns = ks + D;          // [D] updated normaliser
+  float* red = ns + D;         // [kPartials][kCg][5]
+  __shared__ float ss_part;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int c = tid % kCg, rg = tid / kCg, n_cta = gridDim.x;
+  const int h = blockIdx.y, seq = blockIdx.z, col = blockIdx.x * VC + c * 4;
+  const bool col_ok = col < V;
+  cg::cluster_group cluster = cg::this_cluster();
+  pdl_launch_next();
+  pdl_wait_prior();
+  const int t = p.cu_seqlens[seq];
+  const long long slot = p.state_slot[seq];
+  float* Sg = p.S + (slot * H + h) * D * V + col;
+  float* ng = p.n + (slot * H + h) * D;
+  float* mg = p.m + slot * H + h;
+  float4 S[kAhead];
+  auto fetch = [&](int i0) {
+#pragma unroll
+    for (int j = 0; j < kAhead; ++j) {
+      const int r = rg + (i0 + j) * kRg;
+      if (r < D && col_ok) S[j] = __ldcs(reinterpret_cast<const float4*>(Sg + static_cast<long long>(r) * V));
+    }
+  };
+  fetch(0);
+  const float inv_cap = 1.f / p.gate_cap;
+  const float ig = p.gate_cap * tanhf(p.gates[t * p.ldg + p.i_off + h] * inv_cap);
+  const float fr = p.gate_cap * tanhf(p.gates[t * p.ldg + p.f_off + h] * inv_cap);
+  const float fg = fminf(fr, 0.f) - log1pf(expf(-fabsf(fr)));      // log sigmoid
+  const float m_old = *mg;
+  const float m = fmaxf(fg + m_old, ig);
+  const float da = expf(fg + m_old - m), db = expf(ig - m);
+  const A* row = static_cast<const A*>(p.proj) + t * p.ldp;
+  for (int i = tid; i < D; i += kThreads) {
+    const float k = elem_to_f(row[p.k_off + h * D + i]) * db;
+    qs[i] = elem_to_f(row[p.q_off + h * D + i]) * p.q_scale;
+    ks[i] = k;
+    ns[i] = fmaf(da, ng[i], k);
+  }
+  float v4[4] = {0.f, 0.f, 0.f, 0.f};
+  if (col_ok) {
+#pragma unroll
+    for (int j = 0; j < 4; ++j) v4[j] = elem_to_f(row[p.v_off + h * V + col + j]);
+  }
+  __syncthreads();
+  float acc[5] = {0.f, 0.f, 0.f, 0.f, 0.f};
+  const int per = (D + kRg - 1) / kRg;
+  for (int i0 = 0; i0 < per; i0 += kAhead) {
+#pragma unroll
+    for (int j = 0; j < kAhead; ++j) {
+      const int r = rg + (i0 + j) * kRg;
+      if (r < D) {
+        const float kb = ks[r], qr = qs[r];
+        if (col_ok) {
+          float4 s = S[j];
+          s.x = fmaf(da, s.x, kb * v4[0]);
+          s.y = fmaf(da, s.y, kb * v4[1]);
+          s.z = fmaf(da, s.z, kb * v4[2]);
+          s.w = fmaf(da, s.w, kb * v4[3]);
+          if (p.write_state) __stcs(reinterpret_cast<float4*>(Sg + static_cast<long long>(r) * V), s);
+          acc[0] = fmaf(s.x, qr, acc[0]);
+          acc[1] = fmaf(s.y, qr, acc[1]);
+          acc[2] = fmaf(s.z, qr, acc[2]);
+          acc[3] = fmaf(s.w, qr, acc[3]);
+        }
+        acc[4] = fmaf(ns[r], qr, acc[4]);
+      }
+    }
+    if (i0 + kAhead < per) fetch(i0 + kAhead);
+  }
+  if constexpr (kCg < 32) {
+#pragma unroll
+    for (int e = 0; e < 5; ++e)
+#pragma unroll
+      for (int o = kCg; o < 32; o <<= 1) acc[e] += __shfl_xor_sync(0xffffffffu, acc[e], o);
+  }
+  if (lane < kCg) {
+    float* dst = red + (warp * kCg + c) * 5;
+#pragma unroll
+    for (int e = 0; e < 5; ++e) dst[e] = acc[e];
+  }
+  __syncthreads();
+  float o4[4] = {0.f, 0.f, 0.f, 0.f};
+  if (tid < 32) {
+    float sq = 0.f;
+    if (tid < kCg) {
+      float den = 0.f;
+      for (int w = 0; w < kPartials; ++w) {
+        const float* src = red + (w * kCg + tid) * 5;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o4[e] += src[e];
+        den += src[4];
+      }
+      const float inv = 1.f / (fmaxf(fabsf(den), expf(-m)) + 1e-6f);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        o4[e] *= inv;
+        sq += o4[e] * o4[e];
+      }
+    }
+    sq = warp_sum(sq);
+    if (tid == 0) ss_part = sq;
+  }
+  float total = 0.f;
+  if (n_cta > 1) {
+    cluster.sync();
+    if (tid < 32)
+      for (int r = 0; r < n_cta; ++r) total += *cluster.map_shared_rank(&ss_part, r);
+  } else {
+    __syncthreads();
+    total = ss_part;
+  }
+  if (tid < kCg && col_ok) {
+    const float inv = 1.f / sqrtf(total / static_cast<float>(p.vdim_true) + p.eps);
+    const A* gr = row + p.g_off + h * V + col;
+    A* dst = static_cast<A*>(p.out) + t * p.ldo + h * V + col;
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+      dst[e] = elem_from_f<A>(o4[e] * inv * p.norm[h * V + col + e] * sigmoid_of<A>(elem_to_f(gr[e])));
+  }
+  if (blockIdx.x == 0 && p.write_state) {   // (every CTA of the cluster has read n and m: it passed the cluster barrier)
+    for (int i = tid; i < D; i += kThreads) ng[i] = ns[i];
+    if (tid == 0) *mg = m;
+  }
+  if (n_cta > 1) cluster.sync();   // nobody leaves while a neighbour may still read its sum
+}
+
+template <typename A, int VC>
+cudaError_t launch_decode(const MlstmArgs& a) {
+  const size_t smem = sizeof(float) * (3 * static_cast<size_t>(a.dim) + kThreads / 32 * (VC / 4) * 5);
+  const int n_cta = (a.vdim + VC - 1) / VC;
+  return launch_kernel(mlstm_decode_kernel<A, VC>, dim3(n_cta, a.n_heads, a.n_seq), dim3(kThreads), smem, a.stream, a.pdl, n_cta, a);
+}
+
 template <typename A, int VC, int R>
 cudaError_t launch(const MlstmArgs& a) {
   constexpr int kCg = VC / 4;
@@ -188,6 +331,10 @@ cudaError_t launch(const MlstmArgs& a) {
 template <typename A>
 const char* dispatch(const MlstmArgs& a) {
   cudaError_t e;
+  if (a.one_token) {
+    e = a.vdim <= 8 * 64 ? launch_decode<A, 64>(a) : launch_decode<A, 128>(a);
+    return e == cudaSuccess ? nullptr : cudaGetErrorString(e);
+  }
   if (a.vdim <= 8 * 64) {         // 16 row groups
     if (a.dim <= 64) e = launch<A, 64, 4>(a);
     else if (a.dim <= 128) e = launch<A, 64, 8>(a);

@@ -230,9 +230,9 @@ class LayeredModel:
 
     @staticmethod
     def pick_split(ws, T: int, max_kv_len: int, window: int, sm_count: int = 148) -> Tuple[int, int]:
-        """Keys per split (a multiple of 32) and splits per token: about three CTAs per SM when the step is small."""
+        """Keys per split (a multiple of 32) and splits per token: two CTAs per SM when the step is small."""
         keys = min(max_kv_len, window) if window > 0 else max_kv_len
-        want = max(1, min(3 * sm_count // T, ws.split_rows // T, 64))
+        want = max(1, min(2 * sm_count // T, ws.split_rows // T, 64))
         split = max(64, pad_to(-(-keys // want), 32))
         return split, -(-keys // split)
 
@@ -249,7 +249,7 @@ class LayeredModel:
         out = ws.mix[:T, : H * Vp]
         self.ops.mlstm(proj, 0, H * Dp, 2 * H * Dp, H * (2 * Dp + Vp), gates, 0, H, m.vdim, m.dim ** -0.5, m.gate_cap,
                        self.cfg.rms_eps, self.w[f"{p}/mix/norm"], b.cu_seqlens, b.state_slot, S, n, mx, out, write_state,
-                       chunk_ws, self.pdl)
+                       chunk_ws, self.pdl, b.one_token_per_seq)
         return out
 
     # ------------------------------------------------------------------ forward

@@ -113,7 +113,8 @@ class Paged:
 
 GEOMETRIES = [  # heads, kv heads, key width, value width, window, page
     (4, 4, 32, 32, 8, 16), (6, 2, 48, 80, 40, 64), (3, 1, 16, 16, 1, 8), (16, 4, 128, 128, 100, 64), (20, 5, 64, 96, 33, 32),
-    (32, 8, 128, 64, 64, 64), (8, 8, 64, 64, 0, 16), (2, 1, 16, 272, 50, 64), (34, 17, 32, 32, 20, 16)]
+    (32, 8, 128, 64, 64, 64), (8, 8, 64, 64, 0, 16), (2, 1, 16, 272, 50, 64), (34, 17, 32, 32, 20, 16),
+    (4, 2, 160, 128, 30, 16), (12, 1, 80, 48, 21, 64), (16, 16, 64, 64, 90, 16), (7, 7, 48, 256, 11, 32)]
 
 
 @pytest.mark.parametrize("geo", GEOMETRIES)
@@ -252,7 +253,8 @@ def run_memory(ops, geo, dt, chunked, portions, inputs, cap, eps, slots=5):
             ws.fill_(0xff)      # NaN patterns: nothing may be read before it is written
         ops.mlstm(proj, 0, H * D, 2 * H * D, H * (2 * D + V), gates, 0, H, V, D ** -0.5, cap, eps, norm.cuda(),
                   torch.tensor(cu, dtype=torch.int32, device="cuda"),
-                  torch.tensor([slots - 1 - s for s in seqs], dtype=torch.int32, device="cuda"), S, n, m, out, True, ws, False)
+                  torch.tensor([slots - 1 - s for s in seqs], dtype=torch.int32, device="cuda"), S, n, m, out, True, ws, False,
+                  max(step) == 1)
         for j, s in enumerate(seqs):
             outs[s].append(f64(out[cu[j]:cu[j + 1]]))
     return [np.concatenate(o) for o in outs], (f64(S), f64(n), f64(m))
@@ -278,7 +280,7 @@ def test_matrix_memory(ops, geo, dt, i_shift, f_shift):
         o = K.rms(K.mlstm_recurrence(f64(x[0][s]) * D ** -0.5, f64(x[1][s]), f64(x[2][s]), ig, fg), eps).reshape(n, H * V)
         want.append(o * f64(norm) * K.sigmoid(f64(x[3][s]).reshape(n, H * V)))
     whole = [lens]
-    cut = [[64, 0, 3, 2], [2, 1, 61, 63], [83, 0, 0, 11], [1, 0, 0, 1]]
+    cut = [[64, 0, 3, 2], [2, 1, 60, 63], [82, 0, 0, 11], [1, 0, 1, 0], [1, 0, 0, 1]]
     tol = 2e-5 if dt == torch.float32 else 1.2e-2
     states = []
     for chunked in ((False, True) if dt == torch.bfloat16 and ops.mlstm_chunked_supported(D, V) else (False,)):
