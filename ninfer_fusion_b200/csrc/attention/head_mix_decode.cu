@@ -115,7 +115,7 @@ __global__ void __launch_bounds__(NW * 32) head_mix_decode_kernel(const HeadMixA
 #pragma unroll
       for (int e = 0; e < 4; ++e) o[j][n][e] = 0.f;
   }
-  const float inv_cap = p.softcap > 0.f ? p.scale / p.softcap : 0.f;
+  const float cap_k = p.softcap > 0.f ? 2.f * kLog2e * p.scale / p.softcap : 0.f;
   const uint32_t q_a = smem_u32(q_s);
   __syncthreads();
 
@@ -148,7 +148,7 @@ __global__ void __launch_bounds__(NW * 32) head_mix_decode_kernel(const HeadMixA
           const int r = r4 + (e >> 1) * 8;
           if (r < R) {
             float s = c[n][e];
-            s = p.softcap > 0.f ? p.softcap * tanh_of<bf16>(s * inv_cap) : s * p.scale;
+            s = p.softcap > 0.f ? softcap_fast(s, cap_k, p.softcap) : s * p.scale;
             cs[(g * R + r) * kLdS + n * 8 + c4 * 2 + (e & 1)] = s;
           }
         }

@@ -1,6 +1,6 @@
 // Head-mixing attention for prompt portions (bf16 operands, tensor cores).  A mixed score needs every head's score of
 // the same (query, key), while the weighted sum over values is per head, so the work is cut in two kernels that meet in
-// an L2-sized scratch of fp32 scores:
+// a scratch of fp32 scores:
 //
 //   scores   one warp = 16 queries x 8 NT keys x ALL heads (two kernels: query heads resident in shared memory, or, for
 //            head counts and widths that do not fit there, every operand from global memory).  The scores of one head come out of mma.sync in registers,
@@ -101,7 +101,7 @@ __global__ void __launch_bounds__(256) head_mix_scores_kernel(const PrefillParam
   for (int h = 0; h < HMAX; ++h)
 #pragma unroll
     for (int j = 0; j < NT * 4; ++j) acc[h][j] = 0.f;
-  const float inv_cap = a.softcap > 0.f ? a.scale / a.softcap : 0.f;
+  const float cap_k = a.softcap > 0.f ? 2.f * kLog2e * a.scale / a.softcap : 0.f;
   for (int g = 0; g < H; ++g) {
     float c[NT * 4];
 #pragma unroll
@@ -122,7 +122,7 @@ __global__ void __launch_bounds__(256) head_mix_scores_kernel(const PrefillParam
     }
     if (a.softcap > 0.f) {
 #pragma unroll
-      for (int j = 0; j < NT * 4; ++j) c[j] = a.softcap * tanh_of<bf16>(c[j] * inv_cap);
+      for (int j = 0; j < NT * 4; ++j) c[j] = softcap_fast(c[j], cap_k, a.softcap);
     } else {
 #pragma unroll
       for (int j = 0; j < NT * 4; ++j) c[j] *= a.scale;
@@ -186,12 +186,13 @@ __device__ __forceinline__ void unpack2(unsigned long long v, float& x, float& y
   asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(v));
 }
 
-template <int HMAX, int NT, int KS>   // KS: upper bound of dim / 16
+// KS: dim / 16 (EXACT) or an upper bound of it.
+template <int HMAX, int NT, int KS, bool EXACT>
 __global__ void __launch_bounds__(256) head_mix_scores_resident_kernel(const PrefillParams p, int iters) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
   const HeadMixArgs& a = p.a;
   const int H = a.n_heads, G = a.n_kv, R = H / G, D = a.dim, P = a.page_size, W = a.window;
-  const int ldq = D + 8, steps = D / 16;
+  const int ldq = (EXACT ? KS * 16 : D) + 8, steps = EXACT ? KS : D / 16;
   float2* mix_s = reinterpret_cast<float2*>(smem_raw);                             // [H][HMAX]: (mix[h, g], mix[h, g])
   bf16* q_s = reinterpret_cast<bf16*>(smem_raw + sizeof(float2) * H * HMAX);       // [H][16][ldq], k order of the fragments
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r4 = lane >> 2, c4 = lane & 3;
@@ -234,7 +235,7 @@ __global__ void __launch_bounds__(256) head_mix_scores_resident_kernel(const Pre
   }
   __syncthreads();
   const uint32_t q_a = smem_u32(q_s) + ((lane & 15) * ldq + (lane >> 4) * 8) * 2;
-  const float inv_cap = a.softcap > 0.f ? a.scale / a.softcap : 0.f;
+  const float cap_k = a.softcap > 0.f ? 2.f * kLog2e * a.scale / a.softcap : 0.f;
   const long long k_head = static_cast<long long>(P) * D;
   for (int it = 0; it < iters; ++it) {
     const int tile0 = cta0 + it * span + warp * NT;
@@ -272,28 +273,32 @@ __global__ void __launch_bounds__(256) head_mix_scores_resident_kernel(const Pre
     load_k(0, kf);
     for (int g = 0; g < G; ++g) {
       if (g + 1 < G) load_k(g + 1, kn);
+#pragma unroll 2
       for (int r = 0; r < R; ++r) {
         const int hq = g * R + r;
         const uint32_t qa = q_a + hq * 16 * ldq * 2;
-        float c[NT][4];
+        float c[NT][4], c2[NT][4];   // two accumulation chains
 #pragma unroll
         for (int n = 0; n < NT; ++n)
 #pragma unroll
-          for (int e = 0; e < 4; ++e) c[n][e] = 0.f;
+          for (int e = 0; e < 4; ++e) c[n][e] = c2[n][e] = 0.f;
 #pragma unroll
         for (int s = 0; s < KS; ++s) {
           if (s < steps) {
             uint32_t af[4];
             ldsm_x4(qa + s * 32, af);
 #pragma unroll
-            for (int n = 0; n < NT; ++n) mma_bf16_16816(c[n], af, kf[n][s][0], kf[n][s][1]);
+            for (int n = 0; n < NT; ++n) mma_bf16_16816((s & 1) ? c2[n] : c[n], af, kf[n][s][0], kf[n][s][1]);
           }
         }
         unsigned long long cp[NT * 2];
 #pragma unroll
         for (int n = 0; n < NT; ++n) {
 #pragma unroll
-          for (int e = 0; e < 4; ++e) c[n][e] = a.softcap > 0.f ? a.softcap * tanh_of<bf16>(c[n][e] * inv_cap) : c[n][e] * a.scale;
+          for (int e = 0; e < 4; ++e) {
+            c[n][e] += c2[n][e];
+            c[n][e] = a.softcap > 0.f ? softcap_fast(c[n][e], cap_k, a.softcap) : c[n][e] * a.scale;
+          }
           cp[2 * n] = pack2(c[n][0], c[n][1]);
           cp[2 * n + 1] = pack2(c[n][2], c[n][3]);
         }
@@ -347,19 +352,20 @@ __global__ void __launch_bounds__(256) head_mix_scores_resident_kernel(const Pre
 
 constexpr int kVTile = 64;   // keys per V tile
 
-// VT: 16-wide value column tiles per CTA.  blockDim 128: warp = query tile.  grid: (query block, head, value chunk)
+// VT: 16-wide value column tiles per CTA.  blockDim 128: warp = query tile.  grid: (head, query block, value chunk)
 template <int VT>
-__global__ void __launch_bounds__(128) head_mix_values_kernel(const PrefillParams p) {
+__global__ void __launch_bounds__(128, VT <= 8 ? 4 : 2) head_mix_values_kernel(const PrefillParams p) {
   constexpr int kLd = VT * 16 + 8;
   extern __shared__ __align__(16) bf16 v_s[];   // [2][kVTile][kLd]
   const HeadMixArgs& a = p.a;
   const int H = a.n_heads, G = a.n_kv, V = a.vdim, P = a.page_size, W = a.window;
-  const int h = blockIdx.y, g = h / (H / G), v0 = blockIdx.z * VT * 16;
+  const int h = blockIdx.x, g = h / (H / G), v0 = blockIdx.z * VT * 16;
   pdl_launch_next();
   pdl_wait_prior();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int qt = warp;
-  const BlockRange br(p, p.blk0 + blockIdx.x);
+  const int blk = gridDim.y - 1 - blockIdx.y;   // later blocks of a sequence see more keys: longest first
+  const BlockRange br(p, p.blk0 + blk);
   const bool live = qt * 16 < br.cnt;
   const int first = live ? br.first_tile(qt, W) : 1, last = live ? br.last_tile(qt) : 0;
   const int r4 = lane >> 2, c4 = lane & 3;
@@ -367,16 +373,26 @@ __global__ void __launch_bounds__(128) head_mix_values_kernel(const PrefillParam
   const int* table = a.block_table + static_cast<long long>(br.row) * a.table_ld;
   const bf16* vp = static_cast<const bf16*>(a.v_pages) + static_cast<long long>(g) * P * V;
   const uint32_t vs_base = smem_u32(v_s);
+  // a warp stages 16 rows of every V tile, kRows at a time; lane L < 16 looks up the page of row L / kRows * 4 kRows +
+  // warp * kRows + L % kRows once
+  constexpr int kRows = 32 / (VT * 2);
+  const int col = (lane % (VT * 2)) * 8;
+  const bool col_ok = v0 + col < V;
   auto stage = [&](int vt) {
-    const uint32_t dst = vs_base + (vt & 1) * (kVTile * kLd * 2);
-    for (int i = threadIdx.x; i < kVTile * VT * 2; i += 128) {
-      const int r = i / (VT * 2), c = (i % (VT * 2)) * 8;
-      const int key = br.k0 + vt * kVTile + r;
-      bool ok = key >= br.lo && key <= br.last && v0 + c < V;
-      const int page = ok ? table[key / P] : -1;
-      ok = ok && page >= 0;
-      const bf16* src = ok ? vp + (static_cast<long long>(page) * G * P + key % P) * V + v0 + c : vp;
-      cp_async16(dst + (r * kLd + c) * 2, src, ok);
+    int row = -1;
+    {
+      const int L = lane & 15, key = br.k0 + vt * kVTile + L / kRows * (4 * kRows) + warp * kRows + L % kRows;
+      if (key >= br.lo && key <= br.last) {
+        const int page = table[key / P];
+        row = page < 0 ? -1 : page * G * P + key % P;
+      }
+    }
+    const uint32_t dst = vs_base + (vt & 1) * (kVTile * kLd * 2) + ((warp * kRows + lane / (VT * 2)) * kLd + col) * 2;
+#pragma unroll
+    for (int i = 0; i < 16 / kRows; ++i) {
+      const int r = __shfl_sync(0xffffffffu, row, i * kRows + lane / (VT * 2));
+      const bool ok = r >= 0 && col_ok;
+      cp_async16(dst + i * (4 * kRows * kLd * 2), ok ? vp + static_cast<long long>(r) * V + v0 + col : vp, ok);
     }
     cp_async_commit();
   };
@@ -386,26 +402,37 @@ __global__ void __launch_bounds__(128) head_mix_values_kernel(const PrefillParam
 #pragma unroll
     for (int e = 0; e < 4; ++e) o[n][e] = 0.f;
   float m[2] = {-CUDART_INF_F, -CUDART_INF_F}, l[2] = {0.f, 0.f};
-  const float4* sc = p.scratch + ((static_cast<long long>(blockIdx.x) * p.n_tiles) * 4 + qt) * H * 32 + h * 32 + lane;
+  const float4* sc = p.scratch + ((static_cast<long long>(blk) * p.n_tiles) * 4 + qt) * H * 32 + h * 32 + lane;
   const long long sc_tile = static_cast<long long>(4) * H * 32;
+  // scores of half a V tile, fetched one half ahead of their use
+  auto fetch = [&](int half, float4* s) {
+    if (half * 4 > last || half * 4 + 3 < first) return;
+#pragma unroll
+    for (int n = 0; n < 4; ++n) {
+      const int tile = half * 4 + n;
+      s[n] = (tile >= first && tile <= last) ? __ldcs(sc + tile * sc_tile)
+                                             : make_float4(-CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F);
+    }
+  };
+  float4 nxt[4];
+  fetch(0, nxt);
   stage(0);
   for (int vt = 0; vt < n_vt; ++vt) {
-    const bool mine = vt * 8 <= last && vt * 8 + 7 >= first;
-    float4 s[8];
-    if (mine) {
-#pragma unroll
-      for (int n = 0; n < 8; ++n) {
-        const int tile = vt * 8 + n;
-        s[n] = (tile >= first && tile <= last) ? sc[tile * sc_tile]
-                                               : make_float4(-CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F);
-      }
-    }
     if (vt + 1 < n_vt) { stage(vt + 1); cp_async_wait<1>(); } else { cp_async_wait<0>(); }
     __syncthreads();
-    if (mine) {
+    const uint32_t tile_base = vs_base + (vt & 1) * (kVTile * kLd * 2) + ((lane & 15) * kLd + (lane >> 4) * 8) * 2;
+#pragma unroll
+    for (int hf = 0; hf < 2; ++hf) {
+      const int half = vt * 2 + hf;
+      float4 s[4];
+#pragma unroll
+      for (int n = 0; n < 4; ++n)     // scaled for 2^x
+        s[n] = make_float4(nxt[n].x * kLog2e, nxt[n].y * kLog2e, nxt[n].z * kLog2e, nxt[n].w * kLog2e);
+      fetch(half + 1, nxt);
+      if (half * 4 > last || half * 4 + 3 < first) continue;
       float mx0 = m[0], mx1 = m[1];
 #pragma unroll
-      for (int n = 0; n < 8; ++n) {
+      for (int n = 0; n < 4; ++n) {
         mx0 = fmaxf(mx0, fmaxf(s[n].x, s[n].y));
         mx1 = fmaxf(mx1, fmaxf(s[n].z, s[n].w));
       }
@@ -414,26 +441,27 @@ __global__ void __launch_bounds__(128) head_mix_values_kernel(const PrefillParam
         mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, d));
         mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, d));
       }
-      // a row without a visible key so far keeps maximum -inf; its weights are exp(-inf - 0) = 0
+      // a row without a visible key so far keeps maximum -inf; its weights are 2^(-inf - 0) = 0
       const float b0 = mx0 == -CUDART_INF_F ? 0.f : mx0, b1 = mx1 == -CUDART_INF_F ? 0.f : mx1;
-      const float cr0 = __expf(m[0] - b0), cr1 = __expf(m[1] - b1);
-      m[0] = mx0;
-      m[1] = mx1;
-      l[0] *= cr0;
-      l[1] *= cr1;
+      if (__any_sync(0xffffffffu, mx0 > m[0] || mx1 > m[1])) {   // some row has a new maximum
+        const float cr0 = ex2_fast(m[0] - b0), cr1 = ex2_fast(m[1] - b1);
+        m[0] = mx0;
+        m[1] = mx1;
+        l[0] *= cr0;
+        l[1] *= cr1;
 #pragma unroll
-      for (int n = 0; n < VT * 2; ++n) {
-        o[n][0] *= cr0; o[n][1] *= cr0; o[n][2] *= cr1; o[n][3] *= cr1;
+        for (int n = 0; n < VT * 2; ++n) {
+          o[n][0] *= cr0; o[n][1] *= cr0; o[n][2] *= cr1; o[n][3] *= cr1;
+        }
       }
-      const uint32_t tile_base = vs_base + (vt & 1) * (kVTile * kLd * 2);
 #pragma unroll
-      for (int kk = 0; kk < 4; ++kk) {
+      for (int kk = 0; kk < 2; ++kk) {
         float w[8];
 #pragma unroll
         for (int u = 0; u < 2; ++u) {
           const float4 x = s[2 * kk + u];
-          w[4 * u] = __expf(x.x - b0); w[4 * u + 1] = __expf(x.y - b0);
-          w[4 * u + 2] = __expf(x.z - b1); w[4 * u + 3] = __expf(x.w - b1);
+          w[4 * u] = ex2_fast(x.x - b0); w[4 * u + 1] = ex2_fast(x.y - b0);
+          w[4 * u + 2] = ex2_fast(x.z - b1); w[4 * u + 3] = ex2_fast(x.w - b1);
           l[0] += w[4 * u] + w[4 * u + 1];
           l[1] += w[4 * u + 2] + w[4 * u + 3];
         }
@@ -441,7 +469,7 @@ __global__ void __launch_bounds__(128) head_mix_values_kernel(const PrefillParam
 #pragma unroll
         for (int n = 0; n < VT; ++n) {
           uint32_t b[4];
-          ldsm_x4_trans(tile_base + ((kk * 16 + (lane & 15)) * kLd + n * 16 + (lane >> 4) * 8) * 2, b);
+          ldsm_x4_trans(tile_base + ((hf * 32 + kk * 16) * kLd + n * 16) * 2, b);
           mma_bf16_16816(o[2 * n], af, b[0], b[1]);
           mma_bf16_16816(o[2 * n + 1], af, b[2], b[3]);
         }
@@ -460,7 +488,7 @@ __global__ void __launch_bounds__(128) head_mix_values_kernel(const PrefillParam
     const int i = qt * 16 + r4 + r * 8;
     if (i >= br.cnt) continue;
     const long long t = br.t0 + i;
-    float f = head_mix_finish(m[r], l[r], a.sink);
+    float f = head_mix_finish(m[r] * (1.f / kLog2e), l[r], a.sink);
     if (a.gate != nullptr) f *= sigmoid_of<bf16>(a.gate[t * a.ld_gate + h]);
     bf16* dst = static_cast<bf16*>(a.out) + t * a.ldo + static_cast<long long>(h) * V + v0 + c4 * 2;
 #pragma unroll
@@ -494,9 +522,9 @@ size_t resident_smem(int H, int hmax, int D) {
   return sizeof(float2) * static_cast<size_t>(H) * hmax + sizeof(bf16) * static_cast<size_t>(H) * 16 * (D + 8);
 }
 
-template <int HMAX, int NT, int KS>
+template <int HMAX, int NT, int KS, bool EXACT>
 cudaError_t launch_resident(const PrefillParams& p, int n_blocks) {
-  auto kern = head_mix_scores_resident_kernel<HMAX, NT, KS>;
+  auto kern = head_mix_scores_resident_kernel<HMAX, NT, KS, EXACT>;
   const size_t smem = resident_smem(p.a.n_heads, HMAX, p.a.dim);
   if (smem > 48 * 1024) {
     const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
@@ -513,8 +541,10 @@ cudaError_t launch_resident(const PrefillParams& p, int n_blocks) {
 
 template <int HMAX, int NT>
 cudaError_t launch_resident_dim(const PrefillParams& p, int n_blocks) {
-  if (p.a.dim <= 64) return launch_resident<HMAX, NT, 4>(p, n_blocks);
-  return launch_resident<HMAX, NT, 8>(p, n_blocks);
+  if (p.a.dim == 64) return launch_resident<HMAX, NT, 4, true>(p, n_blocks);
+  if (p.a.dim == 128) return launch_resident<HMAX, NT, 8, true>(p, n_blocks);
+  if (p.a.dim < 64) return launch_resident<HMAX, NT, 4, false>(p, n_blocks);
+  return launch_resident<HMAX, NT, 8, false>(p, n_blocks);
 }
 
 template <int VT>
@@ -527,7 +557,7 @@ cudaError_t launch_values(const PrefillParams& p, int n_blocks) {
     if (e != cudaSuccess) return e;
     attr_set = true;
   }
-  const dim3 grid(n_blocks, p.a.n_heads, (p.a.vdim + VT * 16 - 1) / (VT * 16));
+  const dim3 grid(p.a.n_heads, n_blocks, (p.a.vdim + VT * 16 - 1) / (VT * 16));
   return launch_kernel(kern, grid, dim3(128), smem, p.a.stream, p.a.pdl, 1, p);
 }
 
@@ -542,7 +572,7 @@ const char* head_mix_prefill(const HeadMixArgs& a, const int* blk_start, const i
   if (a.T <= 0 || n_blocks <= 0) return nullptr;
   if (a.f32) return "head_mix_prefill: bf16 only";
   if (a.dim % 16 || a.vdim % 16 || a.n_kv <= 0 || a.n_heads % a.n_kv) return "head_mix_prefill: bad head geometry";
-  if (a.n_heads > 512) return "head_mix_prefill: too many heads";
+  if (a.n_heads > 512 || n_blocks > 65535) return "head_mix_prefill: too many heads or query blocks";
   if (a.ldq % 4 || a.ldo % 2) return "head_mix_prefill: misaligned rows";
   PrefillParams p;
   p.a = a;
@@ -551,8 +581,9 @@ const char* head_mix_prefill(const HeadMixArgs& a, const int* blk_start, const i
   p.scratch = static_cast<float4*>(scratch);
   p.n_tiles = tiles_for(max_keys, a.window);
   const int64_t per_block = head_mix_prefill_scratch(a.n_heads, max_keys, a.window, 1);
-  const int at_once = static_cast<int>(scratch_bytes / per_block < n_blocks ? scratch_bytes / per_block : n_blocks);
-  if (at_once < 1) return "head_mix_prefill: the scratch does not hold one query block";
+  const int fit = static_cast<int>(scratch_bytes / per_block < n_blocks ? scratch_bytes / per_block : n_blocks);
+  if (fit < 1) return "head_mix_prefill: the scratch does not hold one query block";
+  const int launches = (n_blocks + fit - 1) / fit, at_once = (n_blocks + launches - 1) / launches;   // equal shares
   for (p.blk0 = 0; p.blk0 < n_blocks; p.blk0 += at_once) {
     const int n = n_blocks - p.blk0 < at_once ? n_blocks - p.blk0 : at_once;
     cudaError_t e;

@@ -40,6 +40,24 @@ __device__ __forceinline__ void store8(float* p, const float* v) {
   reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
 }
 
+// Hardware 2^x and 1 / x (subnormals flushed): the building blocks of exponentials whose argument is already scaled.
+__device__ __forceinline__ float ex2_fast(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float rcp_fast(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+constexpr float kLog2e = 1.4426950408889634f;
+
+// cap * tanh(x * scale / cap) with k = 2 log2(e) scale / cap: cap - 2 cap / (1 + 2^(k x)).
+__device__ __forceinline__ float softcap_fast(float x, float k, float cap) {
+  return fmaf(-2.f * cap, rcp_fast(ex2_fast(x * k) + 1.f), cap);
+}
+
 // exp / tanh / sigmoid in the precision that goes with the element type: the library functions with 32-bit
 // activations, the hardware exponential otherwise (absolute error of tanh about 1e-7).
 template <typename A>

@@ -55,7 +55,7 @@ __device__ __forceinline__ void chunk_of(const MlstmArgs& p, int slot, int& seq,
   if (len < 0 || slot < chunk_base(p.cu_seqlens, lo)) len = 0;
 }
 
-__global__ void __launch_bounds__(256) mlstm_gates_kernel(const MlstmArgs p, const ChunkWs w) {
+__global__ void __launch_bounds__(1024) mlstm_gates_kernel(const MlstmArgs p, const ChunkWs w) {
   pdl_launch_next();
   pdl_wait_prior();
   const int seq = blockIdx.x, h = blockIdx.y, H = p.n_heads;
@@ -64,7 +64,7 @@ __global__ void __launch_bounds__(256) mlstm_gates_kernel(const MlstmArgs p, con
   const int nc = (te - tb + L - 1) / L, base = chunk_base(p.cu_seqlens, seq);
   const float inv_cap = 1.f / p.gate_cap;
   float* m_state = p.m + static_cast<long long>(p.state_slot[seq]) * H + h;
-  for (int c = warp; c < nc; c += 8) {
+  for (int c = warp; c < nc; c += static_cast<int>(blockDim.x >> 5)) {
     float f[2], u[2], ig[2];
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
@@ -186,7 +186,8 @@ __global__ void __launch_bounds__(256) mlstm_contrib_kernel(const MlstmArgs p, c
   if (v0 == 0 && tid < nd) {
     float a = 0.f;
     const bf16* kc = proj + t0 * p.ldp + p.k_off + h * D + d0 + tid;
-    for (int s = 0; s < len; ++s) a = fmaf(wt[s], __bfloat162float(kc[s * p.ldp]), a);
+#pragma unroll 16
+    for (int s = 0; s < L; ++s) a = fmaf(wt[s], s < len ? __bfloat162float(kc[s * p.ldp]) : 0.f, a);
     w.Un[ch * D + d0 + tid] = a;
   }
   cp_async_wait<0>();
@@ -301,11 +302,13 @@ __global__ void __launch_bounds__(256) mlstm_scan_kernel(const MlstmArgs p, cons
   }
 }
 
-// NT: 8-wide value tiles per warp (8 warps cover V).  grid: (chunk slot, head)
-template <int NT>
-__global__ void __launch_bounds__(256, NT >= 8 ? 1 : 2) mlstm_output_kernel(const MlstmArgs p, const ChunkWs w) {
+// NW warps, NT: 8-wide value tiles per warp (NW warps cover V).  grid: (chunk slot, head)
+template <int NW, int NT>
+__global__ void __launch_bounds__(NW * 32, NW == 8 ? 2 : 1) mlstm_output_kernel(const MlstmArgs p, const ChunkWs w) {
   extern __shared__ __align__(16) bf16 smem_b[];
-  __shared__ float Fs[L], us[L], ms[L], inter[L], den_s[2][L], den_state[L], ss_s[8][L];
+  __shared__ float Fs[L], us[L], ms[L], inter[L], den_s[NW / 4][L], den_state[L], ss_s[NW][L];
+  constexpr int kThreads = NW * 32;
+  constexpr int kKn = L / (NW / 4) / 8;    // 8-key tiles per warp of the intra-chunk weights
   const int H = p.n_heads, D = p.dim, V = p.vdim;
   const int ldq = D + 8, ldv = V + 8;
   constexpr int ldp = L + 8;
@@ -323,7 +326,7 @@ __global__ void __launch_bounds__(256, NT >= 8 ? 1 : 2) mlstm_output_kernel(cons
   const long long ch = static_cast<long long>(slot) * H + h;
   const bf16* proj = static_cast<const bf16*>(p.proj);
   const uint32_t qs_a = smem_u32(qs), ks_a = smem_u32(ks), vs_a = smem_u32(vs), ps_a = smem_u32(ps);
-  for (int i = tid; i < L * (D / 8); i += 256) {
+  for (int i = tid; i < L * (D / 8); i += kThreads) {
     const int s = i / (D / 8), c = (i % (D / 8)) * 8;
     const bool ok = s < len;
     const bf16* row = proj + (t0 + (ok ? s : 0)) * p.ldp + h * D + c;
@@ -331,7 +334,7 @@ __global__ void __launch_bounds__(256, NT >= 8 ? 1 : 2) mlstm_output_kernel(cons
     cp_async16(ks_a + (s * ldq + c) * 2, row + p.k_off, ok);
   }
   cp_async_commit();
-  for (int i = tid; i < L * (V / 8); i += 256) {
+  for (int i = tid; i < L * (V / 8); i += kThreads) {
     const int s = i / (V / 8), c = (i % (V / 8)) * 8;
     const bool ok = s < len;
     cp_async16(vs_a + (s * ldv + c) * 2, proj + (t0 + (ok ? s : 0)) * p.ldp + p.v_off + h * V + c, ok);
@@ -347,18 +350,18 @@ __global__ void __launch_bounds__(256, NT >= 8 ? 1 : 2) mlstm_output_kernel(cons
   }
   cp_async_wait<1>();
   __syncthreads();
-  // ---- intra-chunk weights: warp = 16 queries x 32 keys ----
+  // ---- intra-chunk weights: warp = 16 queries x 8 kKn keys ----
   {
     const int mt = warp & 3, nh = warp >> 2;
-    float c[4][4] = {};
-    if (nh * 32 <= mt * 16 + 15) {   // not entirely above the diagonal
+    float c[kKn][4] = {};
+    if (nh * (kKn * 8) <= mt * 16 + 15) {   // not entirely above the diagonal
       for (int d = 0; d < D; d += 16) {
         uint32_t a[4];
         ldsm_x4(qs_a + ((mt * 16 + (lane & 15)) * ldq + d + (lane >> 4) * 8) * 2, a);
 #pragma unroll
-        for (int n = 0; n < 2; ++n) {
+        for (int n = 0; n < kKn / 2; ++n) {
           uint32_t b[4];
-          ldsm_x4(ks_a + ((nh * 32 + n * 16 + (lane & 7) + (lane >> 4) * 8) * ldq + d + ((lane >> 3) & 1) * 8) * 2, b);
+          ldsm_x4(ks_a + ((nh * (kKn * 8) + n * 16 + (lane & 7) + (lane >> 4) * 8) * ldq + d + ((lane >> 3) & 1) * 8) * 2, b);
           mma_bf16_16816(c[2 * n], a, b[0], b[1]);
           mma_bf16_16816(c[2 * n + 1], a, b[2], b[3]);
         }
@@ -366,17 +369,17 @@ __global__ void __launch_bounds__(256, NT >= 8 ? 1 : 2) mlstm_output_kernel(cons
     }
     float sum[2] = {0.f, 0.f};
 #pragma unroll
-    for (int n = 0; n < 4; ++n) {
+    for (int n = 0; n < kKn; ++n) {
       float x[4];
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int t = mt * 16 + r4 + (e >> 1) * 8, s = nh * 32 + n * 8 + c4 * 2 + (e & 1);
+        const int t = mt * 16 + r4 + (e >> 1) * 8, s = nh * (kKn * 8) + n * 8 + c4 * 2 + (e & 1);
         x[e] = s <= t ? c[n][e] * p.q_scale * expf(Fs[t] + us[s] - ms[t]) : 0.f;
         sum[e >> 1] += x[e];
       }
 #pragma unroll
       for (int r = 0; r < 2; ++r)
-        *reinterpret_cast<uint32_t*>(ps + (mt * 16 + r4 + r * 8) * ldp + nh * 32 + n * 8 + c4 * 2) =
+        *reinterpret_cast<uint32_t*>(ps + (mt * 16 + r4 + r * 8) * ldp + nh * (kKn * 8) + n * 8 + c4 * 2) =
             pack_bf16x2(x[2 * r], x[2 * r + 1]);
     }
 #pragma unroll
@@ -386,9 +389,9 @@ __global__ void __launch_bounds__(256, NT >= 8 ? 1 : 2) mlstm_output_kernel(cons
       if (c4 == 0) den_s[nh][mt * 16 + r4 + r * 8] = sum[r];
     }
   }
-  // ---- n_0 . q: warp = eight queries ----
-  for (int j = 0; j < 8; ++j) {
-    const int t = warp * 8 + j;
+  // ---- n_0 . q: warp = L / NW queries ----
+  for (int j = 0; j < L / NW; ++j) {
+    const int t = warp * (L / NW) + j;
     float d = 0.f;
     for (int i = lane * 8; i < D; i += 256) {
       float q[8], n[8];
@@ -478,7 +481,9 @@ __global__ void __launch_bounds__(256, NT >= 8 ? 1 : 2) mlstm_output_kernel(cons
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
       const int t = m * 16 + r4 + r * 8;
-      const float den = den_s[0][t] + den_s[1][t] + inter[t] * den_state[t];
+      float den = inter[t] * den_state[t];
+#pragma unroll
+      for (int i = 0; i < NW / 4; ++i) den += den_s[i][t];
       const float inv = 1.f / (fmaxf(fabsf(den), expf(-ms[t])) + 1e-6f);
       float sq = 0.f;
 #pragma unroll
@@ -503,7 +508,7 @@ __global__ void __launch_bounds__(256, NT >= 8 ? 1 : 2) mlstm_output_kernel(cons
       if (t >= len) continue;
       float tot = 0.f;
 #pragma unroll
-      for (int i = 0; i < 8; ++i) tot += ss_s[i][t];
+      for (int i = 0; i < NW; ++i) tot += ss_s[i][t];
       const float inv = 1.f / sqrtf(tot / static_cast<float>(p.vdim_true) + p.eps);
       const bf16* gr = proj + (t0 + t) * p.ldp + p.g_off + h * V;
       bf16* dst = static_cast<bf16*>(p.out) + (t0 + t) * p.ldo + h * V;
@@ -560,12 +565,12 @@ cudaError_t allow_smem(K kern, size_t smem) {
                           : cudaSuccess;
 }
 
-template <int NT>
+template <int NW, int NT>
 cudaError_t launch_output(const MlstmArgs& a, const ChunkWs& w, int nc) {
   const size_t smem = output_smem(a.dim, a.vdim);
-  const cudaError_t e = allow_smem(mlstm_output_kernel<NT>, smem);
+  const cudaError_t e = allow_smem(mlstm_output_kernel<NW, NT>, smem);
   if (e != cudaSuccess) return e;
-  return launch_kernel(mlstm_output_kernel<NT>, dim3(nc, a.n_heads), dim3(256), smem, a.stream, a.pdl, 1, a, w);
+  return launch_kernel(mlstm_output_kernel<NW, NT>, dim3(nc, a.n_heads), dim3(NW * 32), smem, a.stream, a.pdl, 1, a, w);
 }
 
 template <int MT>
@@ -599,7 +604,7 @@ const char* mlstm_chunked(const MlstmArgs& a, void* workspace, int64_t workspace
   if (carve(&w, static_cast<char*>(workspace), a.T, a.n_seq, a.n_heads, a.dim, a.vdim) > workspace_bytes)
     return "mlstm_chunked: workspace too small";
   const int nc = a.T / L + a.n_seq;
-  cudaError_t e = launch_kernel(mlstm_gates_kernel, dim3(a.n_seq, a.n_heads), dim3(256), 0, a.stream, a.pdl, 1, a, w);
+  cudaError_t e = launch_kernel(mlstm_gates_kernel, dim3(a.n_seq, a.n_heads), dim3(a.T >= 8 * L * a.n_seq ? 1024 : 256), 0, a.stream, a.pdl, 1, a, w);
   if (e != cudaSuccess) return cudaGetErrorString(e);
   e = a.dim <= 128 ? launch_contrib<1>(a, w, nc) : launch_contrib<2>(a, w, nc);
   if (e != cudaSuccess) return cudaGetErrorString(e);
@@ -607,10 +612,10 @@ const char* mlstm_chunked(const MlstmArgs& a, void* workspace, int64_t workspace
   e = launch_kernel(mlstm_scan_kernel, dim3(blocks, a.n_heads, a.n_seq), dim3(256), 0, a.stream, a.pdl, 1, a, w);
   if (e != cudaSuccess) return cudaGetErrorString(e);
   const int nt = (a.vdim / 8 + 7) / 8;
-  if (nt <= 1) e = launch_output<1>(a, w, nc);
-  else if (nt <= 2) e = launch_output<2>(a, w, nc);
-  else if (nt <= 4) e = launch_output<4>(a, w, nc);
-  else e = launch_output<8>(a, w, nc);
+  if (nt <= 1) e = launch_output<8, 1>(a, w, nc);
+  else if (nt <= 2) e = launch_output<8, 2>(a, w, nc);
+  else if (nt <= 4) e = launch_output<16, 2>(a, w, nc);
+  else e = launch_output<16, 4>(a, w, nc);
   return e == cudaSuccess ? nullptr : cudaGetErrorString(e);
 }
 

@@ -25,7 +25,7 @@ from .layered_config import AttentionMixer, LayeredConfig, MatrixMemoryMixer, pa
 
 ACT_XIELU = 3              # csrc/gemm/gemm.h GemmActivation
 PREFILL_MIN_TOKENS = 8     # shorter portions take the token-by-token kernels
-SCORE_SCRATCH_BYTES = 96 << 20   # fp32 scores in flight between the two prefill attention kernels (stays in L2)
+SCORE_SCRATCH_BYTES = 1 << 30    # fp32 scores in flight between the two prefill attention kernels
 
 
 # ---------------------------------------------------------------------------------------------- weight packing

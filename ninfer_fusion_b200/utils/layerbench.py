@@ -16,6 +16,7 @@ from ..models.architectures import LAYERED_REGISTRY, random_layered_weights
 from ..models.config import ModelConfig
 from ..models.weights import random_weights
 from ..runtime.generator import Generator
+from ..models.layered import SCORE_SCRATCH_BYTES
 from .opbench import L2Flusher, measured_peaks, time_op
 
 
@@ -157,7 +158,7 @@ def _attention_rows(k: _Kernels, ops, model, ws, cfg, hyb, batch: int, new: int,
     if new > 1:
         bs, bc = _blocks(batch, new, int(ops.head_mix_block_tokens()))
         one = int(ops.head_mix_prefill_scratch(H, total, m.window, 1))
-        scratch = torch.empty(max(one, min(one * bs.numel(), 96 << 20)), dtype=torch.uint8, device="cuda")
+        scratch = torch.empty(max(one, min(one * bs.numel(), SCORE_SCRATCH_BYTES)), dtype=torch.uint8, device="cuda")
         k.add(f"attention {tag}", "design", lambda: ops.head_mix_prefill(*args, bs, bc, total, scratch, False),
               batch * min(total, seen + new) * G * (D + V) * 2 + io, macs)
     else:
