@@ -69,11 +69,14 @@ def _throughput(cfg, weights, batch: int, prompt: int, steps: int) -> Dict[str, 
 class _Kernels:
     """Times closures cold and puts them against their roofline."""
 
-    def __init__(self, iters: int):
+    def __init__(self, iters: int, only: str = ""):
+        self.only = only
         self.flush, self.iters, self.rows = L2Flusher(), iters, []
         self.bw, self.fl, self.how = measured_peaks()
 
     def add(self, what: str, model: str, fn, n_bytes: float, macs: float = 0.0) -> None:
+        if self.only not in f"{model}: {what}":
+            return
         med, _ = time_op(fn, iters=self.iters, flush=self.flush)
         t_b, t_f = n_bytes / self.bw, 2.0 * macs / self.fl
         self.rows.append({"kernel": what, "model": model, "us": round(med * 1e6, 1), "bound": "bytes" if t_b >= t_f else "math",
@@ -221,7 +224,7 @@ def _memory_rows(k: _Kernels, ops, cfg, hyb, batch: int, new: int, tag: str) -> 
           2 * ssm.numel() * 4 + conv.numel() * 2 + 2 * T * vd * 2, 2.0 * T * hv * d * d)
 
 
-def compare(name: str, layers: int = 0, iters: int = 10, throughput: bool = True) -> Dict[str, object]:
+def compare(name: str, layers: int = 0, iters: int = 10, throughput: bool = True, only: str = "") -> Dict[str, object]:
     cfg = LAYERED_REGISTRY[name]
     if layers:
         cfg = cfg.shrink(layers)
@@ -233,7 +236,7 @@ def compare(name: str, layers: int = 0, iters: int = 10, throughput: bool = True
     model = LayeredModel(cfg, weights, "cuda:0")
     ws = LayeredWorkspace(cfg, 64, 64, "cuda:0", torch.bfloat16)
     ops = model._raw_ops
-    k = _Kernels(iters)
+    k = _Kernels(iters, only)
     for T, tag in ((32, "decode x32"), (2048, "prefill 2048")):
         _gemm_rows(k, ops, model.status.tensor, cfg, hyb, T, tag)
     _attention_rows(k, ops, model, ws, cfg, hyb, 32, 1, 2048, "decode x32")
@@ -247,7 +250,7 @@ def compare(name: str, layers: int = 0, iters: int = 10, throughput: bool = True
     for r in rows:
         pair.setdefault(r["kernel"], {})[r["model"]] = r
     res["kernels"] = rows
-    res["farther_than_hybrid"] = {n: round(p["hybrid"]["fraction"] / p["design"]["fraction"], 2) for n, p in pair.items()}
+    res["farther_than_hybrid"] = {n: round(p["hybrid"]["fraction"] / p["design"]["fraction"], 2) for n, p in pair.items() if len(p) == 2}
     if throughput:
         res["throughput"] = {}
         w2 = random_weights(hyb, "cuda:0", seed=0)
@@ -255,3 +258,21 @@ def compare(name: str, layers: int = 0, iters: int = 10, throughput: bool = True
             res["throughput"][f"{batch} x {prompt}"] = {"design": _throughput(cfg, weights, batch, prompt, 32),
                                                         "hybrid": _throughput(hyb, w2, batch, prompt, 32)}
     return res
+
+
+def main(argv=None) -> int:
+    import argparse
+    import json
+    ap = argparse.ArgumentParser(description="kernel timings of a layer-list geometry beside the hybrid's")
+    ap.add_argument("model", choices=sorted(LAYERED_REGISTRY))
+    ap.add_argument("--layers", type=int, default=4)
+    ap.add_argument("--iters", type=int, default=10)
+    ap.add_argument("--only", default="", help="only kernels whose 'design: name' or 'hybrid: name' contains this")
+    args = ap.parse_args(argv)
+    for r in compare(args.model, args.layers, args.iters, False, args.only)["kernels"]:
+        print(json.dumps(r))
+    return 0
+
+
+if __name__ == "__main__":
+    raise SystemExit(main())

@@ -113,7 +113,7 @@ class Paged:
 
 GEOMETRIES = [  # heads, kv heads, key width, value width, window, page
     (4, 4, 32, 32, 8, 16), (6, 2, 48, 80, 40, 64), (3, 1, 16, 16, 1, 8), (16, 4, 128, 128, 100, 64), (20, 5, 64, 96, 33, 32),
-    (32, 8, 128, 64, 64, 64), (8, 8, 64, 64, 0, 16), (2, 1, 16, 272, 50, 64), (34, 17, 32, 32, 20, 16),
+    (32, 8, 128, 64, 64, 64), (8, 8, 64, 48, 0, 16), (2, 1, 16, 272, 50, 64), (34, 17, 32, 32, 20, 16),
     (4, 2, 160, 128, 30, 16), (12, 1, 80, 48, 21, 64), (16, 16, 64, 64, 90, 16), (7, 7, 48, 256, 11, 32)]
 
 
@@ -224,7 +224,7 @@ def test_qk_norm_and_append(ops, dt):
         assert torch.equal(vp[pg, 0, r].cpu(), proj[t, (H + G) * Dp:])
 
 
-MEMORIES = [(1, 16, 16), (4, 48, 64), (3, 80, 48), (2, 128, 80), (2, 256, 512), (1, 512, 256), (2, 64, 640)]
+MEMORIES = [(1, 16, 16), (5, 48, 96), (3, 80, 48), (2, 128, 80), (2, 256, 512), (1, 512, 256), (2, 64, 640)]
 
 
 def run_memory(ops, geo, dt, chunked, portions, inputs, cap, eps, slots=5):
