@@ -28,12 +28,12 @@ BUILD = ROOT / "build" / "obj"
 LIB = PKG / "_C.so"
 
 # model family -> sources (relative to csrc) of its stand-alone library
-SUBSETS = {
-    "layered": ("common/tensor_map.cpp", "core_bindings.cpp", "layered_bindings.cpp", "gemm/gemm_bf16.cu", "gemm/gemm_f32.cu",
-                "pointwise/rows32.cu", "attention/qkv_append.cu", "attention/head_mix_token.cu", "attention/head_mix_decode.cu",
-                "attention/head_mix_prefill.cu", "mlstm/mlstm_recurrent.cu", "mlstm/mlstm_chunked.cu",
-                "sampling/sampling.cu", "runtime/page_pool.cpp"),
-}
+_LAYERED = ("common/tensor_map.cpp", "core_bindings.cpp", "layered_bindings.cpp", "gemm/gemm_bf16.cu", "gemm/gemm_f32.cu",
+            "pointwise/rows32.cu", "pointwise/sandwich_rows.cu", "sampling/sampling.cu", "runtime/page_pool.cpp")
+_HEAD_MIX = ("head_mix_bindings.cpp", "attention/qkv_append.cu", "attention/head_mix_token.cu", "attention/head_mix_decode.cu",
+             "attention/head_mix_prefill.cu", "mlstm/mlstm_recurrent.cu", "mlstm/mlstm_chunked.cu")
+_LATENT = ("latent_bindings.cpp", "attention/latent_prep.cu", "attention/latent_token.cu", "gated/gated_recurrent.cu", "gated/gated_chunked.cu")
+SUBSETS = {"head_mix": _LAYERED + _HEAD_MIX, "latent": _LAYERED + _LATENT, "layered": _LAYERED + _HEAD_MIX + _LATENT}
 
 
 def library_path(subset: str = "") -> Path:

@@ -31,6 +31,18 @@ inline T* ptr_or_null(OptT t) {
   return t.has_value() && t->defined() ? static_cast<T*>(t->data_ptr()) : nullptr;
 }
 
+// Activation tensors are bf16 or fp32.
+inline bool act_f32(const Tensor& t, const char* name) {
+  need_cuda(t, name);
+  TORCH_CHECK(t.scalar_type() == at::kBFloat16 || t.scalar_type() == at::kFloat, name, " must be bf16 or fp32");
+  return t.scalar_type() == at::kFloat;
+}
+inline void need_vec(const Tensor& t, at::ScalarType dt, int64_t n, const char* name) {
+  need(t, dt, name);
+  TORCH_CHECK(t.is_contiguous() && t.numel() >= n, name, " is too small or not contiguous");
+}
+
+
 inline int64_t sm_count() {
   static int n = 0;
   if (n == 0) n = at::cuda::getCurrentDeviceProperties()->multiProcessorCount;

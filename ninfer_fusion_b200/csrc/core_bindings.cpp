@@ -12,7 +12,7 @@ void gemm_bf16(const Tensor& x, const Tensor& w, OptT out, int64_t epi, OptT res
   need(x, at::kBFloat16, "x"); need(w, at::kBFloat16, "w");
   need_rows(x, "x"); need_rows(w, "w");
   TORCH_CHECK(x.size(1) == w.size(1), "gemm_bf16: K mismatch");
-  TORCH_CHECK(act >= 0 && act <= 3 && (act == 0 || epi == nfb::kEpiStore), "gemm_bf16: activation needs the store epilogue");
+  TORCH_CHECK(act >= 0 && act <= 4 && (act == 0 || epi == nfb::kEpiStore), "gemm_bf16: activation needs the store epilogue");
   c10::cuda::CUDAGuard guard(x.device());
   nfb::GemmArgs a;
   a.w = w.data_ptr(); a.N = w.size(0); a.K = w.size(1); a.ldw = w.stride(0);

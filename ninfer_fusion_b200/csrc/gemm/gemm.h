@@ -52,7 +52,8 @@ struct GemmGather {
 };
 
 // kActXielu: z > 0: a z^2 + z / 2;  z <= 0: b (exp(z) - 1 - z) + z / 2, with (a, b) = act_params[0..1] (both positive).
-enum GemmActivation : int { kActNone = 0, kActGeluTanh = 1, kActGeluErf = 2, kActXielu = 3 };
+// kActRelu2: max(z, 0)^2.
+enum GemmActivation : int { kActNone = 0, kActGeluTanh = 1, kActGeluErf = 2, kActXielu = 3, kActRelu2 = 4 };
 
 constexpr int kMaxRanks = 8;
 

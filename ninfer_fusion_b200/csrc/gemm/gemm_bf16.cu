@@ -131,6 +131,7 @@ __device__ __forceinline__ float gelu(float x, int mode) {
 __device__ __forceinline__ float activate(float z, int mode, float a, float b) {
   if (mode == kActXielu)
     return z > 0.f ? (a * z + 0.5f) * z : b * (__expf(z) - 1.f - z) + 0.5f * z;
+  if (mode == kActRelu2) return z > 0.f ? z * z : 0.f;
   return gelu(z, mode);
 }
 

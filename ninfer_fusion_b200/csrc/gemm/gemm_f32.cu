@@ -15,6 +15,7 @@ __device__ __forceinline__ float act_f32(float z, int mode, const float* prm) {
     case kActGeluTanh: return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
     case kActGeluErf: return 0.5f * z * (1.f + erff(z * 0.7071067811865476f));
     case kActXielu: return z > 0.f ? (prm[0] * z + 0.5f) * z : prm[1] * (expm1f(z) - z) + 0.5f * z;
+    case kActRelu2: return z > 0.f ? z * z : 0.f;
     default: return z;
   }
 }

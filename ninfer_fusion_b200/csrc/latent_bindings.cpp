@@ -1,0 +1,135 @@
+// torch.ops.nfb200.*: latent attention and gated linear memory (layer-list decoders, models/layered.py).  Activations are
+// bf16 or fp32; every op takes its element type from its tensors.
+#include "attention/latent.h"
+#include "binding_util.h"
+#include "gated/gated.h"
+
+namespace {
+
+using namespace nfb_bind;
+
+const double* freq_ptr(const Tensor& freq, int64_t rot_true) {
+  need_vec(freq, at::kDouble, rot_true / 2, "freq");
+  return static_cast<const double*>(freq.data_ptr());
+}
+void need_pages(const Tensor& pages, at::ScalarType dt, int64_t width) {
+  need(pages, dt, "pages");
+  TORCH_CHECK(pages.dim() == 4 && pages.is_contiguous() && pages.size(1) == 1 && pages.size(3) == width,
+              "latent pages must be [pages, 1, page size, latent + rotated part]");
+}
+void need_table(const Tensor& table) {
+  need(table, at::kInt, "block_table");
+  TORCH_CHECK(table.dim() == 2 && table.stride(1) == 1, "block_table must be [rows, pages]");
+}
+
+void latent_prep(const Tensor& proj, int64_t q_rank_true, int64_t rank_true, int64_t rot_true, const Tensor& q_norm,
+                 const Tensor& kv_norm, double eps, const Tensor& freq, const Tensor& table_row, const Tensor& cache_pos,
+                 const Tensor& block_table, const Tensor& q_latent, const Tensor& pages, bool pdl) {
+  nfb::LatentPrepArgs a;
+  a.f32 = act_f32(proj, "proj");
+  const int64_t T = proj.size(0);
+  need_rows(proj, "proj"); need_rows(q_latent, "q_latent"); need(q_latent, proj.scalar_type(), "q_latent"); need_table(block_table);
+  const int64_t qr = q_latent.size(1), rank = kv_norm.numel(), rot = proj.size(1) - qr - rank;
+  TORCH_CHECK(q_latent.size(0) == T && rot >= 0, "latent_prep: projection columns");
+  need_pages(pages, proj.scalar_type(), rank + rot);
+  need_vec(q_norm, at::kFloat, qr, "q_norm"); need_vec(kv_norm, at::kFloat, rank, "kv_norm");
+  need_vec(table_row, at::kInt, T, "table_row"); need_vec(cache_pos, at::kInt, T, "cache_pos");
+  a.proj = proj.data_ptr(); a.ldp = proj.stride(0); a.T = static_cast<int>(T);
+  a.q_rank = static_cast<int>(qr); a.q_rank_true = static_cast<int>(q_rank_true);
+  a.rank = static_cast<int>(rank); a.rank_true = static_cast<int>(rank_true);
+  a.rot = static_cast<int>(rot); a.rot_true = static_cast<int>(rot_true);
+  a.q_norm = static_cast<const float*>(q_norm.data_ptr()); a.kv_norm = static_cast<const float*>(kv_norm.data_ptr());
+  a.eps = static_cast<float>(eps); a.freq = freq_ptr(freq, rot_true);
+  a.table_row = static_cast<const int*>(table_row.data_ptr()); a.cache_pos = static_cast<const int*>(cache_pos.data_ptr());
+  a.block_table = static_cast<const int*>(block_table.data_ptr()); a.table_ld = static_cast<int>(block_table.stride(0));
+  a.page_size = static_cast<int>(pages.size(2));
+  a.q_latent = q_latent.data_ptr(); a.ldq = q_latent.stride(0); a.pages = pages.data_ptr();
+  c10::cuda::CUDAGuard guard(proj.device());
+  a.stream = cur_stream(); a.pdl = pdl;
+  chk(nfb::latent_prep(a));
+}
+
+nfb::LatentArgs latent_args(const Tensor& q, const Tensor& pages, const Tensor& block_table, const Tensor& table_row,
+                            const Tensor& kv_len, int64_t n_heads, int64_t rank, int64_t rot_true, double scale, const Tensor& freq,
+                            OptT sink, const Tensor& out, bool pdl) {
+  nfb::LatentArgs a;
+  a.f32 = act_f32(q, "q");
+  need_rows(q, "q"); need_rows(out, "out"); need(out, q.scalar_type(), "out"); need_table(block_table);
+  const int64_t T = q.size(0), rot = pages.size(3) - rank;
+  need_pages(pages, q.scalar_type(), rank + rot);
+  TORCH_CHECK(n_heads > 0 && q.size(1) % n_heads == 0 && q.size(1) / n_heads >= rot && out.size(0) == T, "latent attention: shapes");
+  need_vec(table_row, at::kInt, T, "table_row"); need_vec(kv_len, at::kInt, T, "kv_len");
+  if (sink.has_value() && sink->defined()) need_vec(*sink, at::kFloat, n_heads, "sink");
+  a.q = q.data_ptr(); a.ldq = q.stride(0); a.pages = pages.data_ptr();
+  a.block_table = static_cast<const int*>(block_table.data_ptr()); a.table_ld = static_cast<int>(block_table.stride(0));
+  a.table_row = static_cast<const int*>(table_row.data_ptr()); a.kv_len = static_cast<const int*>(kv_len.data_ptr());
+  a.T = static_cast<int>(T); a.n_heads = static_cast<int>(n_heads); a.rank = static_cast<int>(rank); a.rot = static_cast<int>(rot);
+  a.dim = static_cast<int>(q.size(1) / n_heads - rot); a.rot_true = static_cast<int>(rot_true);
+  a.page_size = static_cast<int>(pages.size(2)); a.scale = static_cast<float>(scale); a.freq = freq_ptr(freq, rot_true);
+  a.sink = ptr_or_null<const float>(sink); a.out = out.data_ptr(); a.ldo = out.stride(0);
+  a.stream = cur_stream(); a.pdl = pdl;
+  return a;
+}
+
+void latent_token_attention(const Tensor& q_latent, const Tensor& q, const Tensor& pages, const Tensor& block_table,
+                            const Tensor& table_row, const Tensor& kv_len, int64_t n_heads, int64_t rot_true, double scale,
+                            const Tensor& freq, OptT sink, const Tensor& out, bool pdl) {
+  c10::cuda::CUDAGuard guard(q.device());
+  need_rows(q_latent, "q_latent"); need(q_latent, q.scalar_type(), "q_latent");
+  const int64_t rank = q_latent.size(1) / n_heads;
+  nfb::LatentArgs a = latent_args(q, pages, block_table, table_row, kv_len, n_heads, rank, rot_true, scale, freq, sink, out, pdl);
+  TORCH_CHECK(q_latent.size(0) == a.T && out.size(1) == n_heads * rank, "latent attention: shapes");
+  a.q_latent = q_latent.data_ptr(); a.ldl = q_latent.stride(0);
+  chk(nfb::latent_token_attention(a));
+}
+
+void gated_memory(const Tensor& proj, int64_t q_off, int64_t v_off, const Tensor& gates, const Tensor& lower, int64_t vdim_true,
+                  double eps, const Tensor& norm, const Tensor& cu_seqlens, const Tensor& state_slot, const Tensor& S,
+                  const Tensor& out, bool write_state, OptT chunk_ws, bool pdl, bool one_token) {
+  nfb::GatedArgs a;
+  a.f32 = act_f32(proj, "proj");
+  need_rows(proj, "proj"); need_rows(out, "out"); need(out, proj.scalar_type(), "out");
+  need(gates, at::kFloat, "gates"); need_rows(gates, "gates"); need(S, at::kFloat, "S");
+  TORCH_CHECK(S.dim() == 4 && S.is_contiguous(), "gated memory: state must be [slots, heads, dim, vdim]");
+  const int64_t T = proj.size(0), H = S.size(1), D = S.size(2), V = S.size(3), B = state_slot.numel(), cols = proj.size(1);
+  TORCH_CHECK(out.size(0) == T && out.size(1) == H * V && gates.size(0) == T && gates.size(1) >= H * D, "gated memory: out / gates shape");
+  TORCH_CHECK(q_off >= 0 && q_off + H * D <= cols && v_off >= 0 && v_off + H * V <= cols, "gated memory: projection columns");
+  TORCH_CHECK(vdim_true > 0 && vdim_true <= V, "gated memory: value width");
+  need_vec(lower, at::kFloat, H * D, "lower"); need_vec(norm, at::kFloat, V, "norm");
+  need_vec(cu_seqlens, at::kInt, B + 1, "cu_seqlens"); need_vec(state_slot, at::kInt, B, "state_slot");
+  a.proj = proj.data_ptr(); a.ldp = proj.stride(0); a.q_off = static_cast<int>(q_off); a.v_off = static_cast<int>(v_off);
+  a.gates = static_cast<const float*>(gates.data_ptr()); a.ldg = gates.stride(0); a.lower = static_cast<const float*>(lower.data_ptr());
+  a.n_heads = static_cast<int>(H); a.dim = static_cast<int>(D); a.vdim = static_cast<int>(V); a.vdim_true = static_cast<int>(vdim_true);
+  a.eps = static_cast<float>(eps); a.norm = static_cast<const float*>(norm.data_ptr());
+  a.cu_seqlens = static_cast<const int*>(cu_seqlens.data_ptr()); a.state_slot = static_cast<const int*>(state_slot.data_ptr());
+  a.T = static_cast<int>(T); a.n_seq = static_cast<int>(B); a.S = static_cast<float*>(S.data_ptr());
+  a.out = out.data_ptr(); a.ldo = out.stride(0); a.write_state = write_state;
+  TORCH_CHECK(!one_token || T == B, "gated memory: one token per sequence expected");
+  a.one_token = one_token;
+  c10::cuda::CUDAGuard guard(proj.device());
+  a.stream = cur_stream(); a.pdl = pdl;
+  if (chunk_ws.has_value() && chunk_ws->defined()) {
+    need_cuda(*chunk_ws, "chunk_ws");
+    chk(nfb::gated_chunked(a, chunk_ws->data_ptr(), chunk_ws->numel() * chunk_ws->element_size()));
+  } else {
+    chk(nfb::gated_recurrent(a));
+  }
+}
+
+int64_t gated_chunked_workspace_bytes(int64_t T, int64_t n_seq, int64_t n_heads, int64_t dim, int64_t vdim) {
+  return nfb::gated_chunked_workspace_bytes(static_cast<int>(T), static_cast<int>(n_seq), static_cast<int>(n_heads),
+                                            static_cast<int>(dim), static_cast<int>(vdim));
+}
+bool gated_chunked_supported(int64_t dim, int64_t vdim) {
+  return nfb::gated_chunked_supported(static_cast<int>(dim), static_cast<int>(vdim));
+}
+
+}  // namespace
+
+TORCH_LIBRARY_FRAGMENT(nfb200, m) {
+  m.def("latent_prep(Tensor proj, int q_rank_true, int rank_true, int rot_true, Tensor q_norm, Tensor kv_norm, float eps, Tensor freq, Tensor table_row, Tensor cache_pos, Tensor block_table, Tensor q_latent, Tensor pages, bool pdl) -> ()", &latent_prep);
+  m.def("latent_token_attention(Tensor q_latent, Tensor q, Tensor pages, Tensor block_table, Tensor table_row, Tensor kv_len, int n_heads, int rot_true, float scale, Tensor freq, Tensor? sink, Tensor out, bool pdl) -> ()", &latent_token_attention);
+  m.def("gated_memory(Tensor proj, int q_off, int v_off, Tensor gates, Tensor lower, int vdim_true, float eps, Tensor norm, Tensor cu_seqlens, Tensor state_slot, Tensor S, Tensor out, bool write_state, Tensor? chunk_ws, bool pdl, bool one_token=False) -> ()", &gated_memory);
+  m.def("gated_chunked_workspace_bytes(int T, int n_seq, int n_heads, int dim, int vdim) -> int", &gated_chunked_workspace_bytes);
+  m.def("gated_chunked_supported(int dim, int vdim) -> bool", &gated_chunked_supported);
+}

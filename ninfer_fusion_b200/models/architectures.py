@@ -8,10 +8,10 @@ import json
 import os
 from typing import Dict
 
-from . import kuzanex
+from . import kuzanex, tebivik
 from .layered_config import LayeredConfig
 
-DESIGNS = {m.ARCHITECTURE: m for m in (kuzanex,)}
+DESIGNS = {m.ARCHITECTURE: m for m in (kuzanex, tebivik)}
 LAYERED_REGISTRY: Dict[str, LayeredConfig] = {name: c for m in DESIGNS.values() for name, c in m.CONFIGS.items()}
 
 

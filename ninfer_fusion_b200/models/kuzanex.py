@@ -98,12 +98,8 @@ def tensor_shapes(cfg: LayeredConfig) -> Iterator[Tuple[str, tuple]]:
 
 def check_tensors(cfg: LayeredConfig, shape_of) -> None:
     """Every tensor of the configuration is there in its shape; `shape_of(name)` returns None for a missing one."""
-    for name, shape in tensor_shapes(cfg):
-        have = shape_of(name)
-        if have is None:
-            raise ValueError(f"checkpoint has no tensor '{name}'")
-        if tuple(have) != shape:
-            raise ValueError(f"tensor '{name}' has shape {list(have)}, the configuration asks for {list(shape)}")
+    from .layered import check_tensor_shapes
+    check_tensor_shapes(tensor_shapes(cfg), shape_of)
 
 
 def pack(cfg: LayeredConfig, tensors, dtype, device="cpu") -> dict:

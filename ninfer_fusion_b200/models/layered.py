@@ -1,15 +1,16 @@
 """Decoders described as a list of layers (`models/layered_config.py`): weight packing and the forward pass on the
 native kernels.
 
-A layer is a mixer (head-mixing attention or matrix memory) and an optional feed-forward, each followed by the
-norm-after-the-sum step ``x <- rms_norm(alpha x + f(x)) * gain`` on a 32-bit residual stream.  Every size and constant
-is a field of the layer's description; which mechanisms a mixer has (biases, query / key norm, soft cap, distance bias,
-mixing across heads, sink, window, head gate) is too, so a design is a mapping onto these fields
-(`models/kuzanex.py`) and not a model file of its own.
+A layer is a mixer (head-mixing attention, latent attention, matrix memory or gated linear memory) and an optional
+feed-forward on a 32-bit residual stream.  A sublayer meets the stream in one of two ways: the norm after the sum,
+``x <- rms_norm(alpha x + f(x)) * gain``, or norms around it, ``x <- x + mult * norm(f(norm(x)))``, with an optional
+causal convolution in front of every mixer.  Layers can run several times with the same weights; cache and state belong
+to layer runs.  Every size and constant is a field of the description, so a design is a mapping onto these fields
+(`models/kuzanex.py`, `models/tebivik.py`) and not a model file of its own.
 
-The engine side is the hybrid runtime's: one ragged token batch per step (`runtime/batch.py`), K / V rows in the paged
-cache (one geometry per layer), recurrent state in per-sequence slots, preallocated buffers so that a decode step can be
-captured in a CUDA graph.  Activations are bf16 (tcgen05 GEMMs, tensor-core prefill kernels) or, for exact runs, fp32.
+The engine side is the hybrid runtime's: one ragged token batch per step (`runtime/batch.py`), K / V or latent rows in the
+paged cache (one geometry per run), recurrent state in per-sequence slots, preallocated buffers so that a decode step can
+be captured in a CUDA graph.  Activations are bf16 (tcgen05 GEMMs, tensor-core prefill kernels) or, for exact runs, fp32.
 Head widths are padded to multiples of 16 and the model width to a multiple of 8 when the weights are packed: zero rows
 and columns change no product, and every norm divides by the true width.
 """
@@ -21,9 +22,11 @@ import torch
 
 from .._lib import StatusWord, load_native
 from .hybrid import EPI_STORE, LaunchCounter, StepBatch
-from .layered_config import AttentionMixer, LayeredConfig, MatrixMemoryMixer, pad_to
+from .layered_config import (ATTENTION_KINDS, AttentionMixer, GatedMemoryMixer, LatentAttentionMixer, LayeredConfig,
+                             MatrixMemoryMixer, pad_to)
 
-ACT_XIELU = 3              # csrc/gemm/gemm.h GemmActivation
+ACTIVATIONS = {"xielu": 3, "relu2": 4}     # csrc/gemm/gemm.h GemmActivation
+BLOCK_TOKENS = 64          # query tokens per attention block of a step (kHeadMixBlock, kLatentBlock)
 PREFILL_MIN_TOKENS = 8     # shorter portions take the token-by-token kernels
 SCORE_SCRATCH_BYTES = 1 << 30    # fp32 scores in flight between the two prefill attention kernels
 
@@ -57,68 +60,140 @@ def distance_slopes(heads: int) -> torch.Tensor:
     return torch.tensor([2.0 ** (-8.0 * (h + 1) / heads) for h in range(heads)], dtype=torch.float64)
 
 
+def check_tensor_shapes(expected, shape_of) -> None:
+    """Every (name, shape) of `expected` is there; `shape_of(name)` returns None for a missing tensor."""
+    for name, shape in expected:
+        have = shape_of(name)
+        if have is None:
+            raise ValueError(f"checkpoint has no tensor '{name}'")
+        if tuple(have) != shape:
+            raise ValueError(f"tensor '{name}' has shape {list(have)}, the configuration asks for {list(shape)}")
+
+
+def _pack_attention(w, p, m: AttentionMixer, get, n_out: int, hp: int, device):
+    H, G, D, V, Dp, Vp = m.heads, m.kv_heads, m.dim, m.vdim, m.dim_p, m.vdim_p
+    rows = [_pad_head_rows(get("q"), H, D, Dp, hp), _pad_head_rows(get("k"), G, D, Dp, hp), _pad_head_rows(get("v"), G, V, Vp, hp)]
+    bias = torch.zeros(n_out, dtype=torch.float32, device=device)
+    if m.head_gate:
+        rows.append(_pad2(get("g"), H, hp))
+    if m.bias:
+        b = torch.cat([_pad_head_vec(get("q_bias"), H, D, Dp), _pad_head_vec(get("k_bias"), G, D, Dp),
+                       _pad_head_vec(get("v_bias"), G, V, Vp)])
+        bias[: b.numel()] = b
+    if m.qk_norm:
+        w[f"{p}/mix/q_norm"] = _pad_head_vec(get("q_norm"), 1, D, Dp)
+        w[f"{p}/mix/k_norm"] = _pad_head_vec(get("k_norm"), 1, D, Dp)
+    mix = get("talk").double() if m.head_mixing else torch.eye(H, dtype=torch.float64, device=device)
+    if m.head_mixing:
+        w[f"{p}/mix/heads"] = mix.float().contiguous()
+    if m.distance_bias:
+        # mixing is linear: the bias taken off before it is (mix @ slope) taken off after it
+        w[f"{p}/mix/slope"] = (mix @ distance_slopes(H).to(device)).float().contiguous()
+    w[f"{p}/mix/in_bias"] = bias
+    return rows
+
+
+def _pack_matrix_memory(w, p, m: MatrixMemoryMixer, get, n_out: int, hp: int, device):
+    H, D, V, Dp, Vp = m.heads, m.dim, m.vdim, m.dim_p, m.vdim_p
+    bias = torch.zeros(n_out, dtype=torch.float32, device=device)
+    bias[m.main_cols: m.main_cols + H] = get("i_bias").float()
+    bias[m.main_cols + H: m.main_cols + 2 * H] = get("f_bias").float()
+    w[f"{p}/mix/in_bias"] = bias
+    w[f"{p}/mix/norm"] = _pad_head_vec(get("norm"), H, V, Vp)
+    return [_pad_head_rows(get("q"), H, D, Dp, hp), _pad_head_rows(get("k"), H, D, Dp, hp), _pad_head_rows(get("v"), H, V, Vp, hp),
+            _pad_head_rows(get("g"), H, V, Vp, hp), _pad2(get("i"), H, hp), _pad2(get("f"), H, hp)]
+
+
+def _pack_gated_memory(w, p, m: GatedMemoryMixer, get, n_out: int, hp: int, device):
+    H, D, V, Dp, Vp = m.heads, m.dim, m.vdim, m.dim_p, m.vdim_p
+    bias = torch.zeros(n_out, dtype=torch.float32, device=device)
+    bias[m.main_cols: m.main_cols + H * Dp] = _pad_head_vec(get("f_bias"), H, D, Dp)
+    lower = torch.ones((H, Dp), dtype=torch.float32, device=device)       # padded channels forget nothing and take nothing in
+    lower[:, :D] = get("lower").float().reshape(H, D)
+    w[f"{p}/mix/in_bias"] = bias
+    w[f"{p}/mix/lower"] = lower.reshape(-1)
+    w[f"{p}/mix/norm"] = _pad_head_vec(get("norm"), 1, V, Vp)
+    return [_pad_head_rows(get("q"), H, D, Dp, hp), _pad_head_rows(get("v"), H, V, Vp, hp), _pad_head_rows(get("f"), H, D, Dp, hp)]
+
+
+def _pack_latent(w, p, m: LatentAttentionMixer, get, hp: int, dtype, device):
+    H, D, R, V, Q, C = m.heads, m.dim, m.rot_dim, m.vdim, m.q_rank, m.kv_rank
+    Dp, Rp, Vp, Qp, Cp = m.dim_p, m.rot_p, m.vdim_p, m.q_rank_p, m.kv_rank_p
+    uq = get("uq").reshape(H, D + R, Q)
+    q = torch.zeros((H, Dp + Rp, Qp), dtype=uq.dtype, device=device)
+    q[:, :D, :Q] = uq[:, :D]
+    q[:, Dp: Dp + R, :Q] = uq[:, D:]
+    w[f"{p}/mix/uq"] = q.reshape(H * (Dp + Rp), Qp).to(dtype)
+    k, v = _pad_head_rows(get("uk"), H, D, Dp, Cp), _pad_head_rows(get("uv"), H, V, Vp, Cp)
+    w[f"{p}/mix/ukv"] = torch.cat([k, v]).to(dtype)                        # rows: keys of all heads, values of all heads
+    w[f"{p}/mix/uv"] = w[f"{p}/mix/ukv"][H * Dp:].view(H, Vp, Cp)
+    w[f"{p}/mix/uk_t"] = k.reshape(H, Dp, Cp).transpose(1, 2).contiguous().to(dtype)   # takes a query to the latent space
+    w[f"{p}/mix/q_norm"] = _pad_head_vec(get("dq_norm"), 1, Q, Qp)
+    w[f"{p}/mix/kv_norm"] = _pad_head_vec(get("dkv_norm"), 1, C, Cp)
+    w[f"{p}/mix/freq"] = torch.tensor([m.rot_base ** (-2.0 * i / R) for i in range(R // 2)], dtype=torch.float64, device=device)
+    if m.sink:
+        w[f"{p}/mix/sink"] = get("sink").float().contiguous()
+    dkv = get("dkv")
+    return [_pad2(get("dq"), Qp, hp), _pad2(dkv[:C], Cp, hp), _pad2(dkv[C:], Rp, hp)]
+
+
 def pack_weights(cfg: LayeredConfig, get, dtype: torch.dtype = torch.bfloat16, device="cpu") -> Dict[str, torch.Tensor]:
     """Fused, padded weights of the forward pass.  `get(layer, name)` returns a design's tensor by its role (layer -1:
-    the model's own): embed, head, final_norm; norm1, norm2; q, k, v, o, g, q_bias, k_bias, v_bias, q_norm, k_norm,
-    talk; i, f, i_bias, f_bias, norm; up, up_bias, down, down_bias, act."""
-    hp = cfg.hidden_p
+    the model's own): embed, head, final_norm, loop_in, loop_step; norm1, norm1b, norm2, norm2b, conv; the mixers' (see
+    the _pack functions) and o; up, up_bias, down, down_bias, act."""
+    hp, wide = cfg.hidden_p, cfg.residual == "sandwich"
     w: Dict[str, torch.Tensor] = {}
 
     def g(layer, name):
         return get(layer, name).to(device)
 
-    def f32(layer, name):
-        return g(layer, name).float().contiguous()
-    w["text/embed"] = _pad2(g(-1, "embed"), cfg.vocab, hp).to(dtype)
-    w["text/lm_head"] = _pad2(g(-1, "head"), cfg.vocab_p, hp).to(dtype)
-    w["text/final_norm"] = f32(-1, "final_norm").reshape(1)
+    def norm(layer, name):
+        return _pad_head_vec(g(layer, name), 1, cfg.hidden, hp) if wide else g(layer, name).float().contiguous().reshape(1)
+    if cfg.tie_head:
+        w["text/embed"] = w["text/lm_head"] = _pad2(g(-1, "embed"), cfg.vocab_p, hp).to(dtype)
+    else:
+        w["text/embed"] = _pad2(g(-1, "embed"), cfg.vocab, hp).to(dtype)
+        w["text/lm_head"] = _pad2(g(-1, "head"), cfg.vocab_p, hp).to(dtype)
+    w["text/final_norm"] = norm(-1, "final_norm")
+    if cfg.loop is not None:
+        w["text/loop/in_proj"] = _pad_head_cols(g(-1, "loop_in"), 2, cfg.hidden, hp, hp).to(dtype)
+        w["text/loop/step"] = torch.stack([_pad_head_vec(v, 1, cfg.hidden, hp) for v in g(-1, "loop_step")])
     for i, spec in enumerate(cfg.layers):
         m, p = spec.mixer, f"text/layers/{i}"
-        D, V, Dp, Vp, H = m.dim, m.vdim, m.dim_p, m.vdim_p, m.heads
-        w[f"{p}/norm1"] = f32(i, "norm1").reshape(1)
+
+        def mix(name, i=i):
+            return g(i, name)
+        w[f"{p}/norm1"] = norm(i, "norm1")
+        if wide:
+            w[f"{p}/norm1b"] = norm(i, "norm1b")
+        if cfg.conv_taps:
+            w[f"{p}/conv"] = torch.stack([_pad_head_vec(v, 1, cfg.hidden, hp) for v in g(i, "conv").t()])      # [taps, width]
         n_out = pad_to(m.main_cols + m.gate_cols, 2)
-        bias = torch.zeros(n_out, dtype=torch.float32, device=device)
         if m.kind == "attention":
-            G = m.kv_heads
-            rows = [_pad_head_rows(g(i, "q"), H, D, Dp, hp), _pad_head_rows(g(i, "k"), G, D, Dp, hp),
-                    _pad_head_rows(g(i, "v"), G, V, Vp, hp)]
-            if m.head_gate:
-                rows.append(_pad2(g(i, "g"), H, hp))
-            if m.bias:
-                b = torch.cat([_pad_head_vec(g(i, "q_bias"), H, D, Dp), _pad_head_vec(g(i, "k_bias"), G, D, Dp),
-                               _pad_head_vec(g(i, "v_bias"), G, V, Vp)])
-                bias[: b.numel()] = b
-            if m.qk_norm:
-                w[f"{p}/mix/q_norm"] = _pad_head_vec(g(i, "q_norm"), 1, D, Dp)
-                w[f"{p}/mix/k_norm"] = _pad_head_vec(g(i, "k_norm"), 1, D, Dp)
-            mix = g(i, "talk").double() if m.head_mixing else torch.eye(H, dtype=torch.float64, device=device)
-            if m.head_mixing:
-                w[f"{p}/mix/heads"] = mix.float().contiguous()
-            if m.distance_bias:
-                # mixing is linear: the bias taken off before it is (mix @ slope) taken off after it
-                w[f"{p}/mix/slope"] = (mix @ distance_slopes(H).to(device)).float().contiguous()
+            rows = _pack_attention(w, p, m, mix, n_out, hp, device)
+        elif m.kind == "latent_attention":
+            rows = _pack_latent(w, p, m, mix, hp, dtype, device)
+        elif m.kind == "hgrn2":
+            rows = _pack_gated_memory(w, p, m, mix, n_out, hp, device)
         else:
-            rows = [_pad_head_rows(g(i, "q"), H, D, Dp, hp), _pad_head_rows(g(i, "k"), H, D, Dp, hp),
-                    _pad_head_rows(g(i, "v"), H, V, Vp, hp), _pad_head_rows(g(i, "g"), H, V, Vp, hp),
-                    _pad2(g(i, "i"), H, hp), _pad2(g(i, "f"), H, hp)]
-            bias[m.main_cols: m.main_cols + H] = g(i, "i_bias").float()
-            bias[m.main_cols + H: m.main_cols + 2 * H] = g(i, "f_bias").float()
-            w[f"{p}/mix/norm"] = _pad_head_vec(g(i, "norm"), H, V, Vp)
+            rows = _pack_matrix_memory(w, p, m, mix, n_out, hp, device)
         w[f"{p}/mix/in_proj"] = _pad2(torch.cat(rows), n_out, hp).to(dtype)
-        w[f"{p}/mix/in_bias"] = bias
-        w[f"{p}/mix/out_proj"] = _pad_head_cols(g(i, "o"), H, V, Vp, hp).to(dtype)
+        w[f"{p}/mix/out_proj"] = _pad_head_cols(g(i, "o"), m.heads, m.vdim, m.vdim_p, hp).to(dtype)
         if spec.mlp is not None:
             fp = pad_to(spec.mlp.ff, 8)
-            w[f"{p}/norm2"] = f32(i, "norm2").reshape(1)
+            w[f"{p}/norm2"] = norm(i, "norm2")
+            if wide:
+                w[f"{p}/norm2b"] = norm(i, "norm2b")
             w[f"{p}/mlp/up"] = _pad2(g(i, "up"), fp, hp).to(dtype)
             w[f"{p}/mlp/down"] = _pad2(g(i, "down"), hp, fp).to(dtype)
             if spec.mlp.bias:
                 w[f"{p}/mlp/up_bias"] = _pad_head_vec(g(i, "up_bias"), 1, spec.mlp.ff, fp)
                 w[f"{p}/mlp/down_bias"] = _pad_head_vec(g(i, "down_bias"), 1, cfg.hidden, hp)
-            if spec.mlp.activation != "xielu":
+            if spec.mlp.activation not in ACTIVATIONS:
                 raise ValueError(f"layer {i}: unknown feed-forward activation '{spec.mlp.activation}'")
-            a = torch.nn.functional.softplus(g(i, "act").double())
-            w[f"{p}/mlp/act"] = torch.stack([a[0], 0.5 + a[1]]).float().contiguous()
+            if spec.mlp.activation == "xielu":
+                a = torch.nn.functional.softplus(g(i, "act").double())
+                w[f"{p}/mlp/act"] = torch.stack([a[0], 0.5 + a[1]]).float().contiguous()
     return w
 
 
@@ -131,23 +206,45 @@ class LayeredWorkspace:
         T, dev, f32 = max_tokens, device, torch.float32
         mixers = [l.mixer for l in cfg.layers]
         attn = [m for m in mixers if m.kind == "attention"]
+        latent = [m for m in mixers if m.kind == "latent_attention"]
+
+        def rows(cols, dt=dtype):
+            return torch.zeros((T, cols), dtype=dt, device=dev)
+
+        def widest(values, default, mult=64):
+            return pad_to(max(values, default=default), mult)
         self.max_tokens, self.max_logit_rows = T, max_logit_rows
-        self.x = torch.zeros((T, cfg.hidden_p), dtype=f32, device=dev)      # residual stream
-        self.xa = torch.zeros((T, cfg.hidden_p), dtype=dtype, device=dev)   # its copy in the activation type
-        self.delta = torch.zeros((T, cfg.hidden_p), dtype=f32, device=dev)  # output of the running sublayer
-        self.proj = torch.zeros((T, pad_to(max(m.main_cols for m in mixers), 64)), dtype=dtype, device=dev)
-        self.gates = torch.zeros((T, pad_to(max(2, max(m.gate_cols for m in mixers)), 4)), dtype=f32, device=dev)
-        self.mix = torch.zeros((T, pad_to(max(m.out_cols for m in mixers), 64)), dtype=dtype, device=dev)
-        self.q = torch.zeros((T, max((m.heads * m.dim_p for m in attn), default=16)), dtype=dtype, device=dev)
-        self.act = torch.zeros((T, pad_to(max((l.mlp.ff for l in cfg.layers if l.mlp is not None), default=8), 64)),
-                               dtype=dtype, device=dev)
+        self.x = rows(cfg.hidden_p, f32)           # residual stream
+        self.x2 = rows(cfg.hidden_p, f32) if cfg.conv_taps else self.x     # its other copy: a convolution reads rows that its step replaces
+        self.xa = rows(cfg.hidden_p)               # what the next GEMM reads, in the activation type
+        self.pair = rows(2 * cfg.hidden_p) if cfg.loop is not None else None   # [x, embedding output] of a pass's entry
+        self.delta = rows(cfg.hidden_p, f32)       # output of the running sublayer
+        self.proj = rows(widest((m.main_cols for m in mixers), 64))
+        self.gates = rows(widest((m.gate_cols for m in mixers), 2, 4), f32)
+        self.mix = rows(widest((m.out_cols for m in mixers), 64))
+        self.q = rows(max([m.heads * m.dim_p for m in attn] + [m.q_cols for m in latent], default=16))
+        self.act = rows(widest((l.mlp.ff for l in cfg.layers if l.mlp is not None), 8))
+        if latent:
+            self.q_latent = rows(max(m.q_rank_p for m in latent))
+            self.q_abs = rows(max(m.heads * m.kv_rank_p for m in latent))     # absorbed queries, head by head
+            self.o_latent = rows(max(m.heads * m.kv_rank_p for m in latent))  # attended latents
         # split-KV partials: (query token x split) rows of decode-sized steps
         self.split_rows = split_rows
-        self.part_o = torch.empty(split_rows * max((m.out_cols for m in attn), default=0), dtype=f32, device=dev)
-        self.part_ml = torch.empty(split_rows * max((m.heads for m in attn), default=0) * 2, dtype=f32, device=dev)
+        self.part_o = torch.empty(split_rows * max([m.out_cols for m in attn] + [m.heads * m.kv_rank_p for m in latent], default=0),
+                                  dtype=f32, device=dev)
+        self.part_ml = torch.empty(split_rows * max((m.heads for m in attn + latent), default=0) * 2, dtype=f32, device=dev)
         self.logits = torch.zeros((max_logit_rows, cfg.vocab_p), dtype=f32, device=dev)
         self.head_in = torch.zeros((max_logit_rows, cfg.hidden_p), dtype=dtype, device=dev)
         self.next_ids = torch.zeros((max_logit_rows,), dtype=torch.int32, device=dev)
+
+
+def native_subset(cfg: LayeredConfig) -> str:
+    """The stand-alone library (see `_build.SUBSETS`) that has the mixers of this configuration."""
+    kinds = {l.mixer.kind for l in cfg.layers}
+    for name, have in (("head_mix", {"attention", "mlstm"}), ("latent", {"latent_attention", "hgrn2"})):
+        if kinds <= have:
+            return name
+    return "layered"
 
 
 class LayeredModel:
@@ -156,7 +253,7 @@ class LayeredModel:
     def __init__(self, cfg: LayeredConfig, weights: Dict[str, torch.Tensor], device, pdl: bool = False):
         self.cfg, self.w = cfg, weights
         self.device = torch.device(device)
-        self._raw_ops = load_native(subset="layered")
+        self._raw_ops = load_native(subset=native_subset(cfg))
         self.ops = LaunchCounter(self._raw_ops)
         self.status = StatusWord(self.device)
         self.dtype = weights["text/embed"].dtype
@@ -168,9 +265,10 @@ class LayeredModel:
         self.k_row_scale: Dict[int, torch.Tensor] = {}
         self.l2_prefetch = True
         self.prefill_kernels = True     # False: the token-by-token kernels for every size (tests)
-        self.layer_hook = None          # called as hook(layer, x[:T]) after every layer (tests, debugging)
-        self._attn_idx = {l: i for i, l in enumerate(cfg.attn_layers)}
-        self._state_idx = {l: i for i, l in enumerate(cfg.state_layers)}
+        self.layer_hook = None          # called as hook(layer, x[:T]) after every layer run (tests, debugging)
+        self._runs = cfg.runs
+        self._attn_idx = {r: i for i, r in enumerate(cfg.attn_layers)}
+        self._state_idx = {r: i for i, r in enumerate(cfg.state_layers)}
         self._scratch: Dict[str, torch.Tensor] = {}
         self._keep: List[torch.Tensor] = []
 
@@ -199,15 +297,15 @@ class LayeredModel:
         """Fused input projection: [T, main_cols] in the activation type and [T, gate_cols] in fp32."""
         proj = ws.proj[:T, : m.main_cols]
         gates = ws.gates[:T] if m.gate_cols else None
-        self._gemm(ws.xa[:T], self.w[f"{p}/mix/in_proj"], self.w[f"{p}/mix/in_bias"], proj, gates, m.main_cols,
+        self._gemm(ws.xa[:T], self.w[f"{p}/mix/in_proj"], self.w.get(f"{p}/mix/in_bias"), proj, gates, m.main_cols if gates is not None else 0,
                    prefetch=self.w[f"{p}/mix/out_proj"])
         return proj, gates
 
     # ------------------------------------------------------------------ mixers
-    def _attention(self, ws, b: StepBatch, kv, layer: int, T: int, p: str, m: AttentionMixer):
+    def _attention(self, ws, b: StepBatch, kv, run: int, T: int, p: str, m: AttentionMixer):
         ops, w = self.ops, self.w
         proj, gates = self._in_proj(ws, T, p, m)
-        planes = kv.layers[self._attn_idx[layer]]
+        planes = kv.layers[self._attn_idx[run]]
         k_pages, v_pages = planes.typed(self.dtype)
         H, G, Dp, Vp = m.heads, m.kv_heads, m.dim_p, m.vdim_p
         q = ws.q[:T, : H * Dp]
@@ -236,48 +334,143 @@ class LayeredModel:
         split = max(64, pad_to(-(-keys // want), 32))
         return split, -(-keys // split)
 
-    def _matrix_memory(self, ws, b: StepBatch, states, layer: int, T: int, p: str, m: MatrixMemoryMixer,
-                       write_state: bool):
+    def _head_gemm(self, x: torch.Tensor, x_step: int, w: torch.Tensor, out: torch.Tensor) -> None:
+        """out[t, h * N + n] = sum_k w[h, n, k] x[t, h * x_step + k]"""
+        H, N, K = w.shape
+        for h in range(H):
+            self._gemm(x[:, h * x_step: h * x_step + K], w[h], None, out[:, h * N: (h + 1) * N])
+
+    def _latent_attention(self, ws, b: StepBatch, kv, run: int, T: int, p: str, m: LatentAttentionMixer):
+        ops, w, eps = self.ops, self.w, self.cfg.rms_eps
+        proj, _ = self._in_proj(ws, T, p, m)
+        pages, _ = kv.layers[self._attn_idx[run]].typed(self.dtype)
+        c_q, q = ws.q_latent[:T, : m.q_rank_p], ws.q[:T, : m.q_cols]
+        freq, sink = w[f"{p}/mix/freq"], w.get(f"{p}/mix/sink")
+        ops.latent_prep(proj, m.q_rank, m.kv_rank, m.rot_dim, w[f"{p}/mix/q_norm"], w[f"{p}/mix/kv_norm"], eps, freq, b.table_row,
+                        b.cache_pos, kv.table, c_q, pages, self.pdl)
+        self._gemm(c_q, w[f"{p}/mix/uq"], None, q, prefetch=w[f"{p}/mix/uk_t"])
+        out = ws.mix[:T, : m.out_cols]
+        q_abs, o_latent = ws.q_abs[:T, : m.heads * m.kv_rank_p], ws.o_latent[:T, : m.heads * m.kv_rank_p]
+        self._head_gemm(q, m.dim_p + m.rot_p, w[f"{p}/mix/uk_t"], q_abs)
+        ops.latent_token_attention(q_abs, q, pages, kv.table, b.table_row, b.kv_len, m.heads, m.rot_dim, m.scale, freq, sink,
+                                   o_latent, self.pdl)
+        self._head_gemm(o_latent, m.kv_rank_p, w[f"{p}/mix/uv"], out)
+        return out
+
+    def _chunk_workspace(self, b: StepBatch, T: int, kind: str, m) -> "torch.Tensor | None":
+        """Scratch of a memory's chunked prefill kernels; None when the step takes the token-by-token kernel."""
+        supported, size = getattr(self._raw_ops, f"{kind}_chunked_supported"), getattr(self._raw_ops, f"{kind}_chunked_workspace_bytes")
+        if self.f32 or not self.prefill_kernels or b.max_seq_tokens < PREFILL_MIN_TOKENS or not supported(m.dim_p, m.vdim_p):
+            return None
+        return self._grown("chunks", int(size(T, b.n_seqs, m.heads, m.dim_p, m.vdim_p)))
+
+    def _matrix_memory(self, ws, b: StepBatch, states, run: int, T: int, p: str, m: MatrixMemoryMixer, write_state: bool):
         proj, gates = self._in_proj(ws, T, p, m)
-        S, n, mx = states.layers[self._state_idx[layer]]
+        S, n, mx = states.layers[self._state_idx[run]][-3:]
         H, Dp, Vp = m.heads, m.dim_p, m.vdim_p
-        chunk_ws = None
-        if (not self.f32 and self.prefill_kernels and b.max_seq_tokens >= PREFILL_MIN_TOKENS
-                and self._raw_ops.mlstm_chunked_supported(Dp, Vp)):
-            chunk_ws = self._grown("chunks", int(self._raw_ops.mlstm_chunked_workspace_bytes(T, b.n_seqs, H, Dp, Vp)))
-            self.ops.count += 3
+        chunk_ws = self._chunk_workspace(b, T, "mlstm", m)
+        self.ops.count += 3 if chunk_ws is not None else 0
         out = ws.mix[:T, : H * Vp]
         self.ops.mlstm(proj, 0, H * Dp, 2 * H * Dp, H * (2 * Dp + Vp), gates, 0, H, m.vdim, m.dim ** -0.5, m.gate_cap,
                        self.cfg.rms_eps, self.w[f"{p}/mix/norm"], b.cu_seqlens, b.state_slot, S, n, mx, out, write_state,
                        chunk_ws, self.pdl, b.one_token_per_seq)
         return out
 
+    def _gated_memory(self, ws, b: StepBatch, states, run: int, T: int, p: str, m: GatedMemoryMixer, write_state: bool):
+        proj, gates = self._in_proj(ws, T, p, m)
+        S = states.layers[self._state_idx[run]][-1]
+        chunk_ws = self._chunk_workspace(b, T, "gated", m)
+        self.ops.count += 2 if chunk_ws is not None else 0
+        out = ws.mix[:T, : m.out_cols]
+        self.ops.gated_memory(proj, 0, m.heads * m.dim_p, gates, self.w[f"{p}/mix/lower"], m.vdim, self.cfg.rms_eps,
+                              self.w[f"{p}/mix/norm"], b.cu_seqlens, b.state_slot, S, out, write_state, chunk_ws, self.pdl,
+                              b.one_token_per_seq)
+        return out
+
+    def _mixer(self, ws, b: StepBatch, kv, states, run: int, T: int, p: str, m, write_state: bool) -> torch.Tensor:
+        if m.kind in ATTENTION_KINDS:
+            fn = self._attention if m.kind == "attention" else self._latent_attention
+            return fn(ws, b, kv, run, T, p, m)
+        fn = self._gated_memory if m.kind == "hgrn2" else self._matrix_memory
+        return fn(ws, b, states, run, T, p, m, write_state)
+
+    def _feed_forward(self, ws, T: int, p: str, spec, prefetch) -> None:
+        w, up, down = self.w, self.w[f"{p}/mlp/up"], self.w[f"{p}/mlp/down"]
+        act = ws.act[:T, : up.shape[0]]
+        self._gemm(ws.xa[:T], up, w.get(f"{p}/mlp/up_bias"), act, act=ACTIVATIONS[spec.activation], act_params=w.get(f"{p}/mlp/act"),
+                   prefetch=down)
+        self._gemm(act, down, w.get(f"{p}/mlp/down_bias"), out32=ws.delta[:T], prefetch=prefetch)
+
     # ------------------------------------------------------------------ forward
     def forward_hidden(self, ws: LayeredWorkspace, b: StepBatch, kv, states, write_state: bool = True) -> torch.Tensor:
         """Runs all layers; returns the final-normed hidden states [T, hidden (padded)]."""
-        cfg, ops, w = self.cfg, self.ops, self.w
-        T = b.n_tokens
-        if T > ws.max_tokens:
-            raise ValueError(f"step of {T} tokens exceeds the workspace ({ws.max_tokens})")
+        if b.n_tokens > ws.max_tokens:
+            raise ValueError(f"step of {b.n_tokens} tokens exceeds the workspace ({ws.max_tokens})")
+        run = self._forward_sandwich if self.cfg.residual == "sandwich" else self._forward_post_sum
+        return run(ws, b, kv, states, write_state)
+
+    def _next_weights(self, run: int):
+        """What the GEMM after the last one of `run` reads (an L2 hint)."""
+        if run + 1 == len(self._runs):
+            return self.w["text/lm_head"]
+        layer, opens = self._runs[run + 1]
+        return self.w["text/loop/in_proj"] if opens >= 0 else self.w[f"text/layers/{layer}/mix/in_proj"]
+
+    def _forward_post_sum(self, ws, b: StepBatch, kv, states, write_state: bool) -> torch.Tensor:
+        cfg, ops, w, T = self.cfg, self.ops, self.w, b.n_tokens
         x, xa, delta = ws.x[:T], ws.xa[:T], ws.delta[:T]
-        ops.embed_rows32(b.ids, w["text/embed"], x, xa, self.pdl)
-        for layer, spec in enumerate(cfg.layers):
-            p, m = f"text/layers/{layer}", spec.mixer
-            mix = (self._attention(ws, b, kv, layer, T, p, m) if m.kind == "attention" else
-                   self._matrix_memory(ws, b, states, layer, T, p, m, write_state))
-            last = w["text/final_norm"] if layer + 1 == cfg.n_layers else None
-            nxt = w.get(f"text/layers/{layer + 1}/mix/in_proj", w["text/lm_head"])
+        ops.embed_rows32(b.ids, w["text/embed"], x, xa, cfg.embed_scale, self.pdl)
+        for run, (layer, _) in enumerate(self._runs):
+            spec, p = cfg.layers[layer], f"text/layers/{layer}"
+            mix = self._mixer(ws, b, kv, states, run, T, p, spec.mixer, write_state)
+            last, nxt = w["text/final_norm"] if run + 1 == len(self._runs) else None, self._next_weights(run)
             self._gemm(mix, w[f"{p}/mix/out_proj"], None, out32=delta, prefetch=w.get(f"{p}/mlp/up", nxt))
             ops.post_norm_rows(x, delta, xa, cfg.hidden, cfg.residual_alpha, cfg.rms_eps, w[f"{p}/norm1"],
                                last if spec.mlp is None else None, self.pdl)
             if spec.mlp is not None:
-                up, down = w[f"{p}/mlp/up"], w[f"{p}/mlp/down"]
-                act = ws.act[:T, : up.shape[0]]
-                self._gemm(xa, up, w.get(f"{p}/mlp/up_bias"), act, act=ACT_XIELU, act_params=w[f"{p}/mlp/act"], prefetch=down)
-                self._gemm(act, down, w.get(f"{p}/mlp/down_bias"), out32=delta, prefetch=nxt)
+                self._feed_forward(ws, T, p, spec.mlp, nxt)
                 ops.post_norm_rows(x, delta, xa, cfg.hidden, cfg.residual_alpha, cfg.rms_eps, w[f"{p}/norm2"], last, self.pdl)
             if self.layer_hook is not None:
-                self.layer_hook(layer, x[:, : cfg.hidden])
+                self.layer_hook(run, x[:, : cfg.hidden])
+        return xa
+
+    def _forward_sandwich(self, ws, b: StepBatch, kv, states, write_state: bool) -> torch.Tensor:
+        """The residual update of a sublayer waits for the row step in front of the next one (`sandwich_rows`)."""
+        cfg, ops, w, T, hp = self.cfg, self.ops, self.w, b.n_tokens, self.cfg.hidden_p
+        x, other, xa, delta = ws.x[:T], ws.x2[:T], ws.xa[:T], ws.delta[:T]
+        post = None                   # weights of the norm of the sublayer output that waits in `delta`
+
+        def rows(w_next, out, conv_run=-1, layer=0):
+            nonlocal x, other, post
+            conv = (None, None, None, None)
+            if conv_run >= 0 and cfg.conv_taps:
+                state = states.layers[self._state_idx[conv_run]][0] if cfg.conv_taps > 1 else None
+                conv = (w[f"text/layers/{layer}/conv"], state, b.cu_seqlens, b.state_slot)
+            dst = other if conv[0] is not None and post is not None and b.max_seq_tokens > 1 else x
+            ops.sandwich_rows(x, dst, None if post is None else delta, post, w_next, out, cfg.hidden, cfg.norm_groups, cfg.residual_mult,
+                              cfg.rms_eps, *conv, b.max_seq_tokens, write_state, self.pdl)
+            if dst is other:
+                x, other = other, x
+            post = None
+        ops.embed_rows32(b.ids, w["text/embed"], x, ws.pair[:T, hp:] if cfg.loop is not None else xa, cfg.embed_scale, self.pdl)
+        for run, (layer, opens) in enumerate(self._runs):
+            spec, p = cfg.layers[layer], f"text/layers/{layer}"
+            if opens >= 0:
+                rows(None, ws.pair[:T, :hp])
+                self._gemm(ws.pair[:T], w["text/loop/in_proj"], w["text/loop/step"][opens], out32=x, prefetch=w[f"{p}/mix/in_proj"])
+            rows(w[f"{p}/norm1"], xa, run, layer)
+            mix = self._mixer(ws, b, kv, states, run, T, p, spec.mixer, write_state)
+            nxt = self._next_weights(run)
+            self._gemm(mix, w[f"{p}/mix/out_proj"], None, out32=delta, prefetch=w.get(f"{p}/mlp/up", nxt))
+            post = w[f"{p}/norm1b"]
+            if spec.mlp is not None:
+                rows(w[f"{p}/norm2"], xa)
+                self._feed_forward(ws, T, p, spec.mlp, nxt)
+                post = w[f"{p}/norm2b"]
+            if self.layer_hook is not None:
+                rows(None, xa)
+                self.layer_hook(run, x[:, : cfg.hidden])
+        rows(w["text/final_norm"], xa)
         return xa
 
     def head(self, ws: LayeredWorkspace, head_in: torch.Tensor) -> torch.Tensor:

@@ -1,8 +1,10 @@
 """Description of decoders given as a list of layers (read by `models/layered.py`, which runs them).
 
-A layer is a mixer (head-mixing attention or matrix memory) and an optional feed-forward; every size and constant is a
-field, and so is which mechanisms a mixer has.  No torch here: the package table and the host diagnostics read these
-descriptions too."""
+A layer is a mixer (head-mixing attention, latent attention, matrix memory or gated linear memory) and an optional
+feed-forward; every size and constant is a field, and so is which mechanisms a mixer has.  The model's own fields say how
+a sublayer meets the residual stream, what precedes a mixer, and which layers run several times.  Cache and state belong
+to layer RUNS: a layer that runs twice has two of each.  No torch here: the package table and the host diagnostics read
+these descriptions too."""
 from __future__ import annotations
 
 import math
@@ -88,16 +90,121 @@ class MatrixMemoryMixer:
 
 
 @dataclass(frozen=True)
+class LatentAttentionMixer:
+    """Queries through a normed latent; keys and values out of one normed latent row per token, plus one rotated key part
+    that all heads share.  The cache keeps one row per token: [latent, rotated part]."""
+    heads: int
+    dim: int                      # query / key width per head without rotation
+    rot_dim: int                  # rotated query / key width per head
+    vdim: int
+    q_rank: int
+    kv_rank: int
+    scale: float
+    rot_base: float
+    sink: bool = True             # one learned score per head in the softmax denominator
+
+    kind = "latent_attention"
+    kv_heads = 1
+    window = 0
+
+    @property
+    def dim_p(self) -> int:
+        return pad_to(self.dim, 16)
+
+    @property
+    def rot_p(self) -> int:
+        return pad_to(self.rot_dim, 16)
+
+    @property
+    def vdim_p(self) -> int:
+        return pad_to(self.vdim, 16)
+
+    @property
+    def q_rank_p(self) -> int:
+        return pad_to(self.q_rank, 16)
+
+    @property
+    def kv_rank_p(self) -> int:
+        return pad_to(self.kv_rank, 16)
+
+    @property
+    def row_cols(self) -> int:
+        """Width of a cached row."""
+        return self.kv_rank_p + self.rot_p
+
+    @property
+    def main_cols(self) -> int:
+        """Columns of the fused input projection: [query latent, key / value latent, rotated key part]."""
+        return self.q_rank_p + self.row_cols
+
+    gate_cols = 0
+
+    @property
+    def q_cols(self) -> int:
+        """Query columns, head by head [unrotated, rotated]."""
+        return self.heads * (self.dim_p + self.rot_p)
+
+    @property
+    def out_cols(self) -> int:
+        return self.heads * self.vdim_p
+
+
+@dataclass(frozen=True)
+class GatedMemoryMixer:
+    """Linear attention with a forget gate per head and channel, f = lower + (1 - lower) sigmoid(raw), whose complement
+    takes the place of the key (HGRN2)."""
+    heads: int
+    dim: int
+    vdim: int
+
+    kind = "hgrn2"
+
+    @property
+    def dim_p(self) -> int:
+        return pad_to(self.dim, 16)
+
+    @property
+    def vdim_p(self) -> int:
+        return pad_to(self.vdim, 16)
+
+    @property
+    def main_cols(self) -> int:
+        """[q, v]"""
+        return self.heads * (self.dim_p + self.vdim_p)
+
+    @property
+    def gate_cols(self) -> int:
+        """Raw forget gates, fp32."""
+        return self.heads * self.dim_p
+
+    @property
+    def out_cols(self) -> int:
+        return self.heads * self.vdim_p
+
+
+@dataclass(frozen=True)
 class DenseMlp:
     ff: int
-    activation: str = "xielu"     # two learned numbers per layer
+    activation: str = "xielu"     # xielu (two learned numbers per layer) | relu2 (square of relu)
     bias: bool = False
 
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: Union[AttentionMixer, MatrixMemoryMixer]
+    mixer: Union[AttentionMixer, LatentAttentionMixer, MatrixMemoryMixer, GatedMemoryMixer]
     mlp: Optional[DenseMlp] = None
+
+
+@dataclass(frozen=True)
+class LoopSpec:
+    """Layers start .. stop - 1 run `times` times in a row.  Every pass opens with x <- in_proj [x; x0] + step[pass], x0
+    the embedding output."""
+    start: int
+    stop: int
+    times: int
+
+
+ATTENTION_KINDS = ("attention", "latent_attention")
 
 
 @dataclass(frozen=True)
@@ -107,9 +214,16 @@ class LayeredConfig:
     vocab: int
     layers: Tuple[LayerSpec, ...]
     rms_eps: float
-    residual_alpha: float         # x <- norm(residual_alpha * x + f(x))
+    residual_alpha: float         # post_sum: x <- norm(residual_alpha * x + f(x))
     max_context: int = 131072
     architecture: str = ""        # name of the design that maps checkpoints onto this description
+    residual: str = "post_sum"    # post_sum | sandwich: x <- x + residual_mult * norm(f(norm(x)))
+    residual_mult: float = 1.0    # sandwich
+    norm_groups: int = 1          # sandwich: equal parts of a row that are normed by themselves, one weight per column
+    conv_taps: int = 0            # h <- h + causal convolution of h before every mixer, this many taps (0: none)
+    embed_scale: float = 1.0
+    tie_head: bool = False        # logits from the embedding table (without its scale)
+    loop: Optional[LoopSpec] = None
 
     moe = None
     mtp_layers = 0
@@ -128,57 +242,94 @@ class LayeredConfig:
         return pad_to(self.vocab, 8)
 
     @property
+    def runs(self) -> List[Tuple[int, int]]:
+        """Layer runs in order: (layer, pass it opens or -1)."""
+        lp, n = self.loop, len(self.layers)
+        if lp is None:
+            return [(i, -1) for i in range(n)]
+        looped = [(i, t if i == lp.start else -1) for t in range(lp.times) for i in range(lp.start, lp.stop)]
+        return [(i, -1) for i in range(lp.start)] + looped + [(i, -1) for i in range(lp.stop, n)]
+
+    def mixer_of(self, run: int):
+        return self.layers[self.runs[run][0]].mixer
+
+    @property
     def attn_layers(self) -> List[int]:
-        return [i for i, l in enumerate(self.layers) if l.mixer.kind == "attention"]
+        """Layer runs that have a cache (without a loop a run is a layer)."""
+        return [r for r, (i, _) in enumerate(self.runs) if self.layers[i].mixer.kind in ATTENTION_KINDS]
 
     @property
     def state_layers(self) -> List[int]:
-        return [i for i, l in enumerate(self.layers) if l.mixer.kind == "mlstm"]
+        """Layer runs that have recurrent state: a memory, or the inputs that a convolution looks back on."""
+        return [r for r, (i, _) in enumerate(self.runs)
+                if self.conv_taps > 1 or self.layers[i].mixer.kind not in ATTENTION_KINDS]
 
     @property
     def n_kv_heads(self) -> int:
-        return max((self.layers[i].mixer.kv_heads for i in self.attn_layers), default=0)
+        return max((self.mixer_of(r).kv_heads for r in self.attn_layers), default=0)
 
     @property
     def head_dim(self) -> int:
-        return max((self.layers[i].mixer.dim for i in self.attn_layers), default=0)
+        return max((self.mixer_of(r).dim for r in self.attn_layers), default=0)
 
     @property
     def kv_geometry(self) -> List[Tuple[int, int, int]]:
-        """Per attention layer: kv heads, key width, value width of a cache row (padded)."""
-        return [(m.kv_heads, m.dim_p, m.vdim_p) for m in (self.layers[i].mixer for i in self.attn_layers)]
+        """Per attention run: kv heads, key width, value width of a cache row (padded).  A latent row has no separate
+        values."""
+        ms = [self.mixer_of(r) for r in self.attn_layers]
+        return [(1, m.row_cols, 0) if m.kind == "latent_attention" else (m.kv_heads, m.dim_p, m.vdim_p) for m in ms]
 
     @property
     def cache_window(self) -> int:
         """Keys that any layer still looks back on: the widest window, 0 when some layer sees all of the past."""
-        w = [self.layers[i].mixer.window for i in self.attn_layers]
+        w = [self.mixer_of(r).window for r in self.attn_layers]
         return max(w) if w and min(w) > 0 else 0
 
     def state_shapes(self) -> List[List[tuple]]:
-        """Per recurrent layer: shapes (without the slot) of its fp32 state arrays: S, n, m."""
+        """Per run in `state_layers`: shapes (without the slot) of its fp32 state arrays: the convolution's last inputs
+        (oldest first) when there are any, then the memory: S, n, m (matrix memory) or S (gated memory)."""
         out = []
-        for i in self.state_layers:
-            m = self.layers[i].mixer
-            out.append([(m.heads, m.dim_p, m.vdim_p), (m.heads, m.dim_p), (m.heads,)])
+        for r in self.state_layers:
+            m, arrays = self.mixer_of(r), []
+            if self.conv_taps > 1:
+                arrays.append((self.conv_taps - 1, self.hidden_p))
+            if m.kind not in ATTENTION_KINDS:
+                arrays.append((m.heads, m.dim_p, m.vdim_p))
+            if m.kind == "mlstm":
+                arrays += [(m.heads, m.dim_p), (m.heads,)]
+            out.append(arrays)
         return out
 
     def state_bytes_per_slot(self) -> int:
         return sum(4 * math.prod(shape) for layer in self.state_shapes() for shape in layer)
 
     def param_count(self) -> int:
-        n = 2 * self.vocab * self.hidden + 1
+        h, wide = self.hidden, self.residual == "sandwich"
+        norm = h if wide else 1                      # weights of one norm
+        n = (1 if self.tie_head else 2) * self.vocab * h + norm
+        if self.loop is not None:
+            n += 2 * h * h + self.loop.times * h
         for l in self.layers:
             m = l.mixer
+            n += (2 if wide else 1) * norm + self.conv_taps * h + h * m.heads * m.vdim
             if m.kind == "attention":
                 rows = (m.heads + m.kv_heads) * m.dim + m.kv_heads * m.vdim + (m.heads if m.head_gate else 0)
-                n += rows * self.hidden + self.hidden * m.heads * m.vdim + 1
-                n += (m.heads * m.heads if m.head_mixing else 0) + (2 * m.dim if m.qk_norm else 0)
+                n += rows * h + (m.heads * m.heads if m.head_mixing else 0) + (2 * m.dim if m.qk_norm else 0)
+            elif m.kind == "latent_attention":
+                n += (m.q_rank + m.kv_rank + m.rot_dim) * h + m.q_rank + m.kv_rank + (m.heads if m.sink else 0)
+                n += m.heads * (m.dim + m.rot_dim) * m.q_rank + m.heads * (m.dim + m.vdim) * m.kv_rank
+            elif m.kind == "hgrn2":
+                n += (2 * m.heads * m.dim + m.heads * m.vdim) * h + 2 * m.heads * m.dim + m.vdim
             else:
-                n += (2 * m.heads * (m.dim + m.vdim) + 2 * m.heads) * self.hidden + self.hidden * m.heads * m.vdim
-                n += m.heads * m.vdim + 2 * m.heads + 1
+                n += (2 * m.heads * (m.dim + m.vdim) + 2 * m.heads) * h + m.heads * m.vdim + 2 * m.heads
             if l.mlp is not None:
-                n += 2 * self.hidden * l.mlp.ff + 3
+                n += 2 * h * l.mlp.ff + (2 * norm if wide else norm)
+                n += 2 if l.mlp.activation == "xielu" else (l.mlp.ff + h if l.mlp.bias else 0)
         return n
 
     def shrink(self, n_layers: int) -> "LayeredConfig":
-        return replace(self, name=f"{self.name}-{n_layers}L", layers=self.layers[:n_layers])
+        """The first `n_layers` layers; a loop keeps what is left of it."""
+        lp = self.loop
+        if lp is not None:
+            lp = None if lp.start >= n_layers else replace(lp, stop=min(lp.stop, n_layers))
+        return replace(self, name=f"{self.name}-{n_layers}L", layers=self.layers[:n_layers], loop=lp)

@@ -18,7 +18,8 @@ from .architectures import LAYERED_REGISTRY
 from .config import REGISTRY, ModelConfig
 from .layered_config import LayeredConfig
 
-FULL, SLIDING, GDN, MLSTM = "full", "sliding", "gdn", "mlstm"
+FULL, SLIDING, GDN, MLSTM, GATED, LATENT = "full", "sliding", "gdn", "mlstm", "hgrn2", "latent"
+KINDS = (FULL, SLIDING, GDN, MLSTM, GATED, LATENT)
 
 # what the engine's forward pass, kernels and cache can do today
 ENGINE_CAPABILITIES: FrozenSet[str] = frozenset({
@@ -32,12 +33,13 @@ ENGINE_CAPABILITIES: FrozenSet[str] = frozenset({
     "vision-tower",
     # layer-list decoders (models/layered.py)
     "layer-list-schedule", "head-mixing-attention", "attention-sink", "matrix-memory", "post-sum-norm", "xielu-mlp",
+    "latent-attention", "gated-memory", "sandwich-norms", "grouped-norm", "input-convolution", "layer-loop", "relu2-mlp",
 })
 
 
 @dataclass(frozen=True)
 class LayerKind:
-    kind: str                     # FULL | SLIDING | GDN | MLSTM
+    kind: str                     # one of KINDS
     rotary_dim: int = 0           # 0 = no positional rotation on this layer (NoPE)
     rope_theta: float = 0.0
     window: int = 0               # sliding layers
@@ -86,21 +88,27 @@ def _hybrid(cfg: ModelConfig) -> Package:
 
 
 def _layered(cfg: LayeredConfig) -> Package:
-    kinds, needs = [], {"layer-list-schedule", "post-sum-norm"}
+    kinds = []
+    needs = {"layer-list-schedule", "sandwich-norms" if cfg.residual == "sandwich" else "post-sum-norm"}
+    needs |= {c for c, on in (("grouped-norm", cfg.norm_groups > 1), ("input-convolution", cfg.conv_taps), ("layer-loop", cfg.loop)) if on}
     for l in cfg.layers:
         m = l.mixer
         if m.kind == "attention":
             kinds.append(LayerKind(SLIDING if m.window else FULL, 0, 0.0, m.window, m.heads, m.kv_heads, m.dim))
             needs |= {c for c, on in (("sliding-window-attention", m.window), ("head-mixing-attention", m.head_mixing),
                                       ("attention-sink", m.sink), ("qk-norm", m.qk_norm)) if on}
+        elif m.kind == "latent_attention":
+            kinds.append(LayerKind(LATENT, m.rot_dim, m.rot_base, 0, m.heads, 1, m.dim + m.rot_dim))
+            needs |= {"latent-attention"} | ({"attention-sink"} if m.sink else set())
         else:
-            kinds.append(LayerKind(MLSTM, q_heads=m.heads, kv_heads=m.heads, head_dim=m.dim))
-            needs.add("matrix-memory")
+            kinds.append(LayerKind(GATED if m.kind == "hgrn2" else MLSTM, q_heads=m.heads, kv_heads=m.heads, head_dim=m.dim))
+            needs.add("gated-memory" if m.kind == "hgrn2" else "matrix-memory")
         if l.mlp is not None:
             needs.add(f"{l.mlp.activation}-mlp")
     inter = max((l.mlp.ff for l in cfg.layers if l.mlp is not None), default=0)
-    return Package(cfg.name, cfg.hidden, cfg.n_layers, inter, cfg.vocab, tuple(kinds), frozenset(needs), activation="xielu",
-                   config=cfg, notes=f"layer-list decoder ({cfg.architecture})")
+    act = next((l.mlp.activation for l in cfg.layers if l.mlp is not None), "")
+    return Package(cfg.name, cfg.hidden, cfg.n_layers, inter, cfg.vocab, tuple(kinds), frozenset(needs), activation=act,
+                   tie_word_embeddings=cfg.tie_head, config=cfg, notes=f"layer-list decoder ({cfg.architecture})")
 
 
 def _spark() -> Package:
@@ -164,7 +172,7 @@ def construct(model_id: str, have: FrozenSet[str] = ENGINE_CAPABILITIES) -> Mode
         raise PackageRefused(f"{model_id}: the engine lacks {', '.join(miss)}")
     if p.config is None:
         raise PackageRefused(f"{model_id}: registered as a geometry description only")
-    if sum(p.count(k) for k in (FULL, SLIDING, GDN, MLSTM)) != p.n_layers:
+    if sum(p.count(k) for k in KINDS) != p.n_layers:
         raise PackageRefused(f"{model_id}: the layer table does not cover all {p.n_layers} layers")
     return p.config
 
@@ -174,8 +182,8 @@ def construct_oracle(model_id: str, layers: int = 0, vocab: int = 0, hidden_div:
     the GPU gate says about them.  `model_id@N` or `layers` takes the first N layers of the schedule."""
     base, _, n = model_id.partition("@")
     p = lookup(base)
-    if p.count(GDN) or p.count(MLSTM):
-        raise PackageRefused(f"{base}: a GDN hybrid is served by the hybrid runtime, not by the attention-only oracle")
+    if p.n_layers != p.count(FULL) + p.count(SLIDING):
+        raise PackageRefused(f"{base}: a hybrid or layer-list model is served by its own runtime, not by the attention-only oracle")
     n_layers = int(n) if n else int(layers)
     if n_layers or vocab or hidden_div > 1:
         from .all_attention import shrink_package
@@ -186,7 +194,8 @@ def construct_oracle(model_id: str, layers: int = 0, vocab: int = 0, hidden_div:
 def describe(model_id: str) -> dict:
     p = lookup(model_id)
     return {"model_id": p.model_id, "hidden": p.hidden, "layers": p.n_layers, "full": p.count(FULL),
-            "sliding": p.count(SLIDING), "gdn": p.count(GDN), "mlstm": p.count(MLSTM), "intermediate": p.intermediate, "vocab": p.vocab,
+            "sliding": p.count(SLIDING), "gdn": p.count(GDN), "mlstm": p.count(MLSTM),
+            "hgrn2": p.count(GATED), "latent": p.count(LATENT), "intermediate": p.intermediate, "vocab": p.vocab,
             "activation": p.activation, "final_logit_softcap": p.final_logit_softcap,
             "needs": sorted(p.needs), "missing": list(p.missing()), "servable": not p.missing() and p.config is not None,
-            "oracle_runtime": (p.count(GDN) == 0 and p.count(MLSTM) == 0) or isinstance(p.config, ModelConfig), "notes": p.notes}
+            "oracle_runtime": p.n_layers == p.count(FULL) + p.count(SLIDING) or isinstance(p.config, ModelConfig), "notes": p.notes}

@@ -9,7 +9,7 @@ from typing import Optional, Sequence
 import torch
 
 from ..models.hybrid import HybridModel, ShardGeometry, Workspace
-from ..models.layered import LayeredModel, LayeredWorkspace
+from ..models.layered import BLOCK_TOKENS, LayeredModel, LayeredWorkspace
 from ..models.layered_config import LayeredConfig
 from .kv_cache import GdnStatePool, PagedKvCache
 
@@ -53,7 +53,7 @@ def build_runtime(cfg, weights, device, *, rows: int, pages_per_row: int, n_page
                           look_back=cfg.cache_window)
         states = RecurrentStatePool([[(shape, torch.float32) for shape in layer] for layer in cfg.state_shapes()], state_slots, device)
         ws = LayeredWorkspace(cfg, step_tokens, logit_rows, device, model.dtype)
-        return Runtime(model, kv, states, ws, int(model.ops.head_mix_block_tokens()), cfg.vocab, 0)
+        return Runtime(model, kv, states, ws, BLOCK_TOKENS, cfg.vocab, 0)
     model = HybridModel(cfg, weights, device, pdl=pdl, shard=shard)
     model.comm = comm
     g = model.g

@@ -53,10 +53,12 @@ class KvLayerPlanes:
     block_table: Optional[torch.Tensor] = None
 
     def typed(self, dtype: torch.dtype):
-        """K and V planes of an uncoded layer (bf16 / fp32 rows) as [pages, kv heads, page size, width] of `dtype`."""
+        """K and V planes of an uncoded layer (bf16 / fp32 rows) as [pages, kv heads, page size, width] of `dtype`.  A layer
+        whose values are part of its K rows has a V plane of width 0."""
         if self.fmt != (KV_FP32 if dtype == torch.float32 else KV_BF16):
             raise ValueError("the cache format does not match the activation type")
-        return self.k_codes.view(dtype), self.v_codes.view(dtype)
+        k, v = self.k_codes, self.v_codes
+        return k.view(dtype), v.view(dtype) if v.numel() else torch.empty(v.shape, dtype=dtype, device=v.device)
 
     def bytes(self) -> int:
         n = self.k_codes.numel() + self.v_codes.numel()

@@ -84,7 +84,7 @@ def test_embedding_rows(ops, dt):
     table = rnd(1, 37, 40, dtype=dt).cuda()
     ids = torch.tensor([3, 36, 0, 3], dtype=torch.int32, device="cuda")
     x, xa = torch.zeros((4, 40), device="cuda"), torch.zeros((4, 40), dtype=dt, device="cuda")
-    ops.embed_rows32(ids, table, x, xa, False)
+    ops.embed_rows32(ids, table, x, xa, 1.0, False)
     assert torch.equal(x, table[ids.long()].float()) and torch.equal(xa, table[ids.long()])
 
 

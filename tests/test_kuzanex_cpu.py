@@ -73,7 +73,8 @@ def test_packing_pads_heads_with_zeros_and_keeps_products():
 
 
 def test_registry_and_gate():
-    for name, cfg in AR.LAYERED_REGISTRY.items():
+    for name, cfg in kuzanex.CONFIGS.items():
+        assert AR.LAYERED_REGISTRY[name] is cfg
         assert PK.construct(name) is cfg
         d = PK.describe(name)
         assert d["servable"] and d["mlstm"] == len(cfg.state_layers) and d["sliding"] == len(cfg.attn_layers)
