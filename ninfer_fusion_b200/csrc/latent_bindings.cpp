@@ -3,6 +3,7 @@
 #include "attention/latent.h"
 #include "binding_util.h"
 #include "gated/gated.h"
+#include "gemm/head_gemm.h"
 
 namespace {
 
@@ -83,6 +84,51 @@ void latent_token_attention(const Tensor& q_latent, const Tensor& q, const Tenso
   chk(nfb::latent_token_attention(a));
 }
 
+void latent_absorbed_attention(const Tensor& q_latent, const Tensor& q, const Tensor& pages, const Tensor& block_table,
+                               const Tensor& table_row, const Tensor& kv_len, int64_t n_heads, int64_t rot_true, double scale,
+                               const Tensor& freq, OptT sink, const Tensor& out, const Tensor& blk_start, const Tensor& blk_count,
+                               int64_t max_count, const Tensor& token_seq, const Tensor& cu_seqlens, int64_t max_tokens,
+                               int64_t split_keys, int64_t n_splits, OptT part_o, OptT part_ml, bool pdl) {
+  c10::cuda::CUDAGuard guard(q.device());
+  need_rows(q_latent, "q_latent"); need(q_latent, q.scalar_type(), "q_latent");
+  const int64_t rank = q_latent.size(1) / n_heads;
+  nfb::LatentArgs a = latent_args(q, pages, block_table, table_row, kv_len, n_heads, rank, rot_true, scale, freq, sink, out, pdl);
+  TORCH_CHECK(q_latent.size(0) == a.T && out.size(1) == n_heads * rank, "latent attention: shapes");
+  a.q_latent = q_latent.data_ptr(); a.ldl = q_latent.stride(0);
+  nfb::LatentBlocks b;
+  b.n = static_cast<int>(blk_start.numel());
+  need_vec(blk_start, at::kInt, b.n, "blk_start"); need_vec(blk_count, at::kInt, b.n, "blk_count");
+  need_vec(token_seq, at::kInt, a.T, "token_seq"); need(cu_seqlens, at::kInt, "cu_seqlens");
+  b.start = static_cast<const int*>(blk_start.data_ptr()); b.count = static_cast<const int*>(blk_count.data_ptr());
+  b.max_count = static_cast<int>(max_count); b.token_seq = static_cast<const int*>(token_seq.data_ptr());
+  b.cu_seqlens = static_cast<const int*>(cu_seqlens.data_ptr()); b.max_tokens = static_cast<int>(max_tokens);
+  if (n_splits > 1) {
+    TORCH_CHECK(part_o.has_value() && part_o->defined() && part_ml.has_value() && part_ml->defined(), "latent attention: splits need their workspace");
+    need_vec(*part_o, at::kFloat, n_splits * a.T * n_heads * rank, "part_o");
+    need_vec(*part_ml, at::kFloat, n_splits * a.T * n_heads * 2, "part_ml");
+  }
+  chk(nfb::latent_absorbed_attention(a, b, static_cast<int>(split_keys), static_cast<int>(n_splits), ptr_or_null<float>(part_o),
+                                     ptr_or_null<float>(part_ml)));
+}
+bool latent_absorbed_supported(int64_t rank, int64_t rot) {
+  return nfb::latent_absorbed_supported(static_cast<int>(rank), static_cast<int>(rot));
+}
+
+void head_gemm(const Tensor& x, int64_t x_step, const Tensor& w, const Tensor& out, bool pdl) {
+  need(x, at::kBFloat16, "x"); need(w, at::kBFloat16, "w"); need(out, at::kBFloat16, "out");
+  need_rows(x, "x"); need_rows(out, "out");
+  TORCH_CHECK(w.dim() == 3 && w.is_contiguous(), "head_gemm: w must be [heads, N, K]");
+  nfb::HeadGemmArgs a;
+  a.T = static_cast<int>(x.size(0)); a.H = static_cast<int>(w.size(0)); a.N = static_cast<int>(w.size(1)); a.K = static_cast<int>(w.size(2));
+  TORCH_CHECK(x_step >= 0 && x.size(1) >= (a.H - 1) * x_step + a.K && out.size(0) == a.T && out.size(1) == w.size(0) * w.size(1),
+              "head_gemm: shapes");
+  a.x = x.data_ptr(); a.ldx = x.stride(0); a.x_step = static_cast<int>(x_step); a.w = w.data_ptr();
+  a.out = out.data_ptr(); a.ldo = out.stride(0);
+  c10::cuda::CUDAGuard guard(x.device());
+  a.stream = cur_stream(); a.pdl = pdl;
+  chk(nfb::head_gemm(a));
+}
+
 void gated_memory(const Tensor& proj, int64_t q_off, int64_t v_off, const Tensor& gates, const Tensor& lower, int64_t vdim_true,
                   double eps, const Tensor& norm, const Tensor& cu_seqlens, const Tensor& state_slot, const Tensor& S,
                   const Tensor& out, bool write_state, OptT chunk_ws, bool pdl, bool one_token) {
@@ -129,6 +175,9 @@ bool gated_chunked_supported(int64_t dim, int64_t vdim) {
 TORCH_LIBRARY_FRAGMENT(nfb200, m) {
   m.def("latent_prep(Tensor proj, int q_rank_true, int rank_true, int rot_true, Tensor q_norm, Tensor kv_norm, float eps, Tensor freq, Tensor table_row, Tensor cache_pos, Tensor block_table, Tensor q_latent, Tensor pages, bool pdl) -> ()", &latent_prep);
   m.def("latent_token_attention(Tensor q_latent, Tensor q, Tensor pages, Tensor block_table, Tensor table_row, Tensor kv_len, int n_heads, int rot_true, float scale, Tensor freq, Tensor? sink, Tensor out, bool pdl) -> ()", &latent_token_attention);
+  m.def("latent_absorbed_attention(Tensor q_latent, Tensor q, Tensor pages, Tensor block_table, Tensor table_row, Tensor kv_len, int n_heads, int rot_true, float scale, Tensor freq, Tensor? sink, Tensor out, Tensor blk_start, Tensor blk_count, int max_count, Tensor token_seq, Tensor cu_seqlens, int max_tokens, int split_keys, int n_splits, Tensor? part_o, Tensor? part_ml, bool pdl) -> ()", &latent_absorbed_attention);
+  m.def("latent_absorbed_supported(int rank, int rot) -> bool", &latent_absorbed_supported);
+  m.def("head_gemm(Tensor x, int x_step, Tensor w, Tensor out, bool pdl) -> ()", &head_gemm);
   m.def("gated_memory(Tensor proj, int q_off, int v_off, Tensor gates, Tensor lower, int vdim_true, float eps, Tensor norm, Tensor cu_seqlens, Tensor state_slot, Tensor S, Tensor out, bool write_state, Tensor? chunk_ws, bool pdl, bool one_token=False) -> ()", &gated_memory);
   m.def("gated_chunked_workspace_bytes(int T, int n_seq, int n_heads, int dim, int vdim) -> int", &gated_chunked_workspace_bytes);
   m.def("gated_chunked_supported(int dim, int vdim) -> bool", &gated_chunked_supported);

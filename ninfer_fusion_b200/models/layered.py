@@ -334,8 +334,20 @@ class LayeredModel:
         split = max(64, pad_to(-(-keys // want), 32))
         return split, -(-keys // split)
 
+    @staticmethod
+    def pick_latent_split(ws, b: StepBatch, m: LatentAttentionMixer, sm_count: int = 148) -> Tuple[int, int]:
+        """Keys per split (a multiple of 32) and splits per query block: about one CTA per SM when the step is small."""
+        rows = min(b.max_seq_tokens, BLOCK_TOKENS) * m.heads
+        ctas = b.qblk_start.numel() * max(1, -(-rows // 64))
+        want = max(1, min(sm_count // ctas, ws.split_rows // b.n_tokens, 64))
+        split = max(128, pad_to(-(-b.max_kv_len // want), 32))
+        return split, -(-b.max_kv_len // split)
+
     def _head_gemm(self, x: torch.Tensor, x_step: int, w: torch.Tensor, out: torch.Tensor) -> None:
         """out[t, h * N + n] = sum_k w[h, n, k] x[t, h * x_step + k]"""
+        if not self.f32:
+            self.ops.head_gemm(x, x_step, w, out, self.pdl)
+            return
         H, N, K = w.shape
         for h in range(H):
             self._gemm(x[:, h * x_step: h * x_step + K], w[h], None, out[:, h * N: (h + 1) * N])
@@ -352,8 +364,13 @@ class LayeredModel:
         out = ws.mix[:T, : m.out_cols]
         q_abs, o_latent = ws.q_abs[:T, : m.heads * m.kv_rank_p], ws.o_latent[:T, : m.heads * m.kv_rank_p]
         self._head_gemm(q, m.dim_p + m.rot_p, w[f"{p}/mix/uk_t"], q_abs)
-        ops.latent_token_attention(q_abs, q, pages, kv.table, b.table_row, b.kv_len, m.heads, m.rot_dim, m.scale, freq, sink,
-                                   o_latent, self.pdl)
+        args = (q_abs, q, pages, kv.table, b.table_row, b.kv_len, m.heads, m.rot_dim, m.scale, freq, sink, o_latent)
+        if self.f32 or not self._raw_ops.latent_absorbed_supported(m.kv_rank_p, m.rot_p):
+            ops.latent_token_attention(*args, self.pdl)
+        else:
+            split, n = self.pick_latent_split(ws, b, m)
+            ops.latent_absorbed_attention(*args, b.qblk_start, b.qblk_count, min(b.max_seq_tokens, BLOCK_TOKENS), b.token_seq, b.cu_seqlens,
+                                          0, split, n, ws.part_o if n > 1 else None, ws.part_ml if n > 1 else None, self.pdl)
         self._head_gemm(o_latent, m.kv_rank_p, w[f"{p}/mix/uv"], out)
         return out
 
