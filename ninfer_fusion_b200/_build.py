@@ -32,8 +32,8 @@ _LAYERED = ("common/tensor_map.cpp", "core_bindings.cpp", "layered_bindings.cpp"
             "pointwise/rows32.cu", "pointwise/sandwich_rows.cu", "sampling/sampling.cu", "runtime/page_pool.cpp")
 _HEAD_MIX = ("head_mix_bindings.cpp", "attention/qkv_append.cu", "attention/head_mix_token.cu", "attention/head_mix_decode.cu",
              "attention/head_mix_prefill.cu", "mlstm/mlstm_recurrent.cu", "mlstm/mlstm_chunked.cu")
-_LATENT = ("latent_bindings.cpp", "attention/latent_prep.cu", "attention/latent_token.cu", "attention/latent_absorbed.cu", "gemm/head_gemm.cu",
-           "gated/gated_recurrent.cu", "gated/gated_chunked.cu")
+_LATENT = ("latent_bindings.cpp", "attention/latent_prep.cu", "attention/latent_token.cu", "attention/latent_absorbed.cu",
+           "attention/latent_expanded.cu", "gemm/head_gemm.cu", "gated/gated_recurrent.cu", "gated/gated_chunked.cu")
 SUBSETS = {"head_mix": _LAYERED + _HEAD_MIX, "latent": _LAYERED + _LATENT, "layered": _LAYERED + _HEAD_MIX + _LATENT}
 
 

@@ -79,6 +79,20 @@ bool latent_absorbed_supported(int rank, int rot);
 const char* latent_absorbed_attention(const LatentArgs& a, const LatentBlocks& b, int split_keys, int n_splits, float* part_o,
                                       float* part_ml);
 
+// Expanded, bf16 tensor cores, for the sequences the absorbed form leaves out.  latent_gather fills `rows`; the caller makes
+// `kv` from their latents (one GEMM); then latent_expanded_attention writes out [T, n_heads * vdim] of those sequences.
+struct LatentExpand {
+  const int* seqs = nullptr;      // [n_seqs, 3]: block-table row, first row in `rows`, visible positions
+  int n_seqs = 0, max_len = 0;
+  const int* seq_base = nullptr;  // [sequences of the step]: first row in `rows`, -1: not expanded
+  void* rows = nullptr;           // [total, rank + rot]
+  const void* kv = nullptr;       // [total, n_heads * (dim + vdim)]: keys of all heads, values of all heads
+  int vdim = 0;
+};
+bool latent_expanded_supported(int dim, int rot, int vdim);
+const char* latent_gather(const LatentArgs& a, const LatentExpand& x);
+const char* latent_expanded_attention(const LatentArgs& a, const LatentBlocks& b, const LatentExpand& x);
+
 #ifdef __CUDACC__
 // cos and sin of pos * freq, the angle reduced in 64-bit.
 __device__ __forceinline__ void latent_angle(int pos, double freq, float& c, float& s) {

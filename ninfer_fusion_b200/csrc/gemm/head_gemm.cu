@@ -17,7 +17,16 @@ __global__ void __launch_bounds__(kThreads) head_gemm_kernel(const HeadGemmArgs 
   extern __shared__ __align__(16) bf16 smem[];   // [kStages][kT + kN][kLd]
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int n0 = blockIdx.x * kN, h = blockIdx.y, t0 = blockIdx.z * kT;
-  const int n_tok = min(kT, p.T - t0), n_slices = (p.K + kK - 1) / kK;
+  const int n_tok = min(kT, p.T - t0);
+  if (p.max_tokens > 0) {     // (written before the step's first kernel: no need to wait)
+    const int seq = p.token_seq[t0];
+    if (seq == p.token_seq[t0 + n_tok - 1] && p.cu_seqlens[seq + 1] - p.cu_seqlens[seq] >= p.max_tokens) {
+      pdl_launch_next();
+      pdl_wait_prior();
+      return;
+    }
+  }
+  const int n_slices = (p.K + kK - 1) / kK;
   const bf16* w = static_cast<const bf16*>(p.w) + (static_cast<long long>(h) * p.N + n0) * p.K;
   const bf16* x = static_cast<const bf16*>(p.x) + t0 * p.ldx + static_cast<long long>(h) * p.x_step;
   const uint32_t base = smem_u32(smem);

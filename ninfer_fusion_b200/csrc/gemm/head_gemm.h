@@ -13,6 +13,10 @@ struct HeadGemmArgs {
   void* out = nullptr;       // [T, H * N], leading dimension ldo
   int64_t ldo = 0;
   int T = 0, H = 0, N = 0, K = 0;
+  // optional: token tiles that lie inside one sequence of `max_tokens` or more tokens of this step are left out
+  const int* token_seq = nullptr;   // [T]
+  const int* cu_seqlens = nullptr;
+  int max_tokens = 0;
   cudaStream_t stream = nullptr;
   bool pdl = false;
 };

@@ -114,7 +114,59 @@ bool latent_absorbed_supported(int64_t rank, int64_t rot) {
   return nfb::latent_absorbed_supported(static_cast<int>(rank), static_cast<int>(rot));
 }
 
-void head_gemm(const Tensor& x, int64_t x_step, const Tensor& w, const Tensor& out, bool pdl) {
+void latent_gather(const Tensor& pages, const Tensor& block_table, const Tensor& seqs, int64_t max_len, const Tensor& rows, bool pdl) {
+  need(pages, at::kBFloat16, "pages"); need(rows, at::kBFloat16, "rows"); need_table(block_table);
+  need_pages(pages, at::kBFloat16, pages.size(3));
+  need_vec(seqs, at::kInt, seqs.size(0) * 3, "seqs");
+  TORCH_CHECK(rows.dim() == 2 && rows.is_contiguous() && rows.size(1) == pages.size(3), "latent_gather: rows shape");
+  nfb::LatentArgs a;
+  a.pages = pages.data_ptr(); a.rank = static_cast<int>(pages.size(3)); a.rot = 0; a.page_size = static_cast<int>(pages.size(2));
+  a.block_table = static_cast<const int*>(block_table.data_ptr()); a.table_ld = static_cast<int>(block_table.stride(0));
+  nfb::LatentExpand x;
+  x.seqs = static_cast<const int*>(seqs.data_ptr()); x.n_seqs = static_cast<int>(seqs.size(0)); x.max_len = static_cast<int>(max_len);
+  x.rows = rows.data_ptr();
+  c10::cuda::CUDAGuard guard(pages.device());
+  a.stream = cur_stream(); a.pdl = pdl;
+  chk(nfb::latent_gather(a, x));
+}
+
+void latent_expanded_attention(const Tensor& q, const Tensor& rows, const Tensor& kv, const Tensor& kv_len,
+                               int64_t n_heads, int64_t rank, int64_t rot_true, double scale, const Tensor& freq, OptT sink,
+                               const Tensor& out, const Tensor& blk_start, const Tensor& blk_count, int64_t max_count,
+                               const Tensor& token_seq, const Tensor& seq_base, bool pdl) {
+  nfb::LatentArgs a;
+  need(q, at::kBFloat16, "q"); need(rows, at::kBFloat16, "rows"); need(kv, at::kBFloat16, "kv"); need(out, at::kBFloat16, "out");
+  need_rows(q, "q"); need_rows(out, "out");
+  TORCH_CHECK(rows.dim() == 2 && rows.is_contiguous() && kv.dim() == 2 && kv.is_contiguous() && rows.size(0) == kv.size(0),
+              "latent attention: gathered rows");
+  const int64_t T = q.size(0), rot = rows.size(1) - rank;
+  TORCH_CHECK(n_heads > 0 && rot >= 0 && q.size(1) % n_heads == 0 && out.size(1) % n_heads == 0 && out.size(0) == T, "latent attention: shapes");
+  const int64_t dim = q.size(1) / n_heads - rot, vdim = out.size(1) / n_heads;
+  TORCH_CHECK(dim > 0 && kv.size(1) == n_heads * (dim + vdim), "latent attention: expanded columns");
+  need_vec(kv_len, at::kInt, T, "kv_len"); need_vec(token_seq, at::kInt, T, "token_seq");
+  need(seq_base, at::kInt, "seq_base");
+  if (sink.has_value() && sink->defined()) need_vec(*sink, at::kFloat, n_heads, "sink");
+  a.q = q.data_ptr(); a.ldq = q.stride(0); a.kv_len = static_cast<const int*>(kv_len.data_ptr());
+  a.T = static_cast<int>(T); a.n_heads = static_cast<int>(n_heads); a.dim = static_cast<int>(dim); a.rank = static_cast<int>(rank);
+  a.rot = static_cast<int>(rot); a.rot_true = static_cast<int>(rot_true); a.scale = static_cast<float>(scale);
+  a.freq = freq_ptr(freq, rot_true); a.sink = ptr_or_null<const float>(sink); a.out = out.data_ptr(); a.ldo = out.stride(0);
+  nfb::LatentBlocks b;
+  b.n = static_cast<int>(blk_start.numel()); b.max_count = static_cast<int>(max_count);
+  need_vec(blk_start, at::kInt, b.n, "blk_start"); need_vec(blk_count, at::kInt, b.n, "blk_count");
+  b.start = static_cast<const int*>(blk_start.data_ptr()); b.count = static_cast<const int*>(blk_count.data_ptr());
+  b.token_seq = static_cast<const int*>(token_seq.data_ptr());
+  nfb::LatentExpand x;
+  x.seq_base = static_cast<const int*>(seq_base.data_ptr()); x.rows = rows.data_ptr(); x.kv = kv.data_ptr(); x.vdim = static_cast<int>(vdim);
+  c10::cuda::CUDAGuard guard(q.device());
+  a.stream = cur_stream(); a.pdl = pdl;
+  chk(nfb::latent_expanded_attention(a, b, x));
+}
+bool latent_expanded_supported(int64_t dim, int64_t rot, int64_t vdim) {
+  return nfb::latent_expanded_supported(static_cast<int>(dim), static_cast<int>(rot), static_cast<int>(vdim));
+}
+
+void head_gemm(const Tensor& x, int64_t x_step, const Tensor& w, const Tensor& out, OptT token_seq, OptT cu_seqlens, int64_t max_tokens,
+               bool pdl) {
   need(x, at::kBFloat16, "x"); need(w, at::kBFloat16, "w"); need(out, at::kBFloat16, "out");
   need_rows(x, "x"); need_rows(out, "out");
   TORCH_CHECK(w.dim() == 3 && w.is_contiguous(), "head_gemm: w must be [heads, N, K]");
@@ -124,6 +176,12 @@ void head_gemm(const Tensor& x, int64_t x_step, const Tensor& w, const Tensor& o
               "head_gemm: shapes");
   a.x = x.data_ptr(); a.ldx = x.stride(0); a.x_step = static_cast<int>(x_step); a.w = w.data_ptr();
   a.out = out.data_ptr(); a.ldo = out.stride(0);
+  if (max_tokens > 0) {
+    TORCH_CHECK(token_seq.has_value() && cu_seqlens.has_value(), "head_gemm: leaving tokens out needs the sequences");
+    need_vec(*token_seq, at::kInt, a.T, "token_seq"); need(*cu_seqlens, at::kInt, "cu_seqlens");
+    a.token_seq = static_cast<const int*>(token_seq->data_ptr()); a.cu_seqlens = static_cast<const int*>(cu_seqlens->data_ptr());
+    a.max_tokens = static_cast<int>(max_tokens);
+  }
   c10::cuda::CUDAGuard guard(x.device());
   a.stream = cur_stream(); a.pdl = pdl;
   chk(nfb::head_gemm(a));
@@ -177,7 +235,10 @@ TORCH_LIBRARY_FRAGMENT(nfb200, m) {
   m.def("latent_token_attention(Tensor q_latent, Tensor q, Tensor pages, Tensor block_table, Tensor table_row, Tensor kv_len, int n_heads, int rot_true, float scale, Tensor freq, Tensor? sink, Tensor out, bool pdl) -> ()", &latent_token_attention);
   m.def("latent_absorbed_attention(Tensor q_latent, Tensor q, Tensor pages, Tensor block_table, Tensor table_row, Tensor kv_len, int n_heads, int rot_true, float scale, Tensor freq, Tensor? sink, Tensor out, Tensor blk_start, Tensor blk_count, int max_count, Tensor token_seq, Tensor cu_seqlens, int max_tokens, int split_keys, int n_splits, Tensor? part_o, Tensor? part_ml, bool pdl) -> ()", &latent_absorbed_attention);
   m.def("latent_absorbed_supported(int rank, int rot) -> bool", &latent_absorbed_supported);
-  m.def("head_gemm(Tensor x, int x_step, Tensor w, Tensor out, bool pdl) -> ()", &head_gemm);
+  m.def("latent_gather(Tensor pages, Tensor block_table, Tensor seqs, int max_len, Tensor rows, bool pdl) -> ()", &latent_gather);
+  m.def("latent_expanded_attention(Tensor q, Tensor rows, Tensor kv, Tensor kv_len, int n_heads, int rank, int rot_true, float scale, Tensor freq, Tensor? sink, Tensor out, Tensor blk_start, Tensor blk_count, int max_count, Tensor token_seq, Tensor seq_base, bool pdl) -> ()", &latent_expanded_attention);
+  m.def("latent_expanded_supported(int dim, int rot, int vdim) -> bool", &latent_expanded_supported);
+  m.def("head_gemm(Tensor x, int x_step, Tensor w, Tensor out, Tensor? token_seq, Tensor? cu_seqlens, int max_tokens, bool pdl) -> ()", &head_gemm);
   m.def("gated_memory(Tensor proj, int q_off, int v_off, Tensor gates, Tensor lower, int vdim_true, float eps, Tensor norm, Tensor cu_seqlens, Tensor state_slot, Tensor S, Tensor out, bool write_state, Tensor? chunk_ws, bool pdl, bool one_token=False) -> ()", &gated_memory);
   m.def("gated_chunked_workspace_bytes(int T, int n_seq, int n_heads, int dim, int vdim) -> int", &gated_chunked_workspace_bytes);
   m.def("gated_chunked_supported(int dim, int vdim) -> bool", &gated_chunked_supported);

@@ -57,6 +57,10 @@ class StepBatch:
     # multimodal prefill: rows of the step whose embedding is replaced by a vision-tower output row
     embed_rows: Optional[torch.Tensor] = None   # int64 [V]
     embed_vals: Optional[torch.Tensor] = None   # bf16 [V, hidden]
+    # host copies per sequence (block-table row, tokens of this step, visible keys of its last token); models that treat
+    # long and short portions of one step differently keep what they derive from it in `plans`
+    seq_host: Optional[list] = None
+    plans: Optional[dict] = None
 
 
 class Workspace:

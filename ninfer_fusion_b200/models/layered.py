@@ -28,6 +28,7 @@ from .layered_config import (ATTENTION_KINDS, AttentionMixer, GatedMemoryMixer, 
 ACTIVATIONS = {"xielu": 3, "relu2": 4}     # csrc/gemm/gemm.h GemmActivation
 BLOCK_TOKENS = 64          # query tokens per attention block of a step (kHeadMixBlock, kLatentBlock)
 PREFILL_MIN_TOKENS = 8     # shorter portions take the token-by-token kernels
+EXPAND_BYTES = 4 << 30     # keys and values of expanded latents in flight
 SCORE_SCRATCH_BYTES = 1 << 30    # fp32 scores in flight between the two prefill attention kernels
 
 
@@ -343,14 +344,44 @@ class LayeredModel:
         split = max(128, pad_to(-(-b.max_kv_len // want), 32))
         return split, -(-b.max_kv_len // split)
 
-    def _head_gemm(self, x: torch.Tensor, x_step: int, w: torch.Tensor, out: torch.Tensor) -> None:
-        """out[t, h * N + n] = sum_k w[h, n, k] x[t, h * x_step + k]"""
+    def _head_gemm(self, x: torch.Tensor, x_step: int, w: torch.Tensor, out: torch.Tensor, b: StepBatch, max_tokens: int) -> None:
+        """out[t, h * N + n] = sum_k w[h, n, k] x[t, h * x_step + k]; tokens of sequences with `max_tokens` or more may be left out"""
         if not self.f32:
-            self.ops.head_gemm(x, x_step, w, out, self.pdl)
+            self.ops.head_gemm(x, x_step, w, out, b.token_seq, b.cu_seqlens, max_tokens, self.pdl)
             return
         H, N, K = w.shape
         for h in range(H):
             self._gemm(x[:, h * x_step: h * x_step + K], w[h], None, out[:, h * N: (h + 1) * N])
+
+    @staticmethod
+    def expand_tokens(m: LatentAttentionMixer) -> int:
+        """Portion length from which making the keys and values of all visible positions takes fewer multiply-adds than
+        attending in the latent space; 0: never."""
+        wide, heads = 2 * m.kv_rank_p, m.dim_p + m.vdim_p
+        return max(16, -(-m.kv_rank_p * heads // (wide - heads))) if wide > heads else 0
+
+    def _expand_plan(self, b: StepBatch, m: LatentAttentionMixer):
+        """Which sequences of the step take the expanded form: (threshold, [n, 3] of block-table row / first gathered row /
+        positions, first row per sequence or -1, total rows, longest, whether the others are left) or None."""
+        least = self.expand_tokens(m)
+        if (self.f32 or not self.prefill_kernels or b.seq_host is None or not least or b.max_seq_tokens < least
+                or not self._raw_ops.latent_expanded_supported(m.dim_p, m.rot_p, m.vdim_p)):
+            return None
+        key = (least, m.heads * (m.dim_p + m.vdim_p))
+        if key not in b.plans:
+            seqs, base, total = [], [], 0
+            for row, n, end in b.seq_host:
+                base.append(total if n >= least else -1)
+                if n >= least:
+                    seqs.append((row, total, end))
+                    total += end
+            plan = None
+            if total * key[1] * 2 <= EXPAND_BYTES:
+                host = torch.tensor(base + [v for s in seqs for v in s], dtype=torch.int32)
+                dev = (host.pin_memory() if self.device.type == "cuda" else host).to(self.device, non_blocking=True)
+                plan = (least, dev[len(base):].view(-1, 3), dev[: len(base)], total, max(s[2] for s in seqs), len(seqs) < len(base))
+            b.plans[key] = plan
+        return b.plans[key]
 
     def _latent_attention(self, ws, b: StepBatch, kv, run: int, T: int, p: str, m: LatentAttentionMixer):
         ops, w, eps = self.ops, self.w, self.cfg.rms_eps
@@ -362,16 +393,28 @@ class LayeredModel:
                         b.cache_pos, kv.table, c_q, pages, self.pdl)
         self._gemm(c_q, w[f"{p}/mix/uq"], None, q, prefetch=w[f"{p}/mix/uk_t"])
         out = ws.mix[:T, : m.out_cols]
-        q_abs, o_latent = ws.q_abs[:T, : m.heads * m.kv_rank_p], ws.o_latent[:T, : m.heads * m.kv_rank_p]
-        self._head_gemm(q, m.dim_p + m.rot_p, w[f"{p}/mix/uk_t"], q_abs)
-        args = (q_abs, q, pages, kv.table, b.table_row, b.kv_len, m.heads, m.rot_dim, m.scale, freq, sink, o_latent)
-        if self.f32 or not self._raw_ops.latent_absorbed_supported(m.kv_rank_p, m.rot_p):
-            ops.latent_token_attention(*args, self.pdl)
-        else:
-            split, n = self.pick_latent_split(ws, b, m)
-            ops.latent_absorbed_attention(*args, b.qblk_start, b.qblk_count, min(b.max_seq_tokens, BLOCK_TOKENS), b.token_seq, b.cu_seqlens,
-                                          0, split, n, ws.part_o if n > 1 else None, ws.part_ml if n > 1 else None, self.pdl)
-        self._head_gemm(o_latent, m.kv_rank_p, w[f"{p}/mix/uv"], out)
+        plan, blocks = self._expand_plan(b, m), (b.qblk_start, b.qblk_count, min(b.max_seq_tokens, BLOCK_TOKENS))
+        if plan is None or plan[-1]:
+            skip = 0 if plan is None else plan[0]
+            q_abs, o_latent = ws.q_abs[:T, : m.heads * m.kv_rank_p], ws.o_latent[:T, : m.heads * m.kv_rank_p]
+            self._head_gemm(q, m.dim_p + m.rot_p, w[f"{p}/mix/uk_t"], q_abs, b, skip)
+            args = (q_abs, q, pages, kv.table, b.table_row, b.kv_len, m.heads, m.rot_dim, m.scale, freq, sink, o_latent)
+            if self.f32 or not self._raw_ops.latent_absorbed_supported(m.kv_rank_p, m.rot_p):
+                ops.latent_token_attention(*args, self.pdl)
+            else:
+                split, n = self.pick_latent_split(ws, b, m)
+                ops.latent_absorbed_attention(*args, *blocks, b.token_seq, b.cu_seqlens, skip, split, n,
+                                              ws.part_o if n > 1 else None, ws.part_ml if n > 1 else None, self.pdl)
+            self._head_gemm(o_latent, m.kv_rank_p, w[f"{p}/mix/uv"], out, b, skip)
+        if plan is not None:
+            _, seqs, base, total, longest, _ = plan
+            ukv = w[f"{p}/mix/ukv"]
+            rows = self._grown("latent rows", total * m.row_cols * 2)[: total * m.row_cols * 2].view(self.dtype).view(total, m.row_cols)
+            wide = self._grown("latent keys", total * ukv.shape[0] * 2)[: total * ukv.shape[0] * 2].view(self.dtype).view(total, ukv.shape[0])
+            ops.latent_gather(pages, kv.table, seqs, longest, rows, self.pdl)
+            self._gemm(rows[:, : m.kv_rank_p], ukv, None, wide)
+            ops.latent_expanded_attention(q, rows, wide, b.kv_len, m.heads, m.kv_rank_p, m.rot_dim, m.scale, freq, sink, out, *blocks,
+                                          b.token_seq, base, self.pdl)
         return out
 
     def _chunk_workspace(self, b: StepBatch, T: int, kind: str, m) -> "torch.Tensor | None":

@@ -131,4 +131,5 @@ class StepBuffers:
                          max_kv_len=max_kv, n_tokens=T, n_seqs=B,
                          one_token_per_seq=all(len(c.tokens) == 1 for c in chunks),
                          max_seq_tokens=max((len(c.tokens) for c in chunks), default=1),
-                         qblk_start=self._dview("qblk_start", nb), qblk_count=self._dview("qblk_count", nb))
+                         qblk_start=self._dview("qblk_start", nb), qblk_count=self._dview("qblk_count", nb),
+                         seq_host=[(c.table_row, len(c.tokens), c.start_pos + len(c.tokens)) for c in chunks], plans={})
