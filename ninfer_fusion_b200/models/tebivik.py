@@ -169,5 +169,5 @@ T1B = _design("tebivik-1b", 2048, 65536, "mmma" * 4, dict(heads=16, dim=128, rot
               dict(heads=16, dim=128, vdim=128), 8192, (12, 16, 2), 4)
 T7B = _design("tebivik-7b", 4096, 131072, "mmma" * 8, dict(heads=32, dim=128, rot_dim=64, vdim=128, q_rank=1536, kv_rank=512,
                                                              scale=0.0722, rot={"base": 1e4}),
-              dict(heads=32, dim=128, vdim=128), 12288, (28, 32, 2), 8)
+              dict(heads=32, dim=128, vdim=128), 12288, (4, 8, 2), 8)
 CONFIGS = {c.name: c for c in (TINY, T1B, T7B)}

@@ -1,17 +1,20 @@
-"""Layer-list designs beside the hybrid decoder of equal size: model throughput and per-kernel roofline fractions.
+"""Layer-list designs beside the closest other model of equal size: model throughput and per-kernel roofline fractions.
 
 `python bench.py --compare kuzanex-1b` prints one JSON line: prefill and decode tokens/s of the two models through the
 same generator (random weights, bf16), and for every kernel of the design its time, what bounds it, and the same for
-the hybrid's kernel of the like kind at equal size.  Kernels are timed cold (L2 flushed before every launch) with CUDA
+the other model's kernel of the like kind at equal size.  Kuzanex (head-mixing attention, matrix memory) stands beside the
+hybrid decoder, Tebivik (latent attention, gated memory) beside Kuzanex.  Kernels are timed cold (L2 flushed before every launch) with CUDA
 events; the roofline of a kernel is the slower of its algorithmic bytes at the measured copy bandwidth and its
 algorithmic multiply-adds at the measured bf16 GEMM rate.
 """
 from __future__ import annotations
 
+from dataclasses import replace
 from typing import Dict, List
 
 import torch
 
+from ..models import kuzanex
 from ..models.architectures import LAYERED_REGISTRY, random_layered_weights
 from ..models.config import ModelConfig
 from ..models.weights import random_weights
@@ -69,13 +72,15 @@ def _throughput(cfg, weights, batch: int, prompt: int, steps: int) -> Dict[str, 
 class _Kernels:
     """Times closures cold and puts them against their roofline."""
 
-    def __init__(self, iters: int, only: str = ""):
+    def __init__(self, iters: int, only: str = "", names: "Dict[str, str] | None" = None):
         self.only = only
+        self.names = names or {}       # model label of a row -> label to report, "" leaves the row out
         self.flush, self.iters, self.rows = L2Flusher(), iters, []
         self.bw, self.fl, self.how = measured_peaks()
 
     def add(self, what: str, model: str, fn, n_bytes: float, macs: float = 0.0) -> None:
-        if self.only not in f"{model}: {what}":
+        model = self.names.get(model, model)
+        if not model or self.only not in f"{model}: {what}":
             return
         med, _ = time_op(fn, iters=self.iters, flush=self.flush)
         t_b, t_f = n_bytes / self.bw, 2.0 * macs / self.fl
@@ -224,39 +229,146 @@ def _memory_rows(k: _Kernels, ops, cfg, hyb, batch: int, new: int, tag: str) -> 
           2 * ssm.numel() * 4 + conv.numel() * 2 + 2 * T * vd * 2, 2.0 * T * hv * d * d)
 
 
+def equal_size_kuzanex(cfg):
+    """Kuzanex with the width, the layer runs, the heads, the state size and the feed-forwards of a latent / gated-memory
+    configuration; every key is visible."""
+    lat = next(l.mixer for l in cfg.layers if l.mixer.kind == "latent_attention")
+    mem = next(l.mixer for l in cfg.layers if l.mixer.kind == "hgrn2")
+    dim = min(256, 2 * mem.dim)
+    attn = dict(heads=lat.heads, kv_heads=max(1, lat.heads // 4), dim=lat.dim, vdim=lat.vdim, scale=lat.dim ** -0.5, softcap=50.0,
+                mask={"size": 1 << 20})
+    memory = dict(heads=max(1, mem.heads * mem.dim * mem.vdim // (dim * dim)), dim=dim, vdim=dim, gate_cap=15.0)
+    pattern = "".join("a" if cfg.mixer_of(r).kind == "latent_attention" else "m" for r in range(len(cfg.runs)))
+    return replace(kuzanex._design(f"kuzanex-like-{cfg.name}", cfg.hidden, cfg.vocab, pattern, attn, memory, cfg.layers[0].mlp.ff), max_context=cfg.max_context)
+
+
+def _latent_design_rows(k: _Kernels, model, ws, cfg, batch: int, new: int, total: int, tag: str) -> None:
+    """Kernels of a latent / gated-memory design: GEMMs, row steps, attention in the form the step takes, recurrence."""
+    ops, status, w = model._raw_ops, model.status.tensor, model.w
+    at, mt = (next(i for i, l in enumerate(cfg.layers) if l.mixer.kind == kind) for kind in ("latent_attention", "hgrn2"))
+    m, g = cfg.layers[at].mixer, cfg.layers[mt].mixer
+    T, h, P = batch * new, cfg.hidden_p, 64
+    pa, pm = f"text/layers/{at}", f"text/layers/{mt}"
+
+    def gemm(what, weight, x=None, out32_from=None, act=0, bias=None):
+        N, K = weight.shape
+        rows = T if x is None else x.shape[0]
+        x = _rand(rows, K) if x is None else x
+        out = torch.empty((rows, N), dtype=torch.bfloat16, device="cuda")
+        o32 = None if out32_from is None else torch.empty((rows, N - out32_from), device="cuda")
+        splits = int(ops.gemm_pick_splits(rows, N, K, 0))
+        n_out = rows * N * 2 if out32_from is None else rows * (out32_from * 2 + (N - out32_from) * 4)
+        k.add(f"{what} {tag}", "design", lambda: ops.gemm_bf16(x, weight, None if out32_from == 0 else out, 0, None, bias, None, splits, status,
+                                                               False, act, None, None, None, None, None, o32, out32_from or 0),
+              N * K * 2 + rows * K * 2 + n_out, rows * N * K)
+    gemm("input projection (memory)", w[f"{pm}/mix/in_proj"], out32_from=g.main_cols, bias=w[f"{pm}/mix/in_bias"])
+    gemm("input projection (attention)", w[f"{pa}/mix/in_proj"])
+    gemm("query projection", w[f"{pa}/mix/uq"])
+    gemm("output projection", w[f"{pm}/mix/out_proj"], out32_from=0)
+    gemm("feed-forward up", w[f"{pm}/mlp/up"], act=4, bias=w[f"{pm}/mlp/up_bias"])
+    gemm("feed-forward down", w[f"{pm}/mlp/down"], out32_from=0, bias=w[f"{pm}/mlp/down_bias"])
+    if cfg.loop is not None:
+        gemm("loop entry", w["text/loop/in_proj"], out32_from=0)
+    # row steps: in front of a feed-forward (the like of the post-sum norm), and with the convolution
+    x32, x2, d32, xa = torch.randn(T, h, device="cuda"), torch.empty(T, h, device="cuda"), torch.randn(T, h, device="cuda"), _rand(T, h)
+    slots, cu = _ints(torch.arange(batch)), _ints(torch.arange(batch + 1) * new)
+    hist = torch.zeros((batch, cfg.conv_taps - 1, h), device="cuda")
+    common = (w[f"{pm}/norm1b"], w[f"{pm}/norm2"], xa, cfg.hidden, cfg.norm_groups, cfg.residual_mult, 1e-6)
+    k.add(f"residual rows {tag}", "design", lambda: ops.sandwich_rows(x32, x32, d32, *common, None, None, None, None, new, True, False), T * h * 14)
+    dst = x2 if new > 1 else x32
+    k.add(f"residual rows + convolution {tag}", "design",
+          lambda: ops.sandwich_rows(x32, dst, d32, *common, w[f"{pm}/conv"], hist, cu, slots, new, True, False),
+          T * h * 14 + 2 * hist.numel() * 4)
+    # latent attention
+    H, R, C, V, D = m.heads, m.rot_p, m.kv_rank_p, m.vdim_p, m.dim_p
+    per = (total + P - 1) // P
+    row, kv, _ = _tokens(batch, new, total)
+    pos = (kv - 1).int()
+    table = torch.randperm(batch * per, device="cuda").int().view(batch, per)
+    pages = _rand(batch * per, 1, P, C + R)
+    proj, lat, q = _rand(T, m.main_cols), _rand(T, m.q_rank_p), _rand(T, m.q_cols)
+    freq, sink = w[f"{pa}/mix/freq"], w[f"{pa}/mix/sink"]
+    k.add(f"norm + append {tag}", "design", lambda: ops.latent_prep(proj, m.q_rank, m.kv_rank, m.rot_dim, w[f"{pa}/mix/q_norm"], w[f"{pa}/mix/kv_norm"],
+                                                                   1e-6, freq, row, pos, table, lat, pages, False), T * m.main_cols * 4)
+    start, count = _blocks(batch, new, 64)
+    blocks = (start, count, min(new, 64))
+    pairs = batch * _pairs(new, total, 0)
+    if new == 1:
+        from ..runtime.batch import SeqChunk, StepBuffers
+        step = StepBuffers(batch, batch, "cpu", attn_block_tokens=64).build([SeqChunk(i, i, total - 1, [0]) for i in range(batch)])
+        split, n = model.pick_latent_split(ws, step, m)
+        q_abs, o_lat, out = _rand(T, H * C), _rand(T, H * C), _rand(T, H * V)
+        po, ml = torch.empty(T * n * H * C, device="cuda"), torch.empty(T * n * H * 2, device="cuda")
+        k.add(f"attention {tag}", "design", lambda: ops.latent_absorbed_attention(q_abs, q, pages, table, row, kv, H, m.rot_dim, m.scale, freq, sink, o_lat,
+                                                                                *blocks, row, cu, 0, split, n, po, ml, False),
+              batch * total * (C + R) * 2 + T * H * (2 * C + R) * 2, pairs * H * (2 * C + R))
+        uk, uv = w[f"{pa}/mix/uk_t"], w[f"{pa}/mix/uv"]
+        k.add(f"per-head GEMM, queries {tag}", "design", lambda: ops.head_gemm(q, D + R, uk, q_abs, None, None, 0, False),
+              uk.numel() * 2 + T * H * (D + C) * 2, T * uk.numel())
+        k.add(f"per-head GEMM, values {tag}", "design", lambda: ops.head_gemm(o_lat, C, uv, out, None, None, 0, False),
+              uv.numel() * 2 + T * H * (V + C) * 2, T * uv.numel())
+    else:
+        rows = _rand(batch * total, C + R)
+        seqs = _ints([[i, i * total, total] for i in range(batch)])
+        ukv = w[f"{pa}/mix/ukv"]
+        wide, out, base = _rand(batch * total, ukv.shape[0]), _rand(T, H * V), _ints([i * total for i in range(batch)])
+        k.add(f"gather {tag}", "design", lambda: ops.latent_gather(pages, table, seqs, total, rows, False), rows.numel() * 4)
+        gemm("expansion", ukv, x=rows[:, :C])
+        k.add(f"attention {tag}", "design", lambda: ops.latent_expanded_attention(q, rows, wide, kv, H, C, m.rot_dim, m.scale, freq, sink, out, *blocks, row,
+                                                                                base, False),
+              wide.numel() * 2 + batch * total * R * 2 + T * H * (D + R + V) * 2, pairs * H * (D + R + V))
+    # gated memory
+    projm, gates = _rand(T, g.main_cols, s=0.5), torch.randn(T, g.gate_cols, device="cuda") + 3
+    S, out = torch.zeros((batch, g.heads, g.dim_p, g.vdim_p), device="cuda"), _rand(T, g.out_cols)
+    cws = None if new == 1 else torch.empty(int(ops.gated_chunked_workspace_bytes(T, batch, g.heads, g.dim_p, g.vdim_p)), dtype=torch.uint8, device="cuda")
+    k.add(f"recurrence {tag}", "design", lambda: ops.gated_memory(projm, 0, g.heads * g.dim_p, gates, w[f"{pm}/mix/lower"], g.vdim, 1e-6, w[f"{pm}/mix/norm"], cu,
+                                                                 slots, S, out, True, cws, False, new == 1),
+          2 * S.numel() * 4 + projm.numel() * 2 + gates.numel() * 4 + out.numel() * 2, 2.0 * T * g.heads * g.dim_p * g.vdim_p)
+
+
+def _kernels(cfg, other, weights, iters: int, only: str) -> List[dict]:
+    from ..models.layered import LayeredModel, LayeredWorkspace
+    latent = any(l.mixer.kind == "latent_attention" for l in cfg.layers)
+    model = LayeredModel(cfg, weights, "cuda:0")
+    ws = LayeredWorkspace(cfg, 64, 64, "cuda:0", torch.bfloat16)
+    ops = model._raw_ops
+    base, hyb = (other, equal_size_hybrid(other)) if latent else (cfg, other)
+    k = _Kernels(iters, only, {"design": "kuzanex", "hybrid": ""} if latent else None)
+    for T, tag in ((32, "decode x32"), (2048, "prefill 2048")):
+        _gemm_rows(k, ops, model.status.tensor, base, hyb, T, tag)
+    for batch, new, tag in ((32, 1, "decode x32"), (1, 2048, "prefill 2048")):
+        _attention_rows(k, ops, model, ws, base, hyb, batch, new, 2048, tag)
+    for batch, new, tag in ((32, 1, "decode x32"), (1, 2048, "prefill 2048")):
+        _memory_rows(k, ops, base, hyb, batch, new, tag)
+    if latent:
+        k.names = {}
+        for batch, new, tag in ((32, 1, "decode x32"), (1, 2048, "prefill 2048")):
+            _latent_design_rows(k, model, ws, cfg, batch, new, 2048, tag)
+    model.status.check("after the kernel timings")
+    return k.rows
+
+
 def compare(name: str, layers: int = 0, iters: int = 10, throughput: bool = True, only: str = "") -> Dict[str, object]:
     cfg = LAYERED_REGISTRY[name]
     if layers:
         cfg = cfg.shrink(layers)
-    hyb = equal_size_hybrid(cfg)
-    res: Dict[str, object] = {"comparison": cfg.name, "design_params": cfg.param_count(), "hybrid_params": hyb.param_count(), "dtype": "bf16",
+    latent = any(l.mixer.kind == "latent_attention" for l in cfg.layers)
+    other, label = (equal_size_kuzanex(cfg), "kuzanex") if latent else (equal_size_hybrid(cfg), "hybrid")
+    res: Dict[str, object] = {"comparison": cfg.name, "design_params": cfg.param_count(), f"{label}_params": other.param_count(), "dtype": "bf16",
                               "data": "synthetic", "l2": "flushed before every kernel"}
     weights = random_layered_weights(cfg, "cuda:0")
-    from ..models.layered import LayeredModel, LayeredWorkspace
-    model = LayeredModel(cfg, weights, "cuda:0")
-    ws = LayeredWorkspace(cfg, 64, 64, "cuda:0", torch.bfloat16)
-    ops = model._raw_ops
-    k = _Kernels(iters, only)
-    for T, tag in ((32, "decode x32"), (2048, "prefill 2048")):
-        _gemm_rows(k, ops, model.status.tensor, cfg, hyb, T, tag)
-    _attention_rows(k, ops, model, ws, cfg, hyb, 32, 1, 2048, "decode x32")
-    _attention_rows(k, ops, model, ws, cfg, hyb, 1, 2048, 2048, "prefill 2048")
-    _memory_rows(k, ops, cfg, hyb, 32, 1, "decode x32")
-    _memory_rows(k, ops, cfg, hyb, 1, 2048, "prefill 2048")
-    model.status.check("after the kernel timings")
-    del model, ws
-    rows: List[dict] = k.rows
+    rows = _kernels(cfg, other, weights, iters, only)
     pair: Dict[str, dict] = {}
     for r in rows:
         pair.setdefault(r["kernel"], {})[r["model"]] = r
     res["kernels"] = rows
-    res["farther_than_hybrid"] = {n: round(p["hybrid"]["fraction"] / p["design"]["fraction"], 2) for n, p in pair.items() if len(p) == 2}
+    res[f"farther_than_{label}"] = {n: round(p[label]["fraction"] / p["design"]["fraction"], 2) for n, p in pair.items() if len(p) == 2}
     if throughput:
         res["throughput"] = {}
-        w2 = random_weights(hyb, "cuda:0", seed=0)
+        w2 = random_layered_weights(other, "cuda:0") if latent else random_weights(other, "cuda:0", seed=0)
         for batch, prompt in ((1, 2048), (8, 1024), (32, 1024)):
             res["throughput"][f"{batch} x {prompt}"] = {"design": _throughput(cfg, weights, batch, prompt, 32),
-                                                        "hybrid": _throughput(hyb, w2, batch, prompt, 32)}
+                                                        label: _throughput(other, w2, batch, prompt, 32)}
     return res
 
 
