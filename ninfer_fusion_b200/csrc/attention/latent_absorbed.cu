@@ -1,9 +1,12 @@
 // Absorbed latent attention on the tensor cores (bf16): rows of the MMA are (token, head) pairs of one query block, so a
-// cached row is read once for all of them.  One CTA = (split of the keys, up to 16 MT rows, query block), eight warps.
-// Per tile of 32 keys, which live in a cp.async ring:
+// cached row is read once for all of them.  One CTA = (split of the keys, up to 16 MT rows, query block), NW = 8 or 16
+// warps.  Per tile of 4 NW keys, which live in a cp.async ring:
 //   scores   a warp owns eight keys (and a row tile, or half of the width when there is one row tile only)
-//   softmax  a warp owns 2 MT rows, a lane a key; weights go to shared memory in bf16, with the rows' rescale factors
+//   softmax  a warp owns 16 MT / NW rows, a lane one or two keys; weights go to shared memory in bf16, with the rows' rescale
+//            factors
 //   values   a warp owns 8 NT columns of the latent for all rows; the key tile is its own value tile
+// Sixteen warps serve the few rows of a decode step (three barriers per tile, so larger tiles and more warps hide more);
+// eight warps keep the 64 rows of a short portion in registers.
 #include "latent.h"
 
 #include <math_constants.h>
@@ -17,30 +20,30 @@ namespace nfb {
 namespace {
 
 using bf16 = __nv_bfloat16;
-constexpr int KT = 32, kThreads = 256, kLdS = KT + 4, kLdP = KT + 8;
 
 struct Plan {
   int ldk, q, ring, stage, s, p, alpha, len, total;
-  __host__ __device__ Plan(int rows, int width, int stages, int halves) {
+  __host__ __device__ Plan(int rows, int width, int stages, int halves, int keys) {
     ldk = width + 8;
     q = 0;
     ring = q + rows * ldk * 2;
-    stage = KT * ldk * 2;
+    stage = keys * ldk * 2;
     s = ring + stages * stage;
-    p = s + halves * rows * kLdS * 4;
-    alpha = p + rows * kLdP * 2;
+    p = s + halves * rows * (keys + 4) * 4;
+    alpha = p + rows * (keys + 8) * 2;
     len = alpha + rows * 2 * 4;                  // two floats per row: rescale factor / maximum and sum at the end
     total = len + rows * 4;
   }
 };
 
-template <int MT, int NT, int S>
-__global__ void __launch_bounds__(kThreads) latent_absorbed_kernel(const LatentArgs p, const LatentBlocks b, int split_keys, int n_splits,
+template <int NW, int MT, int NT, int S>
+__global__ void __launch_bounds__(NW * 32) latent_absorbed_kernel(const LatentArgs p, const LatentBlocks b, int split_keys, int n_splits,
                                                                     float* __restrict__ part_o, float* __restrict__ part_ml) {
-  constexpr int M = 16 * MT, kHalves = MT == 1 ? 2 : 1, kRows = 2 * MT;
+  constexpr int KT = 4 * NW, kThreads = NW * 32, kLdS = KT + 4, kLdP = KT + 8;
+  constexpr int M = 16 * MT, kHalves = MT == 1 ? 2 : 1, kRows = M / NW, kPer = KT / 32, kLoad = KT / NW;
   extern __shared__ __align__(16) uint8_t smem[];
   const int H = p.n_heads, W = p.rank + p.rot, P = p.page_size;
-  const Plan plan(M, W, S, kHalves);
+  const Plan plan(M, W, S, kHalves, KT);
   bf16* qs = reinterpret_cast<bf16*>(smem + plan.q);
   float* ss = reinterpret_cast<float*>(smem + plan.s);
   bf16* ps = reinterpret_cast<bf16*>(smem + plan.p);
@@ -64,11 +67,11 @@ __global__ void __launch_bounds__(kThreads) latent_absorbed_kernel(const LatentA
   const uint32_t qs_a = smem_u32(qs), ps_a = smem_u32(ps), ring_a = smem_u32(smem) + plan.ring;
   const int ldk = plan.ldk, vecs = W / 8;
 
-  int row_at[KT / 8];          // page * P + place of the warp's rows of the tile to load next, -1: none
+  int row_at[kLoad];          // page * P + place of the warp's rows of the tile to load next, -1: none
   auto look_up = [&](int tile) {
 #pragma unroll
-    for (int j = 0; j < KT / 8; ++j) {
-      const int key = k_begin + tile * KT + j * 8 + warp;
+    for (int j = 0; j < kLoad; ++j) {
+      const int key = k_begin + tile * KT + j * NW + warp;
       const int page = key < k_end ? table[key / P] : -1;
       row_at[j] = page < 0 ? -1 : page * P + key % P;
     }
@@ -76,10 +79,10 @@ __global__ void __launch_bounds__(kThreads) latent_absorbed_kernel(const LatentA
   auto load = [&](int tile) {
     const uint32_t dst = ring_a + (tile % S) * plan.stage;
 #pragma unroll
-    for (int j = 0; j < KT / 8; ++j) {
+    for (int j = 0; j < kLoad; ++j) {
       const bool ok = row_at[j] >= 0;
       const bf16* src = pages + static_cast<long long>(ok ? row_at[j] : 0) * W;
-      for (int c = lane; c < vecs; c += 32) cp_async16(dst + ((j * 8 + warp) * ldk + c * 8) * 2, src + c * 8, ok);
+      for (int c = lane; c < vecs; c += 32) cp_async16(dst + ((j * NW + warp) * ldk + c * 8) * 2, src + c * 8, ok);
     }
   };
 #pragma unroll
@@ -129,7 +132,7 @@ __global__ void __launch_bounds__(kThreads) latent_absorbed_kernel(const LatentA
   for (int i = 0; i < kRows; ++i) { mx[i] = -CUDART_INF_F; l[i] = 0.f; }
   const float scale2 = p.scale * kLog2e;
   const int n_steps = W / 16, col0 = warp * NT * 8;
-  const int nt = warp & 3, grp = warp >> 2;        // eight keys; half of the width (MT = 1) or row tiles grp, grp + 2
+  const int nt = warp % (KT / 8), grp = warp / (KT / 8);        // eight keys; half of the width (MT = 1) or row tiles grp, grp + 2
   const int half = (n_steps / 2 + 1) & ~1;
   const int ks0 = MT == 1 && grp == 1 ? half : 0, ks1 = MT == 1 && grp == 0 ? half : n_steps;
 
@@ -175,20 +178,29 @@ __global__ void __launch_bounds__(kThreads) latent_absorbed_kernel(const LatentA
     const int key = k_begin + tile * KT + lane;
 #pragma unroll
     for (int i = 0; i < kRows; ++i) {
-      const int row = warp * kRows + i;
-      float v = ss[row * kLdS + lane];
-      if constexpr (MT == 1) v += ss[(row + M) * kLdS + lane];
-      v = key < row_len[row] && key < k_end ? v * scale2 : -CUDART_INF_F;
-      float t = v;
+      const int row = warp * kRows + i, limit = min(row_len[row], k_end);
+      float v[kPer], t = -CUDART_INF_F;
+#pragma unroll
+      for (int j = 0; j < kPer; ++j) {
+        v[j] = ss[row * kLdS + lane + 32 * j];
+        if constexpr (MT == 1) v[j] += ss[(row + M) * kLdS + lane + 32 * j];
+        v[j] = key + 32 * j < limit ? v[j] * scale2 : -CUDART_INF_F;
+        t = fmaxf(t, v[j]);
+      }
 #pragma unroll
       for (int off = 16; off > 0; off >>= 1) t = fmaxf(t, __shfl_xor_sync(0xffffffffu, t, off));
       const float m_new = fmaxf(mx[i], t);
       const bool any = m_new > -CUDART_INF_F;
-      const float w = any ? ex2_fast(v - m_new) : 0.f;
       const float f = any ? ex2_fast(mx[i] - m_new) : 1.f;
-      l[i] = l[i] * f + warp_sum(w);
+      float sum = 0.f;
+#pragma unroll
+      for (int j = 0; j < kPer; ++j) {
+        const float w = any ? ex2_fast(v[j] - m_new) : 0.f;
+        sum += w;
+        ps[row * kLdP + lane + 32 * j] = __float2bfloat16(w);
+      }
+      l[i] = l[i] * f + warp_sum(sum);
       mx[i] = m_new;
-      ps[row * kLdP + lane] = __float2bfloat16(w);
       if (lane == 0) alpha[row] = f;
     }
     __syncthreads();
@@ -299,37 +311,38 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentArgs p, c
 
 constexpr int kSmemLimit = 225 * 1024;
 
-template <int MT, int NT, int S>
+template <int NW, int MT, int NT, int S>
 cudaError_t launch(const LatentArgs& a, const LatentBlocks& b, int split_keys, int n_splits, float* part_o, float* part_ml) {
-  const Plan plan(16 * MT, a.rank + a.rot, S, MT == 1 ? 2 : 1);
-  auto kern = latent_absorbed_kernel<MT, NT, S>;
+  const Plan plan(16 * MT, a.rank + a.rot, S, MT == 1 ? 2 : 1, 4 * NW);
+  auto kern = latent_absorbed_kernel<NW, MT, NT, S>;
   const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, plan.total);
   if (e != cudaSuccess) return e;
   const int row_blocks = (b.max_count * a.n_heads + 16 * MT - 1) / (16 * MT);
-  return launch_kernel(kern, dim3(n_splits, row_blocks, b.n), dim3(kThreads), plan.total, a.stream, a.pdl, 1, a, b, split_keys, n_splits,
+  return launch_kernel(kern, dim3(n_splits, row_blocks, b.n), dim3(NW * 32), plan.total, a.stream, a.pdl, 1, a, b, split_keys, n_splits,
                        part_o, part_ml);
 }
 
-template <int MT, int NT>
+template <int NW, int MT, int NT>
 cudaError_t pick_stages(const LatentArgs& a, const LatentBlocks& b, int split_keys, int n_splits, float* part_o, float* part_ml) {
-  if (Plan(16 * MT, a.rank + a.rot, 3, MT == 1 ? 2 : 1).total <= kSmemLimit) return launch<MT, NT, 3>(a, b, split_keys, n_splits, part_o, part_ml);
-  return launch<MT, NT, 2>(a, b, split_keys, n_splits, part_o, part_ml);
+  if (Plan(16 * MT, a.rank + a.rot, 3, MT == 1 ? 2 : 1, 4 * NW).total <= kSmemLimit)
+    return launch<NW, MT, NT, 3>(a, b, split_keys, n_splits, part_o, part_ml);
+  return launch<NW, MT, NT, 2>(a, b, split_keys, n_splits, part_o, part_ml);
 }
 
+// NT: columns per warp / 8 with sixteen warps; eight warps hold twice as many.
 template <int NT>
 cudaError_t pick_rows(const LatentArgs& a, const LatentBlocks& b, int split_keys, int n_splits, float* part_o, float* part_ml) {
   const int rows = b.max_count * a.n_heads;
-  if (rows <= 16) return pick_stages<1, NT>(a, b, split_keys, n_splits, part_o, part_ml);
-  if constexpr (NT <= 8) {
-    if (rows > 32) return pick_stages<4, NT>(a, b, split_keys, n_splits, part_o, part_ml);
-  }
-  return pick_stages<2, NT>(a, b, split_keys, n_splits, part_o, part_ml);
+  if (rows <= 16) return pick_stages<16, 1, NT>(a, b, split_keys, n_splits, part_o, part_ml);
+  if (rows <= 32) return pick_stages<16, 2, NT>(a, b, split_keys, n_splits, part_o, part_ml);
+  return pick_stages<8, 4, 2 * NT>(a, b, split_keys, n_splits, part_o, part_ml);
 }
 
 }  // namespace
 
 bool latent_absorbed_supported(int rank, int rot) {
-  return rank % 16 == 0 && rot % 16 == 0 && rank > 0 && rank <= 512 && Plan(64, rank + rot, 2, 1).total <= kSmemLimit;
+  return rank % 16 == 0 && rot % 16 == 0 && rank > 0 && rank <= 512 && Plan(64, rank + rot, 2, 1, 32).total <= kSmemLimit &&
+         Plan(32, rank + rot, 2, 1, 64).total <= kSmemLimit;
 }
 
 const char* latent_absorbed_attention(const LatentArgs& a, const LatentBlocks& b, int split_keys, int n_splits, float* part_o,
@@ -344,9 +357,8 @@ const char* latent_absorbed_attention(const LatentArgs& a, const LatentBlocks& b
   if (a.n_heads > 4096) return "latent_absorbed_attention: too many heads";
   if (n_splits > 1 && (part_o == nullptr || part_ml == nullptr)) return "latent_absorbed_attention: splits need their workspace";
   cudaError_t e;
-  if (a.rank <= 128) e = pick_rows<2>(a, b, split_keys, n_splits, part_o, part_ml);
-  else if (a.rank <= 256) e = pick_rows<4>(a, b, split_keys, n_splits, part_o, part_ml);
-  else e = pick_rows<8>(a, b, split_keys, n_splits, part_o, part_ml);
+  if (a.rank <= 256) e = pick_rows<2>(a, b, split_keys, n_splits, part_o, part_ml);
+  else e = pick_rows<4>(a, b, split_keys, n_splits, part_o, part_ml);
   if (e == cudaSuccess && n_splits > 1)
     e = launch_kernel(latent_merge_kernel, dim3(a.T, a.n_heads), dim3(128), 0, a.stream, a.pdl, 1, a, b, n_splits, const_cast<const float*>(part_o),
                       const_cast<const float*>(part_ml));

@@ -14,7 +14,7 @@ namespace nfb {
 
 namespace {
 
-constexpr int kBlockTokens = 8;
+constexpr int kBlockTokens = 4;
 
 // How the sum of squares of a group is taken: whole warps lie in one group / whole 8-column vectors do / neither.
 enum GroupMode : int { kWarpGroups = 0, kVectorGroups = 1, kColumnGroups = 2 };
@@ -67,7 +67,7 @@ __device__ __forceinline__ void group_inv(const float (&v)[KV][8], float (&inv)[
 }
 
 template <typename A, int KV, int MODE, bool CONV>
-__global__ void __launch_bounds__(1024) sandwich_kernel(const SandwichArgs p) {
+__global__ void __launch_bounds__(512) sandwich_kernel(const SandwichArgs p) {
   extern __shared__ __align__(16) float smem[];
   const int group_size = p.n_true / p.groups;
   const int n_part = MODE == kWarpGroups ? (p.N + 255) / 256 : (MODE == kVectorGroups ? p.N / 8 : p.N);
@@ -78,24 +78,32 @@ __global__ void __launch_bounds__(1024) sandwich_kernel(const SandwichArgs p) {
   pdl_launch_next();
   pdl_wait_prior();
 
-  float h[KV][8];
-  // h of row t; `store`: the row's new residual is kept
-  auto row = [&](long long t, bool store) {
-    float inv[KV][MODE == kColumnGroups ? 8 : 1];
+  float h[KV][8], x_next[KV][8], d_next[KV][8];
+  auto fetch = [&](long long t) {
 #pragma unroll
     for (int i = 0; i < KV; ++i) {
       const int c = (tid + i * nt) * 8;
-#pragma unroll
-      for (int j = 0; j < 8; ++j) h[i][j] = 0.f;
-      if (c < p.N) load8((p.delta != nullptr ? p.delta : p.x_in) + t * p.N + c, h[i]);
-    }
-    if (p.delta != nullptr) {
-      float x[KV][8];
-#pragma unroll
-      for (int i = 0; i < KV; ++i) {
-        const int c = (tid + i * nt) * 8;
-        if (c < p.N) load8(p.x_in + t * p.N + c, x[i]);
+      if (c < p.N) {
+        load8(p.x_in + t * p.N + c, x_next[i]);
+        if (p.delta != nullptr) load8(p.delta + t * p.N + c, d_next[i]);
       }
+    }
+  };
+  // h of row t, whose inputs have been fetched; fetches those of row `then` (-1: none).  `store`: the new residual is kept
+  auto row = [&](long long t, bool store, long long then) {
+    float inv[KV][MODE == kColumnGroups ? 8 : 1];
+    float x[KV][8];
+#pragma unroll
+    for (int i = 0; i < KV; ++i) {
+      const bool ok = (tid + i * nt) * 8 < p.N;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        x[i][j] = x_next[i][j];
+        h[i][j] = ok ? (p.delta != nullptr ? d_next[i][j] : x[i][j]) : 0.f;
+      }
+    }
+    if (then >= 0) fetch(then);
+    if (p.delta != nullptr) {
       group_inv<KV, MODE>(h, inv, part, inv_s, p, group_size);
 #pragma unroll
       for (int i = 0; i < KV; ++i) {
@@ -126,7 +134,8 @@ __global__ void __launch_bounds__(1024) sandwich_kernel(const SandwichArgs p) {
   A* out = static_cast<A*>(p.out);
   if constexpr (!CONV) {
     const long long t = blockIdx.x;
-    row(t, true);
+    fetch(t);
+    row(t, true, -1);
 #pragma unroll
     for (int i = 0; i < KV; ++i) {
       const int c = (tid + i * nt) * 8;
@@ -145,12 +154,13 @@ __global__ void __launch_bounds__(1024) sandwich_kernel(const SandwichArgs p) {
         if (c < p.N) store8(dst + c, h[i]);
       }
     };
+    fetch(tb + max(i0 - K, 0));
     // history rows of tokens i0 - K .. i0 - 1
     for (int j = 0; j < K; ++j) {
       const int i = i0 - K + j;
       float* dst = hist + ((i + K) % K) * p.N;
       if (i >= 0) {
-        row(tb + i, false);
+        row(tb + i, false, tb + i + 1);
         keep(dst);
       } else {
 #pragma unroll
@@ -165,7 +175,7 @@ __global__ void __launch_bounds__(1024) sandwich_kernel(const SandwichArgs p) {
       }
     }
     for (int i = i0; i < i1; ++i) {
-      row(tb + i, true);
+      row(tb + i, true, i + 1 < i1 ? tb + i + 1 : -1);
 #pragma unroll
       for (int k = 0; k < KV; ++k) {
         const int c = (tid + k * nt) * 8;
@@ -204,7 +214,8 @@ __global__ void __launch_bounds__(1024) sandwich_kernel(const SandwichArgs p) {
           continue;
         }
       }
-      row(tb + i, false);
+      fetch(tb + i);
+      row(tb + i, false, -1);
       keep(state + static_cast<long long>(j) * p.N);
     }
   }
@@ -237,15 +248,15 @@ template <typename A>
 cudaError_t pick_width(const SandwichArgs& a, cudaStream_t stream, bool pdl) {
   const int vecs = a.N / 8;
   if (vecs <= 512) return pick_mode<A, 1>(a, (vecs + 31) / 32 * 32, stream, pdl);
-  if (vecs <= 2048) return pick_mode<A, 2>(a, ((vecs + 1) / 2 + 31) / 32 * 32, stream, pdl);
-  return pick_mode<A, 4>(a, 1024, stream, pdl);
+  if (vecs <= 1024) return pick_mode<A, 2>(a, ((vecs + 1) / 2 + 31) / 32 * 32, stream, pdl);
+  return pick_mode<A, 4>(a, 512, stream, pdl);
 }
 
 }  // namespace
 
 const char* sandwich_rows(const SandwichArgs& a, cudaStream_t stream, bool pdl) {
   if (a.T <= 0) return nullptr;
-  if (a.N % 8 || a.ld_out % 8 || a.n_true <= 0 || a.n_true > a.N || a.N > 32768) return "sandwich_rows: bad row width (up to 32768 columns)";
+  if (a.N % 8 || a.ld_out % 8 || a.n_true <= 0 || a.n_true > a.N || a.N > 16384) return "sandwich_rows: bad row width (up to 16384 columns)";
   if (a.groups < 1 || a.n_true % a.groups || a.groups > 4096) return "sandwich_rows: the width is not a multiple of the groups";
   if (a.delta != nullptr && (a.w_post == nullptr || a.x_out == nullptr)) return "sandwich_rows: a sublayer output needs its norm and a destination";
   if (a.conv_w != nullptr) {

@@ -37,7 +37,7 @@ def ints(x):
 
 # ---------------------------------------------------------------------------- rows
 @pytest.mark.parametrize("dt", DTYPES)
-@pytest.mark.parametrize("n_true,groups", [(150, 6), (96, 3), (150, 1), (2048, 4), (4096, 1), (5000, 8), (9216, 9), (24, 24)])
+@pytest.mark.parametrize("n_true,groups", [(150, 6), (96, 3), (150, 1), (2048, 4), (4096, 1), (5000, 8), (9216, 9), (12288, 3), (24, 24)])
 def test_norms_around_a_sublayer(ops, dt, n_true, groups):
     """Whole warps per group, whole vectors per group, neither; with and without the update and the next norm."""
     T, N, mult, eps = 5, (n_true + 7) // 8 * 8, 0.35, 1e-3
