@@ -1,7 +1,7 @@
 // Absorbed latent attention on the tensor cores (bf16): rows of the MMA are (token, head) pairs of one query block, so a
 // cached row is read once for all of them.  One CTA = (split of the keys, up to 16 MT rows, query block), NW = 8 or 16
 // warps.  Per tile of 4 NW keys, which live in a cp.async ring:
-//   scores   a warp owns eight keys (and a row tile, or half of the width when there is one row tile only)
+//   scores   a warp owns sixteen keys and a quarter of the width, for all rows
 //   softmax  a warp owns 16 MT / NW rows, a lane one or two keys; weights go to shared memory in bf16, with the rows' rescale
 //            factors
 //   values   a warp owns 8 NT columns of the latent for all rows; the key tile is its own value tile
@@ -23,13 +23,13 @@ using bf16 = __nv_bfloat16;
 
 struct Plan {
   int ldk, q, ring, stage, s, p, alpha, len, total;
-  __host__ __device__ Plan(int rows, int width, int stages, int halves, int keys) {
+  __host__ __device__ Plan(int rows, int width, int stages, int keys) {
     ldk = width + 8;
     q = 0;
     ring = q + rows * ldk * 2;
     stage = keys * ldk * 2;
     s = ring + stages * stage;
-    p = s + halves * rows * (keys + 4) * 4;
+    p = s + 4 * rows * (keys + 4) * 4;            // one score array per quarter of the width
     alpha = p + rows * (keys + 8) * 2;
     len = alpha + rows * 2 * 4;                  // two floats per row: rescale factor / maximum and sum at the end
     total = len + rows * 4;
@@ -40,10 +40,10 @@ template <int NW, int MT, int NT, int S>
 __global__ void __launch_bounds__(NW * 32) latent_absorbed_kernel(const LatentArgs p, const LatentBlocks b, int split_keys, int n_splits,
                                                                     float* __restrict__ part_o, float* __restrict__ part_ml) {
   constexpr int KT = 4 * NW, kThreads = NW * 32, kLdS = KT + 4, kLdP = KT + 8;
-  constexpr int M = 16 * MT, kHalves = MT == 1 ? 2 : 1, kRows = M / NW, kPer = KT / 32, kLoad = KT / NW;
+  constexpr int M = 16 * MT, kRows = M / NW, kPer = KT / 32, kLoad = KT / NW;
   extern __shared__ __align__(16) uint8_t smem[];
   const int H = p.n_heads, W = p.rank + p.rot, P = p.page_size;
-  const Plan plan(M, W, S, kHalves, KT);
+  const Plan plan(M, W, S, KT);
   bf16* qs = reinterpret_cast<bf16*>(smem + plan.q);
   float* ss = reinterpret_cast<float*>(smem + plan.s);
   bf16* ps = reinterpret_cast<bf16*>(smem + plan.p);
@@ -132,9 +132,8 @@ __global__ void __launch_bounds__(NW * 32) latent_absorbed_kernel(const LatentAr
   for (int i = 0; i < kRows; ++i) { mx[i] = -CUDART_INF_F; l[i] = 0.f; }
   const float scale2 = p.scale * kLog2e;
   const int n_steps = W / 16, col0 = warp * NT * 8;
-  const int nt = warp % (KT / 8), grp = warp / (KT / 8);        // eight keys; half of the width (MT = 1) or row tiles grp, grp + 2
-  const int half = (n_steps / 2 + 1) & ~1;
-  const int ks0 = MT == 1 && grp == 1 ? half : 0, ks1 = MT == 1 && grp == 0 ? half : n_steps;
+  const int kg = warp % (KT / 16), quarter = warp / (KT / 16), q_steps = (n_steps + 3) / 4;
+  const int ks0 = quarter * q_steps, ks1 = min(n_steps, ks0 + q_steps);
 
   for (int tile = 0; tile < n_tiles; ++tile) {
     cp_async_wait<S - 2>();
@@ -144,34 +143,33 @@ __global__ void __launch_bounds__(NW * 32) latent_absorbed_kernel(const LatentAr
     look_up(tile + S);
     const uint32_t kt = ring_a + (tile % S) * plan.stage;
     // ---- scores ----
-    constexpr int kTiles = MT == 4 ? 2 : 1;
-    float c[kTiles][2][4];
+    float c[MT][2][4];
 #pragma unroll
-    for (int i = 0; i < kTiles; ++i)
+    for (int i = 0; i < MT; ++i)
 #pragma unroll
       for (int e = 0; e < 4; ++e) c[i][0][e] = c[i][1][e] = 0.f;
-    const uint32_t b_at = kt + ((nt * 8 + (lane & 7)) * ldk + (lane >> 3) * 8) * 2;
-    const uint32_t a_at = qs_a + (((MT == 1 ? 0 : grp) * 16 + (lane & 15)) * ldk + (lane >> 4) * 8) * 2;
-#pragma unroll 2
-    for (int ks = ks0; ks < ks1; ks += 2) {
+    const uint32_t b_at = kt + ((kg * 16 + (lane & 7) + (lane >> 4) * 8) * ldk + ((lane >> 3) & 1) * 8) * 2;
+    const uint32_t a_at = qs_a + ((lane & 15) * ldk + (lane >> 4) * 8) * 2;
+#pragma unroll 3
+    for (int ks = ks0; ks < ks1; ++ks) {
       uint32_t bk[4];
-      ldsm_x4(b_at + ks * 32, bk);                 // two steps of sixteen columns
+      ldsm_x4(b_at + ks * 32, bk);
 #pragma unroll
-      for (int i = 0; i < kTiles; ++i) {
+      for (int i = 0; i < MT; ++i) {
         uint32_t a[4];
-        ldsm_x4(a_at + i * (32 * ldk * 2) + ks * 32, a);
+        ldsm_x4(a_at + i * (16 * ldk * 2) + ks * 32, a);
         mma_bf16_16816(c[i][0], a, bk[0], bk[1]);
-        if (ks + 1 < ks1) {
-          ldsm_x4(a_at + i * (32 * ldk * 2) + ks * 32 + 32, a);
-          mma_bf16_16816(c[i][1], a, bk[2], bk[3]);
-        }
+        mma_bf16_16816(c[i][1], a, bk[2], bk[3]);
       }
     }
 #pragma unroll
-    for (int i = 0; i < kTiles; ++i) {
-      const int row = (MT == 1 ? grp * M : (grp + 2 * i) * 16) + r4;
-      *reinterpret_cast<float2*>(ss + row * kLdS + nt * 8 + c4 * 2) = make_float2(c[i][0][0] + c[i][1][0], c[i][0][1] + c[i][1][1]);
-      *reinterpret_cast<float2*>(ss + (row + 8) * kLdS + nt * 8 + c4 * 2) = make_float2(c[i][0][2] + c[i][1][2], c[i][0][3] + c[i][1][3]);
+    for (int i = 0; i < MT; ++i) {
+#pragma unroll
+      for (int n = 0; n < 2; ++n) {
+        float* dst = ss + (quarter * M + i * 16 + r4) * kLdS + kg * 16 + n * 8 + c4 * 2;
+        *reinterpret_cast<float2*>(dst) = make_float2(c[i][n][0], c[i][n][1]);
+        *reinterpret_cast<float2*>(dst + 8 * kLdS) = make_float2(c[i][n][2], c[i][n][3]);
+      }
     }
     __syncthreads();
     // ---- softmax ----
@@ -182,8 +180,8 @@ __global__ void __launch_bounds__(NW * 32) latent_absorbed_kernel(const LatentAr
       float v[kPer], t = -CUDART_INF_F;
 #pragma unroll
       for (int j = 0; j < kPer; ++j) {
-        v[j] = ss[row * kLdS + lane + 32 * j];
-        if constexpr (MT == 1) v[j] += ss[(row + M) * kLdS + lane + 32 * j];
+        const float* sp = ss + row * kLdS + lane + 32 * j;
+        v[j] = (sp[0] + sp[M * kLdS]) + (sp[2 * M * kLdS] + sp[3 * M * kLdS]);
         v[j] = key + 32 * j < limit ? v[j] * scale2 : -CUDART_INF_F;
         t = fmaxf(t, v[j]);
       }
@@ -313,7 +311,7 @@ constexpr int kSmemLimit = 225 * 1024;
 
 template <int NW, int MT, int NT, int S>
 cudaError_t launch(const LatentArgs& a, const LatentBlocks& b, int split_keys, int n_splits, float* part_o, float* part_ml) {
-  const Plan plan(16 * MT, a.rank + a.rot, S, MT == 1 ? 2 : 1, 4 * NW);
+  const Plan plan(16 * MT, a.rank + a.rot, S, 4 * NW);
   auto kern = latent_absorbed_kernel<NW, MT, NT, S>;
   const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, plan.total);
   if (e != cudaSuccess) return e;
@@ -324,7 +322,7 @@ cudaError_t launch(const LatentArgs& a, const LatentBlocks& b, int split_keys, i
 
 template <int NW, int MT, int NT>
 cudaError_t pick_stages(const LatentArgs& a, const LatentBlocks& b, int split_keys, int n_splits, float* part_o, float* part_ml) {
-  if (Plan(16 * MT, a.rank + a.rot, 3, MT == 1 ? 2 : 1, 4 * NW).total <= kSmemLimit)
+  if (Plan(16 * MT, a.rank + a.rot, 3, 4 * NW).total <= kSmemLimit)
     return launch<NW, MT, NT, 3>(a, b, split_keys, n_splits, part_o, part_ml);
   return launch<NW, MT, NT, 2>(a, b, split_keys, n_splits, part_o, part_ml);
 }
@@ -341,8 +339,8 @@ cudaError_t pick_rows(const LatentArgs& a, const LatentBlocks& b, int split_keys
 }  // namespace
 
 bool latent_absorbed_supported(int rank, int rot) {
-  return rank % 16 == 0 && rot % 16 == 0 && rank > 0 && rank <= 512 && Plan(64, rank + rot, 2, 1, 32).total <= kSmemLimit &&
-         Plan(32, rank + rot, 2, 1, 64).total <= kSmemLimit;
+  return rank % 16 == 0 && rot % 16 == 0 && rank > 0 && rank <= 512 && Plan(64, rank + rot, 2, 32).total <= kSmemLimit &&
+         Plan(32, rank + rot, 2, 64).total <= kSmemLimit;
 }
 
 const char* latent_absorbed_attention(const LatentArgs& a, const LatentBlocks& b, int split_keys, int n_splits, float* part_o,

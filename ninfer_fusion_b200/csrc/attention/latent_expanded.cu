@@ -52,19 +52,32 @@ __global__ void __launch_bounds__(kThreads) latent_flash_kernel(const LatentArgs
   const bf16* vals = static_cast<const bf16*>(x.kv) + base * ldx + static_cast<long long>(H) * D + static_cast<long long>(h) * V;
   const bf16* rots = static_cast<const bf16*>(x.rows) + static_cast<long long>(base) * (p.rank + R) + p.rank;
   const int kv8 = W / 8, d8 = D / 8, v8 = V / 8;
-  // thread -> (row, lane of the row): 16 threads walk a row
+  // 16 threads walk a row; a thread's rows of a tile are lr, lr + 8, ..., its 16-byte pieces lc, lc + 16, ...
   const int lr = tid >> 4, lc = tid & 15;
-  auto load = [&](int tile) {
-    const uint32_t dk = ring_a + (tile & 1) * stage * 2, dv = dk + KT * ldk * 2;
+  auto copy = [&](uint32_t dst, int ld_dst, const bf16* src, long long ld_src, int left) {   // one piece of the tile's rows
+    if (left >= KT) {
 #pragma unroll
-    for (int j = 0; j < KT / 8; ++j) {
-      const int r = lr + j * 8, key = tile * KT + r;
-      const bool ok = key < len;
-      const long long kr = ok ? key : 0;
-      for (int c = lc; c < kv8; c += 16)
-        cp_async16(dk + (r * ldk + c * 8) * 2, c < d8 ? keys + kr * ldx + c * 8 : rots + kr * (p.rank + R) + (c - d8) * 8, ok);
-      for (int c = lc; c < v8; c += 16) cp_async16(dv + (r * ldv + c * 8) * 2, vals + kr * ldx + c * 8, ok);
+      for (int j = 0; j < KT / 8; ++j) {
+        cp_async16(dst + j * (8 * ld_dst * 2), src, true);
+        src += 8 * ld_src;
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < KT / 8; ++j) {
+        const bool ok = lr + j * 8 < left;
+        cp_async16(dst + j * (8 * ld_dst * 2), ok ? src : keys, ok);
+        src += 8 * ld_src;
+      }
     }
+  };
+  auto load = [&](int tile) {
+    const uint32_t dk = ring_a + (tile & 1) * stage * 2 + lr * ldk * 2, dv = ring_a + ((tile & 1) * stage + KT * ldk + lr * ldv) * 2;
+    const int left = len - tile * KT;
+    const long long first = static_cast<long long>(tile) * KT + lr;
+    const long long ldr = p.rank + R;
+    for (int c = lc; c < kv8; c += 16)
+      copy(dk + c * 16, ldk, c < d8 ? keys + first * ldx + c * 8 : rots + first * ldr + (c - d8) * 8, c < d8 ? ldx : ldr, left);
+    for (int c = lc; c < v8; c += 16) copy(dv + c * 16, ldv, vals + first * ldx + c * 8, ldx, left);
   };
   load(0);
   cp_async_commit();

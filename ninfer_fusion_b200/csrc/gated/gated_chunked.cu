@@ -85,12 +85,15 @@ __global__ void __launch_bounds__(kThreads) gated_contrib_kernel(const GatedArgs
   {
     const float lower = d < nd ? p.lower[h * D + d0 + d] : 1.f;
     const float* g = p.gates + static_cast<long long>(t0 + blk * B) * p.ldg + h * D + d0 + d;
-    float f[B];
+    const int n = d < nd ? min(B, len - blk * B) : 0;    // tokens of the block that exist
+    float f[B], raw[B];
+#pragma unroll
+    for (int j = 0; j < B; ++j) raw[j] = j < n ? __ldg(g + j * p.ldg) : 0.f;
 #pragma unroll
     for (int j = 0; j < B; ++j) {
-      f[j] = 1.f;
-      k[j] = 0.f;
-      if (blk * B + j < len && d < nd) gated_forget(g[j * p.ldg], lower, f[j], k[j]);
+      gated_forget(raw[j], lower, f[j], k[j]);
+      f[j] = j < n ? f[j] : 1.f;
+      k[j] = j < n ? k[j] : 0.f;
     }
 #pragma unroll
     for (int j = B - 1; j >= 0; --j) {
@@ -281,16 +284,19 @@ __global__ void __launch_bounds__(kThreads, NT <= 2 ? 2 : 1) gated_output_kernel
       const float lower = d < nd ? p.lower[h * D + d0 + d] : 1.f;
       const float* g = p.gates + static_cast<long long>(t0 + blk * B) * p.ldg + h * D + d0 + d;
       const bf16* qr = proj + static_cast<long long>(t0 + blk * B) * p.ldp + p.q_off + h * D + d0 + d;
+      const int n = d < nd ? min(B, len - blk * B) : 0;    // tokens of the block that exist
 #pragma unroll
       for (int j = 0; j < B; ++j) {
-        f[j] = 1.f;
-        k[j] = 0.f;
-        q[j] = 0.f;
-        if (blk * B + j < len && d < nd) {
-          gated_forget(g[j * p.ldg], lower, f[j], k[j]);
-          const float z = __bfloat162float(qr[j * p.ldp]);
-          q[j] = z * sigmoid_of<bf16>(z);
-        }
+        f[j] = j < n ? __ldg(g + j * p.ldg) : 0.f;
+        q[j] = j < n ? __bfloat162float(qr[j * p.ldp]) : 0.f;
+      }
+#pragma unroll
+      for (int j = 0; j < B; ++j) {
+        const float raw = f[j];
+        gated_forget(raw, lower, f[j], k[j]);
+        f[j] = j < n ? f[j] : 1.f;
+        k[j] = j < n ? k[j] : 0.f;
+        q[j] = q[j] * sigmoid_of<bf16>(q[j]);
       }
     }
     __syncthreads();            // the last pass is done with the arrays

@@ -14,13 +14,14 @@ namespace nfb {
 
 namespace {
 
-constexpr int kBlockTokens = 4;
+constexpr int kBlockTokens = 8;
 
 // How the sum of squares of a group is taken: whole warps lie in one group / whole 8-column vectors do / neither.
 enum GroupMode : int { kWarpGroups = 0, kVectorGroups = 1, kColumnGroups = 2 };
 
 // 1 / rms of the group of each of the thread's columns: inv[i][j] for column j of vector i (j = 0 stands for all eight
-// unless the mode is kColumnGroups).  `part` and `inv_s` are shared; every thread of the CTA takes part.
+// unless the mode is kColumnGroups).  `part` and `inv_s` are shared, `part` alternates between two arrays from call to call;
+// every thread of the CTA takes part.
 template <int KV, int MODE>
 __device__ __forceinline__ void group_inv(const float (&v)[KV][8], float (&inv)[KV][MODE == kColumnGroups ? 8 : 1], float* part,
                                           float* inv_s, const SandwichArgs& p, int group_size) {
@@ -49,6 +50,19 @@ __device__ __forceinline__ void group_inv(const float (&v)[KV][8], float (&inv)[
   __syncthreads();
   const int units = group_size / kUnit;
   const float inv_n = 1.f / static_cast<float>(group_size);
+  if constexpr (MODE == kWarpGroups) {      // few partial sums per group: every thread adds its own up
+#pragma unroll
+    for (int i = 0; i < KV; ++i) {
+      const int c = (tid + i * nt) * 8;
+      if (c < p.N) {
+        const float* src = part + c / group_size * units;
+        float s = 0.f;
+        for (int u = 0; u < units; ++u) s += src[u];
+        inv[i][0] = 1.f / sqrtf(s * inv_n + p.eps);
+      }
+    }
+    return;
+  }
   for (int g = warp; g < p.groups; g += nt >> 5) {
     float s = 0.f;
     for (int u = lane; u < units; u += 32) s += part[g * units + u];
@@ -67,44 +81,40 @@ __device__ __forceinline__ void group_inv(const float (&v)[KV][8], float (&inv)[
 }
 
 template <typename A, int KV, int MODE, bool CONV>
-__global__ void __launch_bounds__(512) sandwich_kernel(const SandwichArgs p) {
+__global__ void __launch_bounds__(512, KV == 1 ? 2 : 1) sandwich_kernel(const SandwichArgs p) {
   extern __shared__ __align__(16) float smem[];
   const int group_size = p.n_true / p.groups;
   const int n_part = MODE == kWarpGroups ? (p.N + 255) / 256 : (MODE == kVectorGroups ? p.N / 8 : p.N);
   float* part = smem;
-  float* inv_s = part + (n_part + 3) / 4 * 4;
+  float* inv_s = part + (2 * n_part + 3) / 4 * 4;
   float* hist = inv_s + (p.groups + 3) / 4 * 4;      // [taps - 1][N], row of token i at i mod (taps - 1)
   const int tid = threadIdx.x, nt = blockDim.x;
   pdl_launch_next();
   pdl_wait_prior();
 
-  float h[KV][8], x_next[KV][8], d_next[KV][8];
-  auto fetch = [&](long long t) {
-#pragma unroll
-    for (int i = 0; i < KV; ++i) {
-      const int c = (tid + i * nt) * 8;
-      if (c < p.N) {
-        load8(p.x_in + t * p.N + c, x_next[i]);
-        if (p.delta != nullptr) load8(p.delta + t * p.N + c, d_next[i]);
-      }
-    }
-  };
-  // h of row t, whose inputs have been fetched; fetches those of row `then` (-1: none).  `store`: the new residual is kept
-  auto row = [&](long long t, bool store, long long then) {
+  float h[KV][8];
+  int turn = 0;
+  // h of row t; `store`: the row's new residual is kept
+  auto row = [&](long long t, bool store) {
     float inv[KV][MODE == kColumnGroups ? 8 : 1];
     float x[KV][8];
 #pragma unroll
     for (int i = 0; i < KV; ++i) {
-      const bool ok = (tid + i * nt) * 8 < p.N;
+      const int c = (tid + i * nt) * 8;
 #pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        x[i][j] = x_next[i][j];
-        h[i][j] = ok ? (p.delta != nullptr ? d_next[i][j] : x[i][j]) : 0.f;
+      for (int j = 0; j < 8; ++j) h[i][j] = 0.f;
+      if (c < p.N) {
+        load8(p.x_in + t * p.N + c, x[i]);
+        if (p.delta != nullptr) {
+          load8(p.delta + t * p.N + c, h[i]);
+        } else {
+#pragma unroll
+          for (int j = 0; j < 8; ++j) h[i][j] = x[i][j];
+        }
       }
     }
-    if (then >= 0) fetch(then);
     if (p.delta != nullptr) {
-      group_inv<KV, MODE>(h, inv, part, inv_s, p, group_size);
+      group_inv<KV, MODE>(h, inv, part + (turn ^= 1) * n_part, inv_s, p, group_size);
 #pragma unroll
       for (int i = 0; i < KV; ++i) {
         const int c = (tid + i * nt) * 8;
@@ -118,7 +128,7 @@ __global__ void __launch_bounds__(512) sandwich_kernel(const SandwichArgs p) {
       }
     }
     if (p.w_next != nullptr) {
-      group_inv<KV, MODE>(h, inv, part, inv_s, p, group_size);
+      group_inv<KV, MODE>(h, inv, part + (turn ^= 1) * n_part, inv_s, p, group_size);
 #pragma unroll
       for (int i = 0; i < KV; ++i) {
         const int c = (tid + i * nt) * 8;
@@ -134,8 +144,7 @@ __global__ void __launch_bounds__(512) sandwich_kernel(const SandwichArgs p) {
   A* out = static_cast<A*>(p.out);
   if constexpr (!CONV) {
     const long long t = blockIdx.x;
-    fetch(t);
-    row(t, true, -1);
+    row(t, true);
 #pragma unroll
     for (int i = 0; i < KV; ++i) {
       const int c = (tid + i * nt) * 8;
@@ -154,13 +163,12 @@ __global__ void __launch_bounds__(512) sandwich_kernel(const SandwichArgs p) {
         if (c < p.N) store8(dst + c, h[i]);
       }
     };
-    fetch(tb + max(i0 - K, 0));
     // history rows of tokens i0 - K .. i0 - 1
     for (int j = 0; j < K; ++j) {
       const int i = i0 - K + j;
       float* dst = hist + ((i + K) % K) * p.N;
       if (i >= 0) {
-        row(tb + i, false, tb + i + 1);
+        row(tb + i, false);
         keep(dst);
       } else {
 #pragma unroll
@@ -175,7 +183,7 @@ __global__ void __launch_bounds__(512) sandwich_kernel(const SandwichArgs p) {
       }
     }
     for (int i = i0; i < i1; ++i) {
-      row(tb + i, true, i + 1 < i1 ? tb + i + 1 : -1);
+      row(tb + i, true);
 #pragma unroll
       for (int k = 0; k < KV; ++k) {
         const int c = (tid + k * nt) * 8;
@@ -214,8 +222,7 @@ __global__ void __launch_bounds__(512) sandwich_kernel(const SandwichArgs p) {
           continue;
         }
       }
-      fetch(tb + i);
-      row(tb + i, false, -1);
+      row(tb + i, false);
       keep(state + static_cast<long long>(j) * p.N);
     }
   }
@@ -224,7 +231,7 @@ __global__ void __launch_bounds__(512) sandwich_kernel(const SandwichArgs p) {
 template <typename A, int KV, int MODE>
 cudaError_t launch(const SandwichArgs& a, int threads, cudaStream_t stream, bool pdl) {
   const int n_part = MODE == kWarpGroups ? (a.N + 255) / 256 : (MODE == kVectorGroups ? a.N / 8 : a.N);
-  size_t smem = sizeof(float) * ((n_part + 3) / 4 * 4 + (a.groups + 3) / 4 * 4);
+  size_t smem = sizeof(float) * ((2 * n_part + 3) / 4 * 4 + (a.groups + 3) / 4 * 4);
   if (a.conv_w == nullptr) return launch_kernel(sandwich_kernel<A, KV, MODE, false>, dim3(a.T), dim3(threads), smem, stream, pdl, 1, a);
   smem += sizeof(float) * static_cast<size_t>(a.taps - 1) * a.N;
   auto kern = sandwich_kernel<A, KV, MODE, true>;
