@@ -258,14 +258,14 @@ def test_decoding_with_and_without_a_sink(ops, dt):
     """One token of every sequence over hundreds of keys in many splits, first tokens included."""
     lens = [1, 2, 33, 300, 700]
     for sink in (False, True):
-        x = Latent(6, 32, 16, 32, 128, 64, dt, lens, [1] * 5, sink=sink)
-        out = torch.zeros((x.T, 6 * 128), dtype=dt, device="cuda")
-        args = (x.absorb(), x.q, x.pages, x.table, x.row, x.kv_len, 6, 16, x.scale, x.freq, x.sink)
+        x = Latent(7, 32, 16, 48, 112, 64, dt, lens, [1] * 5, sink=sink)
+        out = torch.zeros((x.T, 7 * 112), dtype=dt, device="cuda")
+        args = (x.absorb(), x.q, x.pages, x.table, x.row, x.kv_len, 7, 16, x.scale, x.freq, x.sink)
         ops.latent_token_attention(*args, out, False)
         assert rel(x.expand(out), x.want) < (3e-6 if dt == torch.float32 else 2e-2)
         if dt == torch.bfloat16:
             for split, n in ((704, 1), (128, 6), (32, 22)):
-                po, ml = torch.empty(x.T * n * 6 * 128, device="cuda"), torch.empty(x.T * n * 6 * 2, device="cuda")
+                po, ml = torch.empty(x.T * n * 7 * 112, device="cuda"), torch.empty(x.T * n * 7 * 2, device="cuda")
                 ops.latent_absorbed_attention(*args, out, *x.blocks, x.row, x.cu, 0, split, n, po, ml, False)
                 assert rel(x.expand(out), x.want) < 2e-2
 
