@@ -8,8 +8,8 @@ torch headers; everything is linked into one shared object that
 by a hash of the source, its local headers and the flags, so a rebuild only
 recompiles what changed.  nvcc cross-compiles, so this runs without a GPU.
 
-``build(subset)`` compiles only the sources one model family needs and links
-them into a library of its own (``_C_<subset>.so``): what a fresh checkout does
+``build(subset)`` compiles only the sources one model needs and links them
+into a library of its own (``_C_<part>+<part>.so``): what a fresh checkout does
 when a single model is to be run and the whole library has not been built.
 """
 from __future__ import annotations
@@ -27,14 +27,27 @@ ROOT = PKG.parent
 BUILD = ROOT / "build" / "obj"
 LIB = PKG / "_C.so"
 
-# model family -> sources (relative to csrc) of its stand-alone library
+# part of the layer-list decoders -> sources (relative to csrc) beside the common ones; a model's stand-alone library has the
+# parts that its layers need
 _LAYERED = ("common/tensor_map.cpp", "core_bindings.cpp", "layered_bindings.cpp", "gemm/gemm_bf16.cu", "gemm/gemm_f32.cu",
             "pointwise/rows32.cu", "pointwise/sandwich_rows.cu", "sampling/sampling.cu", "runtime/page_pool.cpp")
-_HEAD_MIX = ("head_mix_bindings.cpp", "attention/qkv_append.cu", "attention/head_mix_token.cu", "attention/head_mix_decode.cu",
-             "attention/head_mix_prefill.cu", "mlstm/mlstm_recurrent.cu", "mlstm/mlstm_chunked.cu")
-_LATENT = ("latent_bindings.cpp", "attention/latent_prep.cu", "attention/latent_token.cu", "attention/latent_absorbed.cu",
-           "attention/latent_expanded.cu", "gemm/head_gemm.cu", "gated/gated_recurrent.cu", "gated/gated_chunked.cu")
-SUBSETS = {"head_mix": _LAYERED + _HEAD_MIX, "latent": _LAYERED + _LATENT, "layered": _LAYERED + _HEAD_MIX + _LATENT}
+PARTS = {
+    "attention": ("attention_bindings.cpp", "attention/qkv_append.cu", "attention/head_mix_token.cu", "attention/head_mix_decode.cu",
+                  "attention/group_attention.cu"),
+    "head_mix": ("head_mix_bindings.cpp", "attention/head_mix_prefill.cu"),
+    "mlstm": ("mlstm_bindings.cpp", "mlstm/mlstm_recurrent.cu", "mlstm/mlstm_chunked.cu"),
+    "latent": ("latent_bindings.cpp", "attention/latent_prep.cu", "attention/latent_token.cu", "attention/latent_absorbed.cu",
+               "attention/latent_expanded.cu", "gemm/head_gemm.cu"),
+    "gated": ("gated_bindings.cpp", "gated/gated_recurrent.cu", "gated/gated_chunked.cu"),
+    "rglru": ("rglru_bindings.cpp", "rglru/rglru_scan.cu"),
+    "streams": ("stream_bindings.cpp", "pointwise/stream_rows.cu"),
+    "moe": ("moe/moe_bindings.cpp", "moe/moe_route.cu", "moe/moe_grouped_gemm.cu", "moe/moe_grouped_gemm_f32.cu"),
+}
+
+
+def subset_sources(subset: str):
+    """Sources of a library named after its parts, "attention+moe+streams"."""
+    return _LAYERED + tuple(f for part in subset.split("+") for f in PARTS[part])
 
 
 def library_path(subset: str = "") -> Path:
@@ -62,7 +75,7 @@ def _headers_digest() -> str:
 
 def _sources(subset: str = ""):
     if subset:
-        files = [CSRC / name for name in SUBSETS[subset]]
+        files = [CSRC / name for name in subset_sources(subset)]
         return [p for p in files if p.suffix == ".cu"], [p for p in files if p.suffix == ".cpp"]
     cu = sorted(CSRC.rglob("*.cu"))
     cpp = sorted(p for p in CSRC.rglob("*.cpp"))
@@ -94,7 +107,7 @@ def _compile(src: Path, cmd_prefix: list[str], tag: str, hdr: str, verbose: bool
 
 
 def build(verbose: bool = True, ptxas_info: bool = False, subset: str = "") -> Path:
-    """Compile (if needed) and link ``_C.so`` (or the library of one model family); returns its path."""
+    """Compile (if needed) and link ``_C.so`` (or a library of some of its parts); returns its path."""
     import torch
     from torch.utils import cpp_extension as ce
 
@@ -112,7 +125,7 @@ def build(verbose: bool = True, ptxas_info: bool = False, subset: str = "") -> P
     for s in cu:
         jobs.append((s, nv, "nvcc"))
     for s in cpp:
-        uses_torch = any(k in s.read_text() for k in ("torch/", "ATen/", "binding_util.h"))
+        uses_torch = any(k in s.read_text() for k in ("torch/", "ATen/", "binding_util.h", "head_mix_args.h"))
         cx = ["g++"] + CXX_FLAGS + inc + ([abi] + torch_inc if uses_torch else [])
         jobs.append((s, cx, "g++ "))
     workers = max(1, min(len(jobs), os.cpu_count() or 4))

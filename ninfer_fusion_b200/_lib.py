@@ -29,7 +29,7 @@ def native_path() -> Path:
 def load_native(build_if_missing: bool = False, subset: str = ""):
     """Load ``_C.so`` once and return ``torch.ops.nfb200``.
 
-    `subset`: a process that runs one model family only may use that family's own library (see ``_build.SUBSETS``)
+    `subset`: a process that runs one model only may use a library of the parts it needs (see ``_build.PARTS``)
     when the full one is not there; it is compiled if need be."""
     global _loaded
     if _loaded is None:

@@ -2,8 +2,8 @@
 //
 //   c_g(i, j)  = cap * tanh(scale * q_g(i) . k_{g / (H/G)}(j) / cap)          (cap = 0: no cap)
 //   s_h(i, j)  = sum_g mix[h, g] * c_g(i, j)  -  slope[h] * (i - j)            (mix = null: the identity)
-//   visible    : 0 <= i - j < window (window = 0: all of the past)
-//   a_h(i, j)  = exp(s_h) / (sink_one + sum_j exp(s_h))
+//   visible    : j <= i, i - j < window (window = 0: all of the past), floor(i / chunk) = floor(j / chunk) (chunk = 0: no chunks)
+//   a_h(i, j)  = exp(s_h) / (sink_one + exp(sinks[h]) + sum_j exp(s_h))        (sinks = null: without them)
 //   out_h(i)   = sigmoid(gate[i, h]) * sum_j a_h(i, j) v(j)                    (gate = null: no gate)
 //
 // `slope` is the bias AFTER mixing: a per-head bias b_g taken off before the mix is slope[h] = sum_g mix[h, g] b_g.
@@ -25,8 +25,9 @@ struct HeadMixArgs {
   const int* table_row = nullptr;   // [T]
   const int* kv_len = nullptr;      // [T] position + 1
   int T = 0;
-  int n_heads = 0, n_kv = 0, dim = 0, vdim = 0, page_size = 0, window = 0;
+  int n_heads = 0, n_kv = 0, dim = 0, vdim = 0, page_size = 0, window = 0, chunk = 0;
   float scale = 1.f, softcap = 0.f, sink = 0.f;   // sink: what is added to the softmax denominator (0 or 1)
+  const float* sinks = nullptr;     // [H] learned scores that only count in the denominator, or null
   const float* mix = nullptr;       // [H, H] row-major, or null
   const float* slope = nullptr;     // [H], or null
   const float* gate = nullptr;      // [T, *] raw gate values of head h at gate[t * ld_gate + h], or null
@@ -46,10 +47,28 @@ const char* head_mix_token_attention(const HeadMixArgs& a, int split_keys, int n
 bool head_mix_decode_supported(const HeadMixArgs& a);
 const char* head_mix_decode(const HeadMixArgs& a, int split_keys, int n_splits, float* part_o, float* part_ml);
 
+// Scores that are scaled dot products and nothing else (no cap, mix, bias, gate), bf16: grouped-query attention on the tensor
+// cores (group_attention.cu).  head_mix_token_attention picks the decode form by itself; it leaves the splits unmerged.
+bool group_attention_supported(const HeadMixArgs& a);
+const char* group_decode(const HeadMixArgs& a, int split_keys, int n_splits, float* part_o, float* part_ml);
+// Query blocks as in head_mix_prefill.
+const char* group_prefill(const HeadMixArgs& a, const int* blk_start, const int* blk_count, int n_blocks);
+
 #ifdef __CUDACC__
+// First position that the query at position len - 1 sees.
+__device__ __forceinline__ int first_visible(int len, int window, int chunk) {
+  int lo = window > 0 ? max(0, len - window) : 0;
+  if (chunk > 0) lo = max(lo, (len - 1) / chunk * chunk);
+  return lo;
+}
 // What the sum of exp(s - m) v, with m the maximum and l the sum of exp(s - m), is multiplied with.
-__device__ __forceinline__ float head_mix_finish(float m, float l, float sink) {
+__device__ __forceinline__ float head_mix_finish(float m, float l, float sink, const float* sinks, int h) {
   if (!(m > -3.0e38f)) return 0.f;   // no visible key
+  if (sinks != nullptr) {
+    const float s = sinks[h], mx = fmaxf(fmaxf(m, s), sink > 0.f ? 0.f : m);
+    const float e = expf(m - mx);
+    return e / (expf(s - mx) + (sink > 0.f ? sink * expf(-mx) : 0.f) + l * e);
+  }
   if (sink <= 0.f) return 1.f / l;
   const float mx = fmaxf(m, 0.f);
   const float e = expf(m - mx);
@@ -79,6 +98,8 @@ struct QkvAppendArgs {
   const int* cache_pos = nullptr;
   const int* block_table = nullptr;
   int table_ld = 0, page_size = 0;
+  const double* freq = nullptr;     // [rot / 2] rotation of neighbours (2i, 2i + 1) of the first `rot` values of q and k heads,
+  int rot = 0;                      // after the norm, by position * freq[i] (angles in 64-bit); 0: none
   void* q_out = nullptr;            // [T, n_heads * dim], leading dimension ldq
   int64_t ldq = 0;
   void* k_pages = nullptr;
@@ -87,7 +108,7 @@ struct QkvAppendArgs {
   cudaStream_t stream = nullptr;
   bool pdl = false;
 };
-// Per-head RMS norm of q and k, k and v rows appended to their pages.
+// Per-head RMS norm and rotation of q and k, k and v rows appended to their pages.
 const char* qkv_append(const QkvAppendArgs& a);
 
 }  // namespace nfb

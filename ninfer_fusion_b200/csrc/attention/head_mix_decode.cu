@@ -55,7 +55,7 @@ __global__ void __launch_bounds__(NW * 32) head_mix_decode_kernel(const HeadMixA
   pdl_launch_next();
   pdl_wait_prior();
   const int len = p.kv_len[t], qpos = len - 1;
-  const int lo = p.window > 0 ? max(0, len - p.window) : 0;
+  const int lo = first_visible(len, p.window, p.chunk);
   const int k_begin = lo + split * split_keys, k_end = min(len, k_begin + split_keys);
   const int n_tiles = k_end > k_begin ? (k_end - k_begin + KT - 1) / KT : 0;
   const int* table = p.block_table + static_cast<long long>(p.table_row[t]) * p.table_ld;
@@ -258,7 +258,7 @@ __global__ void __launch_bounds__(NW * 32) head_mix_decode_kernel(const HeadMixA
           part_ml[at * 2 + 1] = sum;
         }
       } else {
-        float f = head_mix_finish(m[j][r], sum, p.sink);
+        float f = head_mix_finish(m[j][r], sum, p.sink, p.sinks, h);
         if (p.gate != nullptr) f *= sigmoid_of<bf16>(p.gate[t * p.ld_gate + h]);
         bf16* dst = static_cast<bf16*>(p.out) + t * p.ldo + static_cast<long long>(h) * V + c4 * 2;
 #pragma unroll

@@ -488,7 +488,7 @@ __global__ void __launch_bounds__(128, VT <= 8 ? 4 : 2) head_mix_values_kernel(c
     const int i = qt * 16 + r4 + r * 8;
     if (i >= br.cnt) continue;
     const long long t = br.t0 + i;
-    float f = head_mix_finish(m[r] * (1.f / kLog2e), l[r], a.sink);
+    float f = head_mix_finish(m[r] * (1.f / kLog2e), l[r], a.sink, a.sinks, h);
     if (a.gate != nullptr) f *= sigmoid_of<bf16>(a.gate[t * a.ld_gate + h]);
     bf16* dst = static_cast<bf16*>(a.out) + t * a.ldo + static_cast<long long>(h) * V + v0 + c4 * 2;
 #pragma unroll
@@ -570,7 +570,7 @@ int64_t head_mix_prefill_scratch(int n_heads, int max_keys, int window, int bloc
 const char* head_mix_prefill(const HeadMixArgs& a, const int* blk_start, const int* blk_count, int n_blocks, int max_keys,
                              void* scratch, int64_t scratch_bytes) {
   if (a.T <= 0 || n_blocks <= 0) return nullptr;
-  if (a.f32) return "head_mix_prefill: bf16 only";
+  if (a.f32 || a.chunk > 0) return "head_mix_prefill: bf16 without chunks only";
   if (a.dim % 16 || a.vdim % 16 || a.n_kv <= 0 || a.n_heads % a.n_kv) return "head_mix_prefill: bad head geometry";
   if (a.n_heads > 512 || n_blocks > 65535) return "head_mix_prefill: too many heads or query blocks";
   if (a.ldq % 4 || a.ldo % 2) return "head_mix_prefill: misaligned rows";

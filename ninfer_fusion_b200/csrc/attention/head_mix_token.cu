@@ -1,5 +1,5 @@
 // Head-mixing attention, one query token per CTA, on the FP32 pipes (every size, bf16 or 32-bit; bf16 head geometries
-// that suit the tensor cores take head_mix_decode.cu instead): the CTA holds ALL heads of its token, because a mixed score needs every head's score of the same key.  Keys are walked in blocks of 32:
+// that suit the tensor cores take head_mix_decode.cu, or group_attention.cu for plain scores, instead): the CTA holds ALL heads of its token, because a mixed score needs every head's score of the same key.  Keys are walked in blocks of 32:
 //   scores   eight lanes per (key, kv head): 16-byte loads along the key row, reduced by shuffles, soft-capped
 //   mix      one thread per (head, key): the row of the mixing matrix times the column of scores, bias, mask
 //   softmax  one warp per head, lane = key: running maximum and sum
@@ -43,7 +43,7 @@ __global__ void __launch_bounds__(kThreads) head_mix_token_kernel(const HeadMixA
   pdl_wait_prior();
   const int len = p.kv_len[t];
   const int qpos = len - 1;
-  const int lo = p.window > 0 ? max(0, len - p.window) : 0;
+  const int lo = first_visible(len, p.window, p.chunk);
   const int k_begin = lo + split * split_keys;
   const int k_end = min(len, k_begin + split_keys);
   const int* table = p.block_table + static_cast<long long>(p.table_row[t]) * p.table_ld;
@@ -175,7 +175,7 @@ __global__ void __launch_bounds__(kThreads) head_mix_token_kernel(const HeadMixA
     const int it = tid + i * kThreads;
     if (it < items) {
       const int h = it / vecs;
-      float f = head_mix_finish(ms[h], ls[h], p.sink);
+      float f = head_mix_finish(ms[h], ls[h], p.sink, p.sinks, h);
       if (p.gate != nullptr) f *= sigmoid_of<A>(p.gate[t * p.ld_gate + h]);
 #pragma unroll
       for (int j = 0; j < 8; ++j) acc[i][j] *= f;
@@ -209,7 +209,7 @@ __global__ void __launch_bounds__(128) head_mix_merge_kernel(const HeadMixArgs p
 #pragma unroll
     for (int j = 0; j < 8; ++j) o[j] = fmaf(e, v[j], o[j]);
   }
-  float f = head_mix_finish(m, l, p.sink);
+  float f = head_mix_finish(m, l, p.sink, p.sinks, h);
   if (p.gate != nullptr) f *= sigmoid_of<A>(p.gate[t * p.ld_gate + h]);
 #pragma unroll
   for (int j = 0; j < 8; ++j) o[j] *= f;
@@ -275,6 +275,10 @@ const char* head_mix_token_attention(const HeadMixArgs& a, int split_keys, int n
   if (a.ldq % align || a.ldo % align) return "head_mix attention: misaligned rows";
   if (split_keys <= 0 || n_splits <= 0 || (n_splits > 1 && (part_o == nullptr || part_ml == nullptr)))
     return "head_mix attention: bad split";
+  if (group_attention_supported(a)) {
+    if (const char* err = group_decode(a, split_keys, n_splits, part_o, part_ml)) return err;
+    return merge_splits<__nv_bfloat16>(a, n_splits, part_o, part_ml);
+  }
   if (head_mix_decode_supported(a)) {
     if (const char* err = head_mix_decode(a, split_keys, n_splits, part_o, part_ml)) return err;
     return merge_splits<__nv_bfloat16>(a, n_splits, part_o, part_ml);

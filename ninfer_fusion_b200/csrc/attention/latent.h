@@ -1,22 +1,27 @@
 // Latent attention (plain C++ ABI): queries, keys and values come out of low-rank latents.  One cached row per token,
 // [latent c (rank) | rotated key part (rot)], shared by all heads.  With U_k, U_v the per-head expansions of c:
-//   s_h(i, j) = scale * ( q_h(i) . U_k,h c(j)  +  rotate(r_h(i)) . k_rot(j) ),   j <= i
+//   s_h(i, j) = scale * ( q_h(i) . U_k,h c(j)  +  rotate(r_h(i)) . k_rot(j) ),   j <= i and (window > 0) i - j < window
 //   a_h(i, j) = exp(s_h) / ( exp(sink_h) + sum_j exp(s_h) )                       (sink = null: without it)
 //   out_h(i)  = U_v,h sum_j a_h(i, j) c(j)
 // Two forms.  Absorbed: the query is taken to the latent space (q' = U_k,h^T q_h) and the sum over c is expanded
 // afterwards, so a row is read once for all heads: decode and short portions.  Expanded: keys and values of all visible
 // positions are made by one GEMM and attended as ordinary heads: long portions, a third of the multiply-adds at the usual
 // widths.  Rotation: neighbours (2i, 2i + 1) by position * freq[i], angles in 64-bit.
-// Scores, weights and sums are fp32.  Widths are multiples of 16, zero-padded by the producer.
+// A query without rotated part (rot = 0) needs no freq.  Scores, weights and sums are fp32.  Widths are multiples of 16, zero-padded by the producer.
 #pragma once
 #include <cuda_runtime.h>
 #include <stdint.h>
 
+#include "rotary.cuh"
+
 namespace nfb {
 
 struct LatentPrepArgs {
-  const void* proj = nullptr;       // [T, ldp]: query latent (q_rank) | key / value latent (rank) | key part to rotate (rot)
+  // [T, ldp]: query latent (q_rank; 0: none, the queries are not this kernel's) at column 0; at kv_off key / value latent (rank)
+  // | key part to rotate (rot)
+  const void* proj = nullptr;
   int64_t ldp = 0;
+  int kv_off = 0;
   int T = 0;
   int q_rank = 0, q_rank_true = 0, rank = 0, rank_true = 0, rot = 0, rot_true = 0;
   const float* q_norm = nullptr;    // [q_rank]
@@ -48,7 +53,7 @@ struct LatentArgs {
   const int* table_row = nullptr;   // [T]
   const int* kv_len = nullptr;      // [T] position + 1
   int T = 0;
-  int n_heads = 0, dim = 0, rank = 0, rot = 0, rot_true = 0, page_size = 0;
+  int n_heads = 0, dim = 0, rank = 0, rot = 0, rot_true = 0, page_size = 0, window = 0;
   float scale = 1.f;
   const double* freq = nullptr;
   const float* sink = nullptr;      // [H] or null
@@ -82,9 +87,9 @@ const char* latent_absorbed_attention(const LatentArgs& a, const LatentBlocks& b
 // Expanded, bf16 tensor cores, for the sequences the absorbed form leaves out.  latent_gather fills `rows`; the caller makes
 // `kv` from their latents (one GEMM); then latent_expanded_attention writes out [T, n_heads * vdim] of those sequences.
 struct LatentExpand {
-  const int* seqs = nullptr;      // [n_seqs, 3]: block-table row, first row in `rows`, visible positions
-  int n_seqs = 0, max_len = 0;
-  const int* seq_base = nullptr;  // [sequences of the step]: first row in `rows`, -1: not expanded
+  const int* seqs = nullptr;      // [n_seqs, 4]: block-table row, first row in `rows`, first position, positions
+  int n_seqs = 0, max_len = 0;    // max_len: most positions of a sequence
+  const int* seq_base = nullptr;  // [sequences of the step, 2]: first row in `rows` (-1: not expanded), its position
   void* rows = nullptr;           // [total, rank + rot]
   const void* kv = nullptr;       // [total, n_heads * (dim + vdim)]: keys of all heads, values of all heads
   int vdim = 0;
@@ -94,11 +99,7 @@ const char* latent_gather(const LatentArgs& a, const LatentExpand& x);
 const char* latent_expanded_attention(const LatentArgs& a, const LatentBlocks& b, const LatentExpand& x);
 
 #ifdef __CUDACC__
-// cos and sin of pos * freq, the angle reduced in 64-bit.
-__device__ __forceinline__ void latent_angle(int pos, double freq, float& c, float& s) {
-  const double turn = static_cast<double>(pos) * freq * 0.15915494309189535;   // 1 / (2 pi)
-  sincospif(static_cast<float>(2.0 * (turn - rint(turn))), &s, &c);
-}
+__device__ __forceinline__ int latent_first(int len, int window) { return window > 0 ? max(0, len - window) : 0; }
 #endif
 
 }  // namespace nfb

@@ -60,7 +60,8 @@ __global__ void __launch_bounds__(NW * 32) latent_absorbed_kernel(const LatentAr
     if (b.cu_seqlens[seq + 1] - b.cu_seqlens[seq] >= b.max_tokens) return;
   }
   const int max_len = p.kv_len[t0 + (r0 + n_rows - 1) / H];
-  const int k_begin = split * split_keys, k_end = min(max_len, k_begin + split_keys);
+  const int lo = latent_first(p.kv_len[t0 + r0 / H], p.window);       // of the CTA's first row
+  const int k_begin = lo + split * split_keys, k_end = min(max_len, k_begin + split_keys);
   const int n_tiles = k_end > k_begin ? (k_end - k_begin + KT - 1) / KT : 0;
   const int* table = p.block_table + static_cast<long long>(p.table_row[t0]) * p.table_ld;
   const bf16* pages = static_cast<const bf16*>(p.pages);
@@ -111,7 +112,7 @@ __global__ void __launch_bounds__(NW * 32) latent_absorbed_kernel(const LatentAr
       const int t = t0 + (r0 + r) / H, h = (r0 + r) % H;
       const bf16* q = static_cast<const bf16*>(p.q) + t * p.ldq + static_cast<long long>(h) * (p.dim + p.rot) + p.dim + 2 * e;
       float c, s;
-      latent_angle(p.kv_len[t] - 1, p.freq[e], c, s);
+      rotary_angle(p.kv_len[t] - 1, p.freq[e], c, s);
       const float x = __bfloat162float(q[0]), y = __bfloat162float(q[1]);
       u = x * c - y * s;
       v = y * c + x * s;
@@ -176,13 +177,13 @@ __global__ void __launch_bounds__(NW * 32) latent_absorbed_kernel(const LatentAr
     const int key = k_begin + tile * KT + lane;
 #pragma unroll
     for (int i = 0; i < kRows; ++i) {
-      const int row = warp * kRows + i, limit = min(row_len[row], k_end);
+      const int row = warp * kRows + i, limit = min(row_len[row], k_end), first = latent_first(row_len[row], p.window);
       float v[kPer], t = -CUDART_INF_F;
 #pragma unroll
       for (int j = 0; j < kPer; ++j) {
         const float* sp = ss + row * kLdS + lane + 32 * j;
         v[j] = (sp[0] + sp[M * kLdS]) + (sp[2 * M * kLdS] + sp[3 * M * kLdS]);
-        v[j] = key + 32 * j < limit ? v[j] * scale2 : -CUDART_INF_F;
+        v[j] = key + 32 * j < limit && key + 32 * j >= first ? v[j] * scale2 : -CUDART_INF_F;
         t = fmaxf(t, v[j]);
       }
 #pragma unroll

@@ -22,12 +22,13 @@ constexpr int KT = 64, QT = kLatentBlock, kThreads = 128;
 __global__ void __launch_bounds__(256) latent_gather_kernel(const LatentArgs p, const LatentExpand x) {
   pdl_launch_next();
   pdl_wait_prior();
-  const int* s = x.seqs + blockIdx.y * 3;
-  const int pos = blockIdx.x * 8 + (threadIdx.x >> 5), W = p.rank + p.rot;
-  if (pos >= s[2]) return;
+  const int* s = x.seqs + blockIdx.y * 4;
+  const int at = blockIdx.x * 8 + (threadIdx.x >> 5), W = p.rank + p.rot;
+  if (at >= s[3]) return;
+  const int pos = s[2] + at;
   const int page = p.block_table[static_cast<long long>(s[0]) * p.table_ld + pos / p.page_size];
   const uint4* src = reinterpret_cast<const uint4*>(static_cast<const bf16*>(p.pages) + (static_cast<long long>(max(page, 0)) * p.page_size + pos % p.page_size) * W);
-  uint4* dst = reinterpret_cast<uint4*>(static_cast<bf16*>(x.rows) + static_cast<long long>(s[1] + pos) * W);
+  uint4* dst = reinterpret_cast<uint4*>(static_cast<bf16*>(x.rows) + static_cast<long long>(s[1] + at) * W);
   for (int c = threadIdx.x & 31; c < W / 8; c += 32) dst[c] = page < 0 ? make_uint4(0u, 0u, 0u, 0u) : src[c];
 }
 
@@ -43,14 +44,17 @@ __global__ void __launch_bounds__(kThreads) latent_flash_kernel(const LatentArgs
   pdl_launch_next();
   pdl_wait_prior();
   const int h = blockIdx.x, blk = static_cast<int>(gridDim.y) - 1 - static_cast<int>(blockIdx.y);   // later (longer) blocks first
-  const int t0 = b.start[blk], count = b.count[blk], base = x.seq_base[b.token_seq[t0]];
-  if (base < 0) return;
+  const int t0 = b.start[blk], count = b.count[blk], seq = b.token_seq[t0];
+  const int row_of_first = x.seq_base[seq * 2];
+  if (row_of_first < 0) return;
   const int len = p.kv_len[t0 + count - 1], first_len = p.kv_len[t0];
-  const int n_tiles = (len + KT - 1) / KT;
+  const int k_begin = latent_first(first_len, p.window);             // the block's keys: positions k_begin .. len - 1
+  const int n_tiles = (len - k_begin + KT - 1) / KT;
+  const long long base = static_cast<long long>(row_of_first) + k_begin - x.seq_base[seq * 2 + 1];   // row of position k_begin
   const long long ldx = static_cast<long long>(H) * (D + V);
   const bf16* keys = static_cast<const bf16*>(x.kv) + base * ldx + static_cast<long long>(h) * D;
   const bf16* vals = static_cast<const bf16*>(x.kv) + base * ldx + static_cast<long long>(H) * D + static_cast<long long>(h) * V;
-  const bf16* rots = static_cast<const bf16*>(x.rows) + static_cast<long long>(base) * (p.rank + R) + p.rank;
+  const bf16* rots = static_cast<const bf16*>(x.rows) + base * (p.rank + R) + p.rank;
   const int kv8 = W / 8, d8 = D / 8, v8 = V / 8;
   // 16 threads walk a row; a thread's rows of a tile are lr, lr + 8, ..., its 16-byte pieces lc, lc + 16, ...
   const int lr = tid >> 4, lc = tid & 15;
@@ -72,7 +76,7 @@ __global__ void __launch_bounds__(kThreads) latent_flash_kernel(const LatentArgs
   };
   auto load = [&](int tile) {
     const uint32_t dk = ring_a + (tile & 1) * stage * 2 + lr * ldk * 2, dv = ring_a + ((tile & 1) * stage + KT * ldk + lr * ldv) * 2;
-    const int left = len - tile * KT;
+    const int left = len - k_begin - tile * KT;
     const long long first = static_cast<long long>(tile) * KT + lr;
     const long long ldr = p.rank + R;
     for (int c = lc; c < kv8; c += 16)
@@ -93,7 +97,7 @@ __global__ void __launch_bounds__(kThreads) latent_flash_kernel(const LatentArgs
     if (r < count && 2 * e < p.rot_true) {
       const bf16* q = static_cast<const bf16*>(p.q) + (t0 + r) * p.ldq + static_cast<long long>(h) * W + D + 2 * e;
       float c, s;
-      latent_angle(p.kv_len[t0 + r] - 1, p.freq[e], c, s);
+      rotary_angle(p.kv_len[t0 + r] - 1, p.freq[e], c, s);
       const float a = __bfloat162float(q[0]), bb = __bfloat162float(q[1]);
       u = a * c - bb * s;
       v = bb * c + a * s;
@@ -108,6 +112,7 @@ __global__ void __launch_bounds__(kThreads) latent_flash_kernel(const LatentArgs
   float m[2] = {-CUDART_INF_F, -CUDART_INF_F}, l[2] = {0.f, 0.f};
   const int row0 = warp * 16;
   const int rlen[2] = {row0 + r4 < count ? p.kv_len[t0 + row0 + r4] : 0, row0 + r4 + 8 < count ? p.kv_len[t0 + row0 + r4 + 8] : 0};
+  const int rlo[2] = {latent_first(rlen[0], p.window), latent_first(rlen[1], p.window)}, last_lo = latent_first(len, p.window);
   const float scale2 = p.scale * kLog2e;
   for (int tile = 0; tile < n_tiles; ++tile) {
     cp_async_wait<0>();
@@ -132,13 +137,15 @@ __global__ void __launch_bounds__(kThreads) latent_flash_kernel(const LatentArgs
         mma_bf16_16816(s[2 * n + 1], a, k[2], k[3]);
       }
     }
-    const int k0 = tile * KT;
-    if (k0 + KT > first_len) {       // some query of the block does not see all of the tile
+    const int k0 = k_begin + tile * KT;
+    if (k0 + KT > first_len || k0 < last_lo) {       // some query of the block does not see all of the tile
 #pragma unroll
       for (int n = 0; n < KT / 8; ++n)
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
-          if (k0 + n * 8 + c4 * 2 + (e & 1) >= rlen[e >> 1]) s[n][e] = -CUDART_INF_F;
+        for (int e = 0; e < 4; ++e) {
+          const int key = k0 + n * 8 + c4 * 2 + (e & 1);
+          if (key >= rlen[e >> 1] || key < rlo[e >> 1]) s[n][e] = -CUDART_INF_F;
+        }
     }
     float mt[2] = {m[0], m[1]};
 #pragma unroll

@@ -1,4 +1,4 @@
-// Latent attention: norms of the query and key / value latents, rotation of the shared key part and append of the row
+// Latent attention: norms of the query latent (if there is one) and the key / value latent, rotation of the shared key part and append of the row
 // [latent | rotated part] to its cache page.  One warp per (token, latent); a row is read twice, the second time from L1.
 #include "latent.h"
 
@@ -35,10 +35,11 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentPrepArgs p
   pdl_wait_prior();
   const int lane = threadIdx.x & 31;
   const long long item = static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
-  if (item >= 2LL * p.T) return;
-  const int t = static_cast<int>(item >> 1);
+  const int per = p.q_rank > 0 ? 2 : 1;
+  if (item >= static_cast<long long>(per) * p.T) return;
+  const int t = static_cast<int>(item / per);
   const A* row = static_cast<const A*>(p.proj) + t * p.ldp;
-  if (!(item & 1)) {
+  if (item % per != per - 1) {
     norm_row(row, static_cast<A*>(p.q_latent) + t * p.ldq, p.q_norm, p.q_rank, p.q_rank_true, p.eps, lane);
     return;
   }
@@ -46,13 +47,13 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentPrepArgs p
   const int page = p.block_table[static_cast<long long>(p.table_row[t]) * p.table_ld + pos / p.page_size];
   if (page < 0) return;
   A* dst = static_cast<A*>(p.pages) + (static_cast<long long>(page) * p.page_size + pos % p.page_size) * (p.rank + p.rot);
-  norm_row(row + p.q_rank, dst, p.kv_norm, p.rank, p.rank_true, p.eps, lane);
-  const A* r = row + p.q_rank + p.rank;
+  norm_row(row + p.kv_off, dst, p.kv_norm, p.rank, p.rank_true, p.eps, lane);
+  const A* r = row + p.kv_off + p.rank;
   for (int i = lane; i < p.rot / 2; i += 32) {
     float u = 0.f, v = 0.f;
     if (2 * i < p.rot_true) {
       float c, s;
-      latent_angle(pos, p.freq[i], c, s);
+      rotary_angle(pos, p.freq[i], c, s);
       const float a = elem_to_f(r[2 * i]), b = elem_to_f(r[2 * i + 1]);
       u = a * c - b * s;
       v = b * c + a * s;
@@ -69,8 +70,8 @@ const char* latent_prep(const LatentPrepArgs& a) {
   if (a.q_rank % 16 || a.rank % 16 || a.rot % 16 || a.rot_true % 2 || a.rot_true > a.rot || a.rank_true > a.rank ||
       a.q_rank_true > a.q_rank)
     return "latent_prep: widths must be multiples of 16";
-  if (a.ldp % 8 || a.ldq % 8) return "latent_prep: misaligned rows";
-  const dim3 grid(static_cast<unsigned>((2LL * a.T + 7) / 8));
+  if (a.ldp % 8 || a.ldq % 8 || a.kv_off % 8) return "latent_prep: misaligned rows";
+  const dim3 grid(static_cast<unsigned>(((a.q_rank > 0 ? 2LL : 1LL) * a.T + 7) / 8));
   const cudaError_t e = a.f32 ? launch_kernel(latent_prep_kernel<float>, grid, dim3(256), 0, a.stream, a.pdl, 1, a)
                               : launch_kernel(latent_prep_kernel<__nv_bfloat16>, grid, dim3(256), 0, a.stream, a.pdl, 1, a);
   return e == cudaSuccess ? nullptr : cudaGetErrorString(e);

@@ -31,7 +31,7 @@ __global__ void __launch_bounds__(kThreads) latent_token_kernel(const LatentArgs
     float u = 0.f, v = 0.f;
     if (2 * i < p.rot_true) {
       float c, sn;
-      latent_angle(len - 1, p.freq[i], c, sn);
+      rotary_angle(len - 1, p.freq[i], c, sn);
       const float a = elem_to_f(qr[2 * i]), b = elem_to_f(qr[2 * i + 1]);
       u = a * c - b * sn;
       v = b * c + a * sn;
@@ -43,7 +43,7 @@ __global__ void __launch_bounds__(kThreads) latent_token_kernel(const LatentArgs
   const int* table = p.block_table + static_cast<long long>(p.table_row[t]) * p.table_ld;
   const float sink = p.sink != nullptr ? p.sink[h] : -CUDART_INF_F;
   float m = sink, l = p.sink != nullptr ? 1.f : 0.f, o[kMaxCols] = {};
-  for (int k0 = 0; k0 < len; k0 += kKeys) {
+  for (int k0 = latent_first(len, p.window); k0 < len; k0 += kKeys) {
     const int n = min(kKeys, len - k0);
     __syncthreads();
     if (tid < n) {

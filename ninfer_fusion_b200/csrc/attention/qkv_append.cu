@@ -1,10 +1,11 @@
-// Per-head RMS norm of the query and key heads of a fused projection and the append of k / v rows to their cache
+// Per-head RMS norm and rotation of the query and key heads of a fused projection and the append of k / v rows to their cache
 // pages, for layers whose query / key and value widths differ and whose element type is bf16 or fp32.  One warp per
 // (token, head row); values stay in registers between the two passes of the norm.
 #include "head_mix.h"
 
 #include "../common/elem.cuh"
 #include "../common/launch.h"
+#include "rotary.cuh"
 
 namespace nfb {
 
@@ -28,10 +29,10 @@ __global__ void __launch_bounds__(256) qkv_append_kernel(const QkvAppendArgs p) 
   const int width = kind == 2 ? p.vdim : p.dim;
   const A* src = static_cast<const A*>(p.proj) + t * p.ldp + (kind == 0 ? p.q_off : (kind == 1 ? p.k_off : p.v_off)) + r * width;
   A* dst;
+  const int pos = p.cache_pos[t];
   if (kind == 0) {
     dst = static_cast<A*>(p.q_out) + t * p.ldq + r * width;
   } else {
-    const int pos = p.cache_pos[t];
     const int page = p.block_table[static_cast<long long>(p.table_row[t]) * p.table_ld + pos / p.page_size];
     if (page < 0) return;
     dst = static_cast<A*>(kind == 1 ? p.k_pages : p.v_pages) +
@@ -59,6 +60,18 @@ __global__ void __launch_bounds__(256) qkv_append_kernel(const QkvAppendArgs p) 
 #pragma unroll
         for (int j = 0; j < 8; ++j) v[c][j] = v[c][j] * inv * w[at + j];
       }
+      if (kind != 2 && at < p.rot) {
+#pragma unroll
+        for (int j = 0; j < 8; j += 2) {
+          if (at + j < p.rot) {
+            float cs, sn;
+            rotary_angle(pos, p.freq[(at + j) / 2], cs, sn);
+            const float a = v[c][j], b = v[c][j + 1];
+            v[c][j] = a * cs - b * sn;
+            v[c][j + 1] = b * cs + a * sn;
+          }
+        }
+      }
       store8(dst + at, v[c]);
     }
   }
@@ -70,6 +83,7 @@ const char* qkv_append(const QkvAppendArgs& a) {
   if (a.T <= 0) return nullptr;
   if (a.dim % 16 || a.vdim % 16 || a.dim > 1024 || a.vdim > 1024 || a.dim_true <= 0 || a.dim_true > a.dim)
     return "qkv_append: head widths must be multiples of 16 up to 1024";
+  if (a.rot < 0 || a.rot % 2 || a.rot > a.dim_true || (a.rot > 0 && a.freq == nullptr)) return "qkv_append: bad rotation";
   const int align = a.f32 ? 4 : 8;
   if (a.ldp % align || a.ldq % align || a.q_off % 8 || a.k_off % 8 || a.v_off % 8) return "qkv_append: misaligned rows";
   const long long items = static_cast<long long>(a.T) * (a.n_heads + 2 * a.n_kv);

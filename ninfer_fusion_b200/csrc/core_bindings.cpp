@@ -8,11 +8,11 @@ using namespace nfb_bind;
 
 void gemm_bf16(const Tensor& x, const Tensor& w, OptT out, int64_t epi, OptT resid, OptT bias, OptT partial,
                int64_t splits, OptT status, bool pdl, int64_t act, OptT conv_w, OptT conv_state, OptT conv_slot,
-               OptT conv_out, OptT prefetch, OptT out32, int64_t out32_from, OptT act_params) {
+               OptT conv_out, OptT prefetch, OptT out32, int64_t out32_from, OptT act_params, at::ArrayRef<double> glu) {
   need(x, at::kBFloat16, "x"); need(w, at::kBFloat16, "w");
   need_rows(x, "x"); need_rows(w, "w");
   TORCH_CHECK(x.size(1) == w.size(1), "gemm_bf16: K mismatch");
-  TORCH_CHECK(act >= 0 && act <= 4 && (act == 0 || epi == nfb::kEpiStore), "gemm_bf16: activation needs the store epilogue");
+  TORCH_CHECK(act >= 0 && act <= 5 && (act == 0 || epi == nfb::kEpiStore), "gemm_bf16: activation needs the store epilogue");
   c10::cuda::CUDAGuard guard(x.device());
   nfb::GemmArgs a;
   a.w = w.data_ptr(); a.N = w.size(0); a.K = w.size(1); a.ldw = w.stride(0);
@@ -52,6 +52,10 @@ void gemm_bf16(const Tensor& x, const Tensor& w, OptT out, int64_t epi, OptT res
     need(*partial, at::kFloat, "partial");
     TORCH_CHECK(partial->is_contiguous() && partial->numel() >= splits * a.T * a.N, "gemm_bf16: workspace too small");
     a.partial = static_cast<float*>(partial->data_ptr());
+  }
+  if (!glu.empty()) {
+    TORCH_CHECK(glu.size() == 3, "gemm_bf16: glu = limit, slope, shift");
+    a.glu.limit = static_cast<float>(glu[0]); a.glu.slope = static_cast<float>(glu[1]); a.glu.shift = static_cast<float>(glu[2]);
   }
   a.splits = static_cast<int>(splits); a.epi = static_cast<int>(epi); a.act = static_cast<int>(act);
   a.status = ptr_or_null<int>(status);
@@ -132,7 +136,7 @@ void sample_rows(const Tensor& logits, OptT temperature, OptT top_k, OptT top_p,
 }  // namespace
 
 TORCH_LIBRARY_FRAGMENT(nfb200, m) {
-  m.def("gemm_bf16(Tensor x, Tensor w, Tensor? out, int epi, Tensor? resid, Tensor? bias, Tensor? partial, int splits, Tensor? status, bool pdl, int act=0, Tensor? conv_w=None, Tensor? conv_state=None, Tensor? conv_slot=None, Tensor? conv_out=None, Tensor? prefetch=None, Tensor? out32=None, int out32_from=0, Tensor? act_params=None) -> ()", &gemm_bf16);
+  m.def("gemm_bf16(Tensor x, Tensor w, Tensor? out, int epi, Tensor? resid, Tensor? bias, Tensor? partial, int splits, Tensor? status, bool pdl, int act=0, Tensor? conv_w=None, Tensor? conv_state=None, Tensor? conv_slot=None, Tensor? conv_out=None, Tensor? prefetch=None, Tensor? out32=None, int out32_from=0, Tensor? act_params=None, float[] glu=[]) -> ()", &gemm_bf16);
   m.def("gemm_pick_splits(int T, int N, int K, int epi) -> int", &gemm_pick_splits);
   m.def("argmax_rows(Tensor logits, Tensor out, bool pdl) -> ()", &argmax_rows);
   m.def("sample_rows(Tensor logits, Tensor? temperature, Tensor? top_k, Tensor? top_p, Tensor? min_p, Tensor? presence, Tensor? frequency, Tensor? token_counts, Tensor? seeds, Tensor? positions, int purpose, Tensor out, Tensor? out_prob, Tensor? draft_ids=None, Tensor? accepted=None, Tensor? draft_dist_ids=None, Tensor? draft_dist_probs=None, Tensor? out_dist_ids=None, Tensor? out_dist_probs=None) -> ()", &sample_rows);

@@ -3,12 +3,14 @@
 #include <cuda_runtime.h>
 #include <stdint.h>
 
+#include "../common/glu.cuh"
+
 namespace nfb {
 
 enum GemmEpilogue : int {
   kEpiStore = 0,     // out = act(acc (+ bias[n]))
   kEpiResidual = 1,  // out = resid + acc (+ bias[n])
-  kEpiSwiglu = 2,    // W = [gate; up] (N rows), out[T, N/2] = silu(gate) * up
+  kEpiSwiglu = 2,    // W = [gate; up] (N rows), out[T, N/2] = silu(gate) * up, or another gated unit (GemmArgs::glu)
   kEpiPartial = 3,   // partial[z, T, N] = acc over this split's K range (fp32)
   kEpiPushPartial = 4,  // tensor parallel: fp32 partial tiles are stored into the OWNER rank's receive
                         // buffer [src_rank][split][T][N/world] over NVLink, then the owner's arrival
@@ -52,8 +54,8 @@ struct GemmGather {
 };
 
 // kActXielu: z > 0: a z^2 + z / 2;  z <= 0: b (exp(z) - 1 - z) + z / 2, with (a, b) = act_params[0..1] (both positive).
-// kActRelu2: max(z, 0)^2.
-enum GemmActivation : int { kActNone = 0, kActGeluTanh = 1, kActGeluErf = 2, kActXielu = 3, kActRelu2 = 4 };
+// kActRelu2: max(z, 0)^2.  kActSoftcap: a tanh(z b), with (a, b) = act_params[0..1] (cap and 1 / cap).
+enum GemmActivation : int { kActNone = 0, kActGeluTanh = 1, kActGeluErf = 2, kActXielu = 3, kActRelu2 = 4, kActSoftcap = 5 };
 
 constexpr int kMaxRanks = 8;
 
@@ -80,7 +82,8 @@ struct GemmArgs {
   int64_t ldr = 0;
   const float* bias = nullptr;   // [N] fp32, added by kEpiStore and kEpiResidual
   int act = kActNone;            // kEpiStore: out = act(acc + bias)
-  const float* act_params = nullptr;  // kActXielu: two floats on the device
+  const float* act_params = nullptr;  // kActXielu, kActSoftcap: two floats on the device
+  GluParams glu;                 // kEpiSwiglu
   // kEpiStore: columns n >= out32_from are stored as fp32 in out32[t, n - out32_from] instead of bf16 in `out` (gate
   // rows whose consumers work in 32-bit, or a whole 32-bit result with out32_from = 0; `out` may then be null)
   float* out32 = nullptr;

@@ -72,6 +72,7 @@ struct KernelParams {
   int kb_per_split;    // k-blocks handled by one blockIdx.z
   int num_kb;          // ceil(K / 64)
   int swiglu_half;     // N/2 for the SwiGLU epilogue, else 0
+  GluParams glu;
   __nv_bfloat16* out;
   long long ldo;
   const __nv_bfloat16* resid;
@@ -132,6 +133,7 @@ __device__ __forceinline__ float activate(float z, int mode, float a, float b) {
   if (mode == kActXielu)
     return z > 0.f ? (a * z + 0.5f) * z : b * (__expf(z) - 1.f - z) + 0.5f * z;
   if (mode == kActRelu2) return z > 0.f ? z * z : 0.f;
+  if (mode == kActSoftcap) return a * tanhf(z * b);
   return gelu(z, mode);
 }
 
@@ -421,7 +423,7 @@ __global__ void __launch_bounds__(128) gemm_ws_kernel(const __grid_constant__ CU
               const int j = 2 * m + h;
               const float g = v[j];
               const float u = up_s[(c + j) * 64 + r];
-              a[h] = g / (1.f + __expf(-g)) * u;
+              a[h] = gated_unit(g, u, p.glu);
             }
             const float send = (lane & 1) ? a[0] : a[1];
             const float recv = __shfl_xor_sync(0xffffffffu, send, 1);
@@ -942,7 +944,7 @@ __global__ void __launch_bounds__(kPersistThreads, 1) gemm_persist_kernel(const 
               for (int h = 0; h < 2; ++h) {
                 const int j = 2 * m + h;
                 const float g = __uint_as_float(v[j]);
-                o2[h] = g / (1.f + __expf(-g)) * buf[j * 64 + r];
+                o2[h] = gated_unit(g, buf[j * 64 + r], p.glu);
               }
               const float send = (lane & 1) ? o2[0] : o2[1];
               const float recv = __shfl_xor_sync(0xffffffffu, send, 1);
@@ -1294,7 +1296,7 @@ const char* gemm_bf16(const GemmArgs& a) {
   if ((reinterpret_cast<uintptr_t>(a.w) | reinterpret_cast<uintptr_t>(a.x)) & 15)
     return "gemm_bf16: operands must be 16-byte aligned";
   if ((a.N & 1) || (a.ldo & 1)) return "gemm_bf16: N and ldo must be even";
-  if (a.act == kActXielu && a.act_params == nullptr) return "gemm_bf16: xIELU needs its two parameters";
+  if ((a.act == kActXielu || a.act == kActSoftcap) && a.act_params == nullptr) return "gemm_bf16: the activation needs its two parameters";
   if (a.out32 != nullptr) {
     if (a.epi != kEpiStore || a.conv.state != nullptr) return "gemm_bf16: fp32 columns need the plain store epilogue";
     if ((a.ldo32 & 1) || (a.out32_from & 1) || a.out32_from < 0 || a.out32_from >= a.N ||
@@ -1396,6 +1398,7 @@ const char* gemm_bf16(const GemmArgs& a) {
     kp.conv_C = a.conv.C;
   }
   kp.swiglu_half = a.epi == kEpiSwiglu ? kp.N / 2 : 0;
+  kp.glu = a.glu;
   if (a.epi == kEpiSwiglu && (kp.N % 4)) return "gemm_bf16: SwiGLU needs N % 4 == 0";
   kp.out = static_cast<__nv_bfloat16*>(a.out); kp.ldo = a.ldo;
   kp.resid = static_cast<const __nv_bfloat16*>(a.resid); kp.ldr = a.ldr;

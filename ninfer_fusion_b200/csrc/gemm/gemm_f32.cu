@@ -16,6 +16,7 @@ __device__ __forceinline__ float act_f32(float z, int mode, const float* prm) {
     case kActGeluErf: return 0.5f * z * (1.f + erff(z * 0.7071067811865476f));
     case kActXielu: return z > 0.f ? (prm[0] * z + 0.5f) * z : prm[1] * (expm1f(z) - z) + 0.5f * z;
     case kActRelu2: return z > 0.f ? z * z : 0.f;
+    case kActSoftcap: return prm[0] * tanhf(z * prm[1]);
     default: return z;
   }
 }
@@ -82,7 +83,7 @@ __global__ void __launch_bounds__(kThreads) gemm_f32_kernel(const GemmF32Args p)
 
 const char* gemm_f32(const GemmF32Args& a) {
   if (a.T <= 0 || a.N <= 0 || a.K <= 0) return "gemm_f32: empty problem";
-  if (a.act == kActXielu && a.act_params == nullptr) return "gemm_f32: xIELU needs its two parameters";
+  if ((a.act == kActXielu || a.act == kActSoftcap) && a.act_params == nullptr) return "gemm_f32: the activation needs its two parameters";
   if (a.out == nullptr && !(a.out2 != nullptr && a.out2_from == 0)) return "gemm_f32: no output";
   const dim3 grid((a.N + kTile - 1) / kTile, (a.T + kTile - 1) / kTile);
   if (grid.y > 65535) return "gemm_f32: too many tokens";

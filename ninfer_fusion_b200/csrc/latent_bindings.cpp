@@ -1,8 +1,7 @@
-// torch.ops.nfb200.*: latent attention and gated linear memory (layer-list decoders, models/layered.py).  Activations are
-// bf16 or fp32; every op takes its element type from its tensors.
+// torch.ops.nfb200.*: latent attention (layer-list decoders, models/layered.py).  Activations are bf16 or fp32; every op takes
+// its element type from its tensors.
 #include "attention/latent.h"
 #include "binding_util.h"
-#include "gated/gated.h"
 #include "gemm/head_gemm.h"
 
 namespace {
@@ -23,28 +22,36 @@ void need_table(const Tensor& table) {
   TORCH_CHECK(table.dim() == 2 && table.stride(1) == 1, "block_table must be [rows, pages]");
 }
 
-void latent_prep(const Tensor& proj, int64_t q_rank_true, int64_t rank_true, int64_t rot_true, const Tensor& q_norm,
+void latent_prep(const Tensor& proj, int64_t q_rank_true, int64_t rank_true, int64_t rot_true, OptT q_norm,
                  const Tensor& kv_norm, double eps, const Tensor& freq, const Tensor& table_row, const Tensor& cache_pos,
-                 const Tensor& block_table, const Tensor& q_latent, const Tensor& pages, bool pdl) {
+                 const Tensor& block_table, OptT q_latent, const Tensor& pages, bool pdl) {
   nfb::LatentPrepArgs a;
   a.f32 = act_f32(proj, "proj");
   const int64_t T = proj.size(0);
-  need_rows(proj, "proj"); need_rows(q_latent, "q_latent"); need(q_latent, proj.scalar_type(), "q_latent"); need_table(block_table);
-  const int64_t qr = q_latent.size(1), rank = kv_norm.numel(), rot = proj.size(1) - qr - rank;
-  TORCH_CHECK(q_latent.size(0) == T && rot >= 0, "latent_prep: projection columns");
+  need_rows(proj, "proj"); need_table(block_table);
+  TORCH_CHECK(pages.dim() == 4, "latent pages must be [pages, 1, page size, latent + rotated part]");
+  const int64_t rank = kv_norm.numel(), rot = pages.size(3) - rank, off = proj.size(1) - rank - rot;
+  TORCH_CHECK(rot >= 0 && off >= 0, "latent_prep: projection columns");
   need_pages(pages, proj.scalar_type(), rank + rot);
-  need_vec(q_norm, at::kFloat, qr, "q_norm"); need_vec(kv_norm, at::kFloat, rank, "kv_norm");
+  a.kv_off = static_cast<int>(off);
+  if (q_latent.has_value() && q_latent->defined()) {
+    need_rows(*q_latent, "q_latent"); need(*q_latent, proj.scalar_type(), "q_latent");
+    TORCH_CHECK(q_latent->size(0) == T && q_latent->size(1) == off && q_norm.has_value(), "latent_prep: query latent");
+    need_vec(*q_norm, at::kFloat, off, "q_norm");
+    a.q_rank = static_cast<int>(off); a.q_rank_true = static_cast<int>(q_rank_true);
+    a.q_norm = static_cast<const float*>(q_norm->data_ptr()); a.q_latent = q_latent->data_ptr(); a.ldq = q_latent->stride(0);
+  }
+  need_vec(kv_norm, at::kFloat, rank, "kv_norm");
   need_vec(table_row, at::kInt, T, "table_row"); need_vec(cache_pos, at::kInt, T, "cache_pos");
   a.proj = proj.data_ptr(); a.ldp = proj.stride(0); a.T = static_cast<int>(T);
-  a.q_rank = static_cast<int>(qr); a.q_rank_true = static_cast<int>(q_rank_true);
   a.rank = static_cast<int>(rank); a.rank_true = static_cast<int>(rank_true);
   a.rot = static_cast<int>(rot); a.rot_true = static_cast<int>(rot_true);
-  a.q_norm = static_cast<const float*>(q_norm.data_ptr()); a.kv_norm = static_cast<const float*>(kv_norm.data_ptr());
+  a.kv_norm = static_cast<const float*>(kv_norm.data_ptr());
   a.eps = static_cast<float>(eps); a.freq = freq_ptr(freq, rot_true);
   a.table_row = static_cast<const int*>(table_row.data_ptr()); a.cache_pos = static_cast<const int*>(cache_pos.data_ptr());
   a.block_table = static_cast<const int*>(block_table.data_ptr()); a.table_ld = static_cast<int>(block_table.stride(0));
   a.page_size = static_cast<int>(pages.size(2));
-  a.q_latent = q_latent.data_ptr(); a.ldq = q_latent.stride(0); a.pages = pages.data_ptr();
+  a.pages = pages.data_ptr();
   c10::cuda::CUDAGuard guard(proj.device());
   a.stream = cur_stream(); a.pdl = pdl;
   chk(nfb::latent_prep(a));
@@ -52,8 +59,10 @@ void latent_prep(const Tensor& proj, int64_t q_rank_true, int64_t rank_true, int
 
 nfb::LatentArgs latent_args(const Tensor& q, const Tensor& pages, const Tensor& block_table, const Tensor& table_row,
                             const Tensor& kv_len, int64_t n_heads, int64_t rank, int64_t rot_true, double scale, const Tensor& freq,
-                            OptT sink, const Tensor& out, bool pdl) {
+                            OptT sink, const Tensor& out, int64_t window, bool pdl) {
   nfb::LatentArgs a;
+  TORCH_CHECK(window >= 0, "latent attention: window");
+  a.window = static_cast<int>(window);
   a.f32 = act_f32(q, "q");
   need_rows(q, "q"); need_rows(out, "out"); need(out, q.scalar_type(), "out"); need_table(block_table);
   const int64_t T = q.size(0), rot = pages.size(3) - rank;
@@ -74,11 +83,11 @@ nfb::LatentArgs latent_args(const Tensor& q, const Tensor& pages, const Tensor& 
 
 void latent_token_attention(const Tensor& q_latent, const Tensor& q, const Tensor& pages, const Tensor& block_table,
                             const Tensor& table_row, const Tensor& kv_len, int64_t n_heads, int64_t rot_true, double scale,
-                            const Tensor& freq, OptT sink, const Tensor& out, bool pdl) {
+                            const Tensor& freq, OptT sink, const Tensor& out, bool pdl, int64_t window) {
   c10::cuda::CUDAGuard guard(q.device());
   need_rows(q_latent, "q_latent"); need(q_latent, q.scalar_type(), "q_latent");
   const int64_t rank = q_latent.size(1) / n_heads;
-  nfb::LatentArgs a = latent_args(q, pages, block_table, table_row, kv_len, n_heads, rank, rot_true, scale, freq, sink, out, pdl);
+  nfb::LatentArgs a = latent_args(q, pages, block_table, table_row, kv_len, n_heads, rank, rot_true, scale, freq, sink, out, window, pdl);
   TORCH_CHECK(q_latent.size(0) == a.T && out.size(1) == n_heads * rank, "latent attention: shapes");
   a.q_latent = q_latent.data_ptr(); a.ldl = q_latent.stride(0);
   chk(nfb::latent_token_attention(a));
@@ -88,11 +97,11 @@ void latent_absorbed_attention(const Tensor& q_latent, const Tensor& q, const Te
                                const Tensor& table_row, const Tensor& kv_len, int64_t n_heads, int64_t rot_true, double scale,
                                const Tensor& freq, OptT sink, const Tensor& out, const Tensor& blk_start, const Tensor& blk_count,
                                int64_t max_count, const Tensor& token_seq, const Tensor& cu_seqlens, int64_t max_tokens,
-                               int64_t split_keys, int64_t n_splits, OptT part_o, OptT part_ml, bool pdl) {
+                               int64_t split_keys, int64_t n_splits, OptT part_o, OptT part_ml, bool pdl, int64_t window) {
   c10::cuda::CUDAGuard guard(q.device());
   need_rows(q_latent, "q_latent"); need(q_latent, q.scalar_type(), "q_latent");
   const int64_t rank = q_latent.size(1) / n_heads;
-  nfb::LatentArgs a = latent_args(q, pages, block_table, table_row, kv_len, n_heads, rank, rot_true, scale, freq, sink, out, pdl);
+  nfb::LatentArgs a = latent_args(q, pages, block_table, table_row, kv_len, n_heads, rank, rot_true, scale, freq, sink, out, window, pdl);
   TORCH_CHECK(q_latent.size(0) == a.T && out.size(1) == n_heads * rank, "latent attention: shapes");
   a.q_latent = q_latent.data_ptr(); a.ldl = q_latent.stride(0);
   nfb::LatentBlocks b;
@@ -117,7 +126,8 @@ bool latent_absorbed_supported(int64_t rank, int64_t rot) {
 void latent_gather(const Tensor& pages, const Tensor& block_table, const Tensor& seqs, int64_t max_len, const Tensor& rows, bool pdl) {
   need(pages, at::kBFloat16, "pages"); need(rows, at::kBFloat16, "rows"); need_table(block_table);
   need_pages(pages, at::kBFloat16, pages.size(3));
-  need_vec(seqs, at::kInt, seqs.size(0) * 3, "seqs");
+  TORCH_CHECK(seqs.dim() == 2 && seqs.size(1) == 4, "seqs must be [n, 4]");
+  need_vec(seqs, at::kInt, seqs.size(0) * 4, "seqs");
   TORCH_CHECK(rows.dim() == 2 && rows.is_contiguous() && rows.size(1) == pages.size(3), "latent_gather: rows shape");
   nfb::LatentArgs a;
   a.pages = pages.data_ptr(); a.rank = static_cast<int>(pages.size(3)); a.rot = 0; a.page_size = static_cast<int>(pages.size(2));
@@ -133,8 +143,10 @@ void latent_gather(const Tensor& pages, const Tensor& block_table, const Tensor&
 void latent_expanded_attention(const Tensor& q, const Tensor& rows, const Tensor& kv, const Tensor& kv_len,
                                int64_t n_heads, int64_t rank, int64_t rot_true, double scale, const Tensor& freq, OptT sink,
                                const Tensor& out, const Tensor& blk_start, const Tensor& blk_count, int64_t max_count,
-                               const Tensor& token_seq, const Tensor& seq_base, bool pdl) {
+                               const Tensor& token_seq, const Tensor& seq_base, bool pdl, int64_t window) {
   nfb::LatentArgs a;
+  TORCH_CHECK(window >= 0, "latent attention: window");
+  a.window = static_cast<int>(window);
   need(q, at::kBFloat16, "q"); need(rows, at::kBFloat16, "rows"); need(kv, at::kBFloat16, "kv"); need(out, at::kBFloat16, "out");
   need_rows(q, "q"); need_rows(out, "out");
   TORCH_CHECK(rows.dim() == 2 && rows.is_contiguous() && kv.dim() == 2 && kv.is_contiguous() && rows.size(0) == kv.size(0),
@@ -145,6 +157,7 @@ void latent_expanded_attention(const Tensor& q, const Tensor& rows, const Tensor
   TORCH_CHECK(dim > 0 && kv.size(1) == n_heads * (dim + vdim), "latent attention: expanded columns");
   need_vec(kv_len, at::kInt, T, "kv_len"); need_vec(token_seq, at::kInt, T, "token_seq");
   need(seq_base, at::kInt, "seq_base");
+  TORCH_CHECK(seq_base.dim() == 2 && seq_base.size(1) == 2 && seq_base.is_contiguous(), "seq_base must be [sequences, 2]");
   if (sink.has_value() && sink->defined()) need_vec(*sink, at::kFloat, n_heads, "sink");
   a.q = q.data_ptr(); a.ldq = q.stride(0); a.kv_len = static_cast<const int*>(kv_len.data_ptr());
   a.T = static_cast<int>(T); a.n_heads = static_cast<int>(n_heads); a.dim = static_cast<int>(dim); a.rank = static_cast<int>(rank);
@@ -187,59 +200,15 @@ void head_gemm(const Tensor& x, int64_t x_step, const Tensor& w, const Tensor& o
   chk(nfb::head_gemm(a));
 }
 
-void gated_memory(const Tensor& proj, int64_t q_off, int64_t v_off, const Tensor& gates, const Tensor& lower, int64_t vdim_true,
-                  double eps, const Tensor& norm, const Tensor& cu_seqlens, const Tensor& state_slot, const Tensor& S,
-                  const Tensor& out, bool write_state, OptT chunk_ws, bool pdl, bool one_token) {
-  nfb::GatedArgs a;
-  a.f32 = act_f32(proj, "proj");
-  need_rows(proj, "proj"); need_rows(out, "out"); need(out, proj.scalar_type(), "out");
-  need(gates, at::kFloat, "gates"); need_rows(gates, "gates"); need(S, at::kFloat, "S");
-  TORCH_CHECK(S.dim() == 4 && S.is_contiguous(), "gated memory: state must be [slots, heads, dim, vdim]");
-  const int64_t T = proj.size(0), H = S.size(1), D = S.size(2), V = S.size(3), B = state_slot.numel(), cols = proj.size(1);
-  TORCH_CHECK(out.size(0) == T && out.size(1) == H * V && gates.size(0) == T && gates.size(1) >= H * D, "gated memory: out / gates shape");
-  TORCH_CHECK(q_off >= 0 && q_off + H * D <= cols && v_off >= 0 && v_off + H * V <= cols, "gated memory: projection columns");
-  TORCH_CHECK(vdim_true > 0 && vdim_true <= V, "gated memory: value width");
-  need_vec(lower, at::kFloat, H * D, "lower"); need_vec(norm, at::kFloat, V, "norm");
-  need_vec(cu_seqlens, at::kInt, B + 1, "cu_seqlens"); need_vec(state_slot, at::kInt, B, "state_slot");
-  a.proj = proj.data_ptr(); a.ldp = proj.stride(0); a.q_off = static_cast<int>(q_off); a.v_off = static_cast<int>(v_off);
-  a.gates = static_cast<const float*>(gates.data_ptr()); a.ldg = gates.stride(0); a.lower = static_cast<const float*>(lower.data_ptr());
-  a.n_heads = static_cast<int>(H); a.dim = static_cast<int>(D); a.vdim = static_cast<int>(V); a.vdim_true = static_cast<int>(vdim_true);
-  a.eps = static_cast<float>(eps); a.norm = static_cast<const float*>(norm.data_ptr());
-  a.cu_seqlens = static_cast<const int*>(cu_seqlens.data_ptr()); a.state_slot = static_cast<const int*>(state_slot.data_ptr());
-  a.T = static_cast<int>(T); a.n_seq = static_cast<int>(B); a.S = static_cast<float*>(S.data_ptr());
-  a.out = out.data_ptr(); a.ldo = out.stride(0); a.write_state = write_state;
-  TORCH_CHECK(!one_token || T == B, "gated memory: one token per sequence expected");
-  a.one_token = one_token;
-  c10::cuda::CUDAGuard guard(proj.device());
-  a.stream = cur_stream(); a.pdl = pdl;
-  if (chunk_ws.has_value() && chunk_ws->defined()) {
-    need_cuda(*chunk_ws, "chunk_ws");
-    chk(nfb::gated_chunked(a, chunk_ws->data_ptr(), chunk_ws->numel() * chunk_ws->element_size()));
-  } else {
-    chk(nfb::gated_recurrent(a));
-  }
-}
-
-int64_t gated_chunked_workspace_bytes(int64_t T, int64_t n_seq, int64_t n_heads, int64_t dim, int64_t vdim) {
-  return nfb::gated_chunked_workspace_bytes(static_cast<int>(T), static_cast<int>(n_seq), static_cast<int>(n_heads),
-                                            static_cast<int>(dim), static_cast<int>(vdim));
-}
-bool gated_chunked_supported(int64_t dim, int64_t vdim) {
-  return nfb::gated_chunked_supported(static_cast<int>(dim), static_cast<int>(vdim));
-}
-
 }  // namespace
 
 TORCH_LIBRARY_FRAGMENT(nfb200, m) {
-  m.def("latent_prep(Tensor proj, int q_rank_true, int rank_true, int rot_true, Tensor q_norm, Tensor kv_norm, float eps, Tensor freq, Tensor table_row, Tensor cache_pos, Tensor block_table, Tensor q_latent, Tensor pages, bool pdl) -> ()", &latent_prep);
-  m.def("latent_token_attention(Tensor q_latent, Tensor q, Tensor pages, Tensor block_table, Tensor table_row, Tensor kv_len, int n_heads, int rot_true, float scale, Tensor freq, Tensor? sink, Tensor out, bool pdl) -> ()", &latent_token_attention);
-  m.def("latent_absorbed_attention(Tensor q_latent, Tensor q, Tensor pages, Tensor block_table, Tensor table_row, Tensor kv_len, int n_heads, int rot_true, float scale, Tensor freq, Tensor? sink, Tensor out, Tensor blk_start, Tensor blk_count, int max_count, Tensor token_seq, Tensor cu_seqlens, int max_tokens, int split_keys, int n_splits, Tensor? part_o, Tensor? part_ml, bool pdl) -> ()", &latent_absorbed_attention);
+  m.def("latent_prep(Tensor proj, int q_rank_true, int rank_true, int rot_true, Tensor? q_norm, Tensor kv_norm, float eps, Tensor freq, Tensor table_row, Tensor cache_pos, Tensor block_table, Tensor? q_latent, Tensor pages, bool pdl) -> ()", &latent_prep);
+  m.def("latent_token_attention(Tensor q_latent, Tensor q, Tensor pages, Tensor block_table, Tensor table_row, Tensor kv_len, int n_heads, int rot_true, float scale, Tensor freq, Tensor? sink, Tensor out, bool pdl, int window=0) -> ()", &latent_token_attention);
+  m.def("latent_absorbed_attention(Tensor q_latent, Tensor q, Tensor pages, Tensor block_table, Tensor table_row, Tensor kv_len, int n_heads, int rot_true, float scale, Tensor freq, Tensor? sink, Tensor out, Tensor blk_start, Tensor blk_count, int max_count, Tensor token_seq, Tensor cu_seqlens, int max_tokens, int split_keys, int n_splits, Tensor? part_o, Tensor? part_ml, bool pdl, int window=0) -> ()", &latent_absorbed_attention);
   m.def("latent_absorbed_supported(int rank, int rot) -> bool", &latent_absorbed_supported);
   m.def("latent_gather(Tensor pages, Tensor block_table, Tensor seqs, int max_len, Tensor rows, bool pdl) -> ()", &latent_gather);
-  m.def("latent_expanded_attention(Tensor q, Tensor rows, Tensor kv, Tensor kv_len, int n_heads, int rank, int rot_true, float scale, Tensor freq, Tensor? sink, Tensor out, Tensor blk_start, Tensor blk_count, int max_count, Tensor token_seq, Tensor seq_base, bool pdl) -> ()", &latent_expanded_attention);
+  m.def("latent_expanded_attention(Tensor q, Tensor rows, Tensor kv, Tensor kv_len, int n_heads, int rank, int rot_true, float scale, Tensor freq, Tensor? sink, Tensor out, Tensor blk_start, Tensor blk_count, int max_count, Tensor token_seq, Tensor seq_base, bool pdl, int window=0) -> ()", &latent_expanded_attention);
   m.def("latent_expanded_supported(int dim, int rot, int vdim) -> bool", &latent_expanded_supported);
   m.def("head_gemm(Tensor x, int x_step, Tensor w, Tensor out, Tensor? token_seq, Tensor? cu_seqlens, int max_tokens, bool pdl) -> ()", &head_gemm);
-  m.def("gated_memory(Tensor proj, int q_off, int v_off, Tensor gates, Tensor lower, int vdim_true, float eps, Tensor norm, Tensor cu_seqlens, Tensor state_slot, Tensor S, Tensor out, bool write_state, Tensor? chunk_ws, bool pdl, bool one_token=False) -> ()", &gated_memory);
-  m.def("gated_chunked_workspace_bytes(int T, int n_seq, int n_heads, int dim, int vdim) -> int", &gated_chunked_workspace_bytes);
-  m.def("gated_chunked_supported(int dim, int vdim) -> bool", &gated_chunked_supported);
 }

@@ -46,7 +46,7 @@ void gemm_f32(const Tensor& x, const Tensor& w, OptT out, OptT bias, int64_t act
   need(x, at::kFloat, "x"); need(w, at::kFloat, "w");
   need_rows(x, "x"); need_rows(w, "w");
   TORCH_CHECK(x.size(1) == w.size(1), "gemm_f32: K mismatch");
-  TORCH_CHECK(act >= 0 && act <= 4, "gemm_f32: unknown activation");
+  TORCH_CHECK(act >= 0 && act <= 5, "gemm_f32: unknown activation");
   nfb::GemmF32Args a;
   a.w = static_cast<const float*>(w.data_ptr()); a.N = w.size(0); a.K = w.size(1); a.ldw = w.stride(0);
   a.x = static_cast<const float*>(x.data_ptr()); a.T = x.size(0); a.ldx = x.stride(0);

@@ -24,6 +24,8 @@
 #include <cuda_runtime.h>
 #include <stdint.h>
 
+#include "../common/glu.cuh"
+
 namespace nfb {
 
 constexpr int kMoeMaxRanks = 8;
@@ -53,6 +55,21 @@ struct MoeRouteParams {
   float* shared_gate;  // [T] sigmoid of the shared gate logit
 };
 const char* moe_route(const MoeRouteParams& p, cudaStream_t stream);
+
+// Routing by corrected scores (one GPU): s = softmax over all E + identity outputs; the k largest s + correction are chosen
+// (ties: lower number); weight = scale * s, not renormalised.  Choices >= E are identity experts: they get no row (pos = -1).
+struct MoeRouteScoredParams {
+  int T, E, identity, k;
+  const float* logits;      // [T, ld] fp32
+  long long ld;
+  const float* correction;  // [E + identity], or null
+  float scale;
+  int* hist;                // [E], zero on entry
+  int* ids;                 // [T, k]
+  float* weights;           // [T, k]
+  int* pos;                 // [T, k]
+};
+const char* moe_route_scored(const MoeRouteScoredParams& p, cudaStream_t stream, bool pdl);
 
 struct MoePlanParams {
   int world, rank, E, tile_tokens, cap, max_tiles;
@@ -87,7 +104,7 @@ struct MoePushParams {
 const char* moe_push(const MoePushParams& p, cudaStream_t stream);
 
 enum MoeGemmEpilogue : int {
-  kMoeEpiSwiglu = 0,  // W_e = [gate; up], out[row, n] = silu(gate) * up
+  kMoeEpiSwiglu = 0,  // W_e = [gate; up], out[row, n] = gated unit of (gate, up): silu(gate) * up, or as `glu` says
   kMoeEpiReturn = 1,  // out row goes to the source rank's return buffer [token * k + j, N]
 };
 
@@ -104,6 +121,7 @@ struct MoeGemmArgs {
   const MoeState* state = nullptr;
   int epi = kMoeEpiSwiglu;
   void* out = nullptr;      // kMoeEpiSwiglu: [cap, rows_per_expert / 2] bf16
+  GluParams glu;            // kMoeEpiSwiglu (bf16 experts)
   int64_t ldo = 0;
   // kMoeEpiReturn
   int world = 1;
@@ -117,6 +135,9 @@ struct MoeGemmArgs {
   const float* x_scale = nullptr;   // [cap, K / 128]
 };
 const char* moe_gemm(const MoeGemmArgs& a);
+// 32-bit experts: x, w, out and ret are fp32, tiles of 64 rows.  kMoeEpiSwiglu leaves the columns [gate | up] as they are
+// (out [cap, rows_per_expert]); kMoeEpiReturn stores row token * k + j of peer_ret[0].  No TF32, no counters.
+const char* moe_gemm_f32(const MoeGemmArgs& a);
 // Same tile walk over e4m3 weights with 128 x 128 block scales and activations quantised per row and 128-wide k-block.
 const char* moe_gemm_fp8(const MoeGemmArgs& a);
 // Quantises the first min(max_rows, state->total_rows) rows of x [max_rows, K] (state may be null: all rows).

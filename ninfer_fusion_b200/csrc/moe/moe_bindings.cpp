@@ -1,32 +1,9 @@
 // torch.ops.nfb200.moe_* : checked adapters from torch tensors to the mixture-of-experts launchers.
-#include <ATen/ATen.h>
-#include <ATen/cuda/CUDAContext.h>
-#include <c10/cuda/CUDAGuard.h>
-#include <torch/library.h>
-
-#include "moe.h"
+#include "moe_binding_util.h"
 
 namespace {
 
-using at::Tensor;
-using OptT = const std::optional<Tensor>&;
-
-inline cudaStream_t cur_stream() { return at::cuda::getCurrentCUDAStream().stream(); }
-inline void chk(const char* err) { TORCH_CHECK(err == nullptr, err ? err : ""); }
-inline void need(const Tensor& t, at::ScalarType dt, const char* name) {
-  TORCH_CHECK(t.is_cuda(), name, " must be a CUDA tensor");
-  TORCH_CHECK(t.scalar_type() == dt, name, " has the wrong dtype");
-  TORCH_CHECK(t.is_contiguous() || (t.dim() == 2 && t.stride(1) == 1), name, " must have unit inner stride");
-}
-template <typename T>
-inline T* ptr_or_null(OptT t) {
-  return t.has_value() && t->defined() ? static_cast<T*>(t->data_ptr()) : nullptr;
-}
-inline nfb::MoeState* state_ptr(const Tensor& state) {
-  TORCH_CHECK(state.is_cuda() && state.scalar_type() == at::kByte &&
-                  state.numel() >= static_cast<int64_t>(sizeof(nfb::MoeState)), "bad MoE state tensor");
-  return reinterpret_cast<nfb::MoeState*>(state.data_ptr());
-}
+using namespace nfb_moe_bind;
 
 void moe_route(const Tensor& logits, int64_t E, int64_t k, bool norm_topk, bool has_shared_gate, const Tensor& hist,
                const Tensor& ids, const Tensor& weights, const Tensor& pos, OptT shared_gate) {
@@ -49,6 +26,28 @@ void moe_route(const Tensor& logits, int64_t E, int64_t k, bool norm_topk, bool 
     p.shared_gate = static_cast<float*>(shared_gate->data_ptr());
   }
   chk(nfb::moe_route(p, cur_stream()));
+}
+
+void moe_route_scored(const Tensor& logits, int64_t E, int64_t identity, int64_t k, OptT correction, double scale, const Tensor& hist,
+                      const Tensor& ids, const Tensor& weights, const Tensor& pos, bool pdl) {
+  need(logits, at::kFloat, "logits"); need(hist, at::kInt, "hist"); need(ids, at::kInt, "ids");
+  need(weights, at::kFloat, "weights"); need(pos, at::kInt, "pos");
+  const int64_t T = logits.size(0);
+  TORCH_CHECK(logits.dim() == 2 && logits.size(1) >= E + identity, "logits too narrow");
+  TORCH_CHECK(hist.numel() >= E && ids.numel() >= T * k && weights.numel() >= T * k && pos.numel() >= T * k);
+  TORCH_CHECK(ids.is_contiguous() && weights.is_contiguous() && pos.is_contiguous());
+  nfb::MoeRouteScoredParams p = {};
+  if (correction.has_value() && correction->defined()) {
+    need(*correction, at::kFloat, "correction");
+    TORCH_CHECK(correction->is_contiguous() && correction->numel() >= E + identity);
+    p.correction = static_cast<const float*>(correction->data_ptr());
+  }
+  p.T = static_cast<int>(T); p.E = static_cast<int>(E); p.identity = static_cast<int>(identity); p.k = static_cast<int>(k);
+  p.logits = static_cast<const float*>(logits.data_ptr()); p.ld = logits.stride(0); p.scale = static_cast<float>(scale);
+  p.hist = static_cast<int*>(hist.data_ptr()); p.ids = static_cast<int*>(ids.data_ptr());
+  p.weights = static_cast<float*>(weights.data_ptr()); p.pos = static_cast<int*>(pos.data_ptr());
+  c10::cuda::CUDAGuard guard(logits.device());
+  chk(nfb::moe_route_scored(p, cur_stream(), pdl));
 }
 
 // tiles: int32 [3, max_tiles] = (local expert, first row, valid rows) per token tile
@@ -105,11 +104,14 @@ void moe_push(int64_t world, int64_t rank, int64_t E, int64_t cap, const Tensor&
   chk(nfb::moe_push(p, cur_stream()));
 }
 
-// x: [cap, K] expert-sorted rows; w: [local experts, rows per expert, K].
+// x: [cap, K] expert-sorted rows; w: [local experts, rows per expert, K], bf16, or fp32 for 32-bit runs (one GPU).
 void moe_gemm(const Tensor& x, const Tensor& w, int64_t epi, int64_t tile_tokens, int64_t max_tiles, const Tensor& tiles,
               const Tensor& state, OptT out, int64_t world, OptT recv_meta, at::IntArrayRef peer_bases, int64_t ret_off,
-              int64_t ret_flag_off, OptT status) {
-  need(x, at::kBFloat16, "x"); need(w, at::kBFloat16, "w"); need(tiles, at::kInt, "tiles");
+              int64_t ret_flag_off, OptT status, at::ArrayRef<double> glu) {
+  const auto dt = w.scalar_type();
+  TORCH_CHECK(dt == at::kBFloat16 || dt == at::kFloat, "moe_gemm: bf16 or fp32 experts");
+  const bool f32 = dt == at::kFloat;
+  need(x, dt, "x"); need(w, dt, "w"); need(tiles, at::kInt, "tiles");
   TORCH_CHECK(x.dim() == 2 && w.dim() == 3 && w.is_contiguous() && x.size(1) == w.size(2), "moe_gemm: shapes");
   TORCH_CHECK(tiles.dim() == 2 && tiles.size(0) == 3 && tiles.is_contiguous() && max_tiles <= tiles.size(1));
   c10::cuda::CUDAGuard guard(x.device());
@@ -125,8 +127,8 @@ void moe_gemm(const Tensor& x, const Tensor& w, int64_t epi, int64_t tile_tokens
   a.epi = static_cast<int>(epi);
   if (epi == nfb::kMoeEpiSwiglu) {
     TORCH_CHECK(out.has_value() && out->defined(), "moe_gemm: out required");
-    need(*out, at::kBFloat16, "out");
-    TORCH_CHECK(out->dim() == 2 && out->size(0) >= x.size(0) && out->size(1) == w.size(1) / 2, "moe_gemm: out shape");
+    need(*out, dt, "out");
+    TORCH_CHECK(out->dim() == 2 && out->size(0) >= x.size(0) && out->size(1) == (f32 ? w.size(1) : w.size(1) / 2), "moe_gemm: out shape");
     a.out = out->data_ptr(); a.ldo = out->stride(0);
   } else {
     TORCH_CHECK(recv_meta.has_value() && recv_meta->defined(), "moe_gemm: recv_meta required");
@@ -140,63 +142,12 @@ void moe_gemm(const Tensor& x, const Tensor& w, int64_t epi, int64_t tile_tokens
     }
   }
   a.status = ptr_or_null<int>(status);
-  a.stream = cur_stream();
-  chk(nfb::moe_gemm(a));
-}
-
-// fp8 block-scaled variant: x [cap, K] and w [experts, rows, K] are uint8 e4m3 codes.
-void moe_gemm_fp8(const Tensor& x, const Tensor& x_scale, const Tensor& w, const Tensor& w_scale, int64_t epi,
-                  int64_t tile_tokens, int64_t max_tiles, const Tensor& tiles, const Tensor& state, OptT out, int64_t world,
-                  OptT recv_meta, at::IntArrayRef peer_bases, int64_t ret_off, int64_t ret_flag_off, OptT status) {
-  need(x, at::kByte, "x"); need(w, at::kByte, "w"); need(tiles, at::kInt, "tiles");
-  need(x_scale, at::kFloat, "x_scale"); need(w_scale, at::kFloat, "w_scale");
-  TORCH_CHECK(x.dim() == 2 && w.dim() == 3 && w.is_contiguous() && x.size(1) == w.size(2), "moe_gemm_fp8: shapes");
-  TORCH_CHECK(tiles.dim() == 2 && tiles.size(0) == 3 && tiles.is_contiguous() && max_tiles <= tiles.size(1));
-  const int64_t nkb = w.size(2) / 128;
-  TORCH_CHECK(w_scale.is_contiguous() && w_scale.numel() == w.size(0) * (w.size(1) / 128) * nkb, "moe_gemm_fp8: w_scale shape");
-  TORCH_CHECK(x_scale.is_contiguous() && x_scale.numel() >= x.size(0) * nkb, "moe_gemm_fp8: x_scale shape");
-  c10::cuda::CUDAGuard guard(x.device());
-  nfb::MoeGemmArgs a;
-  a.w = w.data_ptr(); a.n_local_experts = static_cast<int>(w.size(0)); a.rows_per_expert = w.size(1);
-  a.K = w.size(2); a.ldw = w.size(2);
-  a.x = x.data_ptr(); a.cap = x.size(0); a.ldx = x.stride(0);
-  a.w_scale = static_cast<const float*>(w_scale.data_ptr()); a.x_scale = static_cast<const float*>(x_scale.data_ptr());
-  a.tile_tokens = static_cast<int>(tile_tokens); a.max_tiles = static_cast<int>(max_tiles);
-  const int* t = static_cast<const int*>(tiles.data_ptr());
-  const int64_t stride = tiles.size(1);
-  a.tile_expert = t; a.tile_row0 = t + stride; a.tile_rows = t + 2 * stride;
-  a.state = state_ptr(state);
-  a.epi = static_cast<int>(epi);
-  if (epi == nfb::kMoeEpiSwiglu) {
-    TORCH_CHECK(out.has_value() && out->defined(), "moe_gemm_fp8: out required");
-    need(*out, at::kBFloat16, "out");
-    TORCH_CHECK(out->dim() == 2 && out->size(0) >= x.size(0) && out->size(1) == w.size(1) / 2, "moe_gemm_fp8: out shape");
-    a.out = out->data_ptr(); a.ldo = out->stride(0);
-  } else {
-    TORCH_CHECK(recv_meta.has_value() && recv_meta->defined(), "moe_gemm_fp8: recv_meta required");
-    need(*recv_meta, at::kInt, "recv_meta");
-    TORCH_CHECK(static_cast<int64_t>(peer_bases.size()) == world && world <= nfb::kMoeMaxRanks, "peer_bases size");
-    a.world = static_cast<int>(world);
-    a.recv_meta = static_cast<const int*>(recv_meta->data_ptr());
-    for (int r = 0; r < world; ++r) {
-      a.peer_ret[r] = reinterpret_cast<__nv_bfloat16*>(peer_bases[r] + ret_off);
-      a.peer_ret_flag[r] = reinterpret_cast<unsigned int*>(peer_bases[r] + ret_flag_off);
-    }
+  if (!glu.empty()) {
+    TORCH_CHECK(glu.size() == 3, "moe_gemm: glu = limit, slope, shift");
+    a.glu.limit = static_cast<float>(glu[0]); a.glu.slope = static_cast<float>(glu[1]); a.glu.shift = static_cast<float>(glu[2]);
   }
-  a.status = ptr_or_null<int>(status);
   a.stream = cur_stream();
-  chk(nfb::moe_gemm_fp8(a));
-}
-
-void moe_quant_rows_block128(const Tensor& x, const Tensor& codes, const Tensor& scales, OptT state) {
-  need(x, at::kBFloat16, "x"); need(codes, at::kByte, "codes"); need(scales, at::kFloat, "scales");
-  TORCH_CHECK(x.dim() == 2 && codes.is_contiguous() && codes.numel() >= x.numel() && scales.is_contiguous() &&
-              scales.numel() >= x.size(0) * (x.size(1) / 128), "moe_quant_rows_block128: shapes");
-  c10::cuda::CUDAGuard guard(x.device());
-  const nfb::MoeState* st = state.has_value() && state->defined() ? state_ptr(*state) : nullptr;
-  chk(nfb::moe_quant_rows_block128(static_cast<const __nv_bfloat16*>(x.data_ptr()), x.stride(0), static_cast<int>(x.size(0)),
-                                   static_cast<int>(x.size(1)), st, static_cast<uint8_t*>(codes.data_ptr()),
-                                   static_cast<float*>(scales.data_ptr()), cur_stream()));
+  chk(f32 ? nfb::moe_gemm_f32(a) : nfb::moe_gemm(a));
 }
 
 void moe_combine(const Tensor& x, const Tensor& weights, const Tensor& ret, int64_t my_base, int64_t ret_flag_off,
@@ -242,9 +193,8 @@ TORCH_LIBRARY_FRAGMENT(nfb200, m) {
   m.def("moe_route(Tensor logits, int E, int k, bool norm_topk, bool has_shared_gate, Tensor hist, Tensor ids, Tensor weights, Tensor pos, Tensor? shared_gate) -> ()", &moe_route);
   m.def("moe_plan(int world, int rank, int E, int tile_tokens, int cap, Tensor hist, int[] peer_bases, int counts_off, int count_flag_off, Tensor send_base, Tensor tiles, Tensor state, Tensor? status) -> ()", &moe_plan);
   m.def("moe_push(int world, int rank, int E, int cap, Tensor x, Tensor ids, Tensor pos, Tensor send_base, int[] peer_bases, int recv_x_off, int recv_meta_off, int arrive_flag_off, Tensor state, Tensor? status) -> ()", &moe_push);
-  m.def("moe_gemm(Tensor x, Tensor w, int epi, int tile_tokens, int max_tiles, Tensor tiles, Tensor state, Tensor? out, int world, Tensor? recv_meta, int[] peer_bases, int ret_off, int ret_flag_off, Tensor? status) -> ()", &moe_gemm);
-  m.def("moe_gemm_fp8(Tensor x, Tensor x_scale, Tensor w, Tensor w_scale, int epi, int tile_tokens, int max_tiles, Tensor tiles, Tensor state, Tensor? out, int world, Tensor? recv_meta, int[] peer_bases, int ret_off, int ret_flag_off, Tensor? status) -> ()", &moe_gemm_fp8);
-  m.def("moe_quant_rows_block128(Tensor x, Tensor codes, Tensor scales, Tensor? state) -> ()", &moe_quant_rows_block128);
+  m.def("moe_gemm(Tensor x, Tensor w, int epi, int tile_tokens, int max_tiles, Tensor tiles, Tensor state, Tensor? out, int world, Tensor? recv_meta, int[] peer_bases, int ret_off, int ret_flag_off, Tensor? status, float[] glu=[]) -> ()", &moe_gemm);
+  m.def("moe_route_scored(Tensor logits, int E, int identity, int k, Tensor? correction, float scale, Tensor hist, Tensor ids, Tensor weights, Tensor pos, bool pdl) -> ()", &moe_route_scored);
   m.def("moe_combine(Tensor x, Tensor weights, Tensor ret, int my_base, int ret_flag_off, Tensor? shared, Tensor? shared_gate, Tensor? norm_w, Tensor? normed, float eps, Tensor state, Tensor? status) -> ()", &moe_combine);
   m.def("moe_state_bytes() -> int", &moe_state_bytes);
   m.def("moe_tile_tokens(float rows_per_expert) -> int", &moe_tile_tokens);

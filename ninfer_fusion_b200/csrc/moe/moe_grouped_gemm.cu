@@ -6,7 +6,7 @@
 // tcgen05.mma -> TMEM -> tcgen05.ld epilogue.  blockIdx.y walks a fixed upper bound of token tiles
 // and CTAs beyond the device-side tile count leave at once, so the launch is graph-capturable although
 // the routing is data dependent.  Epilogues:
-//   SwiGLU : W_e = [gate; up]; 64 gate rows + the matching 64 up rows form one 128-row tile;
+//   gated unit (SwiGLU or a bounded form): W_e = [gate; up]; 64 gate rows + the matching 64 up rows form one 128-row tile;
 //   return : each output row is stored into the return buffer of the rank that owns the token
 //            (peer stores over NVLink), then that rank's arrival counter is advanced by the number
 //            of rows it got from this CTA -- the combine all-to-all happens inside the GEMM.
@@ -53,6 +53,7 @@ struct MoeKernelParams {
   __nv_bfloat16* peer_ret[kMoeMaxRanks];
   unsigned int* peer_ret_flag[kMoeMaxRanks];
   int* status;
+  GluParams glu;
 };
 
 template <int TN, int EPI>
@@ -210,7 +211,7 @@ __global__ void __launch_bounds__(128) moe_gemm_kernel(const __grid_constant__ C
               const int j = 2 * m + h;
               const float g = v[j];
               const float u = up_s[(c + j) * 64 + r];
-              a[h] = g / (1.f + __expf(-g)) * u;
+              a[h] = gated_unit(g, u, p.glu);
             }
             const float send = (lane & 1) ? a[0] : a[1];
             const float recv = __shfl_xor_sync(0xffffffffu, send, 1);
@@ -347,7 +348,7 @@ const char* moe_gemm(const MoeGemmArgs& a) {
   kp.num_kb = static_cast<int>((a.K + kBlockK - 1) / kBlockK);
   kp.rows_per_expert = static_cast<int>(a.rows_per_expert);
   kp.tile_expert = a.tile_expert; kp.tile_row0 = a.tile_row0; kp.tile_rows = a.tile_rows; kp.state = a.state;
-  kp.status = a.status;
+  kp.status = a.status; kp.glu = a.glu;
   dim3 grid;
   grid.y = a.max_tiles;
   if (a.epi == kMoeEpiSwiglu) {
@@ -356,14 +357,14 @@ const char* moe_gemm(const MoeGemmArgs& a) {
     kp.out = static_cast<__nv_bfloat16*>(a.out); kp.ldo = a.ldo;
     grid.x = static_cast<unsigned>(a.rows_per_expert / 2 / 64);
   } else if (a.epi == kMoeEpiReturn) {
-    if (a.rows_per_expert % 128) return "moe_gemm: expert rows must be a multiple of 128";
+    if (a.rows_per_expert % 8) return "moe_gemm: expert rows must be a multiple of 8";
     if (a.world < 1 || a.world > kMoeMaxRanks || a.recv_meta == nullptr) return "moe_gemm: bad return set-up";
     kp.world = a.world; kp.recv_meta = a.recv_meta;
     for (int r = 0; r < a.world; ++r) {
       if (a.peer_ret[r] == nullptr || a.peer_ret_flag[r] == nullptr) return "moe_gemm: missing peer pointer";
       kp.peer_ret[r] = a.peer_ret[r]; kp.peer_ret_flag[r] = a.peer_ret_flag[r];
     }
-    grid.x = static_cast<unsigned>(a.rows_per_expert / 128);
+    grid.x = static_cast<unsigned>((a.rows_per_expert + 127) / 128);
   } else {
     return "moe_gemm: unknown epilogue";
   }

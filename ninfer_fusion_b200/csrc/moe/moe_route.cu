@@ -8,6 +8,7 @@
 #include "moe.h"
 
 #include "../comm/peer_sync.cuh"
+#include "../common/launch.h"
 #include "../common/ptx.cuh"
 
 namespace nfb {
@@ -70,6 +71,66 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(const MoeRo
   }
   if (lane == 0 && p.shared_gate != nullptr)
     p.shared_gate[t] = p.has_shared_gate ? 1.f / (1.f + __expf(-__bfloat162float(row[p.E]))) : 1.f;
+}
+
+// ---------------------------------------------------------------------------------------------
+// moe_route_scored: one warp per token
+// ---------------------------------------------------------------------------------------------
+__global__ void __launch_bounds__(kRouteWarps * 32) moe_route_scored_kernel(const MoeRouteScoredParams p) {
+  pdl_launch_next();
+  pdl_wait_prior();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t = blockIdx.x * kRouteWarps + warp;
+  if (t >= p.T) return;
+  const int n = p.E + p.identity;
+  const float* row = p.logits + static_cast<long long>(t) * p.ld;
+  float s[kPerLane], top = -INFINITY, sum = 0.f;
+#pragma unroll
+  for (int i = 0; i < kPerLane; ++i) {
+    const int e = lane + 32 * i;
+    s[i] = e < n ? row[e] : -INFINITY;
+    top = fmaxf(top, s[i]);
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
+#pragma unroll
+  for (int i = 0; i < kPerLane; ++i) {
+    s[i] = lane + 32 * i < n ? expf(s[i] - top) : 0.f;
+    sum += s[i];
+  }
+  const float inv = 1.f / warp_sum(sum);
+  float c[kPerLane];                               // choice scores
+#pragma unroll
+  for (int i = 0; i < kPerLane; ++i) {
+    const int e = lane + 32 * i;
+    s[i] *= inv;
+    c[i] = e < n ? s[i] + (p.correction != nullptr ? p.correction[e] : 0.f) : -INFINITY;
+  }
+  for (int r = 0; r < p.k; ++r) {
+    float bv = -INFINITY, bs = 0.f;
+    int bi = 0x7fffffff;
+#pragma unroll
+    for (int i = 0; i < kPerLane; ++i) {
+      const int e = lane + 32 * i;
+      if (c[i] > bv || (c[i] == bv && e < bi && e < n)) { bv = c[i]; bs = s[i]; bi = e; }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, bv, o), os = __shfl_xor_sync(0xffffffffu, bs, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+      if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bs = os; bi = oi; }
+    }
+    if (bi >= n) bi = n - 1;                       // (every score a NaN)
+#pragma unroll
+    for (int i = 0; i < kPerLane; ++i)
+      if (lane + 32 * i == bi) c[i] = -INFINITY;
+    if (lane == 0) {
+      const int a = t * p.k + r;
+      p.ids[a] = bi;
+      p.weights[a] = bs * p.scale;
+      p.pos[a] = bi < p.E ? atomicAdd(p.hist + bi, 1) : -1;
+    }
+  }
 }
 
 // ---------------------------------------------------------------------------------------------
@@ -186,6 +247,7 @@ __global__ void __launch_bounds__(kPushThreads) moe_push_kernel(const MoePushPar
   if (!p.state->overflow) {
     for (int a = blockIdx.x * (kPushThreads / 32) + warp; a < n_assign; a += gridDim.x * (kPushThreads / 32)) {
       const int e = p.ids[a];
+      if (e >= p.E) continue;      // an identity expert: no row
       const int dest = e / El;
       const int slot = p.send_base[e] + p.pos[a];
       if (slot >= p.cap) continue;
@@ -315,6 +377,14 @@ const char* moe_route(const MoeRouteParams& p, cudaStream_t stream) {
   return launch_error(cudaGetLastError());
 }
 
+const char* moe_route_scored(const MoeRouteScoredParams& p, cudaStream_t stream, bool pdl) {
+  if (p.T <= 0) return nullptr;
+  const int n = p.E + p.identity;
+  if (p.E < 1 || p.identity < 0 || n > kMoeMaxExperts) return "moe_route: expert count out of range";
+  if (p.k < 1 || p.k > n) return "moe_route: top-k out of range";
+  return launch_error(launch_kernel(moe_route_scored_kernel, dim3((p.T + kRouteWarps - 1) / kRouteWarps), dim3(kRouteWarps * 32), 0, stream, pdl, 1, p));
+}
+
 const char* moe_plan(const MoePlanParams& p, cudaStream_t stream) {
   if (p.world < 1 || p.world > kMoeMaxRanks || p.rank < 0 || p.rank >= p.world) return "moe_plan: bad rank/world";
   if (p.E < 1 || p.E > kMoeMaxExperts || p.E % p.world) return "moe_plan: experts must divide evenly over ranks";
@@ -332,7 +402,7 @@ const char* moe_push(const MoePushParams& p, cudaStream_t stream) {
 
 const char* moe_combine(const MoeCombineParams& p, cudaStream_t stream) {
   if (p.T <= 0) return nullptr;
-  if (p.H % 8) return "moe_combine: hidden size must be a multiple of 8";
+  if (p.H % 128) return "moe_combine: hidden size must be a multiple of 128 (the arrival count is per 128 columns)";
   moe_combine_kernel<<<p.T, kCombineThreads, 0, stream>>>(p);
   return launch_error(cudaGetLastError());
 }

@@ -1,12 +1,13 @@
 """Decoders described as a list of layers (`models/layered_config.py`): weight packing and the forward pass on the
 native kernels.
 
-A layer is a mixer (head-mixing attention, latent attention, matrix memory or gated linear memory) and an optional
-feed-forward on a 32-bit residual stream.  A sublayer meets the stream in one of two ways: the norm after the sum,
-``x <- rms_norm(alpha x + f(x)) * gain``, or norms around it, ``x <- x + mult * norm(f(norm(x)))``, with an optional
-causal convolution in front of every mixer.  Layers can run several times with the same weights; cache and state belong
-to layer runs.  Every size and constant is a field of the description, so a design is a mapping onto these fields
-(`models/kuzanex.py`, `models/tebivik.py`) and not a model file of its own.
+A layer is a mixer (attention with plain or head-mixed scores, latent attention, matrix memory, gated linear memory or gated
+linear recurrence) and an optional feed-forward (dense, or experts: `models/experts.py`) on a 32-bit residual stream.  A
+sublayer meets the stream in one of three ways: the norm after the sum, ``x <- rms_norm(alpha x + f(x)) * gain``, norms
+around it, ``x <- x + mult * norm(f(norm(x)))``, with an optional causal convolution in front of every mixer, or several
+streams that it reads a weighted sum of and mixes.  Layers can run several times with the same weights; cache and state
+belong to layer runs.  Every size and constant is a field of the description, so a design is a mapping onto these fields
+(`models/kuzanex.py`, `models/tebivik.py`, `models/tuzupel.py`) and not a model file of its own.
 
 The engine side is the hybrid runtime's: one ragged token batch per step (`runtime/batch.py`), K / V or latent rows in the
 paged cache (one geometry per run), recurrent state in per-sequence slots, preallocated buffers so that a decode step can
@@ -21,11 +22,13 @@ from typing import Dict, List, Tuple
 import torch
 
 from .._lib import StatusWord, load_native
+from .experts import ExpertWorkspace, pack_experts, run_experts
 from .hybrid import EPI_STORE, LaunchCounter, StepBatch
-from .layered_config import (ATTENTION_KINDS, AttentionMixer, GatedMemoryMixer, LatentAttentionMixer, LayeredConfig,
-                             MatrixMemoryMixer, pad_to)
+from .layered_config import (ATTENTION_KINDS, AttentionMixer, GatedMemoryMixer, GatedRecurrenceMixer, LatentAttentionMixer,
+                             LayeredConfig, MatrixMemoryMixer, pad_to)
 
 ACTIVATIONS = {"xielu": 3, "relu2": 4}     # csrc/gemm/gemm.h GemmActivation
+ACT_SOFTCAP = 5
 BLOCK_TOKENS = 64          # query tokens per attention block of a step (kHeadMixBlock, kLatentBlock)
 PREFILL_MIN_TOKENS = 8     # shorter portions take the token-by-token kernels
 EXPAND_BYTES = 4 << 30     # keys and values of expanded latents in flight
@@ -90,7 +93,12 @@ def _pack_attention(w, p, m: AttentionMixer, get, n_out: int, hp: int, device):
     if m.distance_bias:
         # mixing is linear: the bias taken off before it is (mix @ slope) taken off after it
         w[f"{p}/mix/slope"] = (mix @ distance_slopes(H).to(device)).float().contiguous()
-    w[f"{p}/mix/in_bias"] = bias
+    if m.bias:
+        w[f"{p}/mix/in_bias"] = bias
+    if m.head_sink:
+        w[f"{p}/mix/sink"] = get("sink").float().contiguous()
+    if m.rotary is not None:
+        w[f"{p}/mix/freq"] = torch.tensor(m.rotary.frequencies(), dtype=torch.float64, device=device)
     return rows
 
 
@@ -120,42 +128,78 @@ def _pack_gated_memory(w, p, m: GatedMemoryMixer, get, n_out: int, hp: int, devi
 def _pack_latent(w, p, m: LatentAttentionMixer, get, hp: int, dtype, device):
     H, D, R, V, Q, C = m.heads, m.dim, m.rot_dim, m.vdim, m.q_rank, m.kv_rank
     Dp, Rp, Vp, Qp, Cp = m.dim_p, m.rot_p, m.vdim_p, m.q_rank_p, m.kv_rank_p
-    uq = get("uq").reshape(H, D + R, Q)
-    q = torch.zeros((H, Dp + Rp, Qp), dtype=uq.dtype, device=device)
-    q[:, :D, :Q] = uq[:, :D]
-    q[:, Dp: Dp + R, :Q] = uq[:, D:]
-    w[f"{p}/mix/uq"] = q.reshape(H * (Dp + Rp), Qp).to(dtype)
+    direct = Q == 0                                                        # queries straight from the input
+    uq = (get("q") if direct else get("uq")).reshape(H, D + R, -1)
+    cols = uq.shape[2]
+    q = torch.zeros((H, Dp + Rp, hp if direct else Qp), dtype=uq.dtype, device=device)
+    q[:, :D, :cols] = uq[:, :D]
+    q[:, Dp: Dp + R, :cols] = uq[:, D:]
+    q = q.reshape(H * (Dp + Rp), -1)
     k, v = _pad_head_rows(get("uk"), H, D, Dp, Cp), _pad_head_rows(get("uv"), H, V, Vp, Cp)
     w[f"{p}/mix/ukv"] = torch.cat([k, v]).to(dtype)                        # rows: keys of all heads, values of all heads
     w[f"{p}/mix/uv"] = w[f"{p}/mix/ukv"][H * Dp:].view(H, Vp, Cp)
     w[f"{p}/mix/uk_t"] = k.reshape(H, Dp, Cp).transpose(1, 2).contiguous().to(dtype)   # takes a query to the latent space
-    w[f"{p}/mix/q_norm"] = _pad_head_vec(get("dq_norm"), 1, Q, Qp)
     w[f"{p}/mix/kv_norm"] = _pad_head_vec(get("dkv_norm"), 1, C, Cp)
     w[f"{p}/mix/freq"] = torch.tensor([m.rot_base ** (-2.0 * i / R) for i in range(R // 2)], dtype=torch.float64, device=device)
     if m.sink:
         w[f"{p}/mix/sink"] = get("sink").float().contiguous()
     dkv = get("dkv")
-    return [_pad2(get("dq"), Qp, hp), _pad2(dkv[:C], Cp, hp), _pad2(dkv[C:], Rp, hp)]
+    latent = [_pad2(dkv[:C], Cp, hp), _pad2(dkv[C:], Rp, hp)]
+    if direct:
+        return [q] + latent
+    w[f"{p}/mix/uq"] = q.to(dtype)
+    w[f"{p}/mix/q_norm"] = _pad_head_vec(get("dq_norm"), 1, Q, Qp)
+    return [_pad2(get("dq"), Qp, hp)] + latent
+
+
+def _pack_gated_recurrence(w, p, m: GatedRecurrenceMixer, get, hp: int, dtype, device):
+    B, n, np_ = m.blocks, m.vdim, m.vdim_p
+
+    def vec(v):
+        return _pad_head_vec(v, B, n, np_)
+    # of the gates: per block the rows of r, then of i; padded channels get zero rows and see nothing
+    gates = torch.zeros((B, 2, np_, np_), dtype=torch.float32, device=device)
+    bias = torch.zeros((B, 2, np_), dtype=torch.float32, device=device)
+    for j, r in enumerate(("ra", "ri")):
+        gates[:, j, :n, :n] = get(r).float()
+        bias[:, j, :n] = get(f"{r}_bias").float()
+    w[f"{p}/mix/gates"], w[f"{p}/mix/gate_bias"] = gates.view(B, 2 * np_, np_).to(dtype), bias.view(B, 2 * np_)
+    w[f"{p}/mix/rate"] = vec(8.0 * torch.nn.functional.softplus(get("lam").double()))
+    w[f"{p}/mix/conv"] = torch.stack([vec(v) for v in get("conv").t()])           # [taps, width]
+    w[f"{p}/mix/conv_bias"] = vec(get("conv_bias"))
+    w[f"{p}/mix/in_bias"] = torch.cat([vec(get("y_bias")), vec(get("x_bias"))])
+    return [_pad_head_rows(get("y"), B, n, np_, hp), _pad_head_rows(get("x"), B, n, np_, hp)]
 
 
 def pack_weights(cfg: LayeredConfig, get, dtype: torch.dtype = torch.bfloat16, device="cpu") -> Dict[str, torch.Tensor]:
     """Fused, padded weights of the forward pass.  `get(layer, name)` returns a design's tensor by its role (layer -1:
-    the model's own): embed, head, final_norm, loop_in, loop_step; norm1, norm1b, norm2, norm2b, conv; the mixers' (see
-    the _pack functions) and o; up, up_bias, down, down_bias, act."""
-    hp, wide = cfg.hidden_p, cfg.residual == "sandwich"
+    the model's own): embed, head, final_norm, loop_in, loop_step; norm1, norm1b, norm2, norm2b, conv; hc1_in, hc1_out,
+    hc1_mix, hc2_...; the mixers' (see the _pack functions) and o; up, up_bias, down, down_bias, act; the experts' (see
+    `pack_experts`)."""
+    hp, wide, streams = cfg.hidden_p, cfg.residual == "sandwich", cfg.residual == "streams"
     w: Dict[str, torch.Tensor] = {}
 
     def g(layer, name):
         return get(layer, name).to(device)
 
     def norm(layer, name):
-        return _pad_head_vec(g(layer, name), 1, cfg.hidden, hp) if wide else g(layer, name).float().contiguous().reshape(1)
+        if not (wide or streams):
+            return g(layer, name).float().contiguous().reshape(1)
+        return _pad_head_vec(g(layer, name).float() + cfg.norm_offset, 1, cfg.hidden, hp)
+
+    def hyper(layer, q):
+        for r in ("in", "out", "mix"):
+            w[f"text/layers/{layer}/hc{q}/{r}"] = g(layer, f"hc{q}_{r}").float().contiguous()
     if cfg.tie_head:
         w["text/embed"] = w["text/lm_head"] = _pad2(g(-1, "embed"), cfg.vocab_p, hp).to(dtype)
     else:
         w["text/embed"] = _pad2(g(-1, "embed"), cfg.vocab, hp).to(dtype)
         w["text/lm_head"] = _pad2(g(-1, "head"), cfg.vocab_p, hp).to(dtype)
     w["text/final_norm"] = norm(-1, "final_norm")
+    if streams:
+        w["text/stream_sum"] = torch.ones(cfg.streams, dtype=torch.float32, device=device)
+    if cfg.logit_softcap:
+        w["text/softcap"] = torch.tensor([cfg.logit_softcap, 1.0 / cfg.logit_softcap], dtype=torch.float32, device=device)
     if cfg.loop is not None:
         w["text/loop/in_proj"] = _pad_head_cols(g(-1, "loop_in"), 2, cfg.hidden, hp, hp).to(dtype)
         w["text/loop/step"] = torch.stack([_pad_head_vec(v, 1, cfg.hidden, hp) for v in g(-1, "loop_step")])
@@ -167,6 +211,8 @@ def pack_weights(cfg: LayeredConfig, get, dtype: torch.dtype = torch.bfloat16, d
         w[f"{p}/norm1"] = norm(i, "norm1")
         if wide:
             w[f"{p}/norm1b"] = norm(i, "norm1b")
+        if streams:
+            hyper(i, 1)
         if cfg.conv_taps:
             w[f"{p}/conv"] = torch.stack([_pad_head_vec(v, 1, cfg.hidden, hp) for v in g(i, "conv").t()])      # [taps, width]
         n_out = pad_to(m.main_cols + m.gate_cols, 2)
@@ -176,15 +222,22 @@ def pack_weights(cfg: LayeredConfig, get, dtype: torch.dtype = torch.bfloat16, d
             rows = _pack_latent(w, p, m, mix, hp, dtype, device)
         elif m.kind == "hgrn2":
             rows = _pack_gated_memory(w, p, m, mix, n_out, hp, device)
+        elif m.kind == "rglru":
+            rows = _pack_gated_recurrence(w, p, m, mix, hp, dtype, device)
         else:
             rows = _pack_matrix_memory(w, p, m, mix, n_out, hp, device)
         w[f"{p}/mix/in_proj"] = _pad2(torch.cat(rows), n_out, hp).to(dtype)
         w[f"{p}/mix/out_proj"] = _pad_head_cols(g(i, "o"), m.heads, m.vdim, m.vdim_p, hp).to(dtype)
         if spec.mlp is not None:
-            fp = pad_to(spec.mlp.ff, 8)
             w[f"{p}/norm2"] = norm(i, "norm2")
             if wide:
                 w[f"{p}/norm2b"] = norm(i, "norm2b")
+            if streams:
+                hyper(i, 2)
+        if spec.mlp is not None and spec.mlp.kind == "moe":
+            pack_experts(w, p, spec.mlp, mix, hp, dtype)
+        elif spec.mlp is not None:
+            fp = pad_to(spec.mlp.ff, 8)
             w[f"{p}/mlp/up"] = _pad2(g(i, "up"), fp, hp).to(dtype)
             w[f"{p}/mlp/down"] = _pad2(g(i, "down"), hp, fp).to(dtype)
             if spec.mlp.bias:
@@ -203,8 +256,9 @@ class LayeredWorkspace:
     """Activation buffers for up to `max_tokens` tokens; addresses are stable across steps."""
 
     def __init__(self, cfg: LayeredConfig, max_tokens: int, max_logit_rows: int, device, dtype: torch.dtype,
-                 split_rows: int = 1024):
+                 split_rows: int = 1024, ops=None):
         T, dev, f32 = max_tokens, device, torch.float32
+        moe = [l.mlp for l in cfg.layers if l.mlp is not None and l.mlp.kind == "moe"]
         mixers = [l.mixer for l in cfg.layers]
         attn = [m for m in mixers if m.kind == "attention"]
         latent = [m for m in mixers if m.kind == "latent_attention"]
@@ -215,7 +269,11 @@ class LayeredWorkspace:
         def widest(values, default, mult=64):
             return pad_to(max(values, default=default), mult)
         self.max_tokens, self.max_logit_rows = T, max_logit_rows
-        self.x = rows(cfg.hidden_p, f32)           # residual stream
+        if cfg.residual == "streams":
+            self.streams = torch.zeros((T, cfg.streams, cfg.hidden_p), dtype=f32, device=dev)
+            self.x = self.streams[:, 0]
+        else:
+            self.x = rows(cfg.hidden_p, f32)       # residual stream
         self.x2 = rows(cfg.hidden_p, f32) if cfg.conv_taps else self.x     # its other copy: a convolution reads rows that its step replaces
         self.xa = rows(cfg.hidden_p)               # what the next GEMM reads, in the activation type
         self.pair = rows(2 * cfg.hidden_p) if cfg.loop is not None else None   # [x, embedding output] of a pass's entry
@@ -224,9 +282,14 @@ class LayeredWorkspace:
         self.gates = rows(widest((m.gate_cols for m in mixers), 2, 4), f32)
         self.mix = rows(widest((m.out_cols for m in mixers), 64))
         self.q = rows(max([m.heads * m.dim_p for m in attn] + [m.q_cols for m in latent], default=16))
-        self.act = rows(widest((l.mlp.ff for l in cfg.layers if l.mlp is not None), 8))
+        self.act = rows(widest((l.mlp.ff for l in cfg.layers if l.mlp is not None and l.mlp.kind == "dense"), 8))
+        if moe:
+            self.experts = ExpertWorkspace(moe, cfg.hidden_p, T, dev, dtype, ops or load_native())
+        rec = max((m.out_cols for m in mixers if m.kind == "rglru"), default=0)
+        if rec:
+            self.rec_u = torch.zeros(T * rec, dtype=dtype, device=dev)
         if latent:
-            self.q_latent = rows(max(m.q_rank_p for m in latent))
+            self.q_latent = rows(max(16, max(m.q_rank_p for m in latent)))
             self.q_abs = rows(max(m.heads * m.kv_rank_p for m in latent))     # absorbed queries, head by head
             self.o_latent = rows(max(m.heads * m.kv_rank_p for m in latent))  # attended latents
         # split-KV partials: (query token x split) rows of decode-sized steps
@@ -240,12 +303,15 @@ class LayeredWorkspace:
 
 
 def native_subset(cfg: LayeredConfig) -> str:
-    """The stand-alone library (see `_build.SUBSETS`) that has the mixers of this configuration."""
-    kinds = {l.mixer.kind for l in cfg.layers}
-    for name, have in (("head_mix", {"attention", "mlstm"}), ("latent", {"latent_attention", "hgrn2"})):
-        if kinds <= have:
-            return name
-    return "layered"
+    """The parts of the stand-alone library (see `_build.PARTS`) that this configuration needs."""
+    parts = {{"latent_attention": "latent", "hgrn2": "gated"}.get(l.mixer.kind, l.mixer.kind) for l in cfg.layers}
+    if any(l.mixer.kind == "attention" and not l.mixer.plain_scores for l in cfg.layers):
+        parts.add("head_mix")
+    if any(l.mlp is not None and l.mlp.kind == "moe" for l in cfg.layers):
+        parts |= {"moe", "streams"}                # (the sum over the experts belongs to the row steps)
+    if cfg.residual == "streams":
+        parts.add("streams")
+    return "+".join(sorted(parts))
 
 
 class LayeredModel:
@@ -283,16 +349,17 @@ class LayeredModel:
         return cur
 
     # ------------------------------------------------------------------ GEMM
-    def _gemm(self, x, w, bias, out=None, out32=None, out32_from=0, act=0, act_params=None, prefetch=None):
+    def _gemm(self, x, w, bias, out=None, out32=None, out32_from=0, act=0, act_params=None, prefetch=None, epi=EPI_STORE, glu=()):
         if self.f32:
+            assert epi == EPI_STORE
             self.ops.gemm_f32(x, w, out, bias, act, act_params, out32, out32_from)
             return
         T, (N, K) = x.shape[0], w.shape
-        splits = int(self.ops.gemm_pick_splits(T, N, K, EPI_STORE))
+        splits = int(self.ops.gemm_pick_splits(T, N, K, epi))
         if not (self.l2_prefetch and T <= 64):
             prefetch = None
-        self.ops.gemm_bf16(x, w, out, EPI_STORE, None, bias, None, splits, self.status.tensor, self.pdl, act, None, None, None,
-                           None, prefetch, out32, out32_from, act_params)
+        self.ops.gemm_bf16(x, w, out, epi, None, bias, None, splits, self.status.tensor, self.pdl, act, None, None, None,
+                           None, prefetch, out32, out32_from, act_params, glu)
 
     def _in_proj(self, ws, T, p, m):
         """Fused input projection: [T, main_cols] in the activation type and [T, gate_cols] in fp32."""
@@ -311,27 +378,33 @@ class LayeredModel:
         H, G, Dp, Vp = m.heads, m.kv_heads, m.dim_p, m.vdim_p
         q = ws.q[:T, : H * Dp]
         ops.qkv_append(proj, 0, H * Dp, (H + G) * Dp, H, G, m.dim, w.get(f"{p}/mix/q_norm"), w.get(f"{p}/mix/k_norm"),
-                       self.cfg.rms_eps, b.table_row, b.cache_pos, kv.table, q, k_pages, v_pages, kv.page_size, self.pdl)
-        out = ws.mix[:T, : H * Vp]
+                       self.cfg.rms_eps, b.table_row, b.cache_pos, kv.table, q, k_pages, v_pages, kv.page_size, self.pdl,
+                       w.get(f"{p}/mix/freq"))
+        out, sinks = ws.mix[:T, : H * Vp], w.get(f"{p}/mix/sink")
         shape = (m.window, m.scale, m.softcap, m.sink, w.get(f"{p}/mix/heads"), w.get(f"{p}/mix/slope"),
                  gates if m.head_gate else None, out)
-        if not self.f32 and self.prefill_kernels and b.max_seq_tokens >= PREFILL_MIN_TOKENS:
+        portions = not self.f32 and self.prefill_kernels and b.max_seq_tokens >= PREFILL_MIN_TOKENS
+        if portions and m.plain_scores and self._raw_ops.group_prefill_supported(Dp, Vp):
+            ops.group_prefill(q, k_pages, v_pages, kv.table, b.table_row, b.kv_len, m.window, m.chunk, m.scale, m.sink, sinks, out,
+                              b.qblk_start, b.qblk_count, self.pdl)
+            return out
+        if portions and not m.plain_scores:
             one = int(ops.head_mix_prefill_scratch(H, b.max_kv_len, m.window, 1))
             nb = b.qblk_start.numel()
             scratch = self._grown("scores", max(one, min(one * nb, SCORE_SCRATCH_BYTES)))
             ops.head_mix_prefill(q, k_pages, v_pages, kv.table, b.table_row, b.kv_len, *shape, b.qblk_start, b.qblk_count,
                                  b.max_kv_len, scratch, self.pdl)
             return out
-        split, n = self.pick_split(ws, T, b.max_kv_len, m.window)
+        split, n = self.pick_split(ws, T, b.max_kv_len, m.look_back, ctas=G if m.plain_scores and not self.f32 else 1)
         ops.head_mix_attention(q, k_pages, v_pages, kv.table, b.table_row, b.kv_len, *shape, split, n,
-                               ws.part_o if n > 1 else None, ws.part_ml if n > 1 else None, self.pdl)
+                               ws.part_o if n > 1 else None, ws.part_ml if n > 1 else None, self.pdl, m.chunk, sinks)
         return out
 
     @staticmethod
-    def pick_split(ws, T: int, max_kv_len: int, window: int, sm_count: int = 148) -> Tuple[int, int]:
-        """Keys per split (a multiple of 32) and splits per token: two CTAs per SM when the step is small."""
+    def pick_split(ws, T: int, max_kv_len: int, window: int, sm_count: int = 148, ctas: int = 1) -> Tuple[int, int]:
+        """Keys per split (a multiple of 32) and splits per token, each of `ctas` CTAs: two CTAs per SM when the step is small."""
         keys = min(max_kv_len, window) if window > 0 else max_kv_len
-        want = max(1, min(2 * sm_count // T, ws.split_rows // T, 64))
+        want = max(1, min(2 * sm_count // (T * ctas), ws.split_rows // T, 64))
         split = max(64, pad_to(-(-keys // want), 32))
         return split, -(-keys // split)
 
@@ -341,8 +414,9 @@ class LayeredModel:
         rows = min(b.max_seq_tokens, BLOCK_TOKENS) * m.heads
         ctas = b.qblk_start.numel() * max(1, -(-rows // 64))
         want = max(1, min(sm_count // ctas, ws.split_rows // b.n_tokens, 64))
-        split = max(128, pad_to(-(-b.max_kv_len // want), 32))
-        return split, -(-b.max_kv_len // split)
+        keys = min(b.max_kv_len, m.window + min(b.max_seq_tokens, BLOCK_TOKENS) - 1) if m.window else b.max_kv_len
+        split = max(128, pad_to(-(-keys // want), 32))
+        return split, -(-keys // split)
 
     def _head_gemm(self, x: torch.Tensor, x_step: int, w: torch.Tensor, out: torch.Tensor, b: StepBatch, max_tokens: int) -> None:
         """out[t, h * N + n] = sum_k w[h, n, k] x[t, h * x_step + k]; tokens of sequences with `max_tokens` or more may be left out"""
@@ -361,25 +435,28 @@ class LayeredModel:
         return max(16, -(-m.kv_rank_p * heads // (wide - heads))) if wide > heads else 0
 
     def _expand_plan(self, b: StepBatch, m: LatentAttentionMixer):
-        """Which sequences of the step take the expanded form: (threshold, [n, 3] of block-table row / first gathered row /
-        positions, first row per sequence or -1, total rows, longest, whether the others are left) or None."""
+        """Which sequences of the step take the expanded form: (threshold, [n, 4] of block-table row / first gathered row /
+        first position / positions, first row (or -1) and its position per sequence, total rows, longest, whether the others
+        are left) or None."""
         least = self.expand_tokens(m)
         if (self.f32 or not self.prefill_kernels or b.seq_host is None or not least or b.max_seq_tokens < least
                 or not self._raw_ops.latent_expanded_supported(m.dim_p, m.rot_p, m.vdim_p)):
             return None
-        key = (least, m.heads * (m.dim_p + m.vdim_p))
+        key = (least, m.heads * (m.dim_p + m.vdim_p), m.window)
         if key not in b.plans:
             seqs, base, total = [], [], 0
             for row, n, end in b.seq_host:
-                base.append(total if n >= least else -1)
+                first = max(0, end - n + 1 - m.window) if m.window else 0       # what the portion's first token sees
+                base += [total, first] if n >= least else [-1, 0]
                 if n >= least:
-                    seqs.append((row, total, end))
-                    total += end
+                    seqs.append((row, total, first, end - first))
+                    total += end - first
             plan = None
             if total * key[1] * 2 <= EXPAND_BYTES:
                 host = torch.tensor(base + [v for s in seqs for v in s], dtype=torch.int32)
                 dev = (host.pin_memory() if self.device.type == "cuda" else host).to(self.device, non_blocking=True)
-                plan = (least, dev[len(base):].view(-1, 3), dev[: len(base)], total, max(s[2] for s in seqs), len(seqs) < len(base))
+                plan = (least, dev[len(base):].view(-1, 4), dev[: len(base)].view(-1, 2), total, max(s[3] for s in seqs),
+                        2 * len(seqs) < len(base))
             b.plans[key] = plan
         return b.plans[key]
 
@@ -387,11 +464,13 @@ class LayeredModel:
         ops, w, eps = self.ops, self.w, self.cfg.rms_eps
         proj, _ = self._in_proj(ws, T, p, m)
         pages, _ = kv.layers[self._attn_idx[run]].typed(self.dtype)
-        c_q, q = ws.q_latent[:T, : m.q_rank_p], ws.q[:T, : m.q_cols]
+        c_q = ws.q_latent[:T, : m.q_rank_p] if m.q_rank else None
+        q = ws.q[:T, : m.q_cols] if m.q_rank else proj[:, : m.q_cols]
         freq, sink = w[f"{p}/mix/freq"], w.get(f"{p}/mix/sink")
-        ops.latent_prep(proj, m.q_rank, m.kv_rank, m.rot_dim, w[f"{p}/mix/q_norm"], w[f"{p}/mix/kv_norm"], eps, freq, b.table_row,
+        ops.latent_prep(proj, m.q_rank, m.kv_rank, m.rot_dim, w.get(f"{p}/mix/q_norm"), w[f"{p}/mix/kv_norm"], eps, freq, b.table_row,
                         b.cache_pos, kv.table, c_q, pages, self.pdl)
-        self._gemm(c_q, w[f"{p}/mix/uq"], None, q, prefetch=w[f"{p}/mix/uk_t"])
+        if m.q_rank:
+            self._gemm(c_q, w[f"{p}/mix/uq"], None, q, prefetch=w[f"{p}/mix/uk_t"])
         out = ws.mix[:T, : m.out_cols]
         plan, blocks = self._expand_plan(b, m), (b.qblk_start, b.qblk_count, min(b.max_seq_tokens, BLOCK_TOKENS))
         if plan is None or plan[-1]:
@@ -400,11 +479,11 @@ class LayeredModel:
             self._head_gemm(q, m.dim_p + m.rot_p, w[f"{p}/mix/uk_t"], q_abs, b, skip)
             args = (q_abs, q, pages, kv.table, b.table_row, b.kv_len, m.heads, m.rot_dim, m.scale, freq, sink, o_latent)
             if self.f32 or not self._raw_ops.latent_absorbed_supported(m.kv_rank_p, m.rot_p):
-                ops.latent_token_attention(*args, self.pdl)
+                ops.latent_token_attention(*args, self.pdl, m.window)
             else:
                 split, n = self.pick_latent_split(ws, b, m)
                 ops.latent_absorbed_attention(*args, *blocks, b.token_seq, b.cu_seqlens, skip, split, n,
-                                              ws.part_o if n > 1 else None, ws.part_ml if n > 1 else None, self.pdl)
+                                              ws.part_o if n > 1 else None, ws.part_ml if n > 1 else None, self.pdl, m.window)
             self._head_gemm(o_latent, m.kv_rank_p, w[f"{p}/mix/uv"], out, b, skip)
         if plan is not None:
             _, seqs, base, total, longest, _ = plan
@@ -414,7 +493,7 @@ class LayeredModel:
             ops.latent_gather(pages, kv.table, seqs, longest, rows, self.pdl)
             self._gemm(rows[:, : m.kv_rank_p], ukv, None, wide)
             ops.latent_expanded_attention(q, rows, wide, b.kv_len, m.heads, m.kv_rank_p, m.rot_dim, m.scale, freq, sink, out, *blocks,
-                                          b.token_seq, base, self.pdl)
+                                          b.token_seq, base, self.pdl, m.window)
         return out
 
     def _chunk_workspace(self, b: StepBatch, T: int, kind: str, m) -> "torch.Tensor | None":
@@ -447,14 +526,34 @@ class LayeredModel:
                               b.one_token_per_seq)
         return out
 
+    def _gated_recurrence(self, ws, b: StepBatch, states, run: int, T: int, p: str, m: GatedRecurrenceMixer, write_state: bool):
+        ops, w = self.ops, self.w
+        proj, _ = self._in_proj(ws, T, p, m)
+        ring, S = states.layers[self._state_idx[run]][-2:]
+        C, n, out = m.out_cols, m.vdim_p, ws.mix[:T, : m.out_cols]
+        gates, gate_bias, rate = w[f"{p}/mix/gates"], w[f"{p}/mix/gate_bias"], w[f"{p}/mix/rate"]
+        step = (m.blocks, w[f"{p}/mix/conv"], w[f"{p}/mix/conv_bias"], b.cu_seqlens, b.token_seq, b.cache_pos, b.state_slot, ring)
+        u = ws.rec_u[: T * C].view(T, C)
+        raw = self._grown("gates", 8 * T * C)[: 8 * T * C].view(torch.float32).view(T, 2 * C)
+        ops.rglru_conv(proj, *step, u, self.pdl)
+        for k in range(m.blocks):
+            self._gemm(u[:, k * n: (k + 1) * n], gates[k], gate_bias[k], out32=raw[:, 2 * k * n: 2 * (k + 1) * n])
+        ops.rglru_scan(proj, *step, u, raw, rate, S, out, write_state, self.pdl)
+        return out
+
     def _mixer(self, ws, b: StepBatch, kv, states, run: int, T: int, p: str, m, write_state: bool) -> torch.Tensor:
         if m.kind in ATTENTION_KINDS:
             fn = self._attention if m.kind == "attention" else self._latent_attention
             return fn(ws, b, kv, run, T, p, m)
-        fn = self._gated_memory if m.kind == "hgrn2" else self._matrix_memory
+        fn = {"hgrn2": self._gated_memory, "mlstm": self._matrix_memory, "rglru": self._gated_recurrence}[m.kind]
         return fn(ws, b, states, run, T, p, m, write_state)
 
     def _feed_forward(self, ws, T: int, p: str, spec, prefetch) -> None:
+        """ws.delta <- the feed-forward of ws.xa"""
+        if spec.kind == "moe":
+            y = run_experts(self, ws.experts, T, p, spec, ws.xa[:T], ws.delta[:T], prefetch)
+            self.ops.mixture_rows(*y.values(), ws.delta[:T], self.pdl)
+            return
         w, up, down = self.w, self.w[f"{p}/mlp/up"], self.w[f"{p}/mlp/down"]
         act = ws.act[:T, : up.shape[0]]
         self._gemm(ws.xa[:T], up, w.get(f"{p}/mlp/up_bias"), act, act=ACTIVATIONS[spec.activation], act_params=w.get(f"{p}/mlp/act"),
@@ -466,7 +565,7 @@ class LayeredModel:
         """Runs all layers; returns the final-normed hidden states [T, hidden (padded)]."""
         if b.n_tokens > ws.max_tokens:
             raise ValueError(f"step of {b.n_tokens} tokens exceeds the workspace ({ws.max_tokens})")
-        run = self._forward_sandwich if self.cfg.residual == "sandwich" else self._forward_post_sum
+        run = {"sandwich": self._forward_sandwich, "streams": self._forward_streams, "post_sum": self._forward_post_sum}[self.cfg.residual]
         return run(ws, b, kv, states, write_state)
 
     def _next_weights(self, run: int):
@@ -533,10 +632,49 @@ class LayeredModel:
         rows(w["text/final_norm"], xa)
         return xa
 
+    def _forward_streams(self, ws, b: StepBatch, kv, states, write_state: bool) -> torch.Tensor:
+        """The update of the streams by a sublayer waits for the row step in front of the next one (`stream_rows`); until the
+        first update every stream is the embedding row itself."""
+        cfg, ops, w, T = self.cfg, self.ops, self.w, b.n_tokens
+        xa, delta, X = ws.xa[:T], ws.delta[:T], ws.streams[:T]
+        source, y, update = None, None, (None, None)     # streams, output of the sublayer that waits and its (mix, out)
+
+        def rows(w_in, w_next):
+            nonlocal source, y, update
+            parts = (None, None, None, None, None, None, 0) if y is None else tuple(y.values())
+            ops.stream_rows(source, b.ids, w["text/embed"], None if y is None else X, *parts, *update, w_in, w_next, xa, cfg.hidden,
+                            cfg.rms_eps, self.pdl)
+            if y is not None:
+                source, y, update = X, None, (None, None)
+        for run, (layer, _) in enumerate(self._runs):
+            spec, p = cfg.layers[layer], f"text/layers/{layer}"
+            rows(w[f"{p}/hc1/in"], w[f"{p}/norm1"])
+            mix, nxt = self._mixer(ws, b, kv, states, run, T, p, spec.mixer, write_state), self._next_weights(run)
+            self._gemm(mix, w[f"{p}/mix/out_proj"], None, out32=delta, prefetch=w.get(f"{p}/mlp/router", w.get(f"{p}/mlp/up", nxt)))
+            y, update = self._plain_sum(delta), (w[f"{p}/hc1/mix"], w[f"{p}/hc1/out"])
+            if spec.mlp is not None:
+                rows(w[f"{p}/hc2/in"], w[f"{p}/norm2"])
+                if spec.mlp.kind == "moe":
+                    y = run_experts(self, ws.experts, T, p, spec.mlp, xa, delta, nxt)
+                else:
+                    self._feed_forward(ws, T, p, spec.mlp, nxt)
+                    y = self._plain_sum(delta)
+                update = (w[f"{p}/hc2/mix"], w[f"{p}/hc2/out"])
+            if self.layer_hook is not None:
+                rows(w["text/stream_sum"], w["text/final_norm"])
+                self.layer_hook(run, X.sum(dim=1)[:, : cfg.hidden])
+        rows(w["text/stream_sum"], w["text/final_norm"])
+        return xa
+
+    @staticmethod
+    def _plain_sum(delta) -> dict:
+        return dict(delta=delta, gate=None, choice=None, weight=None, ret=None, h=None, n_experts=0)
+
     def head(self, ws: LayeredWorkspace, head_in: torch.Tensor) -> torch.Tensor:
         """fp32 logits [rows, vocab] of final-normed hidden states (at most `max_logit_rows`)."""
         out = ws.logits[: head_in.shape[0]]
-        self._gemm(head_in, self.w["text/lm_head"], None, out32=out)
+        act = ACT_SOFTCAP if self.cfg.logit_softcap else 0
+        self._gemm(head_in, self.w["text/lm_head"], None, out32=out, act=act, act_params=self.w.get("text/softcap"))
         return out[:, : self.cfg.vocab]
 
     def logits(self, ws: LayeredWorkspace, b: StepBatch, hidden: torch.Tensor) -> torch.Tensor:

@@ -1,8 +1,9 @@
 """Description of decoders given as a list of layers (read by `models/layered.py`, which runs them).
 
-A layer is a mixer (head-mixing attention, latent attention, matrix memory or gated linear memory) and an optional
-feed-forward; every size and constant is a field, and so is which mechanisms a mixer has.  The model's own fields say how
-a sublayer meets the residual stream, what precedes a mixer, and which layers run several times.  Cache and state belong
+A layer is a mixer (attention with shaped or plain scores, latent attention, matrix memory, gated linear memory or gated
+linear recurrence) and an optional feed-forward (dense or a mixture of experts); every size and constant is a field, and so
+is which mechanisms a mixer has.  The model's own fields say how a sublayer meets the residual stream (or streams), what
+precedes a mixer, and which layers run several times.  Cache and state belong
 to layer RUNS: a layer that runs twice has two of each.  No torch here: the package table and the host diagnostics read
 these descriptions too."""
 from __future__ import annotations
@@ -14,6 +15,38 @@ from typing import List, Optional, Tuple, Union
 
 def pad_to(n: int, m: int) -> int:
     return (n + m - 1) // m * m
+
+
+@dataclass(frozen=True)
+class RotaryScaling:
+    """Frequencies whose wavelength is beyond `original` / `low` positions are divided by `factor`, those within `original` /
+    `high` stay, and in between the two are mixed linearly in `original` / wavelength."""
+    factor: float
+    low: float
+    high: float
+    original: float
+
+
+@dataclass(frozen=True)
+class Rotary:
+    """The first `dims` values of a head, neighbours (2i, 2i + 1), turned by position * frequency i."""
+    base: float
+    dims: int
+    scaling: Optional[RotaryScaling] = None
+
+    def frequencies(self) -> List[float]:
+        out = []
+        for i in range(self.dims // 2):
+            f, s = self.base ** (-2.0 * i / self.dims), self.scaling
+            if s is not None:
+                turns = s.original * f / (2.0 * math.pi)          # original / wavelength
+                if turns < s.low:
+                    f /= s.factor
+                elif turns <= s.high:
+                    keep = (turns - s.low) / (s.high - s.low)
+                    f = (1.0 - keep) * f / s.factor + keep * f
+            out.append(f)
+        return out
 
 
 @dataclass(frozen=True)
@@ -31,8 +64,21 @@ class AttentionMixer:
     head_mixing: bool = False     # scores are mixed across heads by a [heads, heads] matrix before the softmax
     sink: float = 0.0             # added to the softmax denominator
     head_gate: bool = False       # sigmoid gate per head on the output
+    chunk: int = 0                # keys of the query's own chunk of this many positions only (counted from 0); 0: no chunks
+    head_sink: bool = False       # one learned score per head in the softmax denominator
+    rotary: Optional[Rotary] = None   # after the norm, on q and k
 
     kind = "attention"
+
+    @property
+    def plain_scores(self) -> bool:
+        """Scaled dot products and nothing else: no cap, bias, mix or gate."""
+        return not (self.softcap or self.distance_bias or self.head_mixing or self.head_gate)
+
+    @property
+    def look_back(self) -> int:
+        """Keys that a query can still look at, itself included; 0: all of the past."""
+        return min(n for n in (self.window, self.chunk) if n) if self.window or self.chunk else 0
 
     @property
     def dim_p(self) -> int:
@@ -91,8 +137,9 @@ class MatrixMemoryMixer:
 
 @dataclass(frozen=True)
 class LatentAttentionMixer:
-    """Queries through a normed latent; keys and values out of one normed latent row per token, plus one rotated key part
-    that all heads share.  The cache keeps one row per token: [latent, rotated part]."""
+    """Queries through a normed latent, or straight from the input (q_rank 0); keys and values out of one normed latent row
+    per token, plus one rotated key part that all heads share (rot_dim 0: none).  The cache keeps one row per token:
+    [latent, rotated part]."""
     heads: int
     dim: int                      # query / key width per head without rotation
     rot_dim: int                  # rotated query / key width per head
@@ -102,10 +149,14 @@ class LatentAttentionMixer:
     scale: float
     rot_base: float
     sink: bool = True             # one learned score per head in the softmax denominator
+    window: int = 0               # keys a query sees, itself included; 0: all of the past
 
     kind = "latent_attention"
     kv_heads = 1
-    window = 0
+
+    @property
+    def look_back(self) -> int:
+        return self.window
 
     @property
     def dim_p(self) -> int:
@@ -134,8 +185,8 @@ class LatentAttentionMixer:
 
     @property
     def main_cols(self) -> int:
-        """Columns of the fused input projection: [query latent, key / value latent, rotated key part]."""
-        return self.q_rank_p + self.row_cols
+        """Columns of the fused input projection: [query latent or queries, key / value latent, rotated key part]."""
+        return (self.q_rank_p if self.q_rank else self.q_cols) + self.row_cols
 
     gate_cols = 0
 
@@ -183,16 +234,97 @@ class GatedMemoryMixer:
 
 
 @dataclass(frozen=True)
+class GatedRecurrenceMixer:
+    """Griffin's recurrent block: a causal convolution in front of a diagonal linear recurrence whose decay and input gates
+    are block-diagonal maps of its input, times a GELU branch."""
+    width: int
+    blocks: int                   # equal parts of the width, each with gate matrices of its own
+    taps: int                     # of the convolution
+
+    kind = "rglru"
+
+    @property
+    def vdim(self) -> int:
+        return self.width // self.blocks
+
+    @property
+    def vdim_p(self) -> int:
+        return pad_to(self.vdim, 16)
+
+    @property
+    def heads(self) -> int:
+        return self.blocks
+
+    @property
+    def main_cols(self) -> int:
+        """[GELU branch, recurrent branch]"""
+        return 2 * self.out_cols
+
+    gate_cols = 0
+
+    @property
+    def out_cols(self) -> int:
+        return self.blocks * self.vdim_p
+
+
+@dataclass(frozen=True)
 class DenseMlp:
     ff: int
     activation: str = "xielu"     # xielu (two learned numbers per layer) | relu2 (square of relu)
     bias: bool = False
 
+    kind = "dense"
+
+
+@dataclass(frozen=True)
+class GatedUnit:
+    """down( g sigmoid(slope g) (u + shift) ) with g = min(gate h, limit), u = clamp(up h, +- limit); limit 0: no bounds."""
+    ff: int
+    limit: float = 0.0
+    slope: float = 1.0
+    shift: float = 0.0
+
+    @property
+    def ff_p(self) -> int:
+        return pad_to(self.ff, 64)
+
+    def params(self, h: int) -> int:
+        return 3 * h * self.ff
+
+
+@dataclass(frozen=True)
+class ExpertMlp:
+    """Mixture of experts: softmax over all router outputs, the `top` largest scores (with a learned correction added for the
+    choice only) times `scale` weigh the chosen experts.  The last `identity` outputs stand for the input itself.  A
+    shared expert runs for every token under a sigmoid gate."""
+    experts: int
+    top: int
+    expert: GatedUnit
+    identity: int = 0
+    scale: float = 1.0
+    shared: Optional[GatedUnit] = None
+
+    kind = "moe"
+
+    @property
+    def choices(self) -> int:
+        return self.experts + self.identity
+
+    @property
+    def router_cols(self) -> int:
+        """Router outputs and the shared expert's gate."""
+        return pad_to(self.choices + (1 if self.shared else 0), 8)
+
+    @property
+    def slots(self) -> int:
+        """Most experts with weights of their own that one token uses."""
+        return min(self.top, self.experts)
+
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: Union[AttentionMixer, LatentAttentionMixer, MatrixMemoryMixer, GatedMemoryMixer]
-    mlp: Optional[DenseMlp] = None
+    mixer: Union[AttentionMixer, LatentAttentionMixer, MatrixMemoryMixer, GatedMemoryMixer, GatedRecurrenceMixer]
+    mlp: Optional[Union[DenseMlp, ExpertMlp]] = None
 
 
 @dataclass(frozen=True)
@@ -217,13 +349,18 @@ class LayeredConfig:
     residual_alpha: float         # post_sum: x <- norm(residual_alpha * x + f(x))
     max_context: int = 131072
     architecture: str = ""        # name of the design that maps checkpoints onto this description
-    residual: str = "post_sum"    # post_sum | sandwich: x <- x + residual_mult * norm(f(norm(x)))
+    # post_sum | sandwich: x <- x + residual_mult * norm(f(norm(x))) | streams: `streams` copies of the embedding output; a
+    # sublayer reads a weighted sum of them, u = sum_s in[s] x_s, and x_t <- sum_s mix[s, t] x_s + out[t] f(norm(u))
+    residual: str = "post_sum"
     residual_mult: float = 1.0    # sandwich
     norm_groups: int = 1          # sandwich: equal parts of a row that are normed by themselves, one weight per column
     conv_taps: int = 0            # h <- h + causal convolution of h before every mixer, this many taps (0: none)
     embed_scale: float = 1.0
     tie_head: bool = False        # logits from the embedding table (without its scale)
     loop: Optional[LoopSpec] = None
+    streams: int = 1
+    norm_offset: float = 0.0      # added to the stored weights of the sublayers' and the final norm
+    logit_softcap: float = 0.0    # logits <- cap tanh(logits / cap); 0: as they are
 
     moe = None
     mtp_layers = 0
@@ -282,18 +419,21 @@ class LayeredConfig:
     @property
     def cache_window(self) -> int:
         """Keys that any layer still looks back on: the widest window, 0 when some layer sees all of the past."""
-        w = [self.mixer_of(r).window for r in self.attn_layers]
+        w = [self.mixer_of(r).look_back for r in self.attn_layers]
         return max(w) if w and min(w) > 0 else 0
 
     def state_shapes(self) -> List[List[tuple]]:
         """Per run in `state_layers`: shapes (without the slot) of its fp32 state arrays: the convolution's last inputs
-        (oldest first) when there are any, then the memory: S, n, m (matrix memory) or S (gated memory)."""
+        (oldest first) when there are any, then the memory: S, n, m (matrix memory), S (gated memory), or the inputs of
+        the last `taps` positions (row position mod taps) and S (gated recurrence)."""
         out = []
         for r in self.state_layers:
             m, arrays = self.mixer_of(r), []
             if self.conv_taps > 1:
                 arrays.append((self.conv_taps - 1, self.hidden_p))
-            if m.kind not in ATTENTION_KINDS:
+            if m.kind == "rglru":
+                arrays += [(m.taps, m.out_cols), (m.out_cols,)]
+            elif m.kind not in ATTENTION_KINDS:
                 arrays.append((m.heads, m.dim_p, m.vdim_p))
             if m.kind == "mlstm":
                 arrays += [(m.heads, m.dim_p), (m.heads,)]
@@ -305,25 +445,34 @@ class LayeredConfig:
 
     def param_count(self) -> int:
         h, wide = self.hidden, self.residual == "sandwich"
-        norm = h if wide else 1                      # weights of one norm
+        norm = 1 if self.residual == "post_sum" else h                      # weights of one norm
+        hyper = self.streams * (self.streams + 2) if self.residual == "streams" else 0
         n = (1 if self.tie_head else 2) * self.vocab * h + norm
         if self.loop is not None:
             n += 2 * h * h + self.loop.times * h
         for l in self.layers:
             m = l.mixer
-            n += (2 if wide else 1) * norm + self.conv_taps * h + h * m.heads * m.vdim
+            n += (2 if wide else 1) * norm + hyper + self.conv_taps * h + h * m.heads * m.vdim
             if m.kind == "attention":
                 rows = (m.heads + m.kv_heads) * m.dim + m.kv_heads * m.vdim + (m.heads if m.head_gate else 0)
                 n += rows * h + (m.heads * m.heads if m.head_mixing else 0) + (2 * m.dim if m.qk_norm else 0)
+                n += m.heads if m.head_sink else 0
             elif m.kind == "latent_attention":
                 n += (m.q_rank + m.kv_rank + m.rot_dim) * h + m.q_rank + m.kv_rank + (m.heads if m.sink else 0)
-                n += m.heads * (m.dim + m.rot_dim) * m.q_rank + m.heads * (m.dim + m.vdim) * m.kv_rank
+                n += m.heads * (m.dim + m.rot_dim) * (m.q_rank or h) + m.heads * (m.dim + m.vdim) * m.kv_rank
+            elif m.kind == "rglru":
+                n += 2 * m.width * (h + 1) + m.width * (m.taps + 1) + 2 * m.width * (m.vdim + 1) + m.width
             elif m.kind == "hgrn2":
                 n += (2 * m.heads * m.dim + m.heads * m.vdim) * h + 2 * m.heads * m.dim + m.vdim
             else:
                 n += (2 * m.heads * (m.dim + m.vdim) + 2 * m.heads) * h + m.heads * m.vdim + 2 * m.heads
             if l.mlp is not None:
-                n += 2 * h * l.mlp.ff + (2 * norm if wide else norm)
+                n += (2 * norm if wide else norm) + hyper
+            if l.mlp is not None and l.mlp.kind == "moe":
+                n += l.mlp.choices * (h + 1) + l.mlp.experts * l.mlp.expert.params(h)
+                n += l.mlp.shared.params(h) + h if l.mlp.shared else 0
+            elif l.mlp is not None:
+                n += 2 * h * l.mlp.ff
                 n += 2 if l.mlp.activation == "xielu" else (l.mlp.ff + h if l.mlp.bias else 0)
         return n
 

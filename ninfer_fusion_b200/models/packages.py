@@ -18,8 +18,8 @@ from .architectures import LAYERED_REGISTRY
 from .config import REGISTRY, ModelConfig
 from .layered_config import LayeredConfig
 
-FULL, SLIDING, GDN, MLSTM, GATED, LATENT = "full", "sliding", "gdn", "mlstm", "hgrn2", "latent"
-KINDS = (FULL, SLIDING, GDN, MLSTM, GATED, LATENT)
+FULL, SLIDING, GDN, MLSTM, GATED, LATENT, CHUNKED, RGLRU = "full", "sliding", "gdn", "mlstm", "hgrn2", "latent", "chunked", "rglru"
+KINDS = (FULL, SLIDING, GDN, MLSTM, GATED, LATENT, CHUNKED, RGLRU)
 
 # what the engine's forward pass, kernels and cache can do today
 ENGINE_CAPABILITIES: FrozenSet[str] = frozenset({
@@ -34,6 +34,8 @@ ENGINE_CAPABILITIES: FrozenSet[str] = frozenset({
     # layer-list decoders (models/layered.py)
     "layer-list-schedule", "head-mixing-attention", "attention-sink", "matrix-memory", "post-sum-norm", "xielu-mlp",
     "latent-attention", "gated-memory", "sandwich-norms", "grouped-norm", "input-convolution", "layer-loop", "relu2-mlp",
+    "residual-streams", "offset-norm", "chunked-attention", "learned-sink", "interleaved-rope", "scaled-rope", "gated-recurrence",
+    "expert-mlp", "identity-experts", "output-softcap",
 })
 
 
@@ -89,26 +91,37 @@ def _hybrid(cfg: ModelConfig) -> Package:
 
 def _layered(cfg: LayeredConfig) -> Package:
     kinds = []
-    needs = {"layer-list-schedule", "sandwich-norms" if cfg.residual == "sandwich" else "post-sum-norm"}
-    needs |= {c for c, on in (("grouped-norm", cfg.norm_groups > 1), ("input-convolution", cfg.conv_taps), ("layer-loop", cfg.loop)) if on}
+    needs = {"layer-list-schedule", {"sandwich": "sandwich-norms", "streams": "residual-streams"}.get(cfg.residual, "post-sum-norm")}
+    needs |= {c for c, on in (("grouped-norm", cfg.norm_groups > 1), ("input-convolution", cfg.conv_taps), ("layer-loop", cfg.loop),
+                              ("offset-norm", cfg.norm_offset), ("output-softcap", cfg.logit_softcap)) if on}
     for l in cfg.layers:
         m = l.mixer
         if m.kind == "attention":
-            kinds.append(LayerKind(SLIDING if m.window else FULL, 0, 0.0, m.window, m.heads, m.kv_heads, m.dim))
-            needs |= {c for c, on in (("sliding-window-attention", m.window), ("head-mixing-attention", m.head_mixing),
-                                      ("attention-sink", m.sink), ("qk-norm", m.qk_norm)) if on}
+            rot = m.rotary
+            kinds.append(LayerKind(CHUNKED if m.chunk else (SLIDING if m.window else FULL), rot.dims if rot else 0, rot.base if rot else 0.0,
+                                   m.look_back, m.heads, m.kv_heads, m.dim))
+            needs |= {c for c, on in (("sliding-window-attention", m.window), ("chunked-attention", m.chunk),
+                                      ("head-mixing-attention", m.head_mixing), ("attention-sink", m.sink),
+                                      ("learned-sink", m.head_sink), ("qk-norm", m.qk_norm), ("interleaved-rope", rot),
+                                      ("scaled-rope", rot and rot.scaling)) if on}
         elif m.kind == "latent_attention":
-            kinds.append(LayerKind(LATENT, m.rot_dim, m.rot_base, 0, m.heads, 1, m.dim + m.rot_dim))
-            needs |= {"latent-attention"} | ({"attention-sink"} if m.sink else set())
+            kinds.append(LayerKind(LATENT, m.rot_dim, m.rot_base, m.window, m.heads, 1, m.dim + m.rot_dim))
+            needs |= {c for c, on in (("latent-attention", True), ("attention-sink", m.sink), ("sliding-window-attention", m.window)) if on}
+        elif m.kind == "rglru":
+            kinds.append(LayerKind(RGLRU, q_heads=m.blocks, kv_heads=m.blocks, head_dim=m.vdim))
+            needs.add("gated-recurrence")
         else:
             kinds.append(LayerKind(GATED if m.kind == "hgrn2" else MLSTM, q_heads=m.heads, kv_heads=m.heads, head_dim=m.dim))
             needs.add("gated-memory" if m.kind == "hgrn2" else "matrix-memory")
-        if l.mlp is not None:
+        if l.mlp is not None and l.mlp.kind == "moe":
+            needs |= {"expert-mlp"} | ({"identity-experts"} if l.mlp.identity else set())
+        elif l.mlp is not None:
             needs.add(f"{l.mlp.activation}-mlp")
-    inter = max((l.mlp.ff for l in cfg.layers if l.mlp is not None), default=0)
-    act = next((l.mlp.activation for l in cfg.layers if l.mlp is not None), "")
+    mlps = [l.mlp for l in cfg.layers if l.mlp is not None]
+    inter = max((f.expert.ff if f.kind == "moe" else f.ff for f in mlps), default=0)
+    act = next(("gated" if f.kind == "moe" else f.activation for f in mlps), "")
     return Package(cfg.name, cfg.hidden, cfg.n_layers, inter, cfg.vocab, tuple(kinds), frozenset(needs), activation=act,
-                   tie_word_embeddings=cfg.tie_head, config=cfg, notes=f"layer-list decoder ({cfg.architecture})")
+                   final_logit_softcap=cfg.logit_softcap, tie_word_embeddings=cfg.tie_head, config=cfg, notes=f"layer-list decoder ({cfg.architecture})")
 
 
 def _spark() -> Package:

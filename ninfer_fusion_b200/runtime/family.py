@@ -52,7 +52,7 @@ def build_runtime(cfg, weights, device, *, rows: int, pages_per_row: int, n_page
         kv = PagedKvCache(cfg, n_pages, page_size, rows, pages_per_row, device, formats=kv_format, geometry=cfg.kv_geometry,
                           look_back=cfg.cache_window)
         states = RecurrentStatePool([[(shape, torch.float32) for shape in layer] for layer in cfg.state_shapes()], state_slots, device)
-        ws = LayeredWorkspace(cfg, step_tokens, logit_rows, device, model.dtype)
+        ws = LayeredWorkspace(cfg, step_tokens, logit_rows, device, model.dtype, ops=model._raw_ops)
         return Runtime(model, kv, states, ws, BLOCK_TOKENS, cfg.vocab, 0)
     model = HybridModel(cfg, weights, device, pdl=pdl, shard=shard)
     model.comm = comm

@@ -240,12 +240,12 @@ def test_latent_attention(ops, geo, dt):
     # ... and attended in the expanded form
     base, seqs, total = [], [], 0
     for s, (n, m) in enumerate(zip(*RAGGED)):
-        base.append(total if m >= 60 else -1)
+        base.append([total if m >= 60 else -1, 0])
         if m >= 60:
-            seqs.append([s, total, n])
+            seqs.append([s, total, 0, n])
             total += n
     rows = torch.zeros((total, C + R), dtype=dt, device="cuda")
-    ops.latent_gather(x.pages, x.table, ints(seqs), max(s[2] for s in seqs), rows, False)
+    ops.latent_gather(x.pages, x.table, ints(seqs), max(s[3] for s in seqs), rows, False)
     c = rows[:, :C].float().cpu()
     kv = torch.cat([torch.einsum("hdc,jc->jhd", x.uk.float(), c).reshape(total, -1), torch.einsum("hvc,jc->jhv", x.uv.float(), c).reshape(total, -1)], 1)
     wide = torch.full((x.T, H * V), 9.0, dtype=dt, device="cuda")

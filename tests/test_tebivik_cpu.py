@@ -24,7 +24,7 @@ def test_configuration_round_trip(name):
     assert sum(int(np.prod(s)) for _, s in tebivik.tensor_shapes(cfg)) == cfg.param_count()
     assert [r for r, _ in cfg.runs] == [i for i, _ in K.layer_order(c)]
     assert [t for _, t in cfg.runs if t >= 0] == list(range(c["loop"]["times"]))
-    assert native_subset(cfg) == "latent"
+    assert native_subset(cfg) == "+".join(sorted({{"latent_attention": "latent", "hgrn2": "gated"}[l["type"]] for l in c["layers"]}))
 
 
 def test_configuration_errors_are_named():
