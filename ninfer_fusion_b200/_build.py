@@ -39,7 +39,7 @@ PARTS = {
     "latent": ("latent_bindings.cpp", "attention/latent_prep.cu", "attention/latent_token.cu", "attention/latent_absorbed.cu",
                "attention/latent_expanded.cu", "gemm/head_gemm.cu"),
     "gated": ("gated_bindings.cpp", "gated/gated_recurrent.cu", "gated/gated_chunked.cu"),
-    "rglru": ("rglru_bindings.cpp", "rglru/rglru_scan.cu"),
+    "rglru": ("rglru_bindings.cpp", "rglru/rglru_scan.cu", "rglru/rglru_fused.cu"),
     "streams": ("stream_bindings.cpp", "pointwise/stream_rows.cu"),
     "moe": ("moe/moe_bindings.cpp", "moe/moe_route.cu", "moe/moe_grouped_gemm.cu", "moe/moe_grouped_gemm_f32.cu"),
 }

@@ -42,4 +42,12 @@ struct RglruArgs {
 const char* rglru_conv(const RglruArgs& a, void* u);
 const char* rglru_scan(const RglruArgs& a, const void* u, const float* raw);
 
+// Convolution and gates inside (bf16; blocks of up to about 500 channels).
+bool rglru_fused_supported(int width);
+// One token per sequence.
+const char* rglru_decode(const RglruArgs& a);
+// Query blocks: up to 64 consecutive tokens of one sequence each, a sequence's blocks in order and all but its last of 64.
+int64_t rglru_chunked_workspace_bytes(int T, int n_seq, int channels);
+const char* rglru_chunked(const RglruArgs& a, const int* blk_start, const int* blk_count, int n_blocks, void* workspace, int64_t bytes);
+
 }  // namespace nfb

@@ -57,9 +57,40 @@ void rglru_scan(const Tensor& proj, int64_t blocks, const Tensor& conv_w, const 
   chk(nfb::rglru_scan(a, u.data_ptr(), static_cast<const float*>(raw.data_ptr())));
 }
 
+// Convolution, gates and recurrence: one token per sequence without a workspace, portions in query blocks with one.
+void rglru(const Tensor& proj, int64_t blocks, const Tensor& conv_w, const Tensor& conv_b, const Tensor& cu_seqlens,
+           const Tensor& token_seq, const Tensor& cache_pos, const Tensor& state_slot, const Tensor& ring, const Tensor& gate_w,
+           const Tensor& gate_b, const Tensor& rate, const Tensor& S, const Tensor& out, const Tensor& blk_start, const Tensor& blk_count,
+           OptT workspace, bool write_state, bool pdl) {
+  c10::cuda::CUDAGuard guard(proj.device());
+  nfb::RglruArgs a = rglru_args(proj, blocks, conv_w, conv_b, cu_seqlens, token_seq, cache_pos, state_slot, ring);
+  need(gate_w, at::kBFloat16, "gate_w");
+  TORCH_CHECK(gate_w.is_contiguous() && gate_w.numel() == blocks * 2 * a.width * a.width, "rglru: gate_w must be [blocks, 2 width, width]");
+  need_vec(gate_b, at::kFloat, blocks * 2 * a.width, "gate_b");
+  a.gate_w = gate_w.data_ptr(); a.gate_b = static_cast<const float*>(gate_b.data_ptr());
+  out_and_state(a, proj, rate, S, out, write_state);
+  a.pdl = pdl;
+  if (!(workspace.has_value() && workspace->defined())) {
+    chk(nfb::rglru_decode(a));
+    return;
+  }
+  const int64_t nb = blk_start.numel();
+  need_vec(blk_start, at::kInt, nb, "blk_start"); need_vec(blk_count, at::kInt, nb, "blk_count"); need_cuda(*workspace, "workspace");
+  TORCH_CHECK(workspace->is_contiguous(), "workspace must be contiguous");
+  chk(nfb::rglru_chunked(a, static_cast<const int*>(blk_start.data_ptr()), static_cast<const int*>(blk_count.data_ptr()), static_cast<int>(nb),
+                         workspace->data_ptr(), workspace->numel() * workspace->element_size()));
+}
+bool rglru_fused_supported(int64_t width) { return nfb::rglru_fused_supported(static_cast<int>(width)); }
+int64_t rglru_chunked_workspace_bytes(int64_t T, int64_t n_seq, int64_t channels) {
+  return nfb::rglru_chunked_workspace_bytes(static_cast<int>(T), static_cast<int>(n_seq), static_cast<int>(channels));
+}
+
 }  // namespace
 
 TORCH_LIBRARY_FRAGMENT(nfb200, m) {
   m.def("rglru_conv(Tensor proj, int blocks, Tensor conv_w, Tensor conv_b, Tensor cu_seqlens, Tensor token_seq, Tensor cache_pos, Tensor state_slot, Tensor ring, Tensor u, bool pdl) -> ()", &rglru_conv);
   m.def("rglru_scan(Tensor proj, int blocks, Tensor conv_w, Tensor conv_b, Tensor cu_seqlens, Tensor token_seq, Tensor cache_pos, Tensor state_slot, Tensor ring, Tensor u, Tensor raw, Tensor rate, Tensor S, Tensor out, bool write_state, bool pdl) -> ()", &rglru_scan);
+  m.def("rglru(Tensor proj, int blocks, Tensor conv_w, Tensor conv_b, Tensor cu_seqlens, Tensor token_seq, Tensor cache_pos, Tensor state_slot, Tensor ring, Tensor gate_w, Tensor gate_b, Tensor rate, Tensor S, Tensor out, Tensor blk_start, Tensor blk_count, Tensor? workspace, bool write_state, bool pdl) -> ()", &rglru);
+  m.def("rglru_fused_supported(int width) -> bool", &rglru_fused_supported);
+  m.def("rglru_chunked_workspace_bytes(int T, int n_seq, int channels) -> int", &rglru_chunked_workspace_bytes);
 }

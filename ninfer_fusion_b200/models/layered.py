@@ -533,6 +533,12 @@ class LayeredModel:
         C, n, out = m.out_cols, m.vdim_p, ws.mix[:T, : m.out_cols]
         gates, gate_bias, rate = w[f"{p}/mix/gates"], w[f"{p}/mix/gate_bias"], w[f"{p}/mix/rate"]
         step = (m.blocks, w[f"{p}/mix/conv"], w[f"{p}/mix/conv_bias"], b.cu_seqlens, b.token_seq, b.cache_pos, b.state_slot, ring)
+        one = b.one_token_per_seq
+        if not self.f32 and self._raw_ops.rglru_fused_supported(n) and (one or self.prefill_kernels):
+            chunk_ws = None if one else self._grown("recurrence", int(self._raw_ops.rglru_chunked_workspace_bytes(T, b.n_seqs, C)))
+            ops.count += 0 if one else 1
+            ops.rglru(proj, *step, gates, gate_bias, rate, S, out, b.qblk_start, b.qblk_count, chunk_ws, write_state, self.pdl)
+            return out
         u = ws.rec_u[: T * C].view(T, C)
         raw = self._grown("gates", 8 * T * C)[: 8 * T * C].view(torch.float32).view(T, 2 * C)
         ops.rglru_conv(proj, *step, u, self.pdl)

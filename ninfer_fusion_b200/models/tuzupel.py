@@ -17,6 +17,8 @@ NORM_OFFSET = 1.0
 
 
 def _mask(c: dict) -> int:
+    if c.get("mask") is None:
+        return 0
     size = int(c["mask"]["size"])
     if size < 1:
         raise ValueError("the mask must leave a query its own key")
@@ -98,7 +100,9 @@ def config_dict(cfg: LayeredConfig) -> dict:
         if m.kind == "rglru":
             mixer = {"width": m.width, "blocks": m.blocks, "conv": m.taps}
         else:
-            mixer = {"heads": m.heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale, "mask": {"size": m.look_back}}
+            mixer = {"heads": m.heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale}
+            if m.look_back:
+                mixer["mask"] = {"size": m.look_back}
         if m.kind == "latent_attention":
             mixer["kv_rank"] = m.kv_rank
         if m.kind == "attention":

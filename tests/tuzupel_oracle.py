@@ -41,6 +41,8 @@ def stream_write(X, y, mix, w_out):
 # ---------------------------------------------------------------------------- attention
 def frequencies(rot):
     """One frequency per pair, slow ones divided by the factor, a ramp in between."""
+    if not rot:
+        return np.zeros(0)
     d = rot["dims"]
     f = rot["base"] ** (-np.arange(0, d, 2) / d)
     sc = rot.get("scaling")
@@ -84,6 +86,10 @@ def sees(T, window=0, chunk=0):
     return m
 
 
+def edge(mx):
+    return mx["mask"]["size"] if mx.get("mask") else 0
+
+
 def softmax_over(s, seen, sink=None):
     """s [..., T, T]; sink [heads] (axis 0 of s) counts once in every denominator."""
     s = np.where(seen, s, -np.inf)
@@ -107,11 +113,11 @@ def attend(q, k, v, scale, seen, sink=None):
 
 def attention(w, p, h, mx, eps):
     H, G, D, V, T = mx["heads"], mx["kv_heads"], mx["dim"], mx["vdim"], h.shape[0]
-    pos, f = np.arange(T, dtype=np.float64), frequencies(mx["rot"])
+    pos, f = np.arange(T, dtype=np.float64), frequencies(mx.get("rot"))
     q = rotate(rms((h @ w[p + "q"].T).reshape(T, H, D), eps) * w[p + "q.norm"], pos, f)
     k = rotate(rms((h @ w[p + "k"].T).reshape(T, G, D), eps) * w[p + "k.norm"], pos, f)
     v = (h @ w[p + "v"].T).reshape(T, G, V)
-    o = attend(q, k, v, mx["scale"], sees(T, chunk=mx["mask"]["size"]), w[p + "sink"])
+    o = attend(q, k, v, mx["scale"], sees(T, chunk=edge(mx)), w[p + "sink"])
     return o.reshape(T, H * V) @ w[p + "o"].T
 
 
@@ -120,7 +126,7 @@ def latent_attention(w, p, h, mx, eps):
     q = (h @ w[p + "q"].T).reshape(T, H, D)
     c = rms(h @ w[p + "dkv"].T, eps) * w[p + "dkv.norm"]
     k, v = (c @ w[p + "uk"].T).reshape(T, H, D), (c @ w[p + "uv"].T).reshape(T, H, V)
-    return attend(q, k, v, mx["scale"], sees(T, window=mx["mask"]["size"])).reshape(T, H * V) @ w[p + "o"].T
+    return attend(q, k, v, mx["scale"], sees(T, window=edge(mx))).reshape(T, H * V) @ w[p + "o"].T
 
 
 # ---------------------------------------------------------------------------- gated linear recurrence
@@ -169,17 +175,35 @@ def expert(w, p, h, limit):
     return glu_clamped(h @ w[p + ".gate"].T, h @ w[p + ".up"].T, limit) @ w[p + ".down"].T
 
 
-def route(z, correction, top, scale):
-    """Router logits [T, experts + identity] -> (choices [T, top], weights [T, top])."""
+def router_scores(z):
+    """Softmax over all router outputs [T, experts + identity]."""
     e = np.exp(z - z.max(axis=-1, keepdims=True))
-    s = e / e.sum(axis=-1, keepdims=True)
-    ids = np.argsort(-(s + correction), axis=-1, kind="stable")[:, :top]
+    return e / e.sum(axis=-1, keepdims=True)
+
+
+def route(z, correction, top, scale, forced=None):
+    """Router logits -> (choices [T, top], weights [T, top]).  `forced`: choices that are made elsewhere."""
+    s = router_scores(z)
+    ids = np.argsort(-(s + correction), axis=-1, kind="stable")[:, :top] if forced is None else forced
     return ids, np.take_along_axis(s, ids, axis=-1) * scale
 
 
-def experts(w, p, h, mlp):
+def shortfall(z, correction, ids):
+    """Per token: by how much the best choice score left out exceeds the worst one taken (<= 0 for the right choice)."""
+    c = router_scores(z) + correction
+    taken = np.zeros(c.shape, dtype=bool)
+    np.put_along_axis(taken, ids, True, axis=-1)
+    assert (taken.sum(axis=-1) == ids.shape[1]).all()          # no expert twice
+    left = np.where(taken, -np.inf, c).max(axis=-1)
+    return left - np.where(taken, c, np.inf).min(axis=-1)
+
+
+def experts(w, p, h, mlp, forced=None, short=None):
     r, E = mlp["router"], mlp["router"]["experts"]
-    ids, wt = route(h @ w[p + "router"].T, w[p + "correction"], r["top"], r["scale"])
+    z = h @ w[p + "router"].T
+    ids, wt = route(z, w[p + "correction"], r["top"], r["scale"], forced)
+    if short is not None:
+        short.append(shortfall(z, w[p + "correction"], ids))
     out = np.zeros_like(h)
     for e in range(E + r["identity"]):
         for j in range(r["top"]):
@@ -193,12 +217,12 @@ def experts(w, p, h, mlp):
 
 
 # ---------------------------------------------------------------------------- model
-def layer(w, cfg, i, X):
+def layer(w, cfg, i, X, forced=None, short=None):
     spec, eps = cfg["layers"][i], cfg["norm"]["eps"]
     mix = {"attention": attention, "latent_attention": latent_attention, "rglru": rglru}[spec["type"]]
     subs = [(1, lambda h: mix(w, f"l{i}.mix.", h, spec["mixer"], eps))]
     if spec["mlp"]:
-        subs.append((2, lambda h: experts(w, f"l{i}.mlp.", h, spec["mlp"])))
+        subs.append((2, lambda h: experts(w, f"l{i}.mlp.", h, spec["mlp"], forced, short)))
     for q, f in subs:
         hc = f"l{i}.hc{q}."
         y = f(norm_about_zero(stream_read(X, w[hc + "in"]), w[f"l{i}.norm{q}"], eps))
@@ -206,12 +230,13 @@ def layer(w, cfg, i, X):
     return X
 
 
-def forward(w, cfg, tokens, want_layers=False):
-    """Logits [T, vocab] of a whole sequence (and the sum of the streams after every layer)."""
+def forward(w, cfg, tokens, want_layers=False, choices=None, short=None):
+    """Logits [T, vocab] of a whole sequence (and the sum of the streams after every layer).  `choices`: layer -> experts
+    [T, top] to use instead of the router's own; `short` collects the shortfall of every layer's choices."""
     x = w["embed"][np.asarray(tokens)]
     X, per = np.repeat(x[:, None, :], cfg["streams"], axis=1), []
     for i in range(len(cfg["layers"])):
-        X = layer(w, cfg, i, X)
+        X = layer(w, cfg, i, X, None if choices is None else choices[i], short)
         per.append(X.sum(axis=1))
     z = norm_about_zero(X.sum(axis=1), w["final.norm"], cfg["norm"]["eps"]) @ w["head"].T
     cap = cfg.get("logit_softcap")
