@@ -23,11 +23,24 @@ __device__ __forceinline__ void rglru_conv8(const RglruArgs& p, const A* x, cons
   }
 }
 
+// exp(x) - 1 for x <= 0 out of the hardware 2^x, a Taylor polynomial near 0 (relative error about 1e-6)
+__device__ __forceinline__ float expm1_fast(float x) {
+  const float near = x * fmaf(x, fmaf(x, fmaf(x, fmaf(x, 1.f / 120.f, 1.f / 24.f), 1.f / 6.f), 0.5f), 1.f);
+  return x > -0.125f ? near : ex2_fast(x * kLog2e) - 1.f;
+}
+
 // a - 1 (a itself would lose what a long memory is made of: its distance from 1) and the input sqrt(1 - a^2) i u of one token
 // and channel; S <- S + (a - 1) S + input.
+template <typename A>
 __device__ __forceinline__ void rglru_gates(float raw_r, float raw_i, float rate, float u, float& em, float& in) {
-  em = expm1f(-rate / (1.f + expf(-raw_r)));
-  in = sqrtf(-em * (2.f + em)) * u / (1.f + expf(-raw_i));
+  if constexpr (sizeof(A) == 4) {
+    em = expm1f(-rate / (1.f + expf(-raw_r)));
+    in = sqrtf(-em * (2.f + em)) * u / (1.f + expf(-raw_i));
+  } else {
+    em = expm1_fast(-rate * rcp_fast(1.f + ex2_fast(-raw_r * kLog2e)));
+    const float v = -em * (2.f + em);
+    in = (v > 0.f ? v * rsqrtf(v) : 0.f) * u * rcp_fast(1.f + ex2_fast(-raw_i * kLog2e));
+  }
 }
 
 template <typename A>

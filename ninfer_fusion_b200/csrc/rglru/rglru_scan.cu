@@ -35,7 +35,7 @@ __global__ void __launch_bounds__(128) rglru_scan_kernel(const RglruArgs p, cons
   for (int t = t0; t < t1; ++t) {
     const float* g = raw + (static_cast<long long>(t) * p.blocks + b) * 2 * p.width + at;
     float em, in;
-    rglru_gates(g[0], g[p.width], rate, elem_to_f(u[static_cast<long long>(t) * C + c]), em, in);
+    rglru_gates<A>(g[0], g[p.width], rate, elem_to_f(u[static_cast<long long>(t) * C + c]), em, in);
     S += fmaf(em, S, in);
     const float y = elem_to_f(static_cast<const A*>(p.proj)[t * p.ldp + c]);
     static_cast<A*>(p.out)[t * p.ldo + c] = elem_from_f<A>(S * gelu_tanh_of<A>(y));

@@ -208,7 +208,7 @@ def describe(model_id: str) -> dict:
     p = lookup(model_id)
     return {"model_id": p.model_id, "hidden": p.hidden, "layers": p.n_layers, "full": p.count(FULL),
             "sliding": p.count(SLIDING), "gdn": p.count(GDN), "mlstm": p.count(MLSTM),
-            "hgrn2": p.count(GATED), "latent": p.count(LATENT), "intermediate": p.intermediate, "vocab": p.vocab,
-            "activation": p.activation, "final_logit_softcap": p.final_logit_softcap,
+            "hgrn2": p.count(GATED), "latent": p.count(LATENT), "chunked": p.count(CHUNKED), "rglru": p.count(RGLRU),
+            "intermediate": p.intermediate, "vocab": p.vocab, "activation": p.activation, "final_logit_softcap": p.final_logit_softcap,
             "needs": sorted(p.needs), "missing": list(p.missing()), "servable": not p.missing() and p.config is not None,
             "oracle_runtime": p.n_layers == p.count(FULL) + p.count(SLIDING) or isinstance(p.config, ModelConfig), "notes": p.notes}

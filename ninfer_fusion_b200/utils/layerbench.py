@@ -3,7 +3,8 @@
 `python bench.py --compare kuzanex-1b` prints one JSON line: prefill and decode tokens/s of the two models through the
 same generator (random weights, bf16), and for every kernel of the design its time, what bounds it, and the same for
 the other model's kernel of the like kind at equal size.  Kuzanex (head-mixing attention, matrix memory) stands beside the
-hybrid decoder, Tebivik (latent attention, gated memory) beside Kuzanex.  Kernels are timed cold (L2 flushed before every launch) with CUDA
+hybrid decoder, Tebivik (latent attention, gated memory) beside Kuzanex, Tuzupel (streams, experts, plain and latent attention,
+gated recurrence) beside the hybrid decoder with experts.  Kernels are timed cold (L2 flushed before every launch) with CUDA
 events; the roofline of a kernel is the slower of its algorithmic bytes at the measured copy bandwidth and its
 algorithmic multiply-adds at the measured bf16 GEMM rate.
 """
@@ -309,9 +310,9 @@ def _latent_design_rows(k: _Kernels, model, ws, cfg, batch: int, new: int, total
               uv.numel() * 2 + T * H * (V + C) * 2, T * uv.numel())
     else:
         rows = _rand(batch * total, C + R)
-        seqs = _ints([[i, i * total, total] for i in range(batch)])
+        seqs = _ints([[i, i * total, 0, total] for i in range(batch)])
         ukv = w[f"{pa}/mix/ukv"]
-        wide, out, base = _rand(batch * total, ukv.shape[0]), _rand(T, H * V), _ints([i * total for i in range(batch)])
+        wide, out, base = _rand(batch * total, ukv.shape[0]), _rand(T, H * V), _ints([[i * total, 0] for i in range(batch)])
         k.add(f"gather {tag}", "design", lambda: ops.latent_gather(pages, table, seqs, total, rows, False), rows.numel() * 4)
         gemm("expansion", ukv, x=rows[:, :C])
         k.add(f"attention {tag}", "design", lambda: ops.latent_expanded_attention(q, rows, wide, kv, H, C, m.rot_dim, m.scale, freq, sink, out, *blocks, row,
@@ -352,17 +353,23 @@ def compare(name: str, layers: int = 0, iters: int = 10, throughput: bool = True
     cfg = LAYERED_REGISTRY[name]
     if layers:
         cfg = cfg.shrink(layers)
-    latent = any(l.mixer.kind == "latent_attention" for l in cfg.layers)
-    other, label = (equal_size_kuzanex(cfg), "kuzanex") if latent else (equal_size_hybrid(cfg), "hybrid")
+    streams = cfg.residual == "streams"
+    latent = not streams and any(l.mixer.kind == "latent_attention" for l in cfg.layers)
+    if streams:
+        from .streambench import equal_size_expert_hybrid, stream_kernels
+        other, label = equal_size_expert_hybrid(cfg), "hybrid"
+    else:
+        other, label = (equal_size_kuzanex(cfg), "kuzanex") if latent else (equal_size_hybrid(cfg), "hybrid")
     res: Dict[str, object] = {"comparison": cfg.name, "design_params": cfg.param_count(), f"{label}_params": other.param_count(), "dtype": "bf16",
                               "data": "synthetic", "l2": "flushed before every kernel"}
     weights = random_layered_weights(cfg, "cuda:0")
-    rows = _kernels(cfg, other, weights, iters, only)
+    rows = stream_kernels(cfg, other, weights, iters, only) if streams else _kernels(cfg, other, weights, iters, only)
     pair: Dict[str, dict] = {}
     for r in rows:
         pair.setdefault(r["kernel"], {})[r["model"]] = r
     res["kernels"] = rows
-    res[f"farther_than_{label}"] = {n: round(p[label]["fraction"] / p["design"]["fraction"], 2) for n, p in pair.items() if len(p) == 2}
+    likes = {n: next(v for m, v in p.items() if m != "design") for n, p in pair.items() if len(p) == 2 and "design" in p}
+    res[f"farther_than_{label}"] = {n: round(like["fraction"] / max(1e-4, pair[n]["design"]["fraction"]), 2) for n, like in likes.items()}
     if throughput:
         res["throughput"] = {}
         w2 = random_layered_weights(other, "cuda:0") if latent else random_weights(other, "cuda:0", seed=0)
