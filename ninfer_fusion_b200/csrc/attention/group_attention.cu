@@ -255,18 +255,22 @@ __global__ void __launch_bounds__(kThreads) group_decode_kernel(const HeadMixArg
     const int page = table[key / P];
     return page < 0 ? -1 : (page * G + g) * P + key % P;
   };
+  // four lanes walk a row, 64 bytes at a time; a lane's rows are lane / 4 and lane / 4 + 8
   auto load = [&](int row, int i) {
-    const uint32_t dst = ring_a + (i % S) * plan.stage;
+    const uint32_t dst = ring_a + (i % S) * plan.stage + (lane & 3) * 16;
 #pragma unroll
-    for (int part = 0; part < 2; ++part) {
-      const int width = part ? V : D, vecs = width / 8, ld = part ? ldv : ldk;
-      const uint32_t to = dst + (part ? DK * ldk * 2 : 0);
-      const bf16* from = part ? vp : kp;
-      for (int x = lane; x < DK * vecs; x += 32) {      // (DK * vecs is a multiple of 32: no lane leaves the loop early)
-        const int key = x / vecs, c = (x % vecs) * 8;
-        const int r = __shfl_sync(0xffffffffu, row, key);
-        cp_async16(to + (key * ld + c) * 2, r >= 0 ? from + static_cast<long long>(r) * width + c : from, r >= 0);
-      }
+    for (int half = 0; half < 2; ++half) {
+      const int key = (lane >> 2) + half * 8, r = __shfl_sync(0xffffffffu, row, key);
+      const bool ok = r >= 0;
+      const bf16* ks = kp + static_cast<long long>(ok ? r : 0) * D + (lane & 3) * 8;
+      const bf16* vs = vp + static_cast<long long>(ok ? r : 0) * V + (lane & 3) * 8;
+      const uint32_t dk = dst + key * ldk * 2, dv = dst + (DK * ldk + key * ldv) * 2;
+#pragma unroll
+      for (int c = 0; c < DT * 16; c += 32)
+        if (c + (lane & 3) * 8 < D) cp_async16(dk + c * 2, ks + c, ok);
+#pragma unroll
+      for (int c = 0; c < VT * 8; c += 32)
+        if (c + (lane & 3) * 8 < V) cp_async16(dv + c * 2, vs + c, ok);
     }
   };
 #pragma unroll

@@ -82,8 +82,9 @@ def _expert_block(k: _Kernels, model, ws, cfg, hyb, T: int, tag: str) -> None:
     f, p, status = cfg.layers[0].mlp, "text/layers/0", model.status.tensor
     E, kk, ff, sf = f.experts, f.top, f.expert.ff_p, f.shared.ff_p
     x, delta, X = _rand(T, h), torch.empty(T, h, device="cuda"), torch.randn(T, S, h, device="cuda")
-    # experts with weights that the step touches, rows that they see
-    used, rows = min(E, T * kk), T * kk * E / f.choices
+    # experts whose weights the step reads, rows that they see
+    chosen = run_experts(model, ws.experts, T, p, f, x, delta)["choice"].flatten()
+    used, rows = int(torch.unique(chosen[chosen < E]).numel()), int((chosen < E).sum())
     weights = (used * ff + sf) * 3 * h * 2
     macs = (rows * ff + T * sf) * 3 * h
 
@@ -103,8 +104,10 @@ def _expert_block(k: _Kernels, model, ws, cfg, hyb, T: int, tag: str) -> None:
     host._gemm = lambda a, b, o, epi=0: ops.gemm_bf16(a, b, o, epi, None, None, None, int(ops.gemm_pick_splits(a.shape[0], *b.shape, epi)), status, False)
     hws.x, hws.normed = _rand(T, h), _rand(T, h)
     norm, normed = _rand(h), _rand(T, h)
-    k.add(f"expert block {tag}", "hybrid", lambda: block.forward(host, hws, T, "l", norm, normed),
-          (min(E, T * kk) * ff + sf) * 3 * h * 2 + T * h * 8 + 2 * T * kk * h * 2, (T * kk * ff + T * sf) * 3 * h)
+    block.forward(host, hws, T, "l", norm, normed)
+    used_h = int(torch.unique(block.ids[:T]).numel())
+    hws.normed = _rand(T, h)
+    k.add(f"expert block {tag}", "hybrid", lambda: block.forward(host, hws, T, "l", norm, normed), (used_h * ff + sf) * 3 * h * 2 + T * h * 8 + 2 * T * kk * h * 2, (T * kk * ff + T * sf) * 3 * h)
     # the grouped GEMMs alone, on the tables that a run leaves (both models take the same kernel; the unit differs)
     e = ws.experts
     run_experts(model, e, T, p, f, x, delta)
