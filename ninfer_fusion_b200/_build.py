@@ -41,6 +41,8 @@ PARTS = {
     "gated": ("gated_bindings.cpp", "gated/gated_recurrent.cu", "gated/gated_chunked.cu"),
     "rglru": ("rglru_bindings.cpp", "rglru/rglru_scan.cu", "rglru/rglru_fused.cu"),
     "streams": ("stream_bindings.cpp", "pointwise/stream_rows.cu"),
+    "branches": ("branch_bindings.cpp", "pointwise/branch_rows.cu"),
+    "ssd": ("ssd_bindings.cpp", "ssd/ssd_token.cu", "ssd/ssd_chunked.cu"),
     "moe": ("moe/moe_bindings.cpp", "moe/moe_route.cu", "moe/moe_grouped_gemm.cu", "moe/moe_grouped_gemm_f32.cu"),
 }
 
@@ -125,7 +127,7 @@ def build(verbose: bool = True, ptxas_info: bool = False, subset: str = "") -> P
     for s in cu:
         jobs.append((s, nv, "nvcc"))
     for s in cpp:
-        uses_torch = any(k in s.read_text() for k in ("torch/", "ATen/", "binding_util.h", "head_mix_args.h"))
+        uses_torch = any(k in s.read_text() for k in ("torch/", "ATen/", "binding_util.h", "head_mix_args.h", "mixture_args.h"))
         cx = ["g++"] + CXX_FLAGS + inc + ([abi] + torch_inc if uses_torch else [])
         jobs.append((s, cx, "g++ "))
     workers = max(1, min(len(jobs), os.cpu_count() or 4))

@@ -447,7 +447,7 @@ cudaError_t launch_prefill(const HeadMixArgs& a, const int* start, const int* co
 }  // namespace
 
 bool group_attention_supported(const HeadMixArgs& a) {
-  return !a.f32 && a.mix == nullptr && a.slope == nullptr && a.gate == nullptr && a.softcap == 0.f && a.dim % 16 == 0 && a.vdim % 16 == 0 &&
+  return !a.f32 && !a.sigmoid && a.mix == nullptr && a.slope == nullptr && a.gate == nullptr && a.softcap == 0.f && a.dim % 16 == 0 && a.vdim % 16 == 0 &&
          a.dim <= 256 && a.vdim <= 256 && a.n_kv > 0 && a.n_heads % a.n_kv == 0 && a.ldq % 8 == 0 && a.ldo % 8 == 0 &&
          a.n_kv * ((a.n_heads / a.n_kv + 15) / 16) <= 65535 && prefill_smem(a.dim, a.vdim) <= kSmemLimit;
 }

@@ -6,12 +6,20 @@
 //   a_h(i, j)  = exp(s_h) / (sink_one + exp(sinks[h]) + sum_j exp(s_h))        (sinks = null: without them)
 //   out_h(i)   = sigmoid(gate[i, h]) * sum_j a_h(i, j) v(j)                    (gate = null: no gate)
 //
+// or, with `sigmoid`, weights that stand by themselves and are mixed instead of the scores:
+//   w_g(i, j)  = sigmoid(scale * q_g(i) . k(j) - log_rate[g] ln(1 + log_step[g] (i - j)) + offset[g])
+//   out_h(i)   = sigmoid(gate[i, h]) * sum_j (sum_g mix[h, g] w_g(i, j)) v(j)          (log_rate, offset = null: without them)
+//
 // `slope` is the bias AFTER mixing: a per-head bias b_g taken off before the mix is slope[h] = sum_g mix[h, g] b_g.
 // Scores, weights and sums are fp32.  K and V live in paged planes [page, kv_head, token in page, width]; widths are
 // multiples of 16, zero-padded by the producer.  q, k, v and out are bf16 or (f32) fp32.
 #pragma once
 #include <cuda_runtime.h>
 #include <stdint.h>
+
+#ifdef __CUDACC__
+#include "../common/elem.cuh"
+#endif
 
 namespace nfb {
 
@@ -30,6 +38,10 @@ struct HeadMixArgs {
   const float* sinks = nullptr;     // [H] learned scores that only count in the denominator, or null
   const float* mix = nullptr;       // [H, H] row-major, or null
   const float* slope = nullptr;     // [H], or null
+  bool sigmoid = false;
+  const float* log_rate = nullptr;  // [H], or null (sigmoid weights only)
+  const float* log_step = nullptr;  // [H], with log_rate
+  const float* offset = nullptr;    // [H], or null (sigmoid weights only)
   const float* gate = nullptr;      // [T, *] raw gate values of head h at gate[t * ld_gate + h], or null
   int64_t ld_gate = 0;
   void* out = nullptr;              // [T, n_heads * vdim], leading dimension ldo
@@ -61,6 +73,29 @@ __device__ __forceinline__ int first_visible(int len, int window, int chunk) {
   if (chunk > 0) lo = max(lo, (len - 1) / chunk * chunk);
   return lo;
 }
+// Numbers of one head that turn a raw score into its sigmoid weight; `fast` keeps them scaled for 2^x.
+struct SigmoidHead {
+  float scale, offset, rate, step;
+  __device__ __forceinline__ SigmoidHead() {}
+  __device__ __forceinline__ SigmoidHead(const HeadMixArgs& p, int h, bool fast) {
+    const float k = fast ? -1.4426950408889634f : 1.f;
+    scale = p.scale * k;
+    offset = p.offset != nullptr ? p.offset[h] * k : 0.f;
+    rate = p.log_rate != nullptr ? p.log_rate[h] : 0.f;
+    step = p.log_rate != nullptr ? p.log_step[h] : 0.f;
+  }
+  // rate * log2(1 + step * d), hardware logarithm
+  __device__ __forceinline__ float bias_fast(float d) const {
+    float y;
+    asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(fmaf(step, fmaxf(d, 0.f), 1.f)));
+    return rate * y;
+  }
+  __device__ __forceinline__ float weight_fast(float s, float bias) const { return rcp_fast(1.f + ex2_fast(fmaf(scale, s, offset + bias))); }
+  // library functions
+  __device__ __forceinline__ float weight(float s, float d) const {
+    return 1.f / (1.f + expf(rate * log1pf(step * fmaxf(d, 0.f)) - fmaf(scale, s, offset)));
+  }
+};
 // What the sum of exp(s - m) v, with m the maximum and l the sum of exp(s - m), is multiplied with.
 __device__ __forceinline__ float head_mix_finish(float m, float l, float sink, const float* sinks, int h) {
   if (!(m > -3.0e38f)) return 0.f;   // no visible key
@@ -81,8 +116,8 @@ __device__ __forceinline__ float head_mix_finish(float m, float l, float sink, c
 // register-fragment order, as many blocks at a time as fit.
 const char* head_mix_prefill(const HeadMixArgs& a, const int* blk_start, const int* blk_count, int n_blocks, int max_keys,
                              void* scratch, int64_t scratch_bytes);
-// Scratch for `blocks` query blocks at a time.
-int64_t head_mix_prefill_scratch(int n_heads, int max_keys, int window, int blocks);
+// Scratch for `blocks` query blocks at a time: fp32 scores, or bf16 weights (sigmoid).
+int64_t head_mix_prefill_scratch(int n_heads, int max_keys, int window, int blocks, bool sigmoid);
 constexpr int kHeadMixBlock = 64;
 
 struct QkvAppendArgs {
@@ -100,6 +135,10 @@ struct QkvAppendArgs {
   int table_ld = 0, page_size = 0;
   const double* freq = nullptr;     // [rot / 2] rotation of neighbours (2i, 2i + 1) of the first `rot` values of q and k heads,
   int rot = 0;                      // after the norm, by position * freq[i] (angles in 64-bit); 0: none
+  bool unit = false;                // q and k are normed without weights (q_norm and k_norm null)
+  void* v_first = nullptr;          // [T, n_kv * vdim] values of an earlier layer: v <- (1 - lambda) v + lambda v_first, or, without a
+  int64_t ld_first = 0;             // lambda, where this layer's values are left for later ones
+  const float* v_lambda = nullptr;  // one number
   void* q_out = nullptr;            // [T, n_heads * dim], leading dimension ldq
   int64_t ldq = 0;
   void* k_pages = nullptr;

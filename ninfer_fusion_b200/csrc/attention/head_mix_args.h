@@ -7,7 +7,8 @@ namespace nfb_bind {
 
 inline nfb::HeadMixArgs head_mix_args(const Tensor& q, const Tensor& k_pages, const Tensor& v_pages, const Tensor& block_table,
                                const Tensor& table_row, const Tensor& kv_len, int64_t window, double scale, double softcap,
-                               double sink, OptT mix, OptT slope, OptT gate, const Tensor& out, bool pdl, int64_t chunk, OptT sinks) {
+                               double sink, OptT mix, OptT slope, OptT gate, const Tensor& out, bool pdl, int64_t chunk, OptT sinks,
+                               bool sigmoid, OptT log_rate, OptT log_step, OptT offset) {
   nfb::HeadMixArgs a;
   a.f32 = act_f32(q, "q");
   const auto dt = q.scalar_type();
@@ -38,6 +39,14 @@ inline nfb::HeadMixArgs head_mix_args(const Tensor& q, const Tensor& k_pages, co
   a.sink = static_cast<float>(sink); a.chunk = static_cast<int>(chunk);
   if (sinks.has_value() && sinks->defined()) need_vec(*sinks, at::kFloat, H, "sinks");
   a.sinks = ptr_or_null<const float>(sinks);
+  for (OptT v : {std::cref(log_rate), std::cref(log_step), std::cref(offset)})
+    if (v.has_value() && v->defined()) need_vec(*v, at::kFloat, H, "numbers per head");
+  a.sigmoid = sigmoid;
+  a.log_rate = ptr_or_null<const float>(log_rate); a.log_step = ptr_or_null<const float>(log_step); a.offset = ptr_or_null<const float>(offset);
+  TORCH_CHECK((a.log_rate == nullptr) == (a.log_step == nullptr), "head_mix attention: a logarithmic bias has two numbers per head");
+  TORCH_CHECK(sigmoid || (a.log_rate == nullptr && a.offset == nullptr), "head_mix attention: logarithmic bias and offset go with sigmoid weights");
+  TORCH_CHECK(!sigmoid || (softcap == 0.0 && sink == 0.0 && a.sinks == nullptr && !(slope.has_value() && slope->defined())),
+              "head_mix attention: sigmoid weights have neither cap nor sink nor slope");
   a.mix = ptr_or_null<const float>(mix); a.slope = ptr_or_null<const float>(slope);
   a.out = out.data_ptr(); a.ldo = out.stride(0);
   a.stream = cur_stream(); a.pdl = pdl;

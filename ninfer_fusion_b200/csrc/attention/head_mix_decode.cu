@@ -3,6 +3,7 @@
 // block barrier on the loads) and multiplies them against all query heads of the group at once, the query heads being
 // the rows of the MMA.  Scores meet in shared memory once per 16-key tile for the mix:
 //   scores(t) | barrier | mix(t) | barrier | softmax + values(t), scores(t + 1) | barrier | ...
+// Sigmoid weights are made where the scores are, and the mixed ones go straight to the values.
 #include "head_mix.h"
 
 #include <math_constants.h>
@@ -36,7 +37,7 @@ struct SmemPlan {
 };
 
 // NW warps, WG kv heads per warp, VT: upper bound of vdim / 16, S: ring stages.
-template <int NW, int WG, int VT, int S>
+template <int NW, int WG, int VT, int S, bool SIG>
 __global__ void __launch_bounds__(NW * 32) head_mix_decode_kernel(const HeadMixArgs p, int split_keys, int n_splits,
                                                                    float* __restrict__ part_o, float* __restrict__ part_ml) {
   extern __shared__ __align__(16) uint8_t smem[];
@@ -116,6 +117,14 @@ __global__ void __launch_bounds__(NW * 32) head_mix_decode_kernel(const HeadMixA
       for (int e = 0; e < 4; ++e) o[j][n][e] = 0.f;
   }
   const float cap_k = p.softcap > 0.f ? 2.f * kLog2e * p.scale / p.softcap : 0.f;
+  SigmoidHead sig[WG][2];       // of the two query heads of each group that this thread's accumulator rows belong to
+  if constexpr (SIG) {
+#pragma unroll
+    for (int j = 0; j < WG; ++j)
+#pragma unroll
+      for (int r = 0; r < 2; ++r)
+        if (warp + j * NW < G && r4 + r * 8 < R) sig[j][r] = SigmoidHead(p, (warp + j * NW) * R + r4 + r * 8, true);
+  }
   const uint32_t q_a = smem_u32(q_s);
   __syncthreads();
 
@@ -148,7 +157,12 @@ __global__ void __launch_bounds__(NW * 32) head_mix_decode_kernel(const HeadMixA
           const int r = r4 + (e >> 1) * 8;
           if (r < R) {
             float s = c[n][e];
-            s = p.softcap > 0.f ? softcap_fast(s, cap_k, p.softcap) : s * p.scale;
+            if constexpr (SIG) {
+              const SigmoidHead& hd = sig[j][e >> 1];
+              s = hd.weight_fast(s, hd.bias_fast(static_cast<float>(qpos - (k_begin + tile * KT + n * 8 + c4 * 2 + (e & 1)))));
+            } else {
+              s = p.softcap > 0.f ? softcap_fast(s, cap_k, p.softcap) : s * p.scale;
+            }
             cs[(g * R + r) * kLdS + n * 8 + c4 * 2 + (e & 1)] = s;
           }
         }
@@ -177,8 +191,8 @@ __global__ void __launch_bounds__(NW * 32) head_mix_decode_kernel(const HeadMixA
         if (h + 1 < H) s1 -= p.slope[h + 1] * d;
       }
       const bool in = kpos < k_end;
-      ss[h * kLdS + key] = in ? s0 : -CUDART_INF_F;
-      ss[(h + 1) * kLdS + key] = in ? s1 : -CUDART_INF_F;
+      ss[h * kLdS + key] = in ? s0 : (SIG ? 0.f : -CUDART_INF_F);
+      ss[(h + 1) * kLdS + key] = in ? s1 : (SIG ? 0.f : -CUDART_INF_F);
     }
     cp_async_wait<2 * S - 1>();
     __syncthreads();
@@ -199,8 +213,9 @@ __global__ void __launch_bounds__(NW * 32) head_mix_decode_kernel(const HeadMixA
           w[r][0] = x.x; w[r][1] = x.y; w[r][2] = y.x; w[r][3] = y.y;
         } else {
 #pragma unroll
-          for (int e = 0; e < 4; ++e) w[r][e] = -CUDART_INF_F;
+          for (int e = 0; e < 4; ++e) w[r][e] = SIG ? 0.f : -CUDART_INF_F;
         }
+        if constexpr (SIG) continue;
         float mx = fmaxf(fmaxf(w[r][0], w[r][1]), fmaxf(w[r][2], w[r][3]));
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
@@ -224,8 +239,10 @@ __global__ void __launch_bounds__(NW * 32) head_mix_decode_kernel(const HeadMixA
           ldsm_x4_trans(va + n * 32, b);
 #pragma unroll
           for (int u = 0; u < 2; ++u) {
-            o[j][2 * n + u][0] *= corr[0]; o[j][2 * n + u][1] *= corr[0];
-            o[j][2 * n + u][2] *= corr[1]; o[j][2 * n + u][3] *= corr[1];
+            if constexpr (!SIG) {
+              o[j][2 * n + u][0] *= corr[0]; o[j][2 * n + u][1] *= corr[0];
+              o[j][2 * n + u][2] *= corr[1]; o[j][2 * n + u][3] *= corr[1];
+            }
             mma_bf16_16816(o[j][2 * n + u], af, b[2 * u], b[2 * u + 1]);
           }
         }
@@ -254,11 +271,11 @@ __global__ void __launch_bounds__(NW * 32) head_mix_decode_kernel(const HeadMixA
         for (int n = 0; n < VT * 2; ++n)
           if (n * 8 < V) *reinterpret_cast<float2*>(dst + n * 8) = make_float2(o[j][n][2 * r], o[j][n][2 * r + 1]);
         if (c4 == 0) {
-          part_ml[at * 2] = m[j][r];
-          part_ml[at * 2 + 1] = sum;
+          part_ml[at * 2] = SIG ? 0.f : m[j][r];
+          part_ml[at * 2 + 1] = SIG ? 1.f : sum;
         }
       } else {
-        float f = head_mix_finish(m[j][r], sum, p.sink, p.sinks, h);
+        float f = SIG ? 1.f : head_mix_finish(m[j][r], sum, p.sink, p.sinks, h);
         if (p.gate != nullptr) f *= sigmoid_of<bf16>(p.gate[t * p.ld_gate + h]);
         bf16* dst = static_cast<bf16*>(p.out) + t * p.ldo + static_cast<long long>(h) * V + c4 * 2;
 #pragma unroll
@@ -269,10 +286,10 @@ __global__ void __launch_bounds__(NW * 32) head_mix_decode_kernel(const HeadMixA
   }
 }
 
-template <int NW, int WG, int VT, int S>
+template <int NW, int WG, int VT, int S, bool SIG>
 const char* launch(const HeadMixArgs& a, int split_keys, int n_splits, float* part_o, float* part_ml) {
   const int smem = SmemPlan(a.n_heads, a.n_kv, a.dim, a.vdim, S).total;
-  auto kern = head_mix_decode_kernel<NW, WG, VT, S>;
+  auto kern = head_mix_decode_kernel<NW, WG, VT, S, SIG>;
   if (smem > 48 * 1024) {
     const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return cudaGetErrorString(e);
@@ -284,15 +301,15 @@ const char* launch(const HeadMixArgs& a, int split_keys, int n_splits, float* pa
 
 constexpr int kMaxSmem = 220 * 1024;
 
-template <int NW, int WG, int VT>
+template <bool SIG, int NW, int WG, int VT>
 const char* launch_stages(const HeadMixArgs& a, int split_keys, int n_splits, float* part_o, float* part_ml) {
   // two CTAs per SM hide each other's barriers better than a deeper ring; the ring takes what is left
   auto fits = [&](int s, int limit) { return SmemPlan(a.n_heads, a.n_kv, a.dim, a.vdim, s).total <= limit; };
-  if (fits(4, kMaxSmem / 2)) return launch<NW, WG, VT, 4>(a, split_keys, n_splits, part_o, part_ml);
+  if (fits(4, kMaxSmem / 2)) return launch<NW, WG, VT, 4, SIG>(a, split_keys, n_splits, part_o, part_ml);
   if (fits(2, kMaxSmem / 2) || !fits(1, kMaxSmem / 2)) {
-    if (fits(2, kMaxSmem)) return launch<NW, WG, VT, 2>(a, split_keys, n_splits, part_o, part_ml);
+    if (fits(2, kMaxSmem)) return launch<NW, WG, VT, 2, SIG>(a, split_keys, n_splits, part_o, part_ml);
   }
-  return launch<NW, WG, VT, 1>(a, split_keys, n_splits, part_o, part_ml);
+  return launch<NW, WG, VT, 1, SIG>(a, split_keys, n_splits, part_o, part_ml);
 }
 
 }  // namespace
@@ -304,17 +321,24 @@ bool head_mix_decode_supported(const HeadMixArgs& a) {
   return a.vdim <= 256 && a.n_kv <= 8;
 }
 
-const char* head_mix_decode(const HeadMixArgs& a, int split_keys, int n_splits, float* part_o, float* part_ml) {
+namespace {
+template <bool SIG>
+const char* pick_shape(const HeadMixArgs& a, int split_keys, int n_splits, float* part_o, float* part_ml) {
   if (a.vdim <= 64) {
-    if (a.n_kv <= 8) return launch_stages<8, 1, 4>(a, split_keys, n_splits, part_o, part_ml);
-    if (a.n_kv <= 16) return launch_stages<16, 1, 4>(a, split_keys, n_splits, part_o, part_ml);
-    return launch_stages<16, 2, 4>(a, split_keys, n_splits, part_o, part_ml);
+    if (a.n_kv <= 8) return launch_stages<SIG, 8, 1, 4>(a, split_keys, n_splits, part_o, part_ml);
+    if (a.n_kv <= 16) return launch_stages<SIG, 16, 1, 4>(a, split_keys, n_splits, part_o, part_ml);
+    return launch_stages<SIG, 16, 2, 4>(a, split_keys, n_splits, part_o, part_ml);
   }
   if (a.vdim <= 128) {
-    if (a.n_kv <= 8) return launch_stages<8, 1, 8>(a, split_keys, n_splits, part_o, part_ml);
-    return launch_stages<16, 1, 8>(a, split_keys, n_splits, part_o, part_ml);
+    if (a.n_kv <= 8) return launch_stages<SIG, 8, 1, 8>(a, split_keys, n_splits, part_o, part_ml);
+    return launch_stages<SIG, 16, 1, 8>(a, split_keys, n_splits, part_o, part_ml);
   }
-  return launch_stages<8, 1, 16>(a, split_keys, n_splits, part_o, part_ml);
+  return launch_stages<SIG, 8, 1, 16>(a, split_keys, n_splits, part_o, part_ml);
+}
+}  // namespace
+
+const char* head_mix_decode(const HeadMixArgs& a, int split_keys, int n_splits, float* part_o, float* part_ml) {
+  return a.sigmoid ? pick_shape<true>(a, split_keys, n_splits, part_o, part_ml) : pick_shape<false>(a, split_keys, n_splits, part_o, part_ml);
 }
 
 }  // namespace nfb

@@ -12,6 +12,9 @@
 //   values   one CTA = (64 queries, head): flash-style running softmax over score fragments read back in the same
 //            order (they are exactly the A operand of the value MMA), V tiles staged with cp.async.
 //
+// Sigmoid weights stand by themselves, so they are made before the mix: the first kernel leaves mixed WEIGHTS as bf16 pairs,
+// half the scratch, and the second one only multiplies them with the values.
+//
 // Query blocks are processed as many at a time as the scratch holds.
 #include "head_mix.h"
 
@@ -33,8 +36,23 @@ struct PrefillParams {
   const int* blk_count;
   int blk0;            // first query block of this launch
   int n_tiles;         // 8-key tiles reserved per query block
-  float4* scratch;     // [block][tile][q tile 0..3][head][lane]
+  float4* scratch;     // [block][tile][q tile 0..3][head][lane]; sigmoid: uint2, weights of rows r4 and r4 + 8 as bf16 pairs
 };
+
+// Sigmoid weights of the accumulators c[NT][4] of one head.  `base` is the distance of element 0 of tile 0: tiles lie 8 keys
+// apart and the two rows of a thread 8 queries, so 2 (NT + 1) logarithms do for 4 NT elements.
+template <int NT>
+__device__ __forceinline__ void sigmoid_tile(float (*c)[4], const SigmoidHead& hd, float base) {
+  float b[NT + 1][2];
+#pragma unroll
+  for (int m = 0; m <= NT; ++m)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) b[m][e] = hd.bias_fast(base + static_cast<float>(8 - 8 * m - e));
+#pragma unroll
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) c[n][e] = hd.weight_fast(c[n][e], b[n + 1 - (e >> 1)][e & 1]);
+}
 
 // Key range of a query block and of one of its 16-query tiles, in 8-key tiles counted from the block's first key.
 struct BlockRange {
@@ -59,7 +77,7 @@ struct BlockRange {
 
 // HMAX: heads rounded up (mixed scores of all of them are live in registers); NT: 8-key tiles per warp.
 // blockDim 256: 8 warps = 4 query tiles x 2 key groups.  grid: (query block, key group pair, group of HMAX output heads)
-template <int HMAX, int NT>
+template <int HMAX, int NT, bool SIG>
 __global__ void __launch_bounds__(256) head_mix_scores_kernel(const PrefillParams p) {
   extern __shared__ __align__(16) float mix_s[];   // [H][HMAX]: mix_s[g][h] = mix[h0 + h, g]
   const HeadMixArgs& a = p.a;
@@ -120,7 +138,10 @@ __global__ void __launch_bounds__(256) head_mix_scores_kernel(const PrefillParam
         mma_bf16_16816(c + 4 * n, af, y.x, y.y);
       }
     }
-    if (a.softcap > 0.f) {
+    if constexpr (SIG) {
+      sigmoid_tile<NT>(reinterpret_cast<float(*)[4]>(c), SigmoidHead(a, g, true),
+                       static_cast<float>(br.first_query(qt) + r4 - (br.k0 + tile0 * 8 + c4 * 2)));
+    } else if (a.softcap > 0.f) {
 #pragma unroll
       for (int j = 0; j < NT * 4; ++j) c[j] = softcap_fast(c[j], cap_k, a.softcap);
     } else {
@@ -155,6 +176,15 @@ __global__ void __launch_bounds__(256) head_mix_scores_kernel(const PrefillParam
       vis[e] = d >= 0 && (W <= 0 || d < W);
     }
     float4* dst = p.scratch + ((static_cast<long long>(blockIdx.x) * p.n_tiles + tile) * 4 + qt) * H * 32 + lane;
+    if constexpr (SIG) {
+      uint2* pairs = reinterpret_cast<uint2*>(p.scratch) + ((static_cast<long long>(blockIdx.x) * p.n_tiles + tile) * 4 + qt) * H * 32 + lane;
+#pragma unroll
+      for (int h = 0; h < HMAX; ++h)
+        if (h0 + h < H)
+          pairs[(h0 + h) * 32] = make_uint2(pack_bf16x2(vis[0] ? acc[h][4 * n] : 0.f, vis[1] ? acc[h][4 * n + 1] : 0.f),
+                                            pack_bf16x2(vis[2] ? acc[h][4 * n + 2] : 0.f, vis[3] ? acc[h][4 * n + 3] : 0.f));
+      continue;
+    }
 #pragma unroll
     for (int h = 0; h < HMAX; ++h) {
       if (h0 + h < H) {
@@ -187,20 +217,23 @@ __device__ __forceinline__ void unpack2(unsigned long long v, float& x, float& y
 }
 
 // KS: dim / 16 (EXACT) or an upper bound of it.
-template <int HMAX, int NT, int KS, bool EXACT>
+template <int HMAX, int NT, int KS, bool EXACT, bool SIG>
 __global__ void __launch_bounds__(256) head_mix_scores_resident_kernel(const PrefillParams p, int iters) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
   const HeadMixArgs& a = p.a;
   const int H = a.n_heads, G = a.n_kv, R = H / G, D = a.dim, P = a.page_size, W = a.window;
   const int ldq = (EXACT ? KS * 16 : D) + 8, steps = EXACT ? KS : D / 16;
   float2* mix_s = reinterpret_cast<float2*>(smem_raw);                             // [H][HMAX]: (mix[h, g], mix[h, g])
-  bf16* q_s = reinterpret_cast<bf16*>(smem_raw + sizeof(float2) * H * HMAX);       // [H][16][ldq], k order of the fragments
+  SigmoidHead* sig_s = reinterpret_cast<SigmoidHead*>(smem_raw + sizeof(float2) * H * HMAX);     // [H], sigmoid weights only
+  bf16* q_s = reinterpret_cast<bf16*>(sig_s + (SIG ? H : 0));                      // [H][16][ldq], k order of the fragments
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r4 = lane >> 2, c4 = lane & 3;
   for (int i = tid; i < H * HMAX; i += 256) {
     const int g = i / HMAX, h = i % HMAX;
     const float m = h < H ? (a.mix != nullptr ? a.mix[h * H + g] : (h == g ? 1.f : 0.f)) : 0.f;
     mix_s[i] = make_float2(m, m);
   }
+  if constexpr (SIG)
+    for (int h = tid; h < H; h += 256) sig_s[h] = SigmoidHead(a, h, true);
   pdl_launch_next();
   pdl_wait_prior();
   const int qt = blockIdx.x & 3;
@@ -269,6 +302,7 @@ __global__ void __launch_bounds__(256) head_mix_scores_resident_kernel(const Pre
     for (int h = 0; h < HMAX; ++h)
 #pragma unroll
       for (int j = 0; j < NT * 2; ++j) acc[h][j] = 0ull;
+    const float base = static_cast<float>(br.first_query(qt) + r4 - (br.k0 + tile0 * 8 + c4 * 2));
     uint32_t kf[NT][KS][2], kn[NT][KS][2];
     load_k(0, kf);
     for (int g = 0; g < G; ++g) {
@@ -297,8 +331,12 @@ __global__ void __launch_bounds__(256) head_mix_scores_resident_kernel(const Pre
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             c[n][e] += c2[n][e];
-            c[n][e] = a.softcap > 0.f ? softcap_fast(c[n][e], cap_k, a.softcap) : c[n][e] * a.scale;
+            if constexpr (!SIG) c[n][e] = a.softcap > 0.f ? softcap_fast(c[n][e], cap_k, a.softcap) : c[n][e] * a.scale;
           }
+        }
+        if constexpr (SIG) sigmoid_tile<NT>(c, sig_s[hq], base);
+#pragma unroll
+        for (int n = 0; n < NT; ++n) {
           cp[2 * n] = pack2(c[n][0], c[n][1]);
           cp[2 * n + 1] = pack2(c[n][2], c[n][3]);
         }
@@ -332,6 +370,19 @@ __global__ void __launch_bounds__(256) head_mix_scores_resident_kernel(const Pre
         vis[e] = d >= 0 && (W <= 0 || d < W);
       }
       float4* dst = p.scratch + ((static_cast<long long>(blockIdx.x >> 2) * p.n_tiles + tile) * 4 + qt) * H * 32 + lane;
+      if constexpr (SIG) {
+        uint2* pairs = reinterpret_cast<uint2*>(p.scratch) + ((static_cast<long long>(blockIdx.x >> 2) * p.n_tiles + tile) * 4 + qt) * H * 32 + lane;
+#pragma unroll
+        for (int h = 0; h < HMAX; ++h) {
+          if (h < H) {
+            float4 o;
+            unpack2(acc[h][2 * n], o.x, o.y);
+            unpack2(acc[h][2 * n + 1], o.z, o.w);
+            pairs[h * 32] = make_uint2(pack_bf16x2(vis[0] ? o.x : 0.f, vis[1] ? o.y : 0.f), pack_bf16x2(vis[2] ? o.z : 0.f, vis[3] ? o.w : 0.f));
+          }
+        }
+        continue;
+      }
 #pragma unroll
       for (int h = 0; h < HMAX; ++h) {
         if (h < H) {
@@ -353,7 +404,7 @@ __global__ void __launch_bounds__(256) head_mix_scores_resident_kernel(const Pre
 constexpr int kVTile = 64;   // keys per V tile
 
 // VT: 16-wide value column tiles per CTA.  blockDim 128: warp = query tile.  grid: (head, query block, value chunk)
-template <int VT>
+template <int VT, bool SIG>
 __global__ void __launch_bounds__(128, VT <= 8 ? 4 : 2) head_mix_values_kernel(const PrefillParams p) {
   constexpr int kLd = VT * 16 + 8;
   extern __shared__ __align__(16) bf16 v_s[];   // [2][kVTile][kLd]
@@ -404,6 +455,15 @@ __global__ void __launch_bounds__(128, VT <= 8 ? 4 : 2) head_mix_values_kernel(c
   float m[2] = {-CUDART_INF_F, -CUDART_INF_F}, l[2] = {0.f, 0.f};
   const float4* sc = p.scratch + ((static_cast<long long>(blk) * p.n_tiles) * 4 + qt) * H * 32 + h * 32 + lane;
   const long long sc_tile = static_cast<long long>(4) * H * 32;
+  const uint2* wt = reinterpret_cast<const uint2*>(p.scratch) + ((static_cast<long long>(blk) * p.n_tiles) * 4 + qt) * H * 32 + h * 32 + lane;
+  // weights of half a V tile, likewise
+  auto fetch_w = [&](int half, uint2* s) {
+#pragma unroll
+    for (int n = 0; n < 4; ++n) {
+      const int tile = half * 4 + n;
+      s[n] = (tile >= first && tile <= last) ? __ldcs(wt + tile * sc_tile) : make_uint2(0u, 0u);
+    }
+  };
   // scores of half a V tile, fetched one half ahead of their use
   auto fetch = [&](int half, float4* s) {
     if (half * 4 > last || half * 4 + 3 < first) return;
@@ -415,7 +475,8 @@ __global__ void __launch_bounds__(128, VT <= 8 ? 4 : 2) head_mix_values_kernel(c
     }
   };
   float4 nxt[4];
-  fetch(0, nxt);
+  uint2 nxt_w[4];
+  if constexpr (SIG) fetch_w(0, nxt_w); else fetch(0, nxt);
   stage(0);
   for (int vt = 0; vt < n_vt; ++vt) {
     if (vt + 1 < n_vt) { stage(vt + 1); cp_async_wait<1>(); } else { cp_async_wait<0>(); }
@@ -424,6 +485,25 @@ __global__ void __launch_bounds__(128, VT <= 8 ? 4 : 2) head_mix_values_kernel(c
 #pragma unroll
     for (int hf = 0; hf < 2; ++hf) {
       const int half = vt * 2 + hf;
+      if constexpr (SIG) {
+        uint2 w[4];
+#pragma unroll
+        for (int n = 0; n < 4; ++n) w[n] = nxt_w[n];
+        fetch_w(half + 1, nxt_w);
+        if (half * 4 > last || half * 4 + 3 < first) continue;
+#pragma unroll
+        for (int kk = 0; kk < 2; ++kk) {
+          const uint32_t af[4] = {w[2 * kk].x, w[2 * kk].y, w[2 * kk + 1].x, w[2 * kk + 1].y};
+#pragma unroll
+          for (int n = 0; n < VT; ++n) {
+            uint32_t b[4];
+            ldsm_x4_trans(tile_base + ((hf * 32 + kk * 16) * kLd + n * 16) * 2, b);
+            mma_bf16_16816(o[2 * n], af, b[0], b[1]);
+            mma_bf16_16816(o[2 * n + 1], af, b[2], b[3]);
+          }
+        }
+        continue;
+      }
       float4 s[4];
 #pragma unroll
       for (int n = 0; n < 4; ++n)     // scaled for 2^x
@@ -488,7 +568,7 @@ __global__ void __launch_bounds__(128, VT <= 8 ? 4 : 2) head_mix_values_kernel(c
     const int i = qt * 16 + r4 + r * 8;
     if (i >= br.cnt) continue;
     const long long t = br.t0 + i;
-    float f = head_mix_finish(m[r] * (1.f / kLog2e), l[r], a.sink, a.sinks, h);
+    float f = SIG ? 1.f : head_mix_finish(m[r] * (1.f / kLog2e), l[r], a.sink, a.sinks, h);
     if (a.gate != nullptr) f *= sigmoid_of<bf16>(a.gate[t * a.ld_gate + h]);
     bf16* dst = static_cast<bf16*>(a.out) + t * a.ldo + static_cast<long long>(h) * V + v0 + c4 * 2;
 #pragma unroll
@@ -504,9 +584,9 @@ int tiles_for(int max_keys, int window) {
   return (keys + 7 + 7) / 8;
 }
 
-template <int HMAX, int NT>
+template <int HMAX, int NT, bool SIG>
 cudaError_t launch_scores(const PrefillParams& p, int n_blocks) {
-  auto kern = head_mix_scores_kernel<HMAX, NT>;
+  auto kern = head_mix_scores_kernel<HMAX, NT, SIG>;
   const size_t smem = sizeof(float) * static_cast<size_t>(p.a.n_heads) * HMAX;
   const int groups = (p.n_tiles + 2 * NT - 1) / (2 * NT);
   const dim3 grid(n_blocks, groups, (p.a.n_heads + HMAX - 1) / HMAX);
@@ -519,12 +599,12 @@ cudaError_t launch_scores(const PrefillParams& p, int n_blocks) {
 
 constexpr size_t kResidentSmem = 200 * 1024;
 size_t resident_smem(int H, int hmax, int D) {
-  return sizeof(float2) * static_cast<size_t>(H) * hmax + sizeof(bf16) * static_cast<size_t>(H) * 16 * (D + 8);
+  return (sizeof(float2) * hmax + sizeof(SigmoidHead)) * static_cast<size_t>(H) + sizeof(bf16) * static_cast<size_t>(H) * 16 * (D + 8);
 }
 
-template <int HMAX, int NT, int KS, bool EXACT>
+template <int HMAX, int NT, int KS, bool EXACT, bool SIG>
 cudaError_t launch_resident(const PrefillParams& p, int n_blocks) {
-  auto kern = head_mix_scores_resident_kernel<HMAX, NT, KS, EXACT>;
+  auto kern = head_mix_scores_resident_kernel<HMAX, NT, KS, EXACT, SIG>;
   const size_t smem = resident_smem(p.a.n_heads, HMAX, p.a.dim);
   if (smem > 48 * 1024) {
     const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
@@ -539,17 +619,17 @@ cudaError_t launch_resident(const PrefillParams& p, int n_blocks) {
   return launch_kernel(kern, grid, dim3(256), smem, p.a.stream, p.a.pdl, 1, p, iters);
 }
 
-template <int HMAX, int NT>
+template <int HMAX, int NT, bool SIG>
 cudaError_t launch_resident_dim(const PrefillParams& p, int n_blocks) {
-  if (p.a.dim == 64) return launch_resident<HMAX, NT, 4, true>(p, n_blocks);
-  if (p.a.dim == 128) return launch_resident<HMAX, NT, 8, true>(p, n_blocks);
-  if (p.a.dim < 64) return launch_resident<HMAX, NT, 4, false>(p, n_blocks);
-  return launch_resident<HMAX, NT, 8, false>(p, n_blocks);
+  if (p.a.dim == 64) return launch_resident<HMAX, NT, 4, true, SIG>(p, n_blocks);
+  if (p.a.dim == 128) return launch_resident<HMAX, NT, 8, true, SIG>(p, n_blocks);
+  if (p.a.dim < 64) return launch_resident<HMAX, NT, 4, false, SIG>(p, n_blocks);
+  return launch_resident<HMAX, NT, 8, false, SIG>(p, n_blocks);
 }
 
-template <int VT>
+template <int VT, bool SIG>
 cudaError_t launch_values(const PrefillParams& p, int n_blocks) {
-  auto kern = head_mix_values_kernel<VT>;
+  auto kern = head_mix_values_kernel<VT, SIG>;
   constexpr int smem = 2 * kVTile * (VT * 16 + 8) * 2;
   static bool attr_set = false;
   if (smem > 48 * 1024 && !attr_set) {
@@ -561,10 +641,29 @@ cudaError_t launch_values(const PrefillParams& p, int n_blocks) {
   return launch_kernel(kern, grid, dim3(128), smem, p.a.stream, p.a.pdl, 1, p);
 }
 
+// Both kernels of `n` query blocks.
+template <bool SIG>
+cudaError_t launch_both(const PrefillParams& p, int n, bool resident) {
+  const int H = p.a.n_heads, V = p.a.vdim;
+  cudaError_t e;
+  if (resident && H <= 8) e = launch_resident_dim<8, 2, SIG>(p, n);
+  else if (resident && H <= 16) e = launch_resident_dim<16, 2, SIG>(p, n);
+  else if (resident) e = launch_resident_dim<32, 1, SIG>(p, n);
+  else if (H <= 4) e = launch_scores<4, 4, SIG>(p, n);
+  else if (H <= 8) e = launch_scores<8, 2, SIG>(p, n);
+  else if (H <= 16) e = launch_scores<16, 2, SIG>(p, n);
+  else e = launch_scores<32, 1, SIG>(p, n);
+  if (e != cudaSuccess) return e;
+  if (V <= 32) return launch_values<2, SIG>(p, n);
+  if (V <= 64) return launch_values<4, SIG>(p, n);
+  if (V <= 128) return launch_values<8, SIG>(p, n);
+  return launch_values<16, SIG>(p, n);
+}
+
 }  // namespace
 
-int64_t head_mix_prefill_scratch(int n_heads, int max_keys, int window, int blocks) {
-  return static_cast<int64_t>(blocks) * tiles_for(max_keys, window) * 4 * n_heads * 32 * 16;
+int64_t head_mix_prefill_scratch(int n_heads, int max_keys, int window, int blocks, bool sigmoid) {
+  return static_cast<int64_t>(blocks) * tiles_for(max_keys, window) * 4 * n_heads * 32 * (sigmoid ? 8 : 16);
 }
 
 const char* head_mix_prefill(const HeadMixArgs& a, const int* blk_start, const int* blk_count, int n_blocks, int max_keys,
@@ -580,7 +679,7 @@ const char* head_mix_prefill(const HeadMixArgs& a, const int* blk_start, const i
   p.blk_count = blk_count;
   p.scratch = static_cast<float4*>(scratch);
   p.n_tiles = tiles_for(max_keys, a.window);
-  const int64_t per_block = head_mix_prefill_scratch(a.n_heads, max_keys, a.window, 1);
+  const int64_t per_block = head_mix_prefill_scratch(a.n_heads, max_keys, a.window, 1, a.sigmoid);
   const int fit = static_cast<int>(scratch_bytes / per_block < n_blocks ? scratch_bytes / per_block : n_blocks);
   if (fit < 1) return "head_mix_prefill: the scratch does not hold one query block";
   const int launches = (n_blocks + fit - 1) / fit, at_once = (n_blocks + launches - 1) / launches;   // equal shares
@@ -588,18 +687,7 @@ const char* head_mix_prefill(const HeadMixArgs& a, const int* blk_start, const i
     const int n = n_blocks - p.blk0 < at_once ? n_blocks - p.blk0 : at_once;
     cudaError_t e;
     const bool resident = a.n_heads <= 32 && a.dim <= 128 && a.ldq % 8 == 0 && resident_smem(a.n_heads, 32, a.dim) <= kResidentSmem;
-    if (resident && a.n_heads <= 8) e = launch_resident_dim<8, 2>(p, n);
-    else if (resident && a.n_heads <= 16) e = launch_resident_dim<16, 2>(p, n);
-    else if (resident) e = launch_resident_dim<32, 1>(p, n);
-    else if (a.n_heads <= 4) e = launch_scores<4, 4>(p, n);
-    else if (a.n_heads <= 8) e = launch_scores<8, 2>(p, n);
-    else if (a.n_heads <= 16) e = launch_scores<16, 2>(p, n);
-    else e = launch_scores<32, 1>(p, n);
-    if (e != cudaSuccess) return cudaGetErrorString(e);
-    if (a.vdim <= 32) e = launch_values<2>(p, n);
-    else if (a.vdim <= 64) e = launch_values<4>(p, n);
-    else if (a.vdim <= 128) e = launch_values<8>(p, n);
-    else e = launch_values<16>(p, n);
+    e = a.sigmoid ? launch_both<true>(p, n, resident) : launch_both<false>(p, n, resident);
     if (e != cudaSuccess) return cudaGetErrorString(e);
   }
   return nullptr;

@@ -2,7 +2,7 @@
 // that suit the tensor cores take head_mix_decode.cu, or group_attention.cu for plain scores, instead): the CTA holds ALL heads of its token, because a mixed score needs every head's score of the same key.  Keys are walked in blocks of 32:
 //   scores   eight lanes per (key, kv head): 16-byte loads along the key row, reduced by shuffles, soft-capped
 //   mix      one thread per (head, key): the row of the mixing matrix times the column of scores, bias, mask
-//   softmax  one warp per head, lane = key: running maximum and sum
+//   softmax  one warp per head, lane = key: running maximum and sum (sigmoid weights need none: they are made before the mix)
 //   values   one thread per (head, eight value columns): 16-byte loads along the value row
 // Splits of the key range are merged by a second kernel (fp32 partial outputs with their maximum and sum).
 #include "head_mix.h"
@@ -20,7 +20,7 @@ constexpr int kThreads = 256;
 constexpr int kKeys = 32;
 constexpr int kMaxItems = 8;   // (head, 8 value columns) items per thread and pass
 
-template <typename A, int NI>
+template <typename A, int NI, bool SIG>
 __global__ void __launch_bounds__(kThreads) head_mix_token_kernel(const HeadMixArgs p, int split_keys, int n_splits,
                                                                    float* __restrict__ part_o, float* __restrict__ part_ml) {
   extern __shared__ __align__(16) float smem[];
@@ -93,8 +93,14 @@ __global__ void __launch_bounds__(kThreads) head_mix_token_kernel(const HeadMixA
           d += __shfl_xor_sync(0xffffffffu, d, 2);
           d += __shfl_xor_sync(0xffffffffu, d, 1);
           if (l8 == 0) {
-            d *= p.scale;
-            if (p.softcap > 0.f) d = p.softcap * tanh_of<A>(d * inv_cap);
+            if constexpr (SIG) {
+              const SigmoidHead hd(p, g * R + r, sizeof(A) == 2);
+              const float dist = static_cast<float>(qpos - (k0 + key));
+              d = sizeof(A) == 2 ? hd.weight_fast(d, hd.bias_fast(dist)) : hd.weight(d, dist);
+            } else {
+              d *= p.scale;
+              if (p.softcap > 0.f) d = p.softcap * tanh_of<A>(d * inv_cap);
+            }
             cs[(g * R + r) * kKeys + key] = d;
           }
         }
@@ -112,11 +118,11 @@ __global__ void __launch_bounds__(kThreads) head_mix_token_kernel(const HeadMixA
         s = cs[i];
       }
       if (p.slope != nullptr) s -= p.slope[h] * static_cast<float>(qpos - (k0 + key));
-      ss[i] = (key < nk && pages[key] >= 0) ? s : -CUDART_INF_F;
+      ss[i] = (key < nk && pages[key] >= 0) ? s : (SIG ? 0.f : -CUDART_INF_F);
     }
     __syncthreads();
     // ---- running softmax: warp = head, lane = key ----
-    for (int h = warp; h < H; h += kThreads / 32) {
+    for (int h = warp; !SIG && h < H; h += kThreads / 32) {
       const float s = ss[h * kKeys + lane];
       const float m_old = ms[h];
       const float m_new = fmaxf(m_old, warp_max(s));
@@ -130,16 +136,19 @@ __global__ void __launch_bounds__(kThreads) head_mix_token_kernel(const HeadMixA
         ms[h] = m_new;
       }
     }
-    __syncthreads();
+    if constexpr (!SIG) __syncthreads();
+    const float* wgt = SIG ? ss : cs;
     // ---- values ----
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
       const int it = tid + i * kThreads;
       if (it < items) {
         const int h = it / vecs, c = (it % vecs) * 8, g = h / R;
-        const float cr = corr[h];
+        if constexpr (!SIG) {
+          const float cr = corr[h];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) acc[i][j] *= cr;
+          for (int j = 0; j < 8; ++j) acc[i][j] *= cr;
+        }
         const A* vb = vp + static_cast<long long>(g) * P * V + c;
 #pragma unroll 8
         for (int key = 0; key < nk; ++key) {
@@ -147,7 +156,7 @@ __global__ void __launch_bounds__(kThreads) head_mix_token_kernel(const HeadMixA
           if (row >= 0) {
             float vv[8];
             load8(vb + static_cast<long long>(row) * V, vv);
-            const float w = cs[h * kKeys + key];
+            const float w = wgt[h * kKeys + key];
 #pragma unroll
             for (int j = 0; j < 8; ++j) acc[i][j] = fmaf(w, vv[j], acc[i][j]);
           }
@@ -165,8 +174,8 @@ __global__ void __launch_bounds__(kThreads) head_mix_token_kernel(const HeadMixA
       if (it < items) store8(part_o + base * H * V + it * 8, acc[i]);
     }
     for (int h = tid; h < H; h += kThreads) {
-      part_ml[(base * H + h) * 2] = ms[h];
-      part_ml[(base * H + h) * 2 + 1] = ls[h];
+      part_ml[(base * H + h) * 2] = SIG ? 0.f : ms[h];
+      part_ml[(base * H + h) * 2 + 1] = SIG ? 1.f : ls[h];
     }
     return;
   }
@@ -175,7 +184,7 @@ __global__ void __launch_bounds__(kThreads) head_mix_token_kernel(const HeadMixA
     const int it = tid + i * kThreads;
     if (it < items) {
       const int h = it / vecs;
-      float f = head_mix_finish(ms[h], ls[h], p.sink, p.sinks, h);
+      float f = SIG ? 1.f : head_mix_finish(ms[h], ls[h], p.sink, p.sinks, h);
       if (p.gate != nullptr) f *= sigmoid_of<A>(p.gate[t * p.ld_gate + h]);
 #pragma unroll
       for (int j = 0; j < 8; ++j) acc[i][j] *= f;
@@ -209,7 +218,7 @@ __global__ void __launch_bounds__(128) head_mix_merge_kernel(const HeadMixArgs p
 #pragma unroll
     for (int j = 0; j < 8; ++j) o[j] = fmaf(e, v[j], o[j]);
   }
-  float f = head_mix_finish(m, l, p.sink, p.sinks, h);
+  float f = p.sigmoid ? 1.f : head_mix_finish(m, l, p.sink, p.sinks, h);
   if (p.gate != nullptr) f *= sigmoid_of<A>(p.gate[t * p.ld_gate + h]);
 #pragma unroll
   for (int j = 0; j < 8; ++j) o[j] *= f;
@@ -225,13 +234,13 @@ const char* merge_splits(const HeadMixArgs& a, int n_splits, const float* part_o
   return e == cudaSuccess ? nullptr : cudaGetErrorString(e);
 }
 
-template <typename A, int NI>
+template <typename A, int NI, bool SIG>
 const char* launch_token(const HeadMixArgs& a, int split_keys, int n_splits, float* part_o, float* part_ml) {
   const int H = a.n_heads, Hp = (H + 3) & ~3;
   const size_t smem = sizeof(float) * (static_cast<size_t>(H) * a.dim + static_cast<size_t>(H) * Hp + 2u * H * kKeys + 3u * H) +
                       sizeof(int) * kKeys;
   if (smem > 227 * 1024) return "head_mix attention: the heads of one token do not fit in shared memory";
-  auto kern = head_mix_token_kernel<A, NI>;
+  auto kern = head_mix_token_kernel<A, NI, SIG>;
   static size_t granted = 48 * 1024;
   if (smem > granted) {
     const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
@@ -256,13 +265,13 @@ const char* launch_token(const HeadMixArgs& a, int split_keys, int n_splits, flo
   return nullptr;
 }
 
-template <typename A>
+template <typename A, bool SIG>
 const char* launch_items(const HeadMixArgs& a, int split_keys, int n_splits, float* part_o, float* part_ml) {
   const int per = (a.n_heads * (a.vdim / 8) + kThreads - 1) / kThreads;
-  if (per <= 1) return launch_token<A, 1>(a, split_keys, n_splits, part_o, part_ml);
-  if (per <= 2) return launch_token<A, 2>(a, split_keys, n_splits, part_o, part_ml);
-  if (per <= 4) return launch_token<A, 4>(a, split_keys, n_splits, part_o, part_ml);
-  if (per <= kMaxItems) return launch_token<A, kMaxItems>(a, split_keys, n_splits, part_o, part_ml);
+  if (per <= 1) return launch_token<A, 1, SIG>(a, split_keys, n_splits, part_o, part_ml);
+  if (per <= 2) return launch_token<A, 2, SIG>(a, split_keys, n_splits, part_o, part_ml);
+  if (per <= 4) return launch_token<A, 4, SIG>(a, split_keys, n_splits, part_o, part_ml);
+  if (per <= kMaxItems) return launch_token<A, kMaxItems, SIG>(a, split_keys, n_splits, part_o, part_ml);
   return "head_mix attention: heads x value width above 16384 is not supported";
 }
 
@@ -283,8 +292,11 @@ const char* head_mix_token_attention(const HeadMixArgs& a, int split_keys, int n
     if (const char* err = head_mix_decode(a, split_keys, n_splits, part_o, part_ml)) return err;
     return merge_splits<__nv_bfloat16>(a, n_splits, part_o, part_ml);
   }
-  return a.f32 ? launch_items<float>(a, split_keys, n_splits, part_o, part_ml)
-               : launch_items<__nv_bfloat16>(a, split_keys, n_splits, part_o, part_ml);
+  if (a.sigmoid)
+    return a.f32 ? launch_items<float, true>(a, split_keys, n_splits, part_o, part_ml)
+                 : launch_items<__nv_bfloat16, true>(a, split_keys, n_splits, part_o, part_ml);
+  return a.f32 ? launch_items<float, false>(a, split_keys, n_splits, part_o, part_ml)
+               : launch_items<__nv_bfloat16, false>(a, split_keys, n_splits, part_o, part_ml);
 }
 
 }  // namespace nfb

@@ -1,5 +1,5 @@
-// Per-head RMS norm and rotation of the query and key heads of a fused projection and the append of k / v rows to their cache
-// pages, for layers whose query / key and value widths differ and whose element type is bf16 or fp32.  One warp per
+// Per-head RMS norm and rotation of the query and key heads of a fused projection, the mix of the values with those of an
+// earlier layer, and the append of k / v rows to their cache pages, for layers whose query / key and value widths differ and whose element type is bf16 or fp32.  One warp per
 // (token, head row); values stay in registers between the two passes of the norm.
 #include "head_mix.h"
 
@@ -51,14 +51,27 @@ __global__ void __launch_bounds__(256) qkv_append_kernel(const QkvAppendArgs p) 
     }
   }
   float inv = 1.f;
-  if (w != nullptr) inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(p.dim_true) + p.eps);
+  const bool normed = w != nullptr || (p.unit && kind != 2);
+  if (normed) inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(p.dim_true) + p.eps);
 #pragma unroll
   for (int c = 0; c < kMaxChunks; ++c) {
     const int at = (c * 32 + lane) * 8;
     if (at < width) {
-      if (w != nullptr) {
+      if (normed) {
 #pragma unroll
-        for (int j = 0; j < 8; ++j) v[c][j] = v[c][j] * inv * w[at + j];
+        for (int j = 0; j < 8; ++j) v[c][j] = v[c][j] * inv * (w != nullptr ? w[at + j] : 1.f);
+      }
+      if (kind == 2 && p.v_first != nullptr) {
+        A* first = static_cast<A*>(p.v_first) + t * p.ld_first + r * width + at;
+        if (p.v_lambda == nullptr) {
+          store8(first, v[c]);
+        } else {
+          const float lambda = *p.v_lambda;
+          float u[8];
+          load8(first, u);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) v[c][j] = (1.f - lambda) * v[c][j] + lambda * u[j];
+        }
       }
       if (kind != 2 && at < p.rot) {
 #pragma unroll
@@ -85,7 +98,7 @@ const char* qkv_append(const QkvAppendArgs& a) {
     return "qkv_append: head widths must be multiples of 16 up to 1024";
   if (a.rot < 0 || a.rot % 2 || a.rot > a.dim_true || (a.rot > 0 && a.freq == nullptr)) return "qkv_append: bad rotation";
   const int align = a.f32 ? 4 : 8;
-  if (a.ldp % align || a.ldq % align || a.q_off % 8 || a.k_off % 8 || a.v_off % 8) return "qkv_append: misaligned rows";
+  if (a.ldp % align || a.ldq % align || a.q_off % 8 || a.k_off % 8 || a.v_off % 8 || a.ld_first % 8) return "qkv_append: misaligned rows";
   const long long items = static_cast<long long>(a.T) * (a.n_heads + 2 * a.n_kv);
   const dim3 grid(static_cast<unsigned>((items + 7) / 8));
   const cudaError_t e = a.f32 ? launch_kernel(qkv_append_kernel<float>, grid, dim3(256), 0, a.stream, a.pdl, 1, a)

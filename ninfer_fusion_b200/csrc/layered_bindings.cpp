@@ -8,7 +8,7 @@ namespace {
 
 using namespace nfb_bind;
 
-void embed_rows32(const Tensor& ids, const Tensor& table, const Tensor& x32, const Tensor& xa, double scale, bool pdl) {
+void embed_rows32(const Tensor& ids, const Tensor& table, const Tensor& x32, const Tensor& xa, double scale, bool pdl, OptT pos, OptT places) {
   const bool f32 = act_f32(table, "table");
   const int64_t T = ids.numel(), N = table.size(1);
   need_vec(ids, at::kInt, T, "ids");
@@ -16,10 +16,18 @@ void embed_rows32(const Tensor& ids, const Tensor& table, const Tensor& x32, con
   need_vec(x32, at::kFloat, T * N, "x32");
   need(xa, table.scalar_type(), "xa"); need_rows(xa, "xa");
   TORCH_CHECK(xa.size(0) == T && xa.size(1) == N, "embed_rows32: xa shape");
+  const void* at = nullptr;
+  int64_t n_places = 0;
+  if (places.has_value() && places->defined()) {
+    TORCH_CHECK(pos.has_value() && pos->defined() && places->dim() == 2 && places->size(1) == N, "embed_rows32: position table");
+    n_places = places->size(0);
+    need_vec(*places, table.scalar_type(), n_places * N, "places"); need_vec(*pos, at::kInt, T, "pos");
+    at = places->data_ptr();
+  }
   c10::cuda::CUDAGuard guard(table.device());
   chk(nfb::embed_rows32(static_cast<const int*>(ids.data_ptr()), table.data_ptr(), static_cast<float*>(x32.data_ptr()),
                         xa.data_ptr(), static_cast<int>(T), static_cast<int>(N), xa.stride(0), static_cast<float>(scale),
-                        static_cast<int>(table.size(0)), f32,
+                        static_cast<int>(table.size(0)), ptr_or_null<const int>(pos), at, static_cast<int>(n_places), f32,
                         cur_stream(), pdl));
 }
 
@@ -115,7 +123,7 @@ void sandwich_rows(const Tensor& x_in, const Tensor& x_out, OptT delta, OptT w_p
 }  // namespace
 
 TORCH_LIBRARY_FRAGMENT(nfb200, m) {
-  m.def("embed_rows32(Tensor ids, Tensor table, Tensor x32, Tensor xa, float scale, bool pdl) -> ()", &embed_rows32);
+  m.def("embed_rows32(Tensor ids, Tensor table, Tensor x32, Tensor xa, float scale, bool pdl, Tensor? pos=None, Tensor? places=None) -> ()", &embed_rows32);
   m.def("post_norm_rows(Tensor x32, Tensor? delta, Tensor xa, int n_true, float alpha, float eps, Tensor? gain, Tensor? final_gain, bool pdl) -> ()", &post_norm_rows);
   m.def("gemm_f32(Tensor x, Tensor w, Tensor? out, Tensor? bias, int act=0, Tensor? act_params=None, Tensor? out32=None, int out32_from=0) -> ()", &gemm_f32);
   m.def("sandwich_rows(Tensor x_in, Tensor x_out, Tensor? delta, Tensor? w_post, Tensor? w_next, Tensor out, int n_true, int groups, float mult, float eps, Tensor? conv_w, Tensor? conv_state, Tensor? cu_seqlens, Tensor? state_slot, int max_seq_tokens, bool write_state, bool pdl) -> ()", &sandwich_rows);

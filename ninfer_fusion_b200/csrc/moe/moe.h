@@ -56,14 +56,18 @@ struct MoeRouteParams {
 };
 const char* moe_route(const MoeRouteParams& p, cudaStream_t stream);
 
-// Routing by corrected scores (one GPU): s = softmax over all E + identity outputs; the k largest s + correction are chosen
-// (ties: lower number); weight = scale * s, not renormalised.  Choices >= E are identity experts: they get no row (pos = -1).
+// Routing by corrected scores (one GPU): s = softmax over all E + identity outputs, or the sigmoid of each; the k largest
+// s + correction are chosen (ties: lower number); weight = scale * s, or scale * s / (sum of the chosen s + 1e-20).  With
+// groups (equal runs of neighbours) only those of the `keep` best groups can be chosen; a group's score is the sum of its two
+// largest corrected scores.  Choices >= E are identity experts: they get no row (pos = -1).
 struct MoeRouteScoredParams {
   int T, E, identity, k;
   const float* logits;      // [T, ld] fp32
   long long ld;
   const float* correction;  // [E + identity], or null
   float scale;
+  int sigmoid, renormalise; // flags
+  int groups, keep;         // 0 or 1 group: all outputs can be chosen
   int* hist;                // [E], zero on entry
   int* ids;                 // [T, k]
   float* weights;           // [T, k]

@@ -29,7 +29,8 @@ void moe_route(const Tensor& logits, int64_t E, int64_t k, bool norm_topk, bool 
 }
 
 void moe_route_scored(const Tensor& logits, int64_t E, int64_t identity, int64_t k, OptT correction, double scale, const Tensor& hist,
-                      const Tensor& ids, const Tensor& weights, const Tensor& pos, bool pdl) {
+                      const Tensor& ids, const Tensor& weights, const Tensor& pos, bool pdl, bool sigmoid, bool renormalise, int64_t groups,
+                      int64_t keep) {
   need(logits, at::kFloat, "logits"); need(hist, at::kInt, "hist"); need(ids, at::kInt, "ids");
   need(weights, at::kFloat, "weights"); need(pos, at::kInt, "pos");
   const int64_t T = logits.size(0);
@@ -44,6 +45,9 @@ void moe_route_scored(const Tensor& logits, int64_t E, int64_t identity, int64_t
   }
   p.T = static_cast<int>(T); p.E = static_cast<int>(E); p.identity = static_cast<int>(identity); p.k = static_cast<int>(k);
   p.logits = static_cast<const float*>(logits.data_ptr()); p.ld = logits.stride(0); p.scale = static_cast<float>(scale);
+  TORCH_CHECK(groups <= 1 || ((E + identity) % groups == 0 && keep >= 1 && keep <= groups && (E + identity) / groups * keep >= k),
+              "moe_route_scored: groups must be equal and the kept ones hold the choices");
+  p.sigmoid = sigmoid ? 1 : 0; p.renormalise = renormalise ? 1 : 0; p.groups = static_cast<int>(groups); p.keep = static_cast<int>(keep);
   p.hist = static_cast<int*>(hist.data_ptr()); p.ids = static_cast<int*>(ids.data_ptr());
   p.weights = static_cast<float*>(weights.data_ptr()); p.pos = static_cast<int*>(pos.data_ptr());
   c10::cuda::CUDAGuard guard(logits.device());
@@ -194,7 +198,7 @@ TORCH_LIBRARY_FRAGMENT(nfb200, m) {
   m.def("moe_plan(int world, int rank, int E, int tile_tokens, int cap, Tensor hist, int[] peer_bases, int counts_off, int count_flag_off, Tensor send_base, Tensor tiles, Tensor state, Tensor? status) -> ()", &moe_plan);
   m.def("moe_push(int world, int rank, int E, int cap, Tensor x, Tensor ids, Tensor pos, Tensor send_base, int[] peer_bases, int recv_x_off, int recv_meta_off, int arrive_flag_off, Tensor state, Tensor? status) -> ()", &moe_push);
   m.def("moe_gemm(Tensor x, Tensor w, int epi, int tile_tokens, int max_tiles, Tensor tiles, Tensor state, Tensor? out, int world, Tensor? recv_meta, int[] peer_bases, int ret_off, int ret_flag_off, Tensor? status, float[] glu=[]) -> ()", &moe_gemm);
-  m.def("moe_route_scored(Tensor logits, int E, int identity, int k, Tensor? correction, float scale, Tensor hist, Tensor ids, Tensor weights, Tensor pos, bool pdl) -> ()", &moe_route_scored);
+  m.def("moe_route_scored(Tensor logits, int E, int identity, int k, Tensor? correction, float scale, Tensor hist, Tensor ids, Tensor weights, Tensor pos, bool pdl, bool sigmoid=False, bool renormalise=False, int groups=0, int keep=0) -> ()", &moe_route_scored);
   m.def("moe_combine(Tensor x, Tensor weights, Tensor ret, int my_base, int ret_flag_off, Tensor? shared, Tensor? shared_gate, Tensor? norm_w, Tensor? normed, float eps, Tensor state, Tensor? status) -> ()", &moe_combine);
   m.def("moe_state_bytes() -> int", &moe_state_bytes);
   m.def("moe_tile_tokens(float rows_per_expert) -> int", &moe_tile_tokens);

@@ -77,6 +77,7 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(const MoeRo
 // moe_route_scored: one warp per token
 // ---------------------------------------------------------------------------------------------
 __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_scored_kernel(const MoeRouteScoredParams p) {
+  __shared__ float group_s[kRouteWarps][kMoeMaxExperts];
   pdl_launch_next();
   pdl_wait_prior();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -84,21 +85,26 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_scored_kernel(cons
   if (t >= p.T) return;
   const int n = p.E + p.identity;
   const float* row = p.logits + static_cast<long long>(t) * p.ld;
-  float s[kPerLane], top = -INFINITY, sum = 0.f;
+  float s[kPerLane], top = -INFINITY, sum = 0.f, inv = 1.f;
 #pragma unroll
   for (int i = 0; i < kPerLane; ++i) {
     const int e = lane + 32 * i;
     s[i] = e < n ? row[e] : -INFINITY;
     top = fmaxf(top, s[i]);
   }
+  if (p.sigmoid) {
 #pragma unroll
-  for (int o = 16; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
+    for (int i = 0; i < kPerLane; ++i) s[i] = 1.f / (1.f + expf(-s[i]));
+  } else {
 #pragma unroll
-  for (int i = 0; i < kPerLane; ++i) {
-    s[i] = lane + 32 * i < n ? expf(s[i] - top) : 0.f;
-    sum += s[i];
+    for (int o = 16; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
+#pragma unroll
+    for (int i = 0; i < kPerLane; ++i) {
+      s[i] = lane + 32 * i < n ? expf(s[i] - top) : 0.f;
+      sum += s[i];
+    }
+    inv = 1.f / warp_sum(sum);
   }
-  const float inv = 1.f / warp_sum(sum);
   float c[kPerLane];                               // choice scores
 #pragma unroll
   for (int i = 0; i < kPerLane; ++i) {
@@ -106,6 +112,41 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_scored_kernel(cons
     s[i] *= inv;
     c[i] = e < n ? s[i] + (p.correction != nullptr ? p.correction[e] : 0.f) : -INFINITY;
   }
+  if (p.groups > 1) {
+    const int size = n / p.groups;
+    float* score = group_s[warp];
+    for (int g = 0; g < p.groups; ++g) {
+      float a = -INFINITY, b = -INFINITY;          // the two largest of the group
+#pragma unroll
+      for (int i = 0; i < kPerLane; ++i) {
+        const int e = lane + 32 * i;
+        if (e >= g * size && e < (g + 1) * size) {
+          b = fmaxf(b, fminf(a, c[i]));
+          a = fmaxf(a, c[i]);
+        }
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float oa = __shfl_xor_sync(0xffffffffu, a, o), ob = __shfl_xor_sync(0xffffffffu, b, o);
+        b = fmaxf(fmaxf(b, ob), fminf(a, oa));
+        a = fmaxf(a, oa);
+      }
+      if (lane == 0) score[g] = size > 1 ? a + b : a;
+    }
+    __syncwarp();
+#pragma unroll
+    for (int i = 0; i < kPerLane; ++i) {
+      const int e = lane + 32 * i;
+      if (e < n) {
+        const int g = e / size;
+        const float mine = score[g];
+        int better = 0;
+        for (int o = 0; o < p.groups; ++o) better += score[o] > mine || (score[o] == mine && o < g) ? 1 : 0;
+        if (better >= p.keep) c[i] = -INFINITY;
+      }
+    }
+  }
+  float chosen = 0.f;
   for (int r = 0; r < p.k; ++r) {
     float bv = -INFINITY, bs = 0.f;
     int bi = 0x7fffffff;
@@ -130,6 +171,11 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_scored_kernel(cons
       p.weights[a] = bs * p.scale;
       p.pos[a] = bi < p.E ? atomicAdd(p.hist + bi, 1) : -1;
     }
+    chosen += bs;
+  }
+  if (p.renormalise) {
+    __syncwarp();
+    for (int r = lane; r < p.k; r += 32) p.weights[t * p.k + r] /= chosen + 1e-20f;
   }
 }
 

@@ -25,18 +25,26 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 template <typename A>
 __global__ void __launch_bounds__(256) embed_rows32_kernel(const int* __restrict__ ids, const A* __restrict__ table,
                                                             float* __restrict__ x32, A* __restrict__ xa, int N, long long ld_xa,
-                                                            float scale, int vocab) {
+                                                            float scale, int vocab, const int* __restrict__ pos,
+                                                            const A* __restrict__ places, int n_places) {
   pdl_launch_next();
   pdl_wait_prior();
   const long long row = blockIdx.x;
   int id = ids[row];
   id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
   const A* src = table + static_cast<long long>(id) * N;
+  const A* place = places == nullptr ? nullptr : places + static_cast<long long>(min(max(pos[row], 0), n_places - 1)) * N;
   for (int c = threadIdx.x * 8; c < N; c += blockDim.x * 8) {
     float v[8];
     load8(src + c, v);
 #pragma unroll
     for (int j = 0; j < 8; ++j) v[j] *= scale;
+    if (place != nullptr) {
+      float u[8];
+      load8(place + c, u);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[j] += u[j];
+    }
     store8(x32 + row * N + c, v);
     store8(xa + row * ld_xa + c, v);
   }
@@ -100,14 +108,17 @@ __global__ void __launch_bounds__(1024) post_norm_kernel(const PostNormArgs p) {
 }  // namespace
 
 const char* embed_rows32(const int* ids, const void* table, float* x32, void* xa, int T, int N, int64_t ld_xa, float scale,
-                         int vocab, bool f32, cudaStream_t stream, bool pdl) {
+                         int vocab, const int* pos, const void* places, int n_places, bool f32, cudaStream_t stream, bool pdl) {
   if (T <= 0) return nullptr;
+  if (places != nullptr && (pos == nullptr || n_places < 1)) return "embed_rows32: a position table needs the positions";
   if (N % 8 || ld_xa % 8) return "embed_rows32: row widths must be multiples of 8";
   const long long ld = ld_xa;
   cudaError_t e = f32 ? launch_kernel(embed_rows32_kernel<float>, dim3(T), dim3(256), 0, stream, pdl, 1, ids,
-                                      static_cast<const float*>(table), x32, static_cast<float*>(xa), N, ld, scale, vocab)
+                                      static_cast<const float*>(table), x32, static_cast<float*>(xa), N, ld, scale, vocab, pos,
+                                      static_cast<const float*>(places), n_places)
                       : launch_kernel(embed_rows32_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, stream, pdl, 1, ids,
-                                      static_cast<const __nv_bfloat16*>(table), x32, static_cast<__nv_bfloat16*>(xa), N, ld, scale, vocab);
+                                      static_cast<const __nv_bfloat16*>(table), x32, static_cast<__nv_bfloat16*>(xa), N, ld, scale, vocab,
+                                      pos, static_cast<const __nv_bfloat16*>(places), n_places);
   return e == cudaSuccess ? nullptr : cudaGetErrorString(e);
 }
 

@@ -5,10 +5,10 @@
 
 namespace nfb {
 
-// x32[t] = scale * table[ids[t]] in fp32, xa[t] = the same in the activation type (leading dimension ld_xa); rows of N
-// values (N % 8 == 0).  f32: table and xa are fp32.
+// x32[t] = scale * table[ids[t]] + places[pos[t]] in fp32 (places null: without it), xa[t] = the same in the activation type
+// (leading dimension ld_xa); rows of N values (N % 8 == 0).  f32: the tables and xa are fp32.  pos must be below n_places.
 const char* embed_rows32(const int* ids, const void* table, float* x32, void* xa, int T, int N, int64_t ld_xa, float scale,
-                         int vocab, bool f32, cudaStream_t stream, bool pdl);
+                         int vocab, const int* pos, const void* places, int n_places, bool f32, cudaStream_t stream, bool pdl);
 
 struct PostNormArgs {
   float* x32;            // [T, N] residual stream, updated in place

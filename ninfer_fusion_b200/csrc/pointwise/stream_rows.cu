@@ -3,53 +3,13 @@
 // streams of a thread's columns stay in registers, so every stream is read and written once.
 #include "stream_rows.h"
 
-#include "../common/elem.cuh"
 #include "../common/glu.cuh"
 #include "../common/launch.h"
+#include "mixture.cuh"
 
 namespace nfb {
 
 namespace {
-
-__device__ __forceinline__ void load4(const float* p, float* v) {
-  const float4 a = *reinterpret_cast<const float4*>(p);
-  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
-}
-__device__ __forceinline__ void load4(const __nv_bfloat16* p, float* v) {
-  const uint2 r = *reinterpret_cast<const uint2*>(p);
-  v[0] = __uint_as_float(r.x << 16); v[1] = __uint_as_float(r.x & 0xffff0000u);
-  v[2] = __uint_as_float(r.y << 16); v[3] = __uint_as_float(r.y & 0xffff0000u);
-}
-__device__ __forceinline__ void store4(float* p, const float* v) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
-__device__ __forceinline__ void store4(__nv_bfloat16* p, const float* v) {
-  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
-}
-
-// y[t, c .. c + 3]; `g` is the shared expert's factor
-template <typename A>
-__device__ __forceinline__ void mixture4(const MixtureParts& p, long long t, int c, int N, float g, float* y) {
-  y[0] = y[1] = y[2] = y[3] = 0.f;
-  if (p.delta != nullptr) {
-    load4(p.delta + t * N + c, y);
-    if (p.gate != nullptr) {
-#pragma unroll
-      for (int e = 0; e < 4; ++e) y[e] *= g;
-    }
-  }
-  if (p.choice == nullptr) return;
-#pragma unroll 4
-  for (int j = 0; j < p.k; ++j) {
-    const int id = p.choice[t * p.k + j];
-    const float w = p.weight[t * p.k + j];
-    float v[4];
-    load4(id < p.n_experts ? static_cast<const A*>(p.ret) + (t * p.k + j) * N + c : static_cast<const A*>(p.h) + t * p.ld_h + c, v);
-#pragma unroll
-    for (int e = 0; e < 4; ++e) y[e] = fmaf(w, v[e], y[e]);
-  }
-}
-__device__ __forceinline__ float mixture_gate(const MixtureParts& p, long long t) {
-  return p.gate == nullptr ? 1.f : 1.f / (1.f + expf(-p.gate[t * p.ld_gate]));
-}
 
 // KV: four-column pieces per thread, SM: upper bound of the streams.
 template <typename A, int KV, int SM>
@@ -193,12 +153,6 @@ cudaError_t pick_streams(const StreamArgs& a, cudaStream_t stream, bool pdl) {
   return pick_width<A, kMaxStreams>(a, stream, pdl);
 }
 
-const char* bad_parts(const MixtureParts& y) {
-  if (y.choice != nullptr && (y.weight == nullptr || y.k < 1 || (y.n_experts > 0 && y.ret == nullptr) || y.h == nullptr || y.ld_h % 8))
-    return "expert sum: missing or misaligned parts";
-  return nullptr;
-}
-
 }  // namespace
 
 const char* stream_rows(const StreamArgs& a, cudaStream_t stream, bool pdl) {
@@ -209,7 +163,7 @@ const char* stream_rows(const StreamArgs& a, cudaStream_t stream, bool pdl) {
   if (a.x_in == nullptr && (a.ids == nullptr || a.table == nullptr || a.vocab < 1)) return "stream_rows: neither streams nor an embedding table";
   if (a.mix != nullptr && a.w_out == nullptr) return "stream_rows: an update needs both of its weights";
   if (a.mix != nullptr && a.y.delta == nullptr && a.y.choice == nullptr) return "stream_rows: an update needs a sublayer's output";
-  if (const char* err = bad_parts(a.y)) return err;
+  if (const char* err = bad_mixture(a.y)) return err;
   const cudaError_t e = a.f32 ? pick_streams<float>(a, stream, pdl) : pick_streams<__nv_bfloat16>(a, stream, pdl);
   return e == cudaSuccess ? nullptr : cudaGetErrorString(e);
 }
@@ -217,7 +171,7 @@ const char* stream_rows(const StreamArgs& a, cudaStream_t stream, bool pdl) {
 const char* mixture_rows(const MixtureParts& y, float* out, int T, int N, bool f32, cudaStream_t stream, bool pdl) {
   if (T <= 0) return nullptr;
   if (N % 8 || out == nullptr) return "mixture_rows: bad row width";
-  if (const char* err = bad_parts(y)) return err;
+  if (const char* err = bad_mixture(y)) return err;
   const cudaError_t e = f32 ? launch_kernel(mixture_rows_kernel<float>, dim3(T), dim3(256), 0, stream, pdl, 1, y, out, N)
                             : launch_kernel(mixture_rows_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, stream, pdl, 1, y, out, N);
   return e == cudaSuccess ? nullptr : cudaGetErrorString(e);

@@ -1,36 +1,10 @@
 // torch.ops.nfb200.*: row steps of decoders with several residual streams, and sums over experts (layer-list decoders,
 // models/layered.py).  Activations are bf16 or fp32; every op takes its element type from its tensors.
-#include "binding_util.h"
-#include "pointwise/stream_rows.h"
+#include "pointwise/mixture_args.h"
 
 namespace {
 
 using namespace nfb_bind;
-
-nfb::MixtureParts parts(int64_t T, int64_t N, at::ScalarType act, OptT delta, OptT gate, OptT choice, OptT weight, OptT ret, OptT h,
-                        int64_t n_experts) {
-  nfb::MixtureParts y;
-  if (delta.has_value() && delta->defined()) {
-    need_vec(*delta, at::kFloat, T * N, "delta");
-    y.delta = static_cast<const float*>(delta->data_ptr());
-  }
-  if (gate.has_value() && gate->defined()) {
-    need(*gate, at::kFloat, "gate"); need_rows(*gate, "gate");
-    TORCH_CHECK(gate->size(0) >= T && gate->size(1) >= 1, "gate shape");
-    y.gate = static_cast<const float*>(gate->data_ptr()); y.ld_gate = gate->stride(0);
-  }
-  if (choice.has_value() && choice->defined()) {
-    TORCH_CHECK(choice->dim() == 2 && weight.has_value() && ret.has_value() && h.has_value(), "expert sum: choices need weights, rows and the input");
-    const int64_t k = choice->size(1);
-    need_vec(*choice, at::kInt, T * k, "choice"); need_vec(*weight, at::kFloat, T * k, "weight"); need_vec(*ret, act, T * k * N, "ret");
-    need(*h, act, "h"); need_rows(*h, "h");
-    TORCH_CHECK(h->size(0) >= T && h->size(1) >= N, "h shape");
-    y.choice = static_cast<const int*>(choice->data_ptr()); y.weight = static_cast<const float*>(weight->data_ptr());
-    y.ret = ret->data_ptr(); y.h = h->data_ptr(); y.ld_h = h->stride(0);
-    y.k = static_cast<int>(k); y.n_experts = static_cast<int>(n_experts);
-  }
-  return y;
-}
 
 // x_in: [T, S, N], or null with ids and the embedding table
 void stream_rows(OptT x_in, OptT ids, OptT table, OptT x_out, OptT delta, OptT gate, OptT choice, OptT weight, OptT ret, OptT h,
@@ -54,7 +28,7 @@ void stream_rows(OptT x_in, OptT ids, OptT table, OptT x_out, OptT delta, OptT g
     need_vec(*x_out, at::kFloat, T * S * N, "x_out");
     a.x_out = static_cast<float*>(x_out->data_ptr());
   }
-  a.y = parts(T, N, out.scalar_type(), delta, gate, choice, weight, ret, h, n_experts);
+  a.y = mixture_parts(T, N, out.scalar_type(), delta, gate, choice, weight, ret, h, n_experts);
   if (mix.has_value() && mix->defined()) {
     TORCH_CHECK(w_out.has_value(), "stream_rows: w_out");
     need_vec(*mix, at::kFloat, S * S, "mix"); need_vec(*w_out, at::kFloat, S, "w_out");
@@ -74,7 +48,7 @@ void mixture_rows(OptT delta, OptT gate, const Tensor& choice, const Tensor& wei
   const int64_t T = out.size(0), N = out.size(1);
   need_vec(out, at::kFloat, T * N, "out");
   const bool f32 = act_f32(h, "h");
-  const nfb::MixtureParts y = parts(T, N, h.scalar_type(), delta, gate, choice, weight, ret, h, n_experts);
+  const nfb::MixtureParts y = mixture_parts(T, N, h.scalar_type(), delta, gate, choice, weight, ret, h, n_experts);
   c10::cuda::CUDAGuard guard(out.device());
   chk(nfb::mixture_rows(y, static_cast<float*>(out.data_ptr()), static_cast<int>(T), static_cast<int>(N), f32, cur_stream(), pdl));
 }

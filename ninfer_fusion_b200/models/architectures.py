@@ -8,10 +8,10 @@ import json
 import os
 from typing import Dict
 
-from . import kuzanex, tebivik, tuzupel
+from . import kuzanex, ratilorn, tebivik, tuzupel
 from .layered_config import LayeredConfig
 
-DESIGNS = {m.ARCHITECTURE: m for m in (kuzanex, tebivik, tuzupel)}
+DESIGNS = {m.ARCHITECTURE: m for m in (kuzanex, tebivik, tuzupel, ratilorn)}
 LAYERED_REGISTRY: Dict[str, LayeredConfig] = {name: c for m in DESIGNS.values() for name, c in m.CONFIGS.items()}
 
 

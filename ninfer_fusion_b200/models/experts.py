@@ -1,11 +1,11 @@
 """Mixture-of-experts feed-forward of the layer-list decoders (`models/layered_config.ExpertMlp`) on one GPU: packing, buffers
 and the launch sequence on the kernels of `csrc/moe`.
 
-    router GEMM (fp32 logits) -> scored routing -> plan (tile table) -> push (rows sorted by expert) -> grouped GEMM with the
+    router GEMM (fp32 logits) -> scored routing (softmax or sigmoid, in groups or not) -> plan (tile table) -> push (rows sorted by expert) -> grouped GEMM with the
     bounded gated unit -> grouped GEMM whose epilogue puts every row in its token's place; the shared expert is a dense pair
     of GEMMs
 
-The sum over a token's experts is left to the row step that follows (`csrc/pointwise/stream_rows.h` MixtureParts): identity
+The sum over a token's experts is left to the row step that follows (`MixtureParts` of `csrc/pointwise/stream_rows.h`): identity
 experts only have a weight there.  In 32-bit runs the same tables feed an fp32 grouped GEMM."""
 from __future__ import annotations
 
@@ -26,19 +26,20 @@ def _pad(w: torch.Tensor, rows: int, cols: int, dtype) -> torch.Tensor:
     return out
 
 
-def _unit(get, name: str, u: GatedUnit, hp: int, dtype):
+def pack_unit(get, prefix: str, u: GatedUnit, hp: int, dtype):
     """[gate; up] and down of one unit, the unit's width padded: zero gate and up rows give zero, whatever the shift."""
-    up = torch.cat([_pad(get(f"{name}.gate"), u.ff_p, hp, dtype), _pad(get(f"{name}.up"), u.ff_p, hp, dtype)])
-    return up, _pad(get(f"{name}.down"), hp, u.ff_p, dtype)
+    up = torch.cat([_pad(get(f"{prefix}gate"), u.ff_p, hp, dtype), _pad(get(f"{prefix}up"), u.ff_p, hp, dtype)])
+    return up, _pad(get(f"{prefix}down"), hp, u.ff_p, dtype)
 
 
 def pack_experts(w: Dict[str, torch.Tensor], p: str, m: ExpertMlp, get, hp: int, dtype) -> None:
-    units = [_unit(get, f"e{e}", m.expert, hp, dtype) for e in range(m.experts)]
+    units = [pack_unit(get, f"e{e}.", m.expert, hp, dtype) for e in range(m.experts)]
     w[f"{p}/mlp/up"], w[f"{p}/mlp/down"] = torch.stack([u for u, _ in units]), torch.stack([d for _, d in units])
     router = [get("router")]
     if m.shared is not None:
-        w[f"{p}/mlp/shared_up"], w[f"{p}/mlp/shared_down"] = _unit(get, "shared", m.shared, hp, dtype)
-        router.append(get("shared_gate"))
+        w[f"{p}/mlp/shared_up"], w[f"{p}/mlp/shared_down"] = pack_unit(get, "shared.", m.shared, hp, dtype)
+        if m.shared_gate:
+            router.append(get("shared_gate"))
     w[f"{p}/mlp/router"] = _pad(torch.cat(router), m.router_cols, hp, dtype)
     w[f"{p}/mlp/correction"] = get("correction").float().contiguous()
 
@@ -76,12 +77,24 @@ class ExpertWorkspace:
         shared = max([m.shared.ff_p for m in specs if m.shared is not None], default=0)
         self.act = torch.zeros(rows * wide, dtype=dtype, device=dev)
         self.shared_act = torch.zeros(T * shared, dtype=dtype, device=dev)
-        if self.f32:           # [gate | up] columns before the unit
-            self.wide, self.shared_wide = (torch.zeros(2 * t.numel(), dtype=dtype, device=dev) for t in (self.act, self.shared_act))
+        # [gate | up] columns before the unit (32-bit runs)
+        self.wide, self.shared_wide = (torch.zeros(2 * t.numel() if self.f32 else 0, dtype=dtype, device=dev) for t in (self.act, self.shared_act))
 
 
 def glu(u: GatedUnit):
     return [u.limit, u.slope, u.shift]
+
+
+def run_unit(model, T: int, u: GatedUnit, up, down, x: torch.Tensor, act: torch.Tensor, wide, out: torch.Tensor, prefetch=None) -> None:
+    """out [T, hp] fp32 <- the unit of x [T, hp].  `act` and (32-bit runs) `wide` are flat buffers."""
+    h = act[: T * u.ff_p].view(T, u.ff_p)
+    if model.f32:
+        both = wide[: 2 * T * u.ff_p].view(T, 2 * u.ff_p)
+        model._gemm(x, up, None, both)
+        model.ops.glu_rows_f32(both, h, *glu(u), model.pdl)
+    else:
+        model._gemm(x, up, None, h, epi=EPI_SWIGLU, glu=glu(u), prefetch=down)
+    model._gemm(h, down, None, out32=out, prefetch=prefetch)
 
 
 def run_experts(model, ws: ExpertWorkspace, T: int, p: str, m: ExpertMlp, x: torch.Tensor, delta: torch.Tensor, prefetch=None) -> dict:
@@ -93,7 +106,8 @@ def run_experts(model, ws: ExpertWorkspace, T: int, p: str, m: ExpertMlp, x: tor
     model._gemm(x, w[f"{p}/mlp/router"], None, out32=logits, prefetch=w[f"{p}/mlp/up"])
     n, rows = T * k, T * m.slots
     ids, pos, weights = ws.ids[:n].view(T, k), ws.pos[:n].view(T, k), ws.weights[:n].view(T, k)
-    ops.moe_route_scored(logits, E, m.identity, k, w[f"{p}/mlp/correction"], m.scale, ws.hist, ids, weights, pos, model.pdl)
+    ops.moe_route_scored(logits, E, m.identity, k, w[f"{p}/mlp/correction"], m.scale, ws.hist, ids, weights, pos, model.pdl, m.sigmoid,
+                         m.renormalise, m.groups, m.keep)
     tile = F32_TILE if ws.f32 else int(model._raw_ops.moe_tile_tokens(T * k / m.choices))
     n_tiles = min(ws.n_tiles, E + (rows + tile - 1) // tile)
     ops.moe_plan(1, 0, E, tile, rows, ws.hist, ws.base, ws.off["counts"], ws.off["count_flag"], ws.send, ws.tiles, ws.state, status)
@@ -112,14 +126,6 @@ def run_experts(model, ws: ExpertWorkspace, T: int, p: str, m: ExpertMlp, x: tor
     ops.moe_gemm(act, down, RETURN, tile, n_tiles, ws.tiles, ws.state, None, 1, ws.meta, *back)
     parts = dict(delta=None, gate=None, choice=ids, weight=weights, ret=ws.ret[: n * hp].view(n, hp), h=x, n_experts=E)
     if m.shared is not None:
-        sf = m.shared.ff_p
-        sact = ws.shared_act[: T * sf].view(T, sf)
-        if ws.f32:
-            wide = ws.shared_wide[: 2 * T * sf].view(T, 2 * sf)
-            model._gemm(x, w[f"{p}/mlp/shared_up"], None, wide)
-            ops.glu_rows_f32(wide, sact, *glu(m.shared), model.pdl)
-        else:
-            model._gemm(x, w[f"{p}/mlp/shared_up"], None, sact, epi=EPI_SWIGLU, glu=glu(m.shared), prefetch=w[f"{p}/mlp/shared_down"])
-        model._gemm(sact, w[f"{p}/mlp/shared_down"], None, out32=delta, prefetch=prefetch)
-        parts.update(delta=delta, gate=logits[:, m.choices: m.choices + 1])
+        run_unit(model, T, m.shared, w[f"{p}/mlp/shared_up"], w[f"{p}/mlp/shared_down"], x, ws.shared_act, ws.shared_wide, delta, prefetch)
+        parts.update(delta=delta, gate=logits[:, m.choices: m.choices + 1] if m.shared_gate else None)
     return parts

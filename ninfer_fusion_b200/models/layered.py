@@ -1,13 +1,14 @@
 """Decoders described as a list of layers (`models/layered_config.py`): weight packing and the forward pass on the
 native kernels.
 
-A layer is a mixer (attention with plain or head-mixed scores, latent attention, matrix memory, gated linear memory or gated
-linear recurrence) and an optional feed-forward (dense, or experts: `models/experts.py`) on a 32-bit residual stream.  A
-sublayer meets the stream in one of three ways: the norm after the sum, ``x <- rms_norm(alpha x + f(x)) * gain``, norms
-around it, ``x <- x + mult * norm(f(norm(x)))``, with an optional causal convolution in front of every mixer, or several
-streams that it reads a weighted sum of and mixes.  Layers can run several times with the same weights; cache and state
+A layer is a mixer (attention with plain or head-mixed scores or sigmoid weights, latent attention, matrix memory, gated
+linear memory, gated linear recurrence, a selective state space, or attention and a state space side by side) and an
+optional feed-forward (dense, or experts: `models/experts.py`) on a 32-bit residual stream.  A sublayer meets the stream in
+one of four ways: the norm after the sum, ``x <- rms_norm(alpha x + f(x)) * gain``, norms around it,
+``x <- x + mult * norm(f(norm(x)))``, with an optional causal convolution in front of every mixer, several streams that it
+reads a weighted sum of and mixes, or a norm on its output only, ``x <- x + norm(f(x))``.  Layers can run several times with the same weights; cache and state
 belong to layer runs.  Every size and constant is a field of the description, so a design is a mapping onto these fields
-(`models/kuzanex.py`, `models/tebivik.py`, `models/tuzupel.py`) and not a model file of its own.
+(`models/kuzanex.py`, `models/tebivik.py`, `models/tuzupel.py`, `models/ratilorn.py`) and not a model file of its own.
 
 The engine side is the hybrid runtime's: one ragged token batch per step (`runtime/batch.py`), K / V or latent rows in the
 paged cache (one geometry per run), recurrent state in per-sequence slots, preallocated buffers so that a decode step can
@@ -22,10 +23,10 @@ from typing import Dict, List, Tuple
 import torch
 
 from .._lib import StatusWord, load_native
-from .experts import ExpertWorkspace, pack_experts, run_experts
+from .experts import ExpertWorkspace, pack_experts, pack_unit, run_experts, run_unit
 from .hybrid import EPI_STORE, LaunchCounter, StepBatch
 from .layered_config import (ATTENTION_KINDS, AttentionMixer, GatedMemoryMixer, GatedRecurrenceMixer, LatentAttentionMixer,
-                             LayeredConfig, MatrixMemoryMixer, pad_to)
+                             LayeredConfig, MatrixMemoryMixer, ParallelMixer, StateSpaceMixer, mixer_parts, pad_to)
 
 ACTIVATIONS = {"xielu": 3, "relu2": 4}     # csrc/gemm/gemm.h GemmActivation
 ACT_SOFTCAP = 5
@@ -95,6 +96,12 @@ def _pack_attention(w, p, m: AttentionMixer, get, n_out: int, hp: int, device):
         w[f"{p}/mix/slope"] = (mix @ distance_slopes(H).to(device)).float().contiguous()
     if m.bias:
         w[f"{p}/mix/in_bias"] = bias
+    if m.sigmoid:
+        w[f"{p}/mix/offset"] = get("offset").float().contiguous()
+    if m.log_bias:
+        w[f"{p}/mix/log_rate"], w[f"{p}/mix/log_step"] = get("log_rate").float().contiguous(), get("log_step").float().contiguous()
+    if m.value_mix:
+        w[f"{p}/mix/v_lambda"] = get("v_lambda").float().reshape(1)
     if m.head_sink:
         w[f"{p}/mix/sink"] = get("sink").float().contiguous()
     if m.rotary is not None:
@@ -171,11 +178,56 @@ def _pack_gated_recurrence(w, p, m: GatedRecurrenceMixer, get, hp: int, dtype, d
     return [_pad_head_rows(get("y"), B, n, np_, hp), _pad_head_rows(get("x"), B, n, np_, hp)]
 
 
+def _pack_state_space(w, p, m: StateSpaceMixer, get, n_out: int, hp: int, device):
+    H, V, Vp, G, N, Np = m.heads, m.vdim, m.vdim_p, m.groups, m.state, m.state_p
+    z, x, b, c, dt = torch.split(get("in"), [H * V, H * V, G * N, G * N, H])
+
+    def channels(v):
+        x, b, c = torch.split(v, [H * V, G * N, G * N])
+        return torch.cat([_pad_head_vec(x, H, V, Vp), _pad_head_vec(b, G, N, Np), _pad_head_vec(c, G, N, Np)])
+    bias = torch.zeros(n_out, dtype=torch.float32, device=device)
+    bias[m.main_cols: m.main_cols + H] = get("dt_bias").float()
+    w[f"{p}/mix/in_bias"] = bias
+    w[f"{p}/mix/conv"] = torch.stack([channels(v) for v in get("conv").t()])           # [taps, channels]
+    w[f"{p}/mix/conv_bias"] = channels(get("conv_bias"))
+    w[f"{p}/mix/rate"] = torch.exp(get("a_log").double()).float().contiguous()
+    w[f"{p}/mix/skip"] = get("skip").float().contiguous()
+    w[f"{p}/mix/norm"] = _pad_head_vec(get("norm"), H, V, Vp)
+    return [_pad_head_rows(z, H, V, Vp, hp), _pad_head_rows(x, H, V, Vp, hp), _pad_head_rows(b, G, N, Np, hp),
+            _pad_head_rows(c, G, N, Np, hp), _pad2(dt, H, hp)]
+
+
+def _pack_parallel(w, p, m: ParallelMixer, get, n_out: int, hp: int, dtype, device):
+    rows, biases = [], []
+    for side, part in (("left", m.left), ("right", m.right)):
+        def of(name, side=side):
+            return get(f"{side}.{name}")
+        cols, q = part.main_cols + part.gate_cols, f"{p}/{side}"
+        rows += _pack_rows(w, q, part, of, cols, hp, dtype, device)
+        bias = w.pop(f"{q}/mix/in_bias", None)
+        biases.append(torch.zeros(cols, dtype=torch.float32, device=device) if bias is None else bias)
+        w[f"{q}/mix/out_proj"] = _pad_head_cols(of("o"), part.heads, part.vdim, part.vdim_p, hp).to(dtype)
+        w[f"{q}/norm"] = _pad_head_vec(of("out"), 1, of("out").numel(), hp)
+    w[f"{p}/mix/in_bias"] = torch.zeros(n_out, dtype=torch.float32, device=device)
+    w[f"{p}/mix/in_bias"][: m.main_cols + m.gate_cols] = torch.cat(biases)
+    return rows
+
+
+def _pack_rows(w, p, m, get, n_out: int, hp: int, dtype, device):
+    """Rows of the fused input projection of a mixer, its other weights into `w`."""
+    if m.kind == "parallel":
+        return _pack_parallel(w, p, m, get, n_out, hp, dtype, device)
+    if m.kind in ("latent_attention", "rglru"):
+        return {"latent_attention": _pack_latent, "rglru": _pack_gated_recurrence}[m.kind](w, p, m, get, hp, dtype, device)
+    pack = {"attention": _pack_attention, "hgrn2": _pack_gated_memory, "ssd": _pack_state_space, "mlstm": _pack_matrix_memory}[m.kind]
+    return pack(w, p, m, get, n_out, hp, device)
+
+
 def pack_weights(cfg: LayeredConfig, get, dtype: torch.dtype = torch.bfloat16, device="cpu") -> Dict[str, torch.Tensor]:
     """Fused, padded weights of the forward pass.  `get(layer, name)` returns a design's tensor by its role (layer -1:
-    the model's own): embed, head, final_norm, loop_in, loop_step; norm1, norm1b, norm2, norm2b, conv; hc1_in, hc1_out,
-    hc1_mix, hc2_...; the mixers' (see the _pack functions) and o; up, up_bias, down, down_bias, act; the experts' (see
-    `pack_experts`)."""
+    the model's own): embed, head, final_norm, positions, loop_in, loop_step; norm1, norm1b, norm2, norm2b, conv; hc1_in, hc1_out,
+    hc1_mix, hc2_...; the mixers' (see the _pack functions) and o, under "left." and "right." where there are two; up, up_bias,
+    down, down_bias, act; gate, up, down; the experts' (see `pack_experts`)."""
     hp, wide, streams = cfg.hidden_p, cfg.residual == "sandwich", cfg.residual == "streams"
     w: Dict[str, torch.Tensor] = {}
 
@@ -183,7 +235,7 @@ def pack_weights(cfg: LayeredConfig, get, dtype: torch.dtype = torch.bfloat16, d
         return get(layer, name).to(device)
 
     def norm(layer, name):
-        if not (wide or streams):
+        if cfg.residual == "post_sum":
             return g(layer, name).float().contiguous().reshape(1)
         return _pad_head_vec(g(layer, name).float() + cfg.norm_offset, 1, cfg.hidden, hp)
 
@@ -195,7 +247,9 @@ def pack_weights(cfg: LayeredConfig, get, dtype: torch.dtype = torch.bfloat16, d
     else:
         w["text/embed"] = _pad2(g(-1, "embed"), cfg.vocab, hp).to(dtype)
         w["text/lm_head"] = _pad2(g(-1, "head"), cfg.vocab_p, hp).to(dtype)
-    w["text/final_norm"] = norm(-1, "final_norm")
+    w["text/final_norm"] = norm(-1, "final_norm") * cfg.logit_scale        # (the head is linear)
+    if cfg.learned_positions:
+        w["text/places"] = _pad2(g(-1, "positions"), cfg.learned_positions, hp).to(dtype)
     if streams:
         w["text/stream_sum"] = torch.ones(cfg.streams, dtype=torch.float32, device=device)
     if cfg.logit_softcap:
@@ -216,18 +270,10 @@ def pack_weights(cfg: LayeredConfig, get, dtype: torch.dtype = torch.bfloat16, d
         if cfg.conv_taps:
             w[f"{p}/conv"] = torch.stack([_pad_head_vec(v, 1, cfg.hidden, hp) for v in g(i, "conv").t()])      # [taps, width]
         n_out = pad_to(m.main_cols + m.gate_cols, 2)
-        if m.kind == "attention":
-            rows = _pack_attention(w, p, m, mix, n_out, hp, device)
-        elif m.kind == "latent_attention":
-            rows = _pack_latent(w, p, m, mix, hp, dtype, device)
-        elif m.kind == "hgrn2":
-            rows = _pack_gated_memory(w, p, m, mix, n_out, hp, device)
-        elif m.kind == "rglru":
-            rows = _pack_gated_recurrence(w, p, m, mix, hp, dtype, device)
-        else:
-            rows = _pack_matrix_memory(w, p, m, mix, n_out, hp, device)
+        rows = _pack_rows(w, p, m, mix, n_out, hp, dtype, device)
         w[f"{p}/mix/in_proj"] = _pad2(torch.cat(rows), n_out, hp).to(dtype)
-        w[f"{p}/mix/out_proj"] = _pad_head_cols(g(i, "o"), m.heads, m.vdim, m.vdim_p, hp).to(dtype)
+        if m.kind != "parallel":
+            w[f"{p}/mix/out_proj"] = _pad_head_cols(g(i, "o"), m.heads, m.vdim, m.vdim_p, hp).to(dtype)
         if spec.mlp is not None:
             w[f"{p}/norm2"] = norm(i, "norm2")
             if wide:
@@ -236,6 +282,8 @@ def pack_weights(cfg: LayeredConfig, get, dtype: torch.dtype = torch.bfloat16, d
                 hyper(i, 2)
         if spec.mlp is not None and spec.mlp.kind == "moe":
             pack_experts(w, p, spec.mlp, mix, hp, dtype)
+        elif spec.mlp is not None and spec.mlp.kind == "glu":
+            w[f"{p}/mlp/up"], w[f"{p}/mlp/down"] = pack_unit(mix, "", spec.mlp, hp, dtype)
         elif spec.mlp is not None:
             fp = pad_to(spec.mlp.ff, 8)
             w[f"{p}/mlp/up"] = _pad2(g(i, "up"), fp, hp).to(dtype)
@@ -260,7 +308,8 @@ class LayeredWorkspace:
         T, dev, f32 = max_tokens, device, torch.float32
         moe = [l.mlp for l in cfg.layers if l.mlp is not None and l.mlp.kind == "moe"]
         mixers = [l.mixer for l in cfg.layers]
-        attn = [m for m in mixers if m.kind == "attention"]
+        parts = [p for m in mixers for p in mixer_parts(m)]
+        attn = [m for m in parts if m.kind == "attention"]
         latent = [m for m in mixers if m.kind == "latent_attention"]
 
         def rows(cols, dt=dtype):
@@ -278,14 +327,20 @@ class LayeredWorkspace:
         self.xa = rows(cfg.hidden_p)               # what the next GEMM reads, in the activation type
         self.pair = rows(2 * cfg.hidden_p) if cfg.loop is not None else None   # [x, embedding output] of a pass's entry
         self.delta = rows(cfg.hidden_p, f32)       # output of the running sublayer
+        self.delta2 = rows(cfg.hidden_p, f32) if len(parts) > len(mixers) else None      # and of the other one beside it
         self.proj = rows(widest((m.main_cols for m in mixers), 64))
         self.gates = rows(widest((m.gate_cols for m in mixers), 2, 4), f32)
         self.mix = rows(widest((m.out_cols for m in mixers), 64))
         self.q = rows(max([m.heads * m.dim_p for m in attn] + [m.q_cols for m in latent], default=16))
+        first = next((cfg.attention_of(r) for r in cfg.value_runs), None)
+        self.v_first = rows(first.kv_heads * first.vdim_p) if first is not None else None      # values that later layers mix in
+        units = [T * l.mlp.ff_p for l in cfg.layers if l.mlp is not None and l.mlp.kind == "glu"]
+        self.unit_act = torch.zeros(max(units, default=0), dtype=dtype, device=dev)
+        self.unit_wide = torch.zeros(2 * max(units, default=0) if dtype == f32 else 0, dtype=dtype, device=dev)
         self.act = rows(widest((l.mlp.ff for l in cfg.layers if l.mlp is not None and l.mlp.kind == "dense"), 8))
         if moe:
             self.experts = ExpertWorkspace(moe, cfg.hidden_p, T, dev, dtype, ops or load_native())
-        rec = max((m.out_cols for m in mixers if m.kind == "rglru"), default=0)
+        rec = max([m.out_cols for m in mixers if m.kind == "rglru"] + [m.conv_cols for m in parts if m.kind == "ssd"], default=0)
         if rec:
             self.rec_u = torch.zeros(T * rec, dtype=dtype, device=dev)
         if latent:
@@ -304,13 +359,16 @@ class LayeredWorkspace:
 
 def native_subset(cfg: LayeredConfig) -> str:
     """The parts of the stand-alone library (see `_build.PARTS`) that this configuration needs."""
-    parts = {{"latent_attention": "latent", "hgrn2": "gated"}.get(l.mixer.kind, l.mixer.kind) for l in cfg.layers}
-    if any(l.mixer.kind == "attention" and not l.mixer.plain_scores for l in cfg.layers):
+    mixers = [m for l in cfg.layers for m in mixer_parts(l.mixer)]
+    parts = {{"latent_attention": "latent", "hgrn2": "gated"}.get(m.kind, m.kind) for m in mixers}
+    if any(m.kind == "attention" and not m.plain_scores for m in mixers):
         parts.add("head_mix")
     if any(l.mlp is not None and l.mlp.kind == "moe" for l in cfg.layers):
         parts |= {"moe", "streams"}                # (the sum over the experts belongs to the row steps)
-    if cfg.residual == "streams":
+    if cfg.residual == "streams" or any(l.mlp is not None and l.mlp.kind == "glu" for l in cfg.layers):
         parts.add("streams")
+    if cfg.residual == "branch":
+        parts.add("branches")
     return "+".join(sorted(parts))
 
 
@@ -319,6 +377,8 @@ class LayeredModel:
 
     def __init__(self, cfg: LayeredConfig, weights: Dict[str, torch.Tensor], device, pdl: bool = False):
         self.cfg, self.w = cfg, weights
+        if cfg.residual != "branch" and any(l.mixer.kind == "parallel" for l in cfg.layers):
+            raise ValueError("mixers side by side need the residual form 'branch'")
         self.device = torch.device(device)
         self._raw_ops = load_native(subset=native_subset(cfg))
         self.ops = LaunchCounter(self._raw_ops)
@@ -336,6 +396,7 @@ class LayeredModel:
         self._runs = cfg.runs
         self._attn_idx = {r: i for i, r in enumerate(cfg.attn_layers)}
         self._state_idx = {r: i for i, r in enumerate(cfg.state_layers)}
+        self._value_runs = cfg.value_runs
         self._scratch: Dict[str, torch.Tensor] = {}
         self._keep: List[torch.Tensor] = []
 
@@ -366,21 +427,24 @@ class LayeredModel:
         proj = ws.proj[:T, : m.main_cols]
         gates = ws.gates[:T] if m.gate_cols else None
         self._gemm(ws.xa[:T], self.w[f"{p}/mix/in_proj"], self.w.get(f"{p}/mix/in_bias"), proj, gates, m.main_cols if gates is not None else 0,
-                   prefetch=self.w[f"{p}/mix/out_proj"])
+                   prefetch=self.w[f"{p}/left/mix/out_proj" if m.kind == "parallel" else f"{p}/mix/out_proj"])
         return proj, gates
 
     # ------------------------------------------------------------------ mixers
-    def _attention(self, ws, b: StepBatch, kv, run: int, T: int, p: str, m: AttentionMixer):
+    def _attention(self, ws, b: StepBatch, kv, run: int, T: int, p: str, m: AttentionMixer, inputs=None, out=None):
+        """`inputs`: the projection's columns and gates when it is made elsewhere; `out`: where the heads' outputs go."""
         ops, w = self.ops, self.w
-        proj, gates = self._in_proj(ws, T, p, m)
+        proj, gates = inputs or self._in_proj(ws, T, p, m)
         planes = kv.layers[self._attn_idx[run]]
         k_pages, v_pages = planes.typed(self.dtype)
         H, G, Dp, Vp = m.heads, m.kv_heads, m.dim_p, m.vdim_p
         q = ws.q[:T, : H * Dp]
         ops.qkv_append(proj, 0, H * Dp, (H + G) * Dp, H, G, m.dim, w.get(f"{p}/mix/q_norm"), w.get(f"{p}/mix/k_norm"),
                        self.cfg.rms_eps, b.table_row, b.cache_pos, kv.table, q, k_pages, v_pages, kv.page_size, self.pdl,
-                       w.get(f"{p}/mix/freq"))
-        out, sinks = ws.mix[:T, : H * Vp], w.get(f"{p}/mix/sink")
+                       w.get(f"{p}/mix/freq"), m.qk_unit, ws.v_first[:T] if m.value_mix else None,
+                       w[f"{p}/mix/v_lambda"] if m.value_mix and run != self._value_runs[0] else None)
+        out, sinks = ws.mix[:T, : H * Vp] if out is None else out, w.get(f"{p}/mix/sink")
+        weights = (m.sigmoid, w.get(f"{p}/mix/log_rate"), w.get(f"{p}/mix/log_step"), w.get(f"{p}/mix/offset"))
         shape = (m.window, m.scale, m.softcap, m.sink, w.get(f"{p}/mix/heads"), w.get(f"{p}/mix/slope"),
                  gates if m.head_gate else None, out)
         portions = not self.f32 and self.prefill_kernels and b.max_seq_tokens >= PREFILL_MIN_TOKENS
@@ -389,15 +453,15 @@ class LayeredModel:
                               b.qblk_start, b.qblk_count, self.pdl)
             return out
         if portions and not m.plain_scores:
-            one = int(ops.head_mix_prefill_scratch(H, b.max_kv_len, m.window, 1))
+            one = int(ops.head_mix_prefill_scratch(H, b.max_kv_len, m.window, 1, m.sigmoid))
             nb = b.qblk_start.numel()
             scratch = self._grown("scores", max(one, min(one * nb, SCORE_SCRATCH_BYTES)))
             ops.head_mix_prefill(q, k_pages, v_pages, kv.table, b.table_row, b.kv_len, *shape, b.qblk_start, b.qblk_count,
-                                 b.max_kv_len, scratch, self.pdl)
+                                 b.max_kv_len, scratch, self.pdl, *weights)
             return out
         split, n = self.pick_split(ws, T, b.max_kv_len, m.look_back, ctas=G if m.plain_scores and not self.f32 else 1)
         ops.head_mix_attention(q, k_pages, v_pages, kv.table, b.table_row, b.kv_len, *shape, split, n,
-                               ws.part_o if n > 1 else None, ws.part_ml if n > 1 else None, self.pdl, m.chunk, sinks)
+                               ws.part_o if n > 1 else None, ws.part_ml if n > 1 else None, self.pdl, m.chunk, sinks, *weights)
         return out
 
     @staticmethod
@@ -547,11 +611,41 @@ class LayeredModel:
         ops.rglru_scan(proj, *step, u, raw, rate, S, out, write_state, self.pdl)
         return out
 
+    def _state_space(self, ws, b: StepBatch, states, run: int, T: int, p: str, m: StateSpaceMixer, write_state: bool, inputs=None, out=None):
+        """`inputs`, `out`: as in `_attention`."""
+        ops, w = self.ops, self.w
+        proj, gates = inputs or self._in_proj(ws, T, p, m)
+        ring, S = states.layers[self._state_idx[run]][-2:]
+        out = ws.mix[:T, : m.out_cols] if out is None else out
+        one = b.one_token_per_seq
+        u = chunk_ws = None
+        if not one:
+            u = ws.rec_u[: T * m.conv_cols].view(T, m.conv_cols)
+            if (not self.f32 and self.prefill_kernels and b.max_seq_tokens >= PREFILL_MIN_TOKENS
+                    and self._raw_ops.ssd_chunked_supported(m.state_p, m.vdim_p)):
+                chunk_ws = self._grown("state space", int(self._raw_ops.ssd_chunked_workspace_bytes(T, b.n_seqs, m.heads, m.state_p, m.vdim_p)))
+            ops.count += 1 if chunk_ws is None else 3
+        ops.ssd(proj, m.out_cols, gates, w[f"{p}/mix/conv"], w[f"{p}/mix/conv_bias"], w[f"{p}/mix/rate"], w[f"{p}/mix/skip"], m.groups,
+                b.cu_seqlens, b.token_seq, b.cache_pos, b.state_slot, ring, S, u, out, write_state, chunk_ws, self.pdl, one)
+        ops.ssd_gated_norm(out, proj, w[f"{p}/mix/norm"], m.heads, m.vdim, m.norm_groups, self.cfg.rms_eps, self.pdl)
+        return out
+
+    def _parallel(self, ws, b: StepBatch, kv, states, run: int, T: int, p: str, m: ParallelMixer, write_state: bool, prefetch) -> dict:
+        """ws.delta, ws.delta2 <- the outputs of both sides; returns them as `branch_rows` takes them."""
+        w, cut, at = self.w, m.left.out_cols, m.left.main_cols
+        proj, gates = self._in_proj(ws, T, p, m)
+        left, right = ws.mix[:T, :cut], ws.mix[:T, cut: cut + m.right.out_cols]
+        self._attention(ws, b, kv, run, T, f"{p}/left", m.left, (proj[:, :at], None), left)
+        self._state_space(ws, b, states, run, T, f"{p}/right", m.right, write_state, (proj[:, at:], gates), right)
+        self._gemm(left, w[f"{p}/left/mix/out_proj"], None, out32=ws.delta[:T], prefetch=w[f"{p}/right/mix/out_proj"])
+        self._gemm(right, w[f"{p}/right/mix/out_proj"], None, out32=ws.delta2[:T], prefetch=prefetch)
+        return dict(branch_a=ws.delta[:T], branch_b=ws.delta2[:T], w_a=w[f"{p}/left/norm"], w_b=w[f"{p}/right/norm"])
+
     def _mixer(self, ws, b: StepBatch, kv, states, run: int, T: int, p: str, m, write_state: bool) -> torch.Tensor:
         if m.kind in ATTENTION_KINDS:
             fn = self._attention if m.kind == "attention" else self._latent_attention
             return fn(ws, b, kv, run, T, p, m)
-        fn = {"hgrn2": self._gated_memory, "mlstm": self._matrix_memory, "rglru": self._gated_recurrence}[m.kind]
+        fn = {"hgrn2": self._gated_memory, "mlstm": self._matrix_memory, "rglru": self._gated_recurrence, "ssd": self._state_space}[m.kind]
         return fn(ws, b, states, run, T, p, m, write_state)
 
     def _feed_forward(self, ws, T: int, p: str, spec, prefetch) -> None:
@@ -561,6 +655,9 @@ class LayeredModel:
             self.ops.mixture_rows(*y.values(), ws.delta[:T], self.pdl)
             return
         w, up, down = self.w, self.w[f"{p}/mlp/up"], self.w[f"{p}/mlp/down"]
+        if spec.kind == "glu":
+            run_unit(self, T, spec, up, down, ws.xa[:T], ws.unit_act, ws.unit_wide, ws.delta[:T], prefetch)
+            return
         act = ws.act[:T, : up.shape[0]]
         self._gemm(ws.xa[:T], up, w.get(f"{p}/mlp/up_bias"), act, act=ACTIVATIONS[spec.activation], act_params=w.get(f"{p}/mlp/act"),
                    prefetch=down)
@@ -571,7 +668,8 @@ class LayeredModel:
         """Runs all layers; returns the final-normed hidden states [T, hidden (padded)]."""
         if b.n_tokens > ws.max_tokens:
             raise ValueError(f"step of {b.n_tokens} tokens exceeds the workspace ({ws.max_tokens})")
-        run = {"sandwich": self._forward_sandwich, "streams": self._forward_streams, "post_sum": self._forward_post_sum}[self.cfg.residual]
+        run = {"sandwich": self._forward_sandwich, "streams": self._forward_streams, "post_sum": self._forward_post_sum,
+               "branch": self._forward_branch}[self.cfg.residual]
         return run(ws, b, kv, states, write_state)
 
     def _next_weights(self, run: int):
@@ -670,6 +768,38 @@ class LayeredModel:
                 rows(w["text/stream_sum"], w["text/final_norm"])
                 self.layer_hook(run, X.sum(dim=1)[:, : cfg.hidden])
         rows(w["text/stream_sum"], w["text/final_norm"])
+        return xa
+
+    def _forward_branch(self, ws, b: StepBatch, kv, states, write_state: bool) -> torch.Tensor:
+        """A sublayer reads the residual itself; the row step behind it norms its output, adds it and makes the next input."""
+        cfg, ops, w, T = self.cfg, self.ops, self.w, b.n_tokens
+        x, xa, delta = ws.x[:T], ws.xa[:T], ws.delta[:T]
+        no_branches = dict(branch_a=None, branch_b=None, w_a=None, w_b=None)
+
+        def rows(y, branches, norm, last):
+            ops.branch_rows(x, *(branches or no_branches).values(), *(y or self._plain_sum(None)).values(), norm,
+                            w["text/final_norm"] if last else None, xa, cfg.hidden, cfg.rms_eps, self.pdl)
+        ops.embed_rows32(b.ids, w["text/embed"], x, xa, cfg.embed_scale, self.pdl, b.cache_pos, w.get("text/places"))
+        for run, (layer, _) in enumerate(self._runs):
+            spec, p, last = cfg.layers[layer], f"text/layers/{layer}", run + 1 == len(self._runs)
+            nxt = self._next_weights(run)
+            after = w.get(f"{p}/mlp/router", w.get(f"{p}/mlp/up", nxt))
+            if spec.mixer.kind == "parallel":
+                y, pair = None, self._parallel(ws, b, kv, states, run, T, p, spec.mixer, write_state, after)
+            else:
+                mix = self._mixer(ws, b, kv, states, run, T, p, spec.mixer, write_state)
+                self._gemm(mix, w[f"{p}/mix/out_proj"], None, out32=delta, prefetch=after)
+                y, pair = self._plain_sum(delta), None
+            rows(y, pair, w[f"{p}/norm1"], last and spec.mlp is None)
+            if spec.mlp is not None:
+                if spec.mlp.kind == "moe":
+                    y = run_experts(self, ws.experts, T, p, spec.mlp, xa, delta, nxt)
+                else:
+                    self._feed_forward(ws, T, p, spec.mlp, nxt)
+                    y = self._plain_sum(delta)
+                rows(y, None, w[f"{p}/norm2"], last)
+            if self.layer_hook is not None:
+                self.layer_hook(run, x[:, : cfg.hidden])
         return xa
 
     @staticmethod

@@ -1,8 +1,8 @@
 """Description of decoders given as a list of layers (read by `models/layered.py`, which runs them).
 
-A layer is a mixer (attention with shaped or plain scores, latent attention, matrix memory, gated linear memory or gated
-linear recurrence) and an optional feed-forward (dense or a mixture of experts); every size and constant is a field, and so
-is which mechanisms a mixer has.  The model's own fields say how a sublayer meets the residual stream (or streams), what
+A layer is a mixer (attention with shaped or plain scores, latent attention, matrix memory, gated linear memory, gated
+linear recurrence, a selective state space, or two of them side by side) and an optional feed-forward (dense or a mixture of
+experts); every size and constant is a field, and so is which mechanisms a mixer has.  The model's own fields say how a sublayer meets the residual stream (or streams), what
 precedes a mixer, and which layers run several times.  Cache and state belong
 to layer RUNS: a layer that runs twice has two of each.  No torch here: the package table and the host diagnostics read
 these descriptions too."""
@@ -67,13 +67,17 @@ class AttentionMixer:
     chunk: int = 0                # keys of the query's own chunk of this many positions only (counted from 0); 0: no chunks
     head_sink: bool = False       # one learned score per head in the softmax denominator
     rotary: Optional[Rotary] = None   # after the norm, on q and k
+    qk_unit: bool = False         # RMS norm of every query and key head without a weight
+    sigmoid: bool = False         # weight sigmoid(score + a learned number per head) instead of a softmax; mixed instead of the scores
+    log_bias: bool = False        # r1_h ln(1 + r2_h (i - j)) taken off the scores, two learned numbers per head (sigmoid weights)
+    value_mix: bool = False       # v <- (1 - l) v + l v_first, l learned, v_first the values of the first such layer (which keeps its own)
 
     kind = "attention"
 
     @property
     def plain_scores(self) -> bool:
-        """Scaled dot products and nothing else: no cap, bias, mix or gate."""
-        return not (self.softcap or self.distance_bias or self.head_mixing or self.head_gate)
+        """Scaled dot products and nothing else: no cap, bias, mix, gate or sigmoid."""
+        return not (self.softcap or self.distance_bias or self.head_mixing or self.head_gate or self.sigmoid)
 
     @property
     def look_back(self) -> int:
@@ -268,6 +272,69 @@ class GatedRecurrenceMixer:
 
 
 @dataclass(frozen=True)
+class StateSpaceMixer:
+    """Selective state space with one decay per head (Mamba-2): a causal convolution with SiLU in front of
+    S <- exp(-rate dt) S + dt x B^T, y = S C + skip x; then y silu(z), normed in equal parts."""
+    heads: int
+    vdim: int                     # channels per head
+    state: int                    # state columns per channel
+    groups: int                   # of heads that share B and C
+    taps: int                     # of the convolution
+    norm_groups: int = 1
+
+    kind = "ssd"
+
+    @property
+    def vdim_p(self) -> int:
+        return pad_to(self.vdim, 16)
+
+    @property
+    def state_p(self) -> int:
+        return pad_to(self.state, 16)
+
+    @property
+    def conv_cols(self) -> int:
+        """Convolved channels: [x, B, C]"""
+        return self.out_cols + 2 * self.groups * self.state_p
+
+    @property
+    def main_cols(self) -> int:
+        """[z, x, B, C]"""
+        return self.out_cols + self.conv_cols
+
+    @property
+    def gate_cols(self) -> int:
+        """Raw step sizes, fp32."""
+        return self.heads
+
+    @property
+    def out_cols(self) -> int:
+        return self.heads * self.vdim_p
+
+
+@dataclass(frozen=True)
+class ParallelMixer:
+    """Attention and a state space side by side on the same input; the layer's output is the mean of the two, each normed by
+    itself first.  One fused input projection: the left columns, the right ones, then the right gates."""
+    left: AttentionMixer
+    right: StateSpaceMixer
+
+    kind = "parallel"
+
+    @property
+    def main_cols(self) -> int:
+        return self.left.main_cols + self.right.main_cols
+
+    @property
+    def gate_cols(self) -> int:
+        return self.right.gate_cols
+
+    @property
+    def out_cols(self) -> int:
+        return self.left.out_cols + self.right.out_cols
+
+
+@dataclass(frozen=True)
 class DenseMlp:
     ff: int
     activation: str = "xielu"     # xielu (two learned numbers per layer) | relu2 (square of relu)
@@ -278,11 +345,16 @@ class DenseMlp:
 
 @dataclass(frozen=True)
 class GatedUnit:
-    """down( g sigmoid(slope g) (u + shift) ) with g = min(gate h, limit), u = clamp(up h, +- limit); limit 0: no bounds."""
+    """down( g sigmoid(slope g) (u + shift) ) with g = min(gate h, limit), u = clamp(up h, +- limit); limit 0: no bounds.
+    An expert, or a layer's dense feed-forward."""
     ff: int
     limit: float = 0.0
     slope: float = 1.0
     shift: float = 0.0
+
+    kind = "glu"
+    activation = "swiglu"
+    bias = False
 
     @property
     def ff_p(self) -> int:
@@ -294,15 +366,22 @@ class GatedUnit:
 
 @dataclass(frozen=True)
 class ExpertMlp:
-    """Mixture of experts: softmax over all router outputs, the `top` largest scores (with a learned correction added for the
-    choice only) times `scale` weigh the chosen experts.  The last `identity` outputs stand for the input itself.  A
-    shared expert runs for every token under a sigmoid gate."""
+    """Mixture of experts: scores are the softmax over all router outputs or the sigmoid of each; the `top` largest scores
+    (with a learned correction added for the choice only) times `scale`, or divided by their sum, weigh the chosen experts.
+    With `groups` (equal runs of neighbours) only experts of the `keep` best groups can be chosen, a group's score being the
+    sum of its two largest corrected scores.  The last `identity` outputs stand for the input itself.  A shared expert runs for
+    every token, under a sigmoid gate or as it is."""
     experts: int
     top: int
     expert: GatedUnit
     identity: int = 0
     scale: float = 1.0
     shared: Optional[GatedUnit] = None
+    shared_gate: bool = True
+    sigmoid: bool = False
+    renormalise: bool = False
+    groups: int = 0
+    keep: int = 0
 
     kind = "moe"
 
@@ -313,7 +392,7 @@ class ExpertMlp:
     @property
     def router_cols(self) -> int:
         """Router outputs and the shared expert's gate."""
-        return pad_to(self.choices + (1 if self.shared else 0), 8)
+        return pad_to(self.choices + (1 if self.shared and self.shared_gate else 0), 8)
 
     @property
     def slots(self) -> int:
@@ -323,8 +402,9 @@ class ExpertMlp:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: Union[AttentionMixer, LatentAttentionMixer, MatrixMemoryMixer, GatedMemoryMixer, GatedRecurrenceMixer]
-    mlp: Optional[Union[DenseMlp, ExpertMlp]] = None
+    mixer: Union[AttentionMixer, LatentAttentionMixer, MatrixMemoryMixer, GatedMemoryMixer, GatedRecurrenceMixer, StateSpaceMixer,
+                 ParallelMixer]
+    mlp: Optional[Union[DenseMlp, GatedUnit, ExpertMlp]] = None
 
 
 @dataclass(frozen=True)
@@ -339,6 +419,20 @@ class LoopSpec:
 ATTENTION_KINDS = ("attention", "latent_attention")
 
 
+def attention_part(m):
+    """The mixer that owns cache rows, or None."""
+    return m.left if m.kind == "parallel" else (m if m.kind in ATTENTION_KINDS else None)
+
+
+def memory_part(m):
+    """The mixer that owns recurrent state, or None."""
+    return m.right if m.kind == "parallel" else (None if m.kind in ATTENTION_KINDS else m)
+
+
+def mixer_parts(m) -> tuple:
+    return (m.left, m.right) if m.kind == "parallel" else (m,)
+
+
 @dataclass(frozen=True)
 class LayeredConfig:
     name: str
@@ -350,7 +444,8 @@ class LayeredConfig:
     max_context: int = 131072
     architecture: str = ""        # name of the design that maps checkpoints onto this description
     # post_sum | sandwich: x <- x + residual_mult * norm(f(norm(x))) | streams: `streams` copies of the embedding output; a
-    # sublayer reads a weighted sum of them, u = sum_s in[s] x_s, and x_t <- sum_s mix[s, t] x_s + out[t] f(norm(u))
+    # sublayer reads a weighted sum of them, u = sum_s in[s] x_s, and x_t <- sum_s mix[s, t] x_s + out[t] f(norm(u)) |
+    # branch: x <- x + norm(f(x))
     residual: str = "post_sum"
     residual_mult: float = 1.0    # sandwich
     norm_groups: int = 1          # sandwich: equal parts of a row that are normed by themselves, one weight per column
@@ -361,6 +456,9 @@ class LayeredConfig:
     streams: int = 1
     norm_offset: float = 0.0      # added to the stored weights of the sublayers' and the final norm
     logit_softcap: float = 0.0    # logits <- cap tanh(logits / cap); 0: as they are
+    logit_scale: float = 1.0
+    learned_positions: int = 0    # rows of a table of position vectors that are added to the embedding: as many positions a
+                                  # sequence can have; 0: no table
 
     moe = None
     mtp_layers = 0
@@ -393,49 +491,66 @@ class LayeredConfig:
     @property
     def attn_layers(self) -> List[int]:
         """Layer runs that have a cache (without a loop a run is a layer)."""
-        return [r for r, (i, _) in enumerate(self.runs) if self.layers[i].mixer.kind in ATTENTION_KINDS]
+        return [r for r, (i, _) in enumerate(self.runs) if attention_part(self.layers[i].mixer) is not None]
 
     @property
     def state_layers(self) -> List[int]:
         """Layer runs that have recurrent state: a memory, or the inputs that a convolution looks back on."""
         return [r for r, (i, _) in enumerate(self.runs)
-                if self.conv_taps > 1 or self.layers[i].mixer.kind not in ATTENTION_KINDS]
+                if self.conv_taps > 1 or memory_part(self.layers[i].mixer) is not None]
+
+    def attention_of(self, run: int):
+        return attention_part(self.mixer_of(run))
+
+    @property
+    def value_runs(self) -> List[int]:
+        """Layer runs whose values are mixed with those of the first of them."""
+        return [r for r in self.attn_layers if getattr(self.attention_of(r), "value_mix", False)]
+
+    @property
+    def position_limit(self) -> int:
+        """Most positions that a sequence can have; 0: no limit of the model's own."""
+        return self.learned_positions
 
     @property
     def n_kv_heads(self) -> int:
-        return max((self.mixer_of(r).kv_heads for r in self.attn_layers), default=0)
+        return max((self.attention_of(r).kv_heads for r in self.attn_layers), default=0)
 
     @property
     def head_dim(self) -> int:
-        return max((self.mixer_of(r).dim for r in self.attn_layers), default=0)
+        return max((self.attention_of(r).dim for r in self.attn_layers), default=0)
 
     @property
     def kv_geometry(self) -> List[Tuple[int, int, int]]:
         """Per attention run: kv heads, key width, value width of a cache row (padded).  A latent row has no separate
         values."""
-        ms = [self.mixer_of(r) for r in self.attn_layers]
+        ms = [self.attention_of(r) for r in self.attn_layers]
         return [(1, m.row_cols, 0) if m.kind == "latent_attention" else (m.kv_heads, m.dim_p, m.vdim_p) for m in ms]
 
     @property
     def cache_window(self) -> int:
         """Keys that any layer still looks back on: the widest window, 0 when some layer sees all of the past."""
-        w = [self.mixer_of(r).look_back for r in self.attn_layers]
+        w = [self.attention_of(r).look_back for r in self.attn_layers]
         return max(w) if w and min(w) > 0 else 0
 
     def state_shapes(self) -> List[List[tuple]]:
         """Per run in `state_layers`: shapes (without the slot) of its fp32 state arrays: the convolution's last inputs
         (oldest first) when there are any, then the memory: S, n, m (matrix memory), S (gated memory), or the inputs of
-        the last `taps` positions (row position mod taps) and S (gated recurrence)."""
+        the last `taps` positions (row position mod taps) and S (gated recurrence, state space)."""
         out = []
         for r in self.state_layers:
-            m, arrays = self.mixer_of(r), []
+            m, arrays = memory_part(self.mixer_of(r)), []
             if self.conv_taps > 1:
                 arrays.append((self.conv_taps - 1, self.hidden_p))
-            if m.kind == "rglru":
+            if m is None:
+                pass
+            elif m.kind == "rglru":
                 arrays += [(m.taps, m.out_cols), (m.out_cols,)]
-            elif m.kind not in ATTENTION_KINDS:
+            elif m.kind == "ssd":
+                arrays += [(m.taps, m.conv_cols), (m.heads, m.vdim_p, m.state_p)]
+            else:
                 arrays.append((m.heads, m.dim_p, m.vdim_p))
-            if m.kind == "mlstm":
+            if m is not None and m.kind == "mlstm":
                 arrays += [(m.heads, m.dim_p), (m.heads,)]
             out.append(arrays)
         return out
@@ -447,33 +562,44 @@ class LayeredConfig:
         h, wide = self.hidden, self.residual == "sandwich"
         norm = 1 if self.residual == "post_sum" else h                      # weights of one norm
         hyper = self.streams * (self.streams + 2) if self.residual == "streams" else 0
-        n = (1 if self.tie_head else 2) * self.vocab * h + norm
+        n = (1 if self.tie_head else 2) * self.vocab * h + norm + self.learned_positions * h
         if self.loop is not None:
             n += 2 * h * h + self.loop.times * h
         for l in self.layers:
-            m = l.mixer
-            n += (2 if wide else 1) * norm + hyper + self.conv_taps * h + h * m.heads * m.vdim
-            if m.kind == "attention":
-                rows = (m.heads + m.kv_heads) * m.dim + m.kv_heads * m.vdim + (m.heads if m.head_gate else 0)
-                n += rows * h + (m.heads * m.heads if m.head_mixing else 0) + (2 * m.dim if m.qk_norm else 0)
-                n += m.heads if m.head_sink else 0
-            elif m.kind == "latent_attention":
-                n += (m.q_rank + m.kv_rank + m.rot_dim) * h + m.q_rank + m.kv_rank + (m.heads if m.sink else 0)
-                n += m.heads * (m.dim + m.rot_dim) * (m.q_rank or h) + m.heads * (m.dim + m.vdim) * m.kv_rank
-            elif m.kind == "rglru":
-                n += 2 * m.width * (h + 1) + m.width * (m.taps + 1) + 2 * m.width * (m.vdim + 1) + m.width
-            elif m.kind == "hgrn2":
-                n += (2 * m.heads * m.dim + m.heads * m.vdim) * h + 2 * m.heads * m.dim + m.vdim
-            else:
-                n += (2 * m.heads * (m.dim + m.vdim) + 2 * m.heads) * h + m.heads * m.vdim + 2 * m.heads
+            n += (2 if wide else 1) * norm + hyper + self.conv_taps * h + sum(self._mixer_params(m) for m in mixer_parts(l.mixer))
+            n += 2 * h if l.mixer.kind == "parallel" else 0
             if l.mlp is not None:
                 n += (2 * norm if wide else norm) + hyper
             if l.mlp is not None and l.mlp.kind == "moe":
                 n += l.mlp.choices * (h + 1) + l.mlp.experts * l.mlp.expert.params(h)
-                n += l.mlp.shared.params(h) + h if l.mlp.shared else 0
+                n += l.mlp.shared.params(h) + (h if l.mlp.shared_gate else 0) if l.mlp.shared else 0
+            elif l.mlp is not None and l.mlp.kind == "glu":
+                n += l.mlp.params(h)
             elif l.mlp is not None:
                 n += 2 * h * l.mlp.ff
                 n += 2 if l.mlp.activation == "xielu" else (l.mlp.ff + h if l.mlp.bias else 0)
+        return n
+
+    def _mixer_params(self, m) -> int:
+        h = self.hidden
+        n = h * m.heads * m.vdim
+        if m.kind == "attention":
+            cols = (m.heads + m.kv_heads) * m.dim + m.kv_heads * m.vdim
+            n += (cols + (m.heads if m.head_gate else 0)) * h
+            n += (m.heads * m.heads if m.head_mixing else 0) + (2 * m.dim if m.qk_norm else 0) + (1 if m.value_mix else 0)
+            n += m.heads * (int(m.head_sink) + int(m.sigmoid) + 2 * int(m.log_bias))
+        elif m.kind == "latent_attention":
+            n += (m.q_rank + m.kv_rank + m.rot_dim) * h + m.q_rank + m.kv_rank + (m.heads if m.sink else 0)
+            n += m.heads * (m.dim + m.rot_dim) * (m.q_rank or h) + m.heads * (m.dim + m.vdim) * m.kv_rank
+        elif m.kind == "rglru":
+            n += 2 * m.width * (h + 1) + m.width * (m.taps + 1) + 2 * m.width * (m.vdim + 1) + m.width
+        elif m.kind == "ssd":
+            inner, conv = m.heads * m.vdim, m.heads * m.vdim + 2 * m.groups * m.state
+            n += (inner + conv + m.heads) * h + conv * (m.taps + 1) + 3 * m.heads + inner
+        elif m.kind == "hgrn2":
+            n += (2 * m.heads * m.dim + m.heads * m.vdim) * h + 2 * m.heads * m.dim + m.vdim
+        else:
+            n += (2 * m.heads * (m.dim + m.vdim) + 2 * m.heads) * h + m.heads * m.vdim + 2 * m.heads
         return n
 
     def shrink(self, n_layers: int) -> "LayeredConfig":

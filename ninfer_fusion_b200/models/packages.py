@@ -18,8 +18,8 @@ from .architectures import LAYERED_REGISTRY
 from .config import REGISTRY, ModelConfig
 from .layered_config import LayeredConfig
 
-FULL, SLIDING, GDN, MLSTM, GATED, LATENT, CHUNKED, RGLRU = "full", "sliding", "gdn", "mlstm", "hgrn2", "latent", "chunked", "rglru"
-KINDS = (FULL, SLIDING, GDN, MLSTM, GATED, LATENT, CHUNKED, RGLRU)
+FULL, SLIDING, GDN, MLSTM, GATED, LATENT, CHUNKED, RGLRU, SSD = "full", "sliding", "gdn", "mlstm", "hgrn2", "latent", "chunked", "rglru", "ssd"
+KINDS = (FULL, SLIDING, GDN, MLSTM, GATED, LATENT, CHUNKED, RGLRU, SSD)
 
 # what the engine's forward pass, kernels and cache can do today
 ENGINE_CAPABILITIES: FrozenSet[str] = frozenset({
@@ -36,6 +36,8 @@ ENGINE_CAPABILITIES: FrozenSet[str] = frozenset({
     "latent-attention", "gated-memory", "sandwich-norms", "grouped-norm", "input-convolution", "layer-loop", "relu2-mlp",
     "residual-streams", "offset-norm", "chunked-attention", "learned-sink", "interleaved-rope", "scaled-rope", "gated-recurrence",
     "expert-mlp", "identity-experts", "output-softcap",
+    "output-norms", "learned-positions", "sigmoid-attention", "log-distance-bias", "value-mixing", "state-space", "parallel-mixers",
+    "grouped-routing",
 })
 
 
@@ -91,22 +93,30 @@ def _hybrid(cfg: ModelConfig) -> Package:
 
 def _layered(cfg: LayeredConfig) -> Package:
     kinds = []
-    needs = {"layer-list-schedule", {"sandwich": "sandwich-norms", "streams": "residual-streams"}.get(cfg.residual, "post-sum-norm")}
+    needs = {"layer-list-schedule", {"sandwich": "sandwich-norms", "streams": "residual-streams", "branch": "output-norms"}.get(cfg.residual, "post-sum-norm")}
     needs |= {c for c, on in (("grouped-norm", cfg.norm_groups > 1), ("input-convolution", cfg.conv_taps), ("layer-loop", cfg.loop),
-                              ("offset-norm", cfg.norm_offset), ("output-softcap", cfg.logit_softcap)) if on}
+                              ("offset-norm", cfg.norm_offset), ("output-softcap", cfg.logit_softcap),
+                              ("learned-positions", cfg.learned_positions)) if on}
     for l in cfg.layers:
-        m = l.mixer
+        # (of two mixers side by side the attention names the layer's kind)
+        m = l.mixer.left if l.mixer.kind == "parallel" else l.mixer
+        if l.mixer.kind == "parallel":
+            needs |= {"parallel-mixers", "state-space"}
         if m.kind == "attention":
             rot = m.rotary
             kinds.append(LayerKind(CHUNKED if m.chunk else (SLIDING if m.window else FULL), rot.dims if rot else 0, rot.base if rot else 0.0,
                                    m.look_back, m.heads, m.kv_heads, m.dim))
             needs |= {c for c, on in (("sliding-window-attention", m.window), ("chunked-attention", m.chunk),
-                                      ("head-mixing-attention", m.head_mixing), ("attention-sink", m.sink),
-                                      ("learned-sink", m.head_sink), ("qk-norm", m.qk_norm), ("interleaved-rope", rot),
+                                      ("head-mixing-attention", m.head_mixing),
+                                      ("sigmoid-attention", m.sigmoid), ("log-distance-bias", m.log_bias), ("value-mixing", m.value_mix), ("attention-sink", m.sink),
+                                      ("learned-sink", m.head_sink), ("qk-norm", m.qk_norm or m.qk_unit), ("interleaved-rope", rot),
                                       ("scaled-rope", rot and rot.scaling)) if on}
         elif m.kind == "latent_attention":
             kinds.append(LayerKind(LATENT, m.rot_dim, m.rot_base, m.window, m.heads, 1, m.dim + m.rot_dim))
             needs |= {c for c, on in (("latent-attention", True), ("attention-sink", m.sink), ("sliding-window-attention", m.window)) if on}
+        elif m.kind == "ssd":
+            kinds.append(LayerKind(SSD, q_heads=m.heads, kv_heads=m.groups, head_dim=m.vdim))
+            needs.add("state-space")
         elif m.kind == "rglru":
             kinds.append(LayerKind(RGLRU, q_heads=m.blocks, kv_heads=m.blocks, head_dim=m.vdim))
             needs.add("gated-recurrence")
@@ -114,7 +124,7 @@ def _layered(cfg: LayeredConfig) -> Package:
             kinds.append(LayerKind(GATED if m.kind == "hgrn2" else MLSTM, q_heads=m.heads, kv_heads=m.heads, head_dim=m.dim))
             needs.add("gated-memory" if m.kind == "hgrn2" else "matrix-memory")
         if l.mlp is not None and l.mlp.kind == "moe":
-            needs |= {"expert-mlp"} | ({"identity-experts"} if l.mlp.identity else set())
+            needs |= {"expert-mlp"} | ({"identity-experts"} if l.mlp.identity else set()) | ({"grouped-routing"} if l.mlp.groups else set())
         elif l.mlp is not None:
             needs.add(f"{l.mlp.activation}-mlp")
     mlps = [l.mlp for l in cfg.layers if l.mlp is not None]

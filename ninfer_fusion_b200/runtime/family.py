@@ -29,6 +29,19 @@ def is_layered(cfg) -> bool:
     return isinstance(cfg, LayeredConfig)
 
 
+def context_limit(cfg, max_context: int) -> int:
+    """`max_context`, or as many positions as the model has vectors for."""
+    limit = getattr(cfg, "position_limit", 0)
+    return min(max_context, limit) if limit else max_context
+
+
+def check_positions(cfg, end: int) -> None:
+    """A sequence may not grow beyond the model's positions."""
+    limit = getattr(cfg, "position_limit", 0)
+    if limit and end > limit:
+        raise ValueError(f"{cfg.name}: position {end - 1} is beyond the model's {limit} positions")
+
+
 def kv_format_for(cfg, weights, kv_format):
     """Layer-list models keep their rows in the activation type."""
     if not is_layered(cfg):

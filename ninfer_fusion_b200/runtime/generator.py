@@ -17,6 +17,7 @@ import torch
 from ..models.config import ModelConfig
 from ..models.hybrid import ShardGeometry, StepBatch
 from .batch import SeqChunk, StepBuffers
+from .family import build_runtime, check_positions, context_limit
 
 
 def context_bucket(n: int) -> int:
@@ -41,11 +42,11 @@ class Generator:
             weights = OffloadedWeights(weights, self.device, int(weight_budget_bytes))
             if weights.plan.offloaded_layers:
                 use_graph = False
+        max_context = context_limit(cfg, max_context)
         self.max_batch, self.max_context = max_batch, max_context
         self.page_size = page_size
         self.prefill_chunk = prefill_chunk
         self.use_graph = use_graph and self.device.type == "cuda"
-        from .family import build_runtime
         pages_per_row = (max_context + page_size - 1) // page_size
         cap = max(prefill_chunk, max_batch)
         rt = build_runtime(cfg, weights, device, rows=max_batch, pages_per_row=pages_per_row,
@@ -102,6 +103,8 @@ class Generator:
         drive the rope; later decode positions are shifted by its rope_delta."""
         if len(prompts) > self.max_batch:
             raise ValueError("too many sequences")
+        for p in prompts:
+            check_positions(self.cfg, len(p))
         self.reset()
         B = len(prompts)
         bufs = self.bufs_prefill
@@ -119,7 +122,7 @@ class Generator:
             self.rows.append(b)
             self.slots.append(self.states.alloc())
             self.lengths.append(0)
-            self.kv.ensure(b, len(prompts[b]) + 1)
+            self.kv.ensure(b, context_limit(self.cfg, len(prompts[b]) + 1))
         self.kv.publish()
         first = [0] * B
         cursor = [0] * B
@@ -174,6 +177,7 @@ class Generator:
 
     def _ensure_pages(self, extra: int = 1) -> None:
         for b, r in enumerate(self.rows):
+            check_positions(self.cfg, self.lengths[b] + extra)
             self.kv.ensure(r, self.lengths[b] + extra)
         self.kv.publish()
 

@@ -17,7 +17,7 @@ from ..utils import trace
 from ..models.config import ModelConfig
 from ..models.hybrid import ShardGeometry, StepBatch
 from .batch import SeqChunk, StepBuffers
-from .family import build_runtime
+from .family import build_runtime, check_positions, context_limit
 from .generator import context_bucket
 from .program import Lane, ProgramBase, SamplingParams
 
@@ -32,6 +32,7 @@ class GpuProgram(ProgramBase):
         """`kv_format` "mixed" (or a per-layer list with "mixed" entries): those layers keep their cells in three
         precision tiers; `mixed_capacity` = cells per tier and layer, `descent` = a kv.descent.DescentConfig that
         `kv_descent_step` applies between rounds (None = cells only move when `kv.descend` is called by hand)."""
+        max_context = context_limit(cfg, max_context)
         super().__init__(cfg, max_lanes, max_context)
         if weight_budget_bytes is not None:
             from .weight_offload import OffloadedWeights
@@ -255,6 +256,8 @@ class GpuProgram(ProgramBase):
         portions of prompts beside single tokens, all in one batch.  Nothing is sampled; returns the wanted logits
         [rows, vocab] fp32 on the host, in the order of the entries and of their places.  Lanes come from `open_empty`."""
         chunks = []
+        for lane, tokens, want in entries:
+            check_positions(self.cfg, lane.n_cached + len(tokens))
         for lane, tokens, want in entries:
             self.kv.advance(lane.row, lane.n_cached, lane.n_cached + len(tokens))
             chunks.append(SeqChunk(lane.row, lane.slot, lane.n_cached, tokens, want=list(want)))
