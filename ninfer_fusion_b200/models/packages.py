@@ -221,4 +221,4 @@ def describe(model_id: str) -> dict:
             "hgrn2": p.count(GATED), "latent": p.count(LATENT), "chunked": p.count(CHUNKED), "rglru": p.count(RGLRU),
             "intermediate": p.intermediate, "vocab": p.vocab, "activation": p.activation, "final_logit_softcap": p.final_logit_softcap,
             "needs": sorted(p.needs), "missing": list(p.missing()), "servable": not p.missing() and p.config is not None,
-            "oracle_runtime": p.n_layers == p.count(FULL) + p.count(SLIDING) or isinstance(p.config, ModelConfig), "notes": p.notes}
+            "oracle_runtime": isinstance(p.config, ModelConfig) or (p.config is None and p.n_layers == p.count(FULL) + p.count(SLIDING)), "notes": p.notes}

@@ -1,0 +1,367 @@
+"""Ratilorn on the GPU through the engine's own step, scheduler and command line, against the plain oracle.
+
+Which experts a token takes can be a close call that rounding decides.  The bf16 runs therefore record the router's choices:
+each has to be right to rounding, and the oracle goes on with the same choices."""
+import json
+import os
+import subprocess
+import sys
+
+import numpy as np
+import pytest
+import torch
+
+import ratilorn_cases as C
+import ratilorn_oracle as K
+from kuzanex_cases import check, err, prompt
+
+pytestmark = pytest.mark.gpu
+ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+DTYPES = [torch.float32, torch.bfloat16]
+
+
+def n_experts(cfg):
+    return sum(l.mlp is not None and l.mlp.kind == "moe" for l in cfg.layers)
+
+
+def program(name, dt, tokens=512, lanes=4, page=16, **kw):
+    from ninfer_fusion_b200.models import ratilorn
+    from ninfer_fusion_b200.runtime.gpu_program import GpuProgram
+    _, cfg, t, _ = C.build(name)
+    w = ratilorn.pack(cfg, t.__getitem__, dt, "cuda:0")
+    kw = {"use_graph": False, "checkpoint_slots": 0, "prefill_chunk": tokens, **kw}
+    prog = GpuProgram(cfg, w, "cuda:0", max_lanes=lanes, max_context=tokens, kv_pages=tokens // page, page_size=page, **kw)
+    prog.choices = []                       # of every layer with experts, in the order of the launches
+    if n_experts(cfg):
+        raw = prog.model.ops.moe_route_scored
+
+        def route(*a):
+            raw(*a)
+            prog.choices.append(a[7].cpu().numpy().astype(np.int64))
+        prog.model.ops._cache["moe_route_scored"] = route
+    return prog
+
+
+_ORACLE = {}
+
+
+def oracle(name, n, seed):
+    key = (name, n, seed)
+    if key not in _ORACLE:
+        c, _, _, w = C.build(name)
+        ids = prompt(n, c["vocab"], seed)
+        _ORACLE[key] = (ids, K.forward(w, c, ids))
+    return _ORACLE[key]
+
+
+def verify(name, ids, got, want, choices, dt, what=""):
+    """Logits of all positions against the oracle's; `choices` as recorded, [layers with experts][T, top]."""
+    if dt == torch.float32:
+        check(got, want, dt, what)
+        return
+    c, _, _, w = C.build(name)
+    layers = [i for i, l in enumerate(c["layers"]) if (l["mlp"] or {}).get("kind") == "moe"]
+    forced, short = {i: None for i in range(len(c["layers"]))}, []
+    forced.update(zip(layers, choices))
+    want = K.forward(w, c, ids, choices=forced, short=short)
+    if short:
+        assert max(s.max() for s in short) < 0.08, (what, [s.max() for s in short])
+        assert np.mean(np.concatenate(short) > 0) < 0.08            # close calls are the exception
+    e = np.sqrt(((got - want - (got - want).mean(1, keepdims=True)) ** 2).mean(1)) / want.std()
+    assert np.isfinite(e).all() and e.max() < 0.08 and (e > 0.04).mean() < 0.05, (what, np.sort(e)[-5:])
+
+
+def run(prog, ids, cuts):
+    """(logits of all positions, choices [layers][T, top])"""
+    prog.choices.clear()
+    lane, out, at = prog.open_empty(), [], 0
+    for n in cuts:
+        n = min(n, len(ids) - at)
+        if n <= 0:
+            break
+        out.append(prog.step([(lane, ids[at:at + n], list(range(n)))]).numpy())
+        at += n
+    assert at == len(ids)
+    prog.close(lane)
+    prog.model.status.check()
+    n_moe = n_experts(prog.cfg)
+    steps = [prog.choices[i: i + n_moe] for i in range(0, len(prog.choices), n_moe)] if n_moe else []
+    return np.concatenate(out), [np.concatenate(x) for x in zip(*steps)]
+
+
+CUTS = {"whole": [10 ** 6], "tokens": [1] * 300, "twos": [2] * 150, "mixed": [3, 64, 1, 1, 17, 2, 65, 1, 7, 8, 9] * 9, "decode": [100] + [1] * 300}
+
+
+@pytest.mark.parametrize("dt", DTYPES)
+@pytest.mark.parametrize("name", sorted(C.CASES))
+def test_every_cut_of_a_prompt_gives_the_oracles_logits(name, dt):
+    """Whole prompt, token by token, portions down to two tokens, decoding past pages and chunks: every form of both attentions
+    and of the state space, the convolution across every border."""
+    ids, want = oracle(name, 141, 1)
+    prog = program(name, dt, tokens=160)
+    for what, cut in CUTS.items():
+        got, choices = run(prog, ids, cut)
+        verify(name, ids, got, want, choices, dt, what)
+    assert prog.kv.pool.free_pages == prog.kv.n_pages          # every page and slot came back
+    assert len(prog._free_rows) == 4 and len(prog.states._free) == 4
+
+
+def test_layers_leave_the_oracles_residual():
+    c, _, _, w = C.build("mixed")
+    ids = prompt(70, c["vocab"], 2)
+    _, per = K.forward(w, c, ids, True)
+    prog = program("mixed", torch.float32)
+    seen = []
+    prog.model.layer_hook = lambda run, x: seen.append(x.cpu().numpy().copy())
+    got, _ = run(prog, ids, [70])
+    assert len(seen) == len(per) == 5
+    for a, b in zip(seen, per):
+        assert np.abs(a - b).max() < 3e-5 * np.abs(b).max()
+    check(got, K.forward(w, c, ids), torch.float32)            # looking on changes nothing
+
+
+@pytest.mark.parametrize("dt", DTYPES)
+@pytest.mark.parametrize("name", ["mixed", "odd", "parallel_only", "sigmoid_only"])
+def test_mixed_batches_equal_each_request_alone(name, dt):
+    """Up to four live requests, portions beside single tokens, requests that pause, pages and slots used again; the pool
+    holds the live requests only."""
+    prog = program(name, dt, tokens=416)
+    rng = np.random.default_rng(3)
+    lens = [33, 141, 1, 64, 90, 17, 128, 2, 55]
+    todo, live, got = list(range(len(lens))), {}, {i: [] for i in range(len(lens))}
+    picks = {i: [] for i in range(len(lens))}
+    while todo or live:
+        while todo and len(live) < 4 and sum(-(-lens[i] // 16) * 16 for i in [*live, todo[0]]) <= 416:
+            live[todo.pop(0)] = [prog.open_empty(), 0]
+        entries, who = [], []
+        for i, (lane, at) in live.items():
+            if rng.random() < 0.2 and len(live) > 1:
+                continue                                        # left out of this step
+            n = min(int(rng.choice([1, 1, 2, 5, 16, 40, 70])), lens[i] - at)
+            entries.append((lane, oracle(name, lens[i], 10 + i)[0][at:at + n], list(range(n))))
+            who.append((i, n))
+        if not entries:
+            continue
+        prog.choices.clear()
+        lg, r = prog.step(entries).numpy(), 0
+        for i, n in who:
+            got[i].append(lg[r:r + n])
+            picks[i].append([x[r:r + n] for x in prog.choices])
+            r += n
+            live[i][1] += n
+            if live[i][1] == lens[i]:
+                prog.close(live.pop(i)[0])
+    for i, n in enumerate(lens):
+        ids, want = oracle(name, n, 10 + i)
+        verify(name, ids, np.concatenate(got[i]), want, [np.concatenate(x) for x in zip(*picks[i])], dt, i)
+    assert prog.kv.pool.free_pages == prog.kv.n_pages
+
+
+@pytest.mark.parametrize("name", ["mixed", "parallel_only", "sigmoid_only"])
+def test_prefill_kernels_and_token_kernels_agree(name):
+    ids, want = oracle(name, 141, 1)
+    prog = program(name, torch.bfloat16)
+    for kernels in (True, False):
+        prog.model.prefill_kernels = kernels
+        got, choices = run(prog, ids, [141])
+        verify(name, ids, got, want, choices, torch.bfloat16)
+
+
+@pytest.mark.parametrize("dt", DTYPES)
+def test_padding_stays_zero_and_only_wanted_places_come_back(dt):
+    ids, want = oracle("odd", 60, 2)
+    prog = program("odd", dt)
+    lane = prog.open_empty()
+    assert prog.step([(lane, ids[:20], [])]).shape == (0, want.shape[1])
+    lg = prog.step([(lane, ids[20:], [39, 0, 7])]).numpy()
+    if dt == torch.float32:
+        check(lg, want[[59, 20, 27]], dt)
+    assert lg.shape == (3, want.shape[1]) and not prog.ws.x[:40, prog.cfg.hidden:].any()
+
+
+@pytest.mark.parametrize("dt", DTYPES)
+@pytest.mark.parametrize("case", ["sigmoid_only", "parallel_only"])
+@pytest.mark.parametrize("far", [1, 2, 15, 16, 63, 64, 65, 200, 400])
+def test_a_key_far_away(case, far, dt):
+    """One layer alone.  The queries of the last token are turned so that the key of the token at position 1 stands out: alone
+    at the end of a portion, decoded, or with the key in a portion of two, the model sees what the oracle sees of it."""
+    from ninfer_fusion_b200.models import ratilorn
+    from ninfer_fusion_b200.runtime.gpu_program import GpuProgram
+    c, cfg, t, _ = C.build(case)
+    one = ratilorn.parse_config(dict(c, layers=[dict(c["layers"][0], mlp=None)], max_positions=512), case)
+    t = {n: v for n, v in t.items() if n.startswith("l0.") or not n.startswith("l")}
+    t["pos"] = t["pos"][:512].contiguous() * 0.25
+    w = {n: v.double().numpy() for n, v in t.items()}
+    cd, m = ratilorn.config_dict(one), one.attention_of(0)
+    p = "l0.mix." + ("left." if case == "parallel_only" else "")
+    h = lambda token, place: w["embed"][token] + w["pos"][place]
+    key = np.repeat((w[p + "k"] @ h(9, 1) + w[p + "k.b"]).reshape(m.kv_heads, m.dim), m.heads // m.kv_heads, axis=0).reshape(-1)
+    last = h(5, far + 1)
+    t[p + "q"] = torch.from_numpy(w[p + "q"] + 8.0 * np.outer(key, last / (last @ last))).to(torch.bfloat16)
+    if case == "sigmoid_only":
+        t["l0.mix.pb"] = t["l0.mix.pb"] - 4.0                   # the other keys hardly count
+    w = {n: v.double().numpy() for n, v in t.items()}
+    ids = [11 if i in (5, 9) else i for i in prompt(far + 2, c["vocab"], 6)]
+    ids[1], ids[far + 1] = 9, 5
+    want = K.forward(w, cd, ids)[-1:]
+    other = list(ids)
+    other[1] = 11
+    assert err(K.forward(w, cd, other)[-1:], want) > 0.05
+    prog = GpuProgram(one, ratilorn.pack(one, t.__getitem__, dt, "cuda:0"), "cuda:0", max_lanes=1, max_context=512, kv_pages=32, page_size=16,
+                      use_graph=False, checkpoint_slots=0, prefill_chunk=512)
+    for cuts in ([far + 2], [far + 1, 1], [2, far], [far, 2]):
+        lane, at = prog.open_empty(), 0
+        for n in cuts:
+            got = prog.step([(lane, ids[at:at + n], [n - 1])]).numpy()
+            at += n
+        prog.close(lane)
+        assert err(got, want) < (3e-5 if dt == torch.float32 else 0.03), cuts
+
+
+def test_positions_end_where_the_table_ends():
+    """437 positions: the last one is served, the next one refused, and the engine admits no longer request."""
+    ids, want = oracle("mixed", 437, 4)
+    prog = program("mixed", torch.float32, tokens=1024)
+    assert prog.max_context == 437 and not prog.can_admit(430, 8) and prog.can_admit(430, 7)
+    lane = prog.open_empty()
+    prog.step([(lane, ids[:430], [])])
+    got = prog.step([(lane, ids[430:], list(range(7)))]).numpy()
+    check(got, want[430:], torch.float32)
+    with pytest.raises(ValueError, match="position 437"):
+        prog.step([(lane, [1], [0])])
+    prog.close(lane)
+
+
+def test_long_decoding_in_32_bit():
+    ids, want = oracle("mixed", 420, 4)
+    prog = program("mixed", torch.float32, tokens=432, page=8)
+    check(run(prog, ids, [30] + [1] * 390)[0], want, torch.float32)
+
+
+# ---------------------------------------------------------------------------- engine
+def engine(name, dt, **kw):
+    from ninfer_fusion_b200.runtime.engine import Engine
+    chunk = kw.get("prefill_chunk", 64)
+
+    def make():
+        prog = program(name, dt, use_graph=True, **{"prefill_chunk": 64, **kw})
+        prog.model.ops._cache.pop("moe_route_scored", None)        # (no recording inside graphs)
+        return prog
+    return Engine(make, prefill_chunk=chunk, prefill_chunk_mode="manual")
+
+
+@pytest.mark.parametrize("name", ["mixed", "odd", "parallel_only", "sigmoid_only"])
+def test_greedy_generation_through_the_scheduler(name):
+    """Six unequal requests over four lanes, decode graphs on: every request's tokens are the oracle's."""
+    from ninfer_fusion_b200.runtime.engine import RequestOptions
+    c, _, _, w = C.build(name)
+    e = engine(name, torch.float32, tokens=256)
+    prompts = [prompt(n, c["vocab"], 40 + n) for n in (70, 1, 33, 9, 100, 18)]
+    hs = [e.submit(p, RequestOptions(max_tokens=12)) for p in prompts]
+    out = [h.wait(timeout=120) for h in hs]
+    assert all(h.finish_reason == "length" for h in hs), [h.error for h in hs]
+    for p, o in zip(prompts, out):
+        assert o == K.greedy(w, c, p, 12)
+    assert e.health()["free_lanes"] == 4
+    assert e.program.kv.pool.free_pages == e.program.kv.n_pages
+    e.shutdown()
+
+
+def test_bf16_generation_follows_the_oracle_step_by_step():
+    """In bf16 a near tie may fall the other way: every emitted token's oracle logit is close to the best."""
+    from ninfer_fusion_b200.runtime.engine import RequestOptions
+    c, _, _, w = C.build("mixed")
+    e = engine("mixed", torch.bfloat16, tokens=256)
+    prompts = [prompt(n, c["vocab"], 60 + n) for n in (80, 5, 31)]
+    hs = [e.submit(p, RequestOptions(max_tokens=30)) for p in prompts]
+    off = 0
+    for p, h in zip(prompts, hs):
+        toks = h.wait(timeout=120)
+        lg = K.forward(w, c, p + toks)[len(p) - 1:-1]
+        assert len(toks) == 30
+        off += sum(lg[j].max() - lg[j][t] > 0.1 * lg[j].std() for j, t in enumerate(toks))
+    assert off <= 9                                  # (an expert chosen the other way at a close call)
+    e.shutdown()
+
+
+def test_sampling_is_reproducible_and_respects_its_parameters():
+    from ninfer_fusion_b200.runtime.engine import RequestOptions
+    from ninfer_fusion_b200.runtime.program import SamplingParams
+    c, _, _, w = C.build("mixed")
+    e = engine("mixed", torch.float32, tokens=256)
+    p = prompt(20, c["vocab"], 3)
+    runs = [e.generate(p, RequestOptions(max_tokens=16, sampling=SamplingParams(temperature=1.5, top_k=8, seed=s))) for s in (1, 1, 2)]
+    assert runs[0] == runs[1] != runs[2]
+    for j, t in enumerate(runs[0]):
+        lg = K.forward(w, c, p + runs[0][:j])[-1]
+        assert (lg > lg[t] + 1e-3 * lg.std()).sum() < 8
+    e.shutdown()
+
+
+@pytest.mark.parametrize("cold", [False, True])
+def test_a_session_continues_from_its_frontier(cold, tmp_path):
+    """Second turn of a session: pages and the state image (state spaces and convolution inputs) are restored, also from a host
+    copy; only the new tokens are prefilled and the result is the same as from scratch."""
+    from ninfer_fusion_b200.runtime.engine import RequestOptions
+    c, _, _, w = C.build("mixed")
+    e = engine("mixed", torch.float32, tokens=512, checkpoint_slots=2)
+    if cold:
+        e.program.host_budget_bytes = 1 << 28
+    p = prompt(150, c["vocab"], 8)
+    first = e.generate(p, RequestOptions(max_tokens=5, session="s"))
+    if cold:
+        while e.program._evict_checkpoint():
+            pass
+        assert e.program.cold_stats["demoted_host"] >= 1
+    turn = p + first + prompt(21, c["vocab"], 9)
+    h = e.submit(turn, RequestOptions(max_tokens=6, session="s"))
+    assert h.wait(timeout=120) == K.greedy(w, c, turn, 6)
+    assert h.cached_tokens >= 150
+    e.shutdown()
+
+
+# ---------------------------------------------------------------------------- command line
+@pytest.fixture(scope="module")
+def folder(tmp_path_factory):
+    from ninfer_fusion_b200.models import architectures as AR
+    path = tmp_path_factory.mktemp("model")
+    _, cfg, t, _ = C.build("mixed")
+    AR.save_folder(str(path), cfg, t)
+    return str(path)
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_trace_run(folder, tmp_path, dtype):
+    (ia, wa), (ib, wb) = oracle("mixed", 90, 14), oracle("mixed", 33, 10)
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": ia[:50], "want": [49, 3]}], "end": []},
+             {"step": 1, "entries": [{"id": "a", "tokens": ia[50:51], "want": [0]}, {"id": "b", "tokens": ib[:32], "want": []}], "end": []},
+             {"step": 2, "entries": [{"id": "b", "tokens": ib[32:], "want": [0]}, {"id": "a", "tokens": ia[51:], "want": [38]}], "end": ["a", "b"]},
+             {"step": 3, "entries": [{"id": "a", "tokens": ib, "want": [5, 32]}], "end": ["a"]}]
+    r = subprocess.run([os.path.join(ROOT, "bin", "trace_run"), "--model", folder, "--dtype", dtype, "--out", str(tmp_path), "--max-tokens", "192"],
+                       input="".join(json.dumps(s) + "\n" for s in steps), capture_output=True, text=True, timeout=240)
+    assert r.returncode == 0, r.stderr
+    assert [x for x in r.stdout.splitlines() if x.startswith("done")] == [f"done {i}" for i in range(4)]
+    want = {0: wa[[49, 3]], 1: wa[[50]], 2: np.stack([wb[32], wa[89]]), 3: wb[[5, 32]]}
+    for i, x in want.items():
+        got = np.fromfile(tmp_path / f"{i}.f32", "<f4").reshape(x.shape)
+        if dtype == "float32":
+            d = got - x
+            d -= d.mean(1, keepdims=True)
+            assert np.sqrt((d * d).mean(1)).max() / wa.std() < 3e-5
+        assert np.isfinite(got).all()
+
+
+def test_generate_command(folder):
+    c, _, _, w = C.build("mixed")
+    p = prompt(20, 200, 5)
+    # the vocabulary is too small for the built-in byte tokenizer: the registered geometry runs the text path
+    r = subprocess.run([sys.executable, "-m", "ninfer_fusion_b200.cli", "generate", "--model", "ratilorn-tiny", "--random-init", "--raw",
+                        "--prompt", "Hello", "--max-tokens", "5", "--print-ids", "--greedy", "--max-context", "256"],
+                       capture_output=True, text=True, cwd=ROOT, timeout=240)
+    assert r.returncode == 0, r.stderr
+    assert len(json.loads(r.stderr.strip().splitlines()[-1])["completion_ids"]) == 5
+    r = subprocess.run([sys.executable, "-m", "ninfer_fusion_b200.cli", "generate", "--model", folder, "--float32", "--prompt-ids",
+                        ",".join(map(str, p)), "--max-tokens", "5", "--print-ids", "--greedy", "--max-context", "256"],
+                       capture_output=True, text=True, cwd=ROOT, timeout=240)
+    assert r.returncode == 0, r.stderr
+    assert json.loads(r.stderr.strip().splitlines()[-1])["completion_ids"] == K.greedy(w, c, p, 5)
