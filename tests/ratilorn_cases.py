@@ -40,7 +40,7 @@ def conf(width, vocab, layers, positions=512, scale=0.7, eps=1e-4):
 
 CASES = {
     "mixed": conf(96, 211, [par((6, 2, 32, 48, 0.3), (4, 32, 48, 2, 4, 2), dense(72)), sig(6, 3, 32, 16, mlp=moe(9, 2, 48, (3, 2))),
-                            par((4, 4, 16, 32, 0.4), (6, 16, 16, 3, 3, 6), moe(8, 3, 24, (4, 2))), sig(4, 2, 48, 32, v_mix=False, mlp=moe(6, 2, 40)),
+                            par((4, 4, 16, 32, 0.4), (6, 16, 16, 3, 3, 2), moe(8, 3, 24, (4, 2))), sig(4, 2, 48, 32, v_mix=False, mlp=moe(6, 2, 40)),
                             sig(9, 3, 16, 16, mlp=moe(8, 2, 32, (2, 1), None))], 437),
     # widths that are no multiple of anything, layers without feed-forward, one expert per token, the last layer ends with its mixer
     "odd": conf(90, 77, [sig(3, 1, 20, 36, mlp=moe(3, 1, 30, None, None)), par((5, 5, 12, 20, 0.5), (3, 20, 24, 1, 1, 4), dense(50)),

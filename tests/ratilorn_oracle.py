@@ -175,28 +175,25 @@ def route(z, correction, r, forced=None):
 
 
 def shortfall(z, correction, r, ids):
-    """Per token: how far the choices are from one that the scores allow (<= 0 for the right choice): the best choice score left
-    out in the chosen groups above the worst one taken, or the best group left out above the worst one used."""
+    """Per token: by how much scores would have to differ for the choices to be right (<= 0: they are): the best choice score
+    left out against the worst one taken, in every group that is used or kept by more than that, and the worst group used against
+    the last one kept."""
     c, groups = sigmoid(z) + correction, r.get("groups")
     taken = np.zeros(c.shape, dtype=bool)
     np.put_along_axis(taken, ids, True, axis=-1)
     assert (taken.sum(axis=-1) == ids.shape[1]).all()          # no expert twice
-    worst = np.where(taken, c, np.inf).min(axis=-1)
+    worst = np.where(taken, c, np.inf).min(axis=-1, keepdims=True)
     if not groups:
-        return np.where(taken, -np.inf, c).max(axis=-1) - worst
+        return np.where(taken, -np.inf, c).max(axis=-1) - worst[:, 0]
     n, keep = groups["count"], groups["keep"]
     parts, hit = c.reshape(len(c), n, -1), taken.reshape(len(c), n, -1)
     score, used = np.sort(parts, axis=-1)[..., -2:].sum(axis=-1), hit.any(axis=-1)
     assert (used.sum(axis=-1) <= keep).all()
-    out = np.empty(len(c))
-    for t in range(len(c)):
-        # the groups used and the best of the others, as many as may be kept
-        order = sorted(range(n), key=lambda g: (not used[t, g], -score[t, g]))[:keep]
-        rest = [g for g in range(n) if g not in order]
-        group = max((score[t, g] for g in rest), default=-np.inf) - min(score[t, g] for g in order)
-        left = max((parts[t, g][~hit[t, g]].max(initial=-np.inf) for g in order), default=-np.inf) - worst[t]
-        out[t] = max(group, left)
-    return out
+    order = -np.sort(-score, axis=-1)
+    last, after = order[:, keep - 1: keep], order[:, keep: keep + 1] if keep < n else np.full((len(c), 1), -np.inf)
+    left = np.where(hit, -np.inf, parts).max(axis=-1) - worst                  # of every group
+    kept = np.where(score >= last, np.minimum(left, score - after), -np.inf)   # a group kept by little need not have been
+    return np.maximum(np.maximum(np.where(used, left, kept).max(axis=-1), (last - np.where(used, score, np.inf)).max(axis=-1)), -1.0)
 
 
 def experts(w, p, h, mlp, forced=None, short=None):
