@@ -302,7 +302,7 @@ def main() -> int:
                     help="multi-GPU plan: tp = tensor parallel (dense default), ep = data parallel + expert parallel (MoE default)")
     ap.add_argument("--compare", default="",
                     help="not the headline benchmark: a layer-list geometry beside the closest other model of equal size (kuzanex-1b, kuzanex-7b: "
-                         "the hybrid decoder; tebivik-1b, tebivik-7b: Kuzanex; tuzupel-1b, tuzupel-7b: the hybrid decoder with experts), throughput and per-kernel roofline fractions, one JSON line (one GPU; --layers shrinks both)")
+                         "the hybrid decoder; tebivik-1b, tebivik-7b: Kuzanex; tuzupel-1b, tuzupel-7b, ratilorn-1b, ratilorn-7b: the hybrid decoder with experts), throughput and per-kernel roofline fractions, one JSON line (one GPU; --layers shrinks both)")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm(args)

@@ -4,7 +4,8 @@
 same generator (random weights, bf16), and for every kernel of the design its time, what bounds it, and the same for
 the other model's kernel of the like kind at equal size.  Kuzanex (head-mixing attention, matrix memory) stands beside the
 hybrid decoder, Tebivik (latent attention, gated memory) beside Kuzanex, Tuzupel (streams, experts, plain and latent attention,
-gated recurrence) beside the hybrid decoder with experts.  Kernels are timed cold (L2 flushed before every launch) with CUDA
+gated recurrence) and Ratilorn (head-mixing sigmoid attention, state space beside attention, experts) beside the hybrid decoder
+with experts and Kuzanex's kernels.  Kernels are timed cold (L2 flushed before every launch) with CUDA
 events; the roofline of a kernel is the slower of its algorithmic bytes at the measured copy bandwidth and its
 algorithmic multiply-adds at the measured bf16 GEMM rate.
 """
@@ -353,17 +354,20 @@ def compare(name: str, layers: int = 0, iters: int = 10, throughput: bool = True
     cfg = LAYERED_REGISTRY[name]
     if layers:
         cfg = cfg.shrink(layers)
-    streams = cfg.residual == "streams"
+    streams, branch = cfg.residual == "streams", cfg.residual == "branch"
     latent = not streams and any(l.mixer.kind == "latent_attention" for l in cfg.layers)
-    if streams:
-        from .streambench import equal_size_expert_hybrid, stream_kernels
-        other, label = equal_size_expert_hybrid(cfg), "hybrid"
+    if streams or branch:
+        from . import branchbench, streambench
+        other, label = (branchbench if branch else streambench).equal_size_expert_hybrid(cfg), "hybrid"
     else:
         other, label = (equal_size_kuzanex(cfg), "kuzanex") if latent else (equal_size_hybrid(cfg), "hybrid")
     res: Dict[str, object] = {"comparison": cfg.name, "design_params": cfg.param_count(), f"{label}_params": other.param_count(), "dtype": "bf16",
                               "data": "synthetic", "l2": "flushed before every kernel"}
     weights = random_layered_weights(cfg, "cuda:0")
-    rows = stream_kernels(cfg, other, weights, iters, only) if streams else _kernels(cfg, other, weights, iters, only)
+    if streams or branch:
+        rows = (branchbench.branch_kernels if branch else streambench.stream_kernels)(cfg, other, weights, iters, only)
+    else:
+        rows = _kernels(cfg, other, weights, iters, only)
     pair: Dict[str, dict] = {}
     for r in rows:
         pair.setdefault(r["kernel"], {})[r["model"]] = r
