@@ -74,8 +74,9 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(const MoeRo
 }
 
 // ---------------------------------------------------------------------------------------------
-// moe_route_scored: one warp per token
+// moe_route_scored: one warp per token; PL: outputs per lane
 // ---------------------------------------------------------------------------------------------
+template <int PL>
 __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_scored_kernel(const MoeRouteScoredParams p) {
   __shared__ float group_s[kRouteWarps][kMoeMaxExperts];
   pdl_launch_next();
@@ -85,29 +86,29 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_scored_kernel(cons
   if (t >= p.T) return;
   const int n = p.E + p.identity;
   const float* row = p.logits + static_cast<long long>(t) * p.ld;
-  float s[kPerLane], top = -INFINITY, sum = 0.f, inv = 1.f;
+  float s[PL], top = -INFINITY, sum = 0.f, inv = 1.f;
 #pragma unroll
-  for (int i = 0; i < kPerLane; ++i) {
+  for (int i = 0; i < PL; ++i) {
     const int e = lane + 32 * i;
     s[i] = e < n ? row[e] : -INFINITY;
     top = fmaxf(top, s[i]);
   }
   if (p.sigmoid) {
 #pragma unroll
-    for (int i = 0; i < kPerLane; ++i) s[i] = 1.f / (1.f + expf(-s[i]));
+    for (int i = 0; i < PL; ++i) s[i] = 1.f / (1.f + expf(-s[i]));
   } else {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
 #pragma unroll
-    for (int i = 0; i < kPerLane; ++i) {
+    for (int i = 0; i < PL; ++i) {
       s[i] = lane + 32 * i < n ? expf(s[i] - top) : 0.f;
       sum += s[i];
     }
     inv = 1.f / warp_sum(sum);
   }
-  float c[kPerLane];                               // choice scores
+  float c[PL];                               // choice scores
 #pragma unroll
-  for (int i = 0; i < kPerLane; ++i) {
+  for (int i = 0; i < PL; ++i) {
     const int e = lane + 32 * i;
     s[i] *= inv;
     c[i] = e < n ? s[i] + (p.correction != nullptr ? p.correction[e] : 0.f) : -INFINITY;
@@ -118,7 +119,7 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_scored_kernel(cons
     for (int g = 0; g < p.groups; ++g) {
       float a = -INFINITY, b = -INFINITY;          // the two largest of the group
 #pragma unroll
-      for (int i = 0; i < kPerLane; ++i) {
+      for (int i = 0; i < PL; ++i) {
         const int e = lane + 32 * i;
         if (e >= g * size && e < (g + 1) * size) {
           b = fmaxf(b, fminf(a, c[i]));
@@ -135,7 +136,7 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_scored_kernel(cons
     }
     __syncwarp();
 #pragma unroll
-    for (int i = 0; i < kPerLane; ++i) {
+    for (int i = 0; i < PL; ++i) {
       const int e = lane + 32 * i;
       if (e < n) {
         const int g = e / size;
@@ -151,7 +152,7 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_scored_kernel(cons
     float bv = -INFINITY, bs = 0.f;
     int bi = 0x7fffffff;
 #pragma unroll
-    for (int i = 0; i < kPerLane; ++i) {
+    for (int i = 0; i < PL; ++i) {
       const int e = lane + 32 * i;
       if (c[i] > bv || (c[i] == bv && e < bi && e < n)) { bv = c[i]; bs = s[i]; bi = e; }
     }
@@ -163,7 +164,7 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_scored_kernel(cons
     }
     if (bi >= n) bi = n - 1;                       // (every score a NaN)
 #pragma unroll
-    for (int i = 0; i < kPerLane; ++i)
+    for (int i = 0; i < PL; ++i)
       if (lane + 32 * i == bi) c[i] = -INFINITY;
     if (lane == 0) {
       const int a = t * p.k + r;
@@ -428,7 +429,11 @@ const char* moe_route_scored(const MoeRouteScoredParams& p, cudaStream_t stream,
   const int n = p.E + p.identity;
   if (p.E < 1 || p.identity < 0 || n > kMoeMaxExperts) return "moe_route: expert count out of range";
   if (p.k < 1 || p.k > n) return "moe_route: top-k out of range";
-  return launch_error(launch_kernel(moe_route_scored_kernel, dim3((p.T + kRouteWarps - 1) / kRouteWarps), dim3(kRouteWarps * 32), 0, stream, pdl, 1, p));
+  const dim3 grid((p.T + kRouteWarps - 1) / kRouteWarps), block(kRouteWarps * 32);
+  if (n <= 32) return launch_error(launch_kernel(moe_route_scored_kernel<1>, grid, block, 0, stream, pdl, 1, p));
+  if (n <= 64) return launch_error(launch_kernel(moe_route_scored_kernel<2>, grid, block, 0, stream, pdl, 1, p));
+  if (n <= 128) return launch_error(launch_kernel(moe_route_scored_kernel<4>, grid, block, 0, stream, pdl, 1, p));
+  return launch_error(launch_kernel(moe_route_scored_kernel<kPerLane>, grid, block, 0, stream, pdl, 1, p));
 }
 
 const char* moe_plan(const MoePlanParams& p, cudaStream_t stream) {

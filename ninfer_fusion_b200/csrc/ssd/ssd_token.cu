@@ -60,8 +60,18 @@ __global__ void __launch_bounds__(kThreads) ssd_decode_kernel(const SsdArgs p, i
       const int c = i < nv ? ch.x0 + v0 + i : (i < nv + N ? ch.b0 + i - nv : ch.c0 + i - nv - N);
       const float now = elem_to_f(in[c]);
       float a = fmaf(p.conv_w[static_cast<long long>(p.taps - 1) * ch.K + c], now, p.conv_b[c]);
-      for (int back = min(p.taps - 1, pos); back >= 1; --back)
-        a = fmaf(p.conv_w[static_cast<long long>(p.taps - 1 - back) * ch.K + c], ring[static_cast<long long>((pos - back) % p.taps) * ch.K + c], a);
+      for (int b0 = 1; b0 < p.taps; b0 += 3) {              // three earlier inputs at a time, their loads side by side
+        float x[3], w[3];
+#pragma unroll
+        for (int j = 0; j < 3; ++j) {
+          const int back = b0 + j;
+          const bool there = back < p.taps && back <= pos;
+          x[j] = there ? ring[static_cast<long long>((pos - back) % p.taps) * ch.K + c] : 0.f;
+          w[j] = there ? p.conv_w[static_cast<long long>(p.taps - 1 - back) * ch.K + c] : 0.f;
+        }
+#pragma unroll
+        for (int j = 0; j < 3; ++j) a = fmaf(w[j], x[j], a);
+      }
       a *= sigmoid_of<A>(a);
       (i < nv ? xs + i : (i < nv + N ? bs + i - nv : cs + i - nv - N))[0] = a;
       if (p.write_state && (i < nv || first)) ring[static_cast<long long>(pos % p.taps) * ch.K + c] = now;
