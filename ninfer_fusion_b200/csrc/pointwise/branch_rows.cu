@@ -29,18 +29,22 @@ __device__ __forceinline__ void block_sums(float (&v)[NS], float (*red)[16]) {
 
 // KV: four-column pieces per thread; PAIR: two branches.
 template <typename A, int KV, bool PAIR>
-__global__ void __launch_bounds__(512) branch_rows_kernel(const BranchRowsArgs p) {
+__global__ void __launch_bounds__(512, KV <= 4 ? 2 : 1) branch_rows_kernel(const BranchRowsArgs p) {
   __shared__ float red[2][2][16];
   const int tid = threadIdx.x, nt = blockDim.x, N = p.N;
-  float w[KV][4], wa[PAIR ? KV : 1][4], wb[PAIR ? KV : 1][4];
+  // the weights come ahead of the rows when there are registers for them
+  constexpr bool kAhead = KV <= 2;
+  float w[kAhead ? KV : 1][4], wa[PAIR && kAhead ? KV : 1][4], wb[PAIR && kAhead ? KV : 1][4];
+  if constexpr (kAhead) {
 #pragma unroll
-  for (int i = 0; i < KV; ++i) {
-    const int c = (tid + i * nt) * 4;
-    if (c < N) {
-      load4(p.w + c, w[i]);
-      if constexpr (PAIR) {
-        load4(p.w_a + c, wa[i]);
-        load4(p.w_b + c, wb[i]);
+    for (int i = 0; i < KV; ++i) {
+      const int c = (tid + i * nt) * 4;
+      if (c < N) {
+        load4(p.w + c, w[i]);
+        if constexpr (PAIR) {
+          load4(p.w_a + c, wa[i]);
+          load4(p.w_b + c, wb[i]);
+        }
       }
     }
   }
@@ -68,14 +72,20 @@ __global__ void __launch_bounds__(512) branch_rows_kernel(const BranchRowsArgs p
     block_sums<2>(s, red[1]);
     const float ia = 0.5f / sqrtf(s[0] * inv_n + p.eps), ib = 0.5f / sqrtf(s[1] * inv_n + p.eps);
 #pragma unroll
-    for (int i = 0; i < KV; ++i)
-      if ((tid + i * nt) * 4 < N) {
+    for (int i = 0; i < KV; ++i) {
+      const int c = (tid + i * nt) * 4, k = kAhead ? i : 0;
+      if (c < N) {
+        if constexpr (!kAhead) {
+          load4(p.w_a + c, wa[0]);
+          load4(p.w_b + c, wb[0]);
+        }
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          y[i][e] = y[i][e] * ia * wa[i][e] + v[i][e] * ib * wb[i][e];
+          y[i][e] = y[i][e] * ia * wa[k][e] + v[i][e] * ib * wb[k][e];
           s1[0] = fmaf(y[i][e], y[i][e], s1[0]);
         }
       }
+    }
   } else {
     const float g = mixture_gate(p.y, t);
 #pragma unroll
@@ -94,11 +104,12 @@ __global__ void __launch_bounds__(512) branch_rows_kernel(const BranchRowsArgs p
   float s2[1] = {0.f};
 #pragma unroll
   for (int i = 0; i < KV; ++i) {
-    const int c = (tid + i * nt) * 4;
+    const int c = (tid + i * nt) * 4, k = kAhead ? i : 0;
     if (c < N) {
+      if constexpr (!kAhead) load4(p.w + c, w[0]);
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        x[i][e] = fmaf(y[i][e] * inv, w[i][e], x[i][e]);
+        x[i][e] = fmaf(y[i][e] * inv, w[k][e], x[i][e]);
         s2[0] = fmaf(x[i][e], x[i][e], s2[0]);
       }
       store4(p.x + t * N + c, x[i]);
@@ -128,6 +139,10 @@ template <typename A, bool PAIR>
 cudaError_t pick_width(const BranchRowsArgs& a, cudaStream_t stream, bool pdl) {
   const int pieces = a.N / 4;
   auto threads = [&](int kv) { return dim3(((pieces + kv - 1) / kv + 31) / 32 * 32); };
+  if (a.T >= 512 && pieces > 256) {       // many rows: small CTAs, several of them per SM between each other's barriers
+    if (pieces <= 512) return launch_kernel(branch_rows_kernel<A, 2, PAIR>, dim3(a.T), threads(2), 0, stream, pdl, 1, a);
+    if (pieces <= 1024) return launch_kernel(branch_rows_kernel<A, 4, PAIR>, dim3(a.T), threads(4), 0, stream, pdl, 1, a);
+  }
   if (pieces <= 512) return launch_kernel(branch_rows_kernel<A, 1, PAIR>, dim3(a.T), threads(1), 0, stream, pdl, 1, a);
   if (pieces <= 1024) return launch_kernel(branch_rows_kernel<A, 2, PAIR>, dim3(a.T), threads(2), 0, stream, pdl, 1, a);
   if (pieces <= 2048) return launch_kernel(branch_rows_kernel<A, 4, PAIR>, dim3(a.T), threads(4), 0, stream, pdl, 1, a);
