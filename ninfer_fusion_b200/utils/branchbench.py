@@ -92,13 +92,13 @@ def _expert_block(k: _Kernels, model, ws, cfg, hyb, T: int, tag: str) -> None:
     at = _first(cfg, lambda l: l.mlp.kind == "moe")
     f, p, status = cfg.layers[at].mlp, f"text/layers/{at}", model.status.tensor
     E, kk, ff, sf = f.experts, f.top, f.expert.ff_p, f.shared.ff_p
-    x, delta, X = _rand(T, h), torch.empty(T, h, device="cuda"), torch.randn(T, h, device="cuda")
+    x, xo, delta, X = _rand(T, h), _rand(T, h), torch.empty(T, h, device="cuda"), torch.randn(T, h, device="cuda")
     used = int(torch.unique(run_experts(model, ws.experts, T, p, f, x, delta)["choice"]).numel())
     rows, weights = T * kk, (used * ff + sf) * 3 * h * 2
 
     def design():
         y = run_experts(model, ws.experts, T, p, f, x, delta)
-        ops.branch_rows(X, None, None, None, None, *y.values(), w[f"{p}/norm2"], None, x, cfg.hidden, 1e-6, False)
+        ops.branch_rows(X, None, None, None, None, *y.values(), w[f"{p}/norm2"], None, xo, cfg.hidden, 1e-6, False)      # (the next run routes the same rows)
     k.add(f"expert block {tag}", "design", design, weights + T * h * 14 + 2 * rows * h * 2, (rows * ff + T * sf) * 3 * h)
     block = MoeBlock(hyb, "cuda:0", T)
     hw = {f"l/moe/{n}": t for n, t in (("router", _rand(E + 1, h, s=0.02)), ("experts_gate_up", w[f"{p}/mlp/up"]), ("experts_down", w[f"{p}/mlp/down"]),
